@@ -1,10 +1,10 @@
 """Host-side bookkeeping of the cache: pages, block tables, groups, state slots.
 
 Keys and values live in pages of ``page_tokens`` tokens.  Layers whose needs are equal
-(``CacheNeed``: all keys, or a window of them, with the same head geometry) form a *group*;
+(``CacheNeed``: all keys, a window of them, or the current chunk's, with the same head geometry) form a *group*;
 every group has its own page pool and every request has one block table per group.  Pages are
 given back when a request ends, when it is preempted, and — in a window group — as soon as
-every key on them is older than the window; freed pages are handed out again (most recently
+every key on them is older than the window (or belongs to a chunk that has passed); freed pages are handed out again (most recently
 freed first).  Beside the pages, every admitted request holds one *slot* for state of fixed
 size; mixers of kind "state" keep their per-request tensors there.
 
@@ -178,6 +178,8 @@ class CacheManager:
         for gi, (need, _) in enumerate(grouped):
             if need.kind == "window" and getattr(need, "keep_first", 0) > 0:
                 self._lib.ember_cache_set_keep(self.core, gi, int(need.keep_first))
+            if need.kind == "window" and getattr(need, "chunk", 0) > 0:
+                self._lib.ember_cache_set_chunk(self.core, gi, int(need.chunk))
         self.groups: List[CacheGroup] = []
         for gi, (need, layers) in enumerate(grouped):
             pool = None
@@ -262,6 +264,11 @@ class CacheManager:
 
     def capacity_tokens(self) -> int:
         paged = [g.pool.n_pages * self.page_tokens for g in self.groups if g.paged and g.need.kind == "full"]
+        return min(paged) if paged else 1 << 30
+
+    def pool_tokens(self) -> int:
+        """Tokens the smallest page pool holds (groups that give pages back early serve longer requests than this)."""
+        paged = [g.pool.n_pages * self.page_tokens for g in self.groups if g.paged]
         return min(paged) if paged else 1 << 30
 
     def check(self) -> str:

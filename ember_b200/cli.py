@@ -79,7 +79,7 @@ def _load(args):
                           max_context=args.max_context or None, strict_weights=args.strict_weights)
     if args.verbose:
         r = llm.runner
-        print(f"[cache: {r.cache.capacity_tokens()} tokens in pages of {r.cache.page_tokens}, "
+        print(f"[cache: {r.cache.pool_tokens()} tokens in pages of {r.cache.page_tokens}, "
               f"{r.storage.bytes() / 2**20:.0f} MiB; context limit {llm.engine.scheduler.max_context}]", file=sys.stderr)
     return llm
 

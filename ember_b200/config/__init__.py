@@ -1,6 +1,6 @@
 """Typed configurations and the architecture registry."""
-from .spec import (AttentionSpec, ConfigError, DynamicTanhSpec, HyperConnectionSpec, TimeMixSpec, GatedDeltaSpec, GatedLinearAttentionSpec, GatedMLPSpec, LatentAttentionSpec,
-                   LayerNormSpec, LayerSpec, MatrixMemorySpec, ModelSpec, NoPositionSpec, ParallelMixerSpec, PartSpec,
+from .spec import (AttentionSpec, BigramEmbeddingSpec, ConcatReentrySpec, ConfigError, DynamicTanhSpec, HyperConnectionSpec, TimeMixSpec, GatedDeltaSpec, GatedLinearAttentionSpec, GatedMLPSpec, LatentAttentionSpec,
+                   LayerNormSpec, LayerSpec, MatrixMemorySpec, MLPSpec, ModelSpec, NoPositionSpec, ParallelMixerSpec, PartSpec,
                    RMSNormSpec, RotarySpec, RoutedMLPSpec, ScheduleEntry, SigmoidAttentionSpec, SigmoidGateSpec,
                    SinkAttentionSpec, StateSpaceSpec, default_schedule)
 from .registry import (config_from_dict, load_config, load_model_spec, register_architecture,
@@ -10,6 +10,7 @@ from .fadosun import FadosunConfig
 from .zufusun import ZufusunConfig
 from .fomanex import FomanexConfig
 from .pepapel import PepapelConfig
+from .filanex import FilanexConfig
 
 __all__ = [
     "AttentionSpec", "ConfigError", "GatedMLPSpec", "LayerSpec", "ModelSpec", "NoPositionSpec", "PartSpec",
@@ -18,5 +19,5 @@ __all__ = [
     "Qwen3Config", "FadosunConfig", "GatedDeltaSpec", "LayerNormSpec", "MatrixMemorySpec", "ParallelMixerSpec",
     "SigmoidAttentionSpec", "SigmoidGateSpec", "StateSpaceSpec", "ZufusunConfig", "GatedLinearAttentionSpec",
     "LatentAttentionSpec", "RoutedMLPSpec", "SinkAttentionSpec", "FomanexConfig", "DynamicTanhSpec", "HyperConnectionSpec",
-    "TimeMixSpec", "PepapelConfig",
+    "TimeMixSpec", "PepapelConfig", "FilanexConfig", "BigramEmbeddingSpec", "ConcatReentrySpec", "MLPSpec",
 ]

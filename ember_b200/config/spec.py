@@ -159,7 +159,8 @@ class SinkAttentionSpec(PartSpec):
     query at position p is multiplied by 1 + q_temp_coef * ln(floor((p + 1) / q_temp_every) + 1)); ``softcap`` > 0
     (score <- softcap * tanh(score / softcap) after the scale); ``chunk`` > 0 (position i sees j <= i only if
     floor(i / chunk) == floor(j / chunk), chunks counted from the sequence's start); ``head_gate`` (head h's output is
-    multiplied by sigmoid(W_g x)_h, tensor ``g`` [heads, hidden])."""
+    multiplied by sigmoid(W_g x)_h, tensor ``g`` [heads, hidden]); ``element_gate`` (the concatenated heads are multiplied
+    element by element by sigmoid(W_g x), tensor ``g`` [heads value_dim, hidden])."""
 
     kind: ClassVar[str] = "sink_attention"
     hidden_size: int = 0
@@ -181,6 +182,7 @@ class SinkAttentionSpec(PartSpec):
     softcap: float = 0.0
     chunk: int = 0
     head_gate: bool = False
+    element_gate: bool = False
 
 
 @dataclass(frozen=True)
@@ -353,6 +355,21 @@ class GatedMLPSpec(PartSpec):
 
 
 @dataclass(frozen=True)
+class MLPSpec(PartSpec):
+    """down( act(up(x)) ), one matrix up and one down; act is "gelu" (0.5 z (1 + erf(z / sqrt 2))).  ``names``: the two
+    tensors' names under the prefix (up, down); ``bias``: both have biases, named like the matrices with ``bias_suffix``
+    behind."""
+
+    kind: ClassVar[str] = "mlp"
+    hidden_size: int = 0
+    intermediate_size: int = 0
+    activation: str = "gelu"
+    names: Tuple[str, str] = ("up_proj.weight", "down_proj.weight")
+    bias: bool = False
+    bias_suffix: str = ".b"
+
+
+@dataclass(frozen=True)
 class RoutedMLPSpec(PartSpec):
     """Mixture of ``experts`` gated feed-forwards (tensors e0.., each gate, up, down, no biases) of which a token uses
     the ``top`` with the largest router logits (tensor ``router``, fp32), weighted by the softmax over those logits
@@ -380,11 +397,41 @@ class RoutedMLPSpec(PartSpec):
     # s + correction, and only outputs of the ``keep_groups`` best groups can be chosen.
     groups: int = 0
     keep_groups: int = 0
+    # ``group_score`` "max" as above, or "top2": a group's score is the sum of its two largest s + correction (of its only
+    # one, in groups of one).  ``renorm_eps`` is added to the sum the weights are divided by under ``renormalize``.
+    group_score: str = "max"
+    renorm_eps: float = 0.0
     # ``identity`` > 0: the router has ``experts`` + ``identity`` outputs; the last ``identity`` are experts without
     # tensors whose output is the token's input itself (times the weight).
     identity: int = 0
     # ``expert`` "gated" as above, or "square_relu": W_down relu(W_up h)^2, tensors e<i>.up and e<i>.down only.
     expert: str = "gated"
+
+
+# --------------------------------------------------------- what is added to the embedded tokens
+@dataclass(frozen=True)
+class BigramEmbeddingSpec(PartSpec):
+    """A hashed embedding of (previous token, token) added to the embedded token: row
+    (mul_prev * previous + mul_cur * token) mod ``buckets`` of a table of ``buckets`` + 1 rows; a sequence's first token
+    takes the last row.  The previous token is a per-request state.  Tensor: prefix + ``name`` [buckets + 1, size]."""
+
+    kind: ClassVar[str] = "bigram"
+    size: int = 0
+    buckets: int = 0
+    mul_prev: int = 1
+    mul_cur: int = 1
+    name: str = "bigram"
+
+
+# --------------------------------------------------------------- what comes ahead of a pass of a loop
+@dataclass(frozen=True)
+class ConcatReentrySpec(PartSpec):
+    """x <- W [x; x0] with x0 the embedding's output: how the stream enters a pass of a looped stretch of layers.
+    Tensor: prefix + ``name`` [size, 2 size], the columns of x first."""
+
+    kind: ClassVar[str] = "concat_linear"
+    size: int = 0
+    name: str = "weight"
 
 
 # ---------------------------------------------------------------------- connections
@@ -458,11 +505,13 @@ class ScheduleEntry:
     """One position in the run order.  ``layer`` indexes ``ModelSpec.layers``; a layer
     may appear more than once.  ``cache_of`` names the layer whose cache this run
     reads and writes; -1 means its own.  ``instance`` tells the caches of one layer apart: a layer
-    that runs several times with the same weights (a loop) keeps one cache or state per pass."""
+    that runs several times with the same weights (a loop) keeps one cache or state per pass.  ``reentry``: the model's
+    re-entry part (``ModelSpec.reentry``) mixes the stream with the embedding's output right before this run."""
 
     layer: int
     cache_of: int = -1
     instance: int = 0
+    reentry: bool = False
 
 
 @dataclass(frozen=True)
@@ -499,6 +548,13 @@ class ModelSpec:
     # the residual stream in ``residual_streams`` copies (hyper-connections): all equal to the embedding's output at the
     # start, read and written by the layers' connections, summed before the final norm
     residual_streams: int = 1
+    # a term added to the embedded (and scaled) tokens in the embedding's own kernel (a hashed bigram embedding); it may
+    # keep a per-request state
+    embedding_term: Optional[PartSpec] = None
+    embedding_term_prefix: str = ""
+    # how the stream is mixed with the embedding's output before the runs of the schedule marked ``reentry``
+    reentry: Optional[PartSpec] = None
+    reentry_prefix: str = ""
 
     def __post_init__(self):
         n = len(self.layers)
@@ -515,6 +571,11 @@ class ModelSpec:
                 raise ConfigError("a schedule entry's cache instance cannot be negative")
         if self.residual_streams < 1:
             raise ConfigError("a model has at least one residual stream")
+        if any(e.reentry for e in self.schedule):
+            if self.reentry is None:
+                raise ConfigError("the schedule re-enters a loop; the model has no re-entry part")
+            if self.residual_streams != 1:
+                raise ConfigError("a re-entry part mixes a single residual stream")
 
 
 def default_schedule(n_layers: int) -> Tuple[ScheduleEntry, ...]:

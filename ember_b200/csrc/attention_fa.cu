@@ -58,6 +58,8 @@ struct FaParams {
     int chunk;                // > 0: a query sees a key only inside its own chunk of positions (chunks counted from position 0)
     float scale_log2;
     float cap_over_scale, scale_over_cap;   // a cap on the scaled scores, cap * tanh(scale s / cap), applied to the raw scores as (cap / scale) tanh(s scale / cap); 0: no cap
+    const float* gate;        // logits of a gate per output element: row t, element head * 128 + d, or null
+    int ld_gate;              // (a multiple of 4, rows 16-byte aligned)
     int n_tiles;
     int* err;
 };
@@ -470,12 +472,23 @@ attention_fa_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
             const float inv = l_run > 0.0f ? 1.0f / l_run : 0.0f;
             const int rq = r / G, rg = r - rq * G;
             __nv_bfloat16* dst = p.out + ((size_t)(row0 + rq) * p.n_heads + kvh * G + rg) * FA_D;
+            const float* gate = p.gate ? p.gate + (size_t)(row0 + rq) * p.ld_gate + (kvh * G + rg) * FA_D : nullptr;
 #pragma unroll
             for (int c = 0; c < FA_D / 32; c++) {
                 uint32_t tu[32];
                 fa_tmem_ld32_nowait(tmem_o + lane_base + (uint32_t)(c * 32), tu);
                 fa_tmem_wait_ld();
                 if (ok && r < rows) {
+                    if (gate) {
+#pragma unroll
+                        for (int e = 0; e < 32; e += 4) {
+                            const float4 gv = __ldg(reinterpret_cast<const float4*>(gate + c * 32 + e));
+                            tu[e] = __float_as_uint(__uint_as_float(tu[e]) / (1.0f + __expf(-gv.x)));
+                            tu[e + 1] = __float_as_uint(__uint_as_float(tu[e + 1]) / (1.0f + __expf(-gv.y)));
+                            tu[e + 2] = __float_as_uint(__uint_as_float(tu[e + 2]) / (1.0f + __expf(-gv.z)));
+                            tu[e + 3] = __float_as_uint(__uint_as_float(tu[e + 3]) / (1.0f + __expf(-gv.w)));
+                        }
+                    }
 #pragma unroll
                     for (int q4 = 0; q4 < 4; q4++) {
                         uint4 packed;
@@ -558,8 +571,10 @@ EMBER_API int ember_attention_fa_tile_queries(int group) { return group >= 1 && 
 
 EMBER_API int ember_attention_fa(const void* q, const void* k_pool, const void* v_pool, void* out, int n_heads, int n_kv,
                                  int D, const int* tiles, int n_tiles, const int* block_table, int max_blocks, int page,
-                                 int num_pages, int window, float scale, int* err, float softcap, int chunk, void* stream) {
+                                 int num_pages, int window, float scale, int* err, float softcap, int chunk, const float* gate, int ld_gate,
+                                 void* stream) {
     if (n_tiles <= 0) return 0;
+    if (gate && ((((uintptr_t)gate) & 15) || ld_gate < n_heads * FA_D || (ld_gate & 3))) return fail("attention_fa: gate rows of %d", ld_gate);
     if (n_heads <= 0 || n_kv <= 0 || n_heads % n_kv) return fail("attention_fa: bad head counts %d/%d", n_heads, n_kv);
     if (!ember_attention_fa_supported(D, n_heads / n_kv, page))
         return fail("attention_fa: head size %d, group %d, page %d are not taken", D, n_heads / n_kv, page);
@@ -573,7 +588,7 @@ EMBER_API int ember_attention_fa(const void* q, const void* k_pool, const void* 
     p.max_blocks = max_blocks; p.page = page; p.num_pages = num_pages; p.n_heads = n_heads; p.n_kv = n_kv;
     p.window = window; p.chunk = chunk < 0 ? 0 : chunk; p.scale_log2 = scale * FA_LOG2E;
     p.cap_over_scale = (softcap > 0.0f && scale > 0.0f) ? softcap / scale : 0.0f;
-    p.scale_over_cap = softcap > 0.0f ? scale / softcap : 0.0f; p.n_tiles = n_tiles; p.err = err;
+    p.scale_over_cap = softcap > 0.0f ? scale / softcap : 0.0f; p.gate = gate; p.ld_gate = ld_gate; p.n_tiles = n_tiles; p.err = err;
     const size_t smem = (size_t)2 * FA_ROWS * 128 + (size_t)(FA_K_STAGES + FA_V_STAGES) * 2 * FA_KT * 128 + 256;
     static bool attr = false;
     if (!attr) {

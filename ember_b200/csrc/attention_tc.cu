@@ -50,6 +50,8 @@ struct AttnTcParams {
     int chunk;                // > 0: a query sees a key only inside its own chunk of positions (chunks counted from position 0)
     float scale_log2;         // softmax scale * log2(e)
     float cap_log2, scale_over_cap;   // a cap on the scaled scores, cap * tanh(score / cap): cap * log2(e) and scale / cap (0: no cap)
+    const float* gate;        // logits of a gate per output element: row t, element head * D + d, or null
+    int ld_gate;
     int n_splits, split_keys;
     int n_tiles;
     int cluster_merge;        // the splits of a tile are a thread-block cluster and are merged in its first block's shared memory
@@ -62,6 +64,9 @@ __device__ __forceinline__ uint32_t s32(const void* p) { return (uint32_t)__cvta
 __device__ __forceinline__ float score_log2(const AttnTcParams& p, float raw) {
     return p.cap_log2 > 0.0f ? p.cap_log2 * tanhf(raw * p.scale_over_cap) : raw * p.scale_log2;
 }
+
+// A result element times the sigmoid of its gate's logit, where the layer has such a gate (`g` points at the row's logits).
+__device__ __forceinline__ float gated(const float* g, int i, float v) { return g ? v / (1.0f + __expf(-__ldg(g + i))) : v; }
 
 __device__ __forceinline__ void ldsm_x4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
@@ -152,8 +157,10 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
     int lo = max(p.window > 0 ? max(0, pos0 - p.window + 1) : 0, p.chunk > 0 ? pos0 - pos0 % p.chunk : 0);
     int hi = pos0 + nq;
     if (p.n_splits > 1) {
-        lo = max(lo, split * p.split_keys);
-        hi = min(hi, (split + 1) * p.split_keys);
+        // splits are ranges of a fixed length from key 0 on, with chunks from the tile that holds the chunk's first key
+        const int base = p.chunk > 0 ? (pos0 - pos0 % p.chunk) / KT * KT : 0;
+        lo = max(lo, base + split * p.split_keys);
+        hi = min(hi, base + (split + 1) * p.split_keys);
     }
     const int k_begin = lo - (lo % KT);
     const int n_kt = hi > k_begin ? (hi - k_begin + KT - 1) / KT : 0;
@@ -369,16 +376,20 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
         if (r_a < rows) {
             const int qi = r_a / G, g = r_a - qi * G;
             __nv_bfloat16* dst = p.out + ((size_t)(row0 + qi) * p.n_heads + kvh * G + g) * D;
+            const float* gt = p.gate ? p.gate + (size_t)(row0 + qi) * p.ld_gate + (kvh * G + g) * D : nullptr;
 #pragma unroll
             for (int j = 0; j < ND; j++)
-                *reinterpret_cast<uint32_t*>(dst + j * 8 + 2 * t4) = pack_bf16(o[j][0] * inv_a, o[j][1] * inv_a);
+                *reinterpret_cast<uint32_t*>(dst + j * 8 + 2 * t4) =
+                    pack_bf16(gated(gt, j * 8 + 2 * t4, o[j][0] * inv_a), gated(gt, j * 8 + 2 * t4 + 1, o[j][1] * inv_a));
         }
         if (r_b < rows) {
             const int qi = r_b / G, g = r_b - qi * G;
             __nv_bfloat16* dst = p.out + ((size_t)(row0 + qi) * p.n_heads + kvh * G + g) * D;
+            const float* gt = p.gate ? p.gate + (size_t)(row0 + qi) * p.ld_gate + (kvh * G + g) * D : nullptr;
 #pragma unroll
             for (int j = 0; j < ND; j++)
-                *reinterpret_cast<uint32_t*>(dst + j * 8 + 2 * t4) = pack_bf16(o[j][2] * inv_b, o[j][3] * inv_b);
+                *reinterpret_cast<uint32_t*>(dst + j * 8 + 2 * t4) =
+                    pack_bf16(gated(gt, j * 8 + 2 * t4, o[j][2] * inv_b), gated(gt, j * 8 + 2 * t4 + 1, o[j][3] * inv_b));
         }
         return;
     }
@@ -401,6 +412,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
     }
     __syncthreads();
     if (merge_in_cluster) atc_cluster_wait();
+    const float* gate_row = p.gate ? p.gate + (size_t)row0 * p.ld_gate + kvh * G * D : nullptr;     // (nq == 1)
     const uint32_t recv_o0 = atc_map_to_rank(s32(recv), 0);
     const uint32_t recv_ml0 = recv_o0 + (uint32_t)(p.n_splits * rows * D) * 4u;
     for (int idx = threadIdx.x; idx < rows * D; idx += ATC_THREADS) {
@@ -419,7 +431,8 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
         }
         // nq == 1: row r is head r of the group
         if (p.n_splits <= 1) {
-            p.out[((size_t)row0 * p.n_heads + kvh * G + r) * D + d] = __float2bfloat16_rn(L > 0.0f ? acc / L : 0.0f);
+            p.out[((size_t)row0 * p.n_heads + kvh * G + r) * D + d] =
+                __float2bfloat16_rn(gated(gate_row, r * D + d, L > 0.0f ? acc / L : 0.0f));
         } else if (merge_in_cluster) {
             atc_st_cluster(recv_o0 + (uint32_t)((split * rows + r) * D + d) * 4u, acc);
             if (d == 0) {
@@ -454,7 +467,8 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
                 L += rml[(sp * rows + r) * 2 + 1] * f;
                 acc = fmaf(ro[((size_t)sp * rows + r) * D + d], f, acc);
             }
-            p.out[((size_t)row0 * p.n_heads + kvh * G + r) * D + d] = __float2bfloat16_rn(L > 0.0f ? acc * (1.0f / L) : 0.0f);
+            p.out[((size_t)row0 * p.n_heads + kvh * G + r) * D + d] =
+                __float2bfloat16_rn(gated(gate_row, r * D + d, L > 0.0f ? acc * (1.0f / L) : 0.0f));
         }
     }
 }
@@ -465,7 +479,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
 // dependent loads before, which is what the kernel's time was at batch 1 with 13 splits).
 __global__ void attention_tc_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                             __nv_bfloat16* __restrict__ out, const int* __restrict__ tiles,
-                                            int n_heads, int n_splits, int D) {
+                                            int n_heads, int n_splits, int D, const float* __restrict__ gate, int ld_gate) {
     extern __shared__ float w_s[];                                         // [n_splits] weights, then 1 / L
     float& inv_s = w_s[n_splits];
     pdl_launch_dependents();
@@ -473,6 +487,7 @@ __global__ void attention_tc_combine_kernel(const float* __restrict__ part_o, co
     const size_t th = blockIdx.x;                                          // tile * n_heads + head
     const int tile = (int)(th / n_heads), head = (int)(th % n_heads);
     const size_t oh = (size_t)tiles[tile * 4 + 1] * n_heads + head;        // the tile's single token row
+    const float* gate_row = gate ? gate + (size_t)tiles[tile * 4 + 1] * ld_gate + head * D : nullptr;
     const float* ml = part_ml + th * n_splits * 2;
     // Up to 16 splits (what the planner makes): a thread's partial sums are requested now, so that they travel
     // while the first warp forms the weights (one trip to memory behind the dependency instead of two).
@@ -509,7 +524,7 @@ __global__ void attention_tc_combine_kernel(const float* __restrict__ part_o, co
 #pragma unroll
         for (int s = 0; s < EARLY; s++)
             if (s < n_splits) o = fmaf(a[s], w_s[s], o);                   // ascending, as below
-        out[oh * D + threadIdx.x] = __float2bfloat16_rn(o * inv);
+        out[oh * D + threadIdx.x] = __float2bfloat16_rn(gated(gate_row, threadIdx.x, o * inv));
     }
     for (int d = (int)threadIdx.x + (early ? (int)blockDim.x : 0); d < D; d += blockDim.x) {
         const float* po = part_o + th * n_splits * D + d;
@@ -523,7 +538,7 @@ __global__ void attention_tc_combine_kernel(const float* __restrict__ part_o, co
             o = fmaf(a3, w_s[s + 3], o);
         }
         for (; s < n_splits; s++) o = fmaf(po[(size_t)s * D], w_s[s], o);
-        out[oh * D + d] = __float2bfloat16_rn(o * inv);
+        out[oh * D + d] = __float2bfloat16_rn(gated(gate_row, d, o * inv));
     }
 }
 
@@ -592,8 +607,9 @@ EMBER_API int ember_attention_tc(const void* q, const void* k_pool, const void* 
                                  int n_heads, int n_kv, int D, const int* tiles, int n_tiles,
                                  const int* block_table, int max_blocks, int page, int num_pages, int window,
                                  float scale, int n_splits, int split_keys, float* part_o, float* part_ml,
-                                 int* err, float softcap, int chunk, void* stream) {
+                                 int* err, float softcap, int chunk, const float* gate, int ld_gate, void* stream) {
     if (n_tiles <= 0) return 0;
+    if (gate && ld_gate < n_heads * D) return fail("attention_tc: gate rows of %d", ld_gate);
     if (softcap < 0.0f) return fail("attention_tc: a score cap of %g", softcap);
     if (n_heads <= 0 || n_kv <= 0 || n_heads % n_kv) return fail("attention_tc: bad head counts %d/%d", n_heads, n_kv);
     const int G = n_heads / n_kv;
@@ -616,6 +632,7 @@ EMBER_API int ember_attention_tc(const void* q, const void* k_pool, const void* 
     p.tiles = tiles; p.block_table = block_table; p.max_blocks = max_blocks; p.page = page; p.num_pages = num_pages;
     p.n_heads = n_heads; p.n_kv = n_kv; p.window = window; p.chunk = chunk < 0 ? 0 : chunk; p.scale_log2 = scale * LOG2E;
     p.cap_log2 = softcap * LOG2E; p.scale_over_cap = softcap > 0.0f ? scale / softcap : 0.0f;
+    p.gate = gate; p.ld_gate = ld_gate;
     p.n_splits = n_splits; p.split_keys = split_keys; p.n_tiles = n_tiles; p.err = err;
     p.cluster_merge = cluster_merge ? 1 : 0;
     cudaStream_t st = (cudaStream_t)stream;
@@ -654,7 +671,7 @@ EMBER_API int ember_attention_tc(const void* q, const void* k_pool, const void* 
     if (n_splits > 1 && !cluster_merge) {
         launch_kernel(attention_tc_combine_kernel, (unsigned)((size_t)n_tiles * n_heads), D, (size_t)(n_splits + 1) * sizeof(float), st,
                       (const float*)part_o,
-                      (const float*)part_ml, (__nv_bfloat16*)out, tiles, n_heads, n_splits, D);
+                      (const float*)part_ml, (__nv_bfloat16*)out, tiles, n_heads, n_splits, D, gate, ld_gate);
         return check_launch("attention_tc_combine");
     }
     return 0;

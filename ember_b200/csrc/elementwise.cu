@@ -33,6 +33,70 @@ __global__ void embed_kernel(const int* __restrict__ tokens, const int* __restri
     for (int i = threadIdx.x; i < H; i += blockDim.x) o[i] = scale * to_float(row[i]);
 }
 
+// The same with a hashed row of (previous token, token) added: row (mul_prev * previous + mul_cur * token) mod buckets of a
+// second table of buckets + 1 rows, the last of which is a sequence's first token's.  A run's first token finds its
+// previous one in the request's state slot (int32); the block of that token also leaves the run's last token there, so the
+// slot is read and written by one thread and nothing depends on the order of blocks.
+struct BigramArgs {
+    const void* table;
+    long long buckets, mul_prev, mul_cur;
+    const int* positions; const int* seq_of; const int* query_start; const int* slots;
+    int* state; int state_stride;      // ints from one slot to the next
+};
+template <typename TW, typename TB>
+__global__ void embed_bigram_kernel(const int* __restrict__ tokens, const int* __restrict__ prev_ids, int n_prev,
+                                    const TW* __restrict__ table, float* __restrict__ out, int H, int V, float scale, BigramArgs g,
+                                    int* __restrict__ err) {
+    __shared__ int picked[2];                                // the token and its bigram row (-1: a token out of range)
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x;
+    if (threadIdx.x == 0) {
+        auto token = [&](int i) {
+            int k = tokens[i];
+            if (k < 0 && prev_ids != nullptr && -k <= n_prev) k = prev_ids[-k - 1];
+            return k;
+        };
+        const int tok = token(t), seq = g.seq_of[t], first = g.query_start[seq];
+        int prev;
+        if (t > first) prev = token(t - 1);
+        else {
+            int* slot = g.state + (size_t)g.slots[seq] * g.state_stride;
+            prev = *slot;
+            *slot = token(g.query_start[seq + 1] - 1);
+        }
+        const bool start = g.positions[t] == 0;
+        const bool bad = tok < 0 || tok >= V || (!start && (prev < 0 || prev >= V));
+        if (bad && err) atomicOr(err, EMBER_ERR_TOKEN_RANGE);
+        picked[0] = tok;
+        picked[1] = bad ? -1 : (start ? (int)g.buckets : (int)((g.mul_prev * prev + g.mul_cur * tok) % g.buckets));
+    }
+    __syncthreads();
+    float* o = out + (size_t)t * H;
+    if (picked[1] < 0) {
+        for (int i = threadIdx.x; i < H; i += blockDim.x) o[i] = 0.0f;
+        return;
+    }
+    const TW* row = table + (size_t)picked[0] * H;
+    const TB* two = (const TB*)g.table + (size_t)picked[1] * H;
+    for (int i = threadIdx.x; i < H; i += blockDim.x) o[i] = scale * to_float(row[i]) + to_float(two[i]);
+}
+
+// out[t, col + i] = x[t, i] (and out[t, col2 + i] with col2 >= 0) in rows of ld: an fp32 row as one half of a wider row in the
+// activations' type, the operand of a product over two concatenated inputs.
+template <typename TO>
+__global__ void place_columns_kernel(const float* __restrict__ x, TO* __restrict__ out, int H, int ld, int col, int col2) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const float* in = x + (size_t)blockIdx.x * H;
+    TO* o = out + (size_t)blockIdx.x * ld;
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+        const TO v = from_float<TO>(in[i]);
+        o[col + i] = v;
+        if (col2 >= 0) o[col2 + i] = v;
+    }
+}
+
 // -------------------------------------------------------------------------------- RMSNorm
 // out[r, i] = w[i] * (x[row(r), i] * (1 / sqrt(mean(x^2) + eps))), statistics in fp32.
 // `rows` (nullable) gathers input rows: the final norm runs only on the rows whose logits
@@ -424,6 +488,43 @@ EMBER_API int ember_embed(const int* tokens, const int* prev_ids, int n_prev, co
     else
         return fail("embed: unsupported table dtype %d", table_dtype);
     return check_launch("embed");
+}
+
+EMBER_API int ember_embed_bigram(const int* tokens, const int* prev_ids, int n_prev, const void* table, const void* bigram,
+                                 int table_dtype, int bigram_dtype, float* out, int T, int H, int V, float scale, long long buckets, long long mul_prev,
+                                 long long mul_cur, const int* positions, const int* seq_of, const int* query_start, const int* slots,
+                                 int* state, int state_stride, int* err, void* stream) {
+    if (T <= 0) return 0;
+    if (H <= 0 || V <= 0) return fail("embed_bigram: bad sizes H=%d V=%d", H, V);
+    const long long most = 1ll << 31;
+    if (buckets <= 0 || buckets >= most || mul_prev < 0 || mul_prev >= most || mul_cur < 0 || mul_cur >= most || state_stride <= 0)
+        return fail("embed_bigram: %lld buckets, multipliers %lld and %lld (each below 2^31)", buckets, mul_prev, mul_cur);
+    cudaStream_t st = (cudaStream_t)stream;
+    const BigramArgs g{bigram, buckets, mul_prev, mul_cur, positions, seq_of, query_start, slots, state, state_stride};
+    const int threads = H >= 1024 ? 256 : 128;
+    if ((table_dtype != EMBER_F32 && table_dtype != EMBER_BF16) || (bigram_dtype != EMBER_F32 && bigram_dtype != EMBER_BF16))
+        return fail("embed_bigram: unsupported table dtypes %d / %d", table_dtype, bigram_dtype);
+    auto run = [&](auto kernel, auto* tab) { launch_kernel(kernel, T, threads, 0, st, tokens, prev_ids, n_prev, tab, out, H, V, scale, g, err); };
+    const bool wide = bigram_dtype == EMBER_F32;
+    if (table_dtype == EMBER_F32) {
+        if (wide) run(embed_bigram_kernel<float, float>, (const float*)table);
+        else run(embed_bigram_kernel<float, __nv_bfloat16>, (const float*)table);
+    } else {
+        if (wide) run(embed_bigram_kernel<__nv_bfloat16, float>, (const __nv_bfloat16*)table);
+        else run(embed_bigram_kernel<__nv_bfloat16, __nv_bfloat16>, (const __nv_bfloat16*)table);
+    }
+    return check_launch("embed_bigram");
+}
+
+EMBER_API int ember_place_columns(const float* x, void* out, int out_dtype, int T, int H, int ld, int col, int col2, void* stream) {
+    if (T <= 0) return 0;
+    if (H <= 0 || col < 0 || col + H > ld || (col2 >= 0 && col2 + H > ld)) return fail("place_columns: %d columns at %d / %d of rows of %d", H, col, col2, ld);
+    cudaStream_t st = (cudaStream_t)stream;
+    const int threads = H >= 1024 ? 256 : 128;
+    if (out_dtype == EMBER_F32) launch_kernel(place_columns_kernel<float>, T, threads, 0, st, x, (float*)out, H, ld, col, col2);
+    else if (out_dtype == EMBER_BF16) launch_kernel(place_columns_kernel<__nv_bfloat16>, T, threads, 0, st, x, (__nv_bfloat16*)out, H, ld, col, col2);
+    else return fail("place_columns: unsupported output dtype %d", out_dtype);
+    return check_launch("place_columns");
 }
 
 EMBER_API int ember_rmsnorm(const float* x, const int* rows, const float* w, float eps, void* out, int out_dtype,

@@ -46,7 +46,8 @@ struct GemmTcParams {
     int num_k_blocks;     // ceil(K / TILE_K)
     int k_blocks_per_split;
     int epilogue;         // 0 store bf16, 1 store fp32, 2 add fp32, 3 act(gate)*up -> bf16
-    int act;              // epilogue 3: 0 silu, 1 relu, 2 gelu (tanh form)
+    int act;              // epilogue 3: 0 silu, 1 relu, 2 gelu (tanh form); epilogue 0: 0 none, 3 gelu (exact, by erf)
+    const float* bias;    // [N] added to the sums of epilogues 0, 1 and 2 (once, whatever the parts of K), or null
     void* out;
     int ldc;
     float* accum;         // atomic split-K target: fp32 [M, accum_ld] (the residual itself for epilogue 2)
@@ -147,9 +148,28 @@ __device__ __forceinline__ float gate_mul(float g, float u, int act) {
     return (act ? fmaxf(g, 0.0f) : g / (1.0f + __expf(-g))) * u;
 }
 
+__device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f)); }
+// A complete sum of output column n as the plain epilogues (0, 1, 2) want it: with its bias, through its activation.
+__device__ __forceinline__ float finish_sum(const GemmTcParams& p, int n, float v) {
+    if (p.bias) v += __ldg(p.bias + n);
+    return p.act == 3 ? gelu_erf(v) : v;
+}
+
 // Fused epilogue of 16 consecutive output columns of one token row (normal orientation):
 // store bf16 / store fp32 / add into the fp32 residual / silu(gate) * up.
-__device__ __forceinline__ void store_chunk_normal(const GemmTcParams& p, int m, int n0, int nv, const float* v) {
+__device__ __forceinline__ void store_finished_chunk(const GemmTcParams& p, int m, int n0, int nv, const float* v);
+// ``first``: these are the sums of the first part of K (the one that brings the bias).
+__device__ __forceinline__ void store_chunk_normal(const GemmTcParams& p, int m, int n0, int nv, float* v, bool first) {
+    if ((p.bias && first) || p.act == 3) {
+        if (p.epilogue != 3) {
+#pragma unroll
+            for (int j = 0; j < 16; j++)
+                if (j < nv) v[j] = finish_sum(p, n0 + j, v[j]);
+        }
+    }
+    store_finished_chunk(p, m, n0, nv, v);
+}
+__device__ __forceinline__ void store_finished_chunk(const GemmTcParams& p, int m, int n0, int nv, const float* v) {
     if (p.epilogue == 0) {
         __nv_bfloat16* dst = (__nv_bfloat16*)p.out + (size_t)m * p.ldc + n0;
         if (nv == 16 && (((uintptr_t)dst) & 15) == 0) {
@@ -641,9 +661,9 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_consta
                         const float other = __shfl_xor_sync(0xffffffffu, x, 1);             // gate rows are even, up rows odd
                         if ((lane & 1) == 0) reinterpret_cast<__nv_bfloat16*>(row)[r >> 1] = __float2bfloat16_rn(gate_mul(x, other, p.act));
                     } else if (p.epilogue == 0) {
-                        reinterpret_cast<__nv_bfloat16*>(row)[r] = __float2bfloat16_rn(x);
+                        reinterpret_cast<__nv_bfloat16*>(row)[r] = __float2bfloat16_rn(finish_sum(p, row_tile * TILE_ROWS + r, x));
                     } else {
-                        reinterpret_cast<float*>(row)[r] = x;
+                        reinterpret_cast<float*>(row)[r] = finish_sum(p, row_tile * TILE_ROWS + r, x);
                     }
                 };
                 // (64 columns a round trip to tensor memory, as the prefill epilogues read, gained nothing here)
@@ -676,7 +696,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_consta
                         float* dst = p.accum + (size_t)m * p.accum_ld + n0;
                         for (int j = 0; j < nv; j++) atomicAdd(dst + j, v[j]);
                     } else {
-                        store_chunk_normal(p, m, n0, nv, v);
+                        store_chunk_normal(p, m, n0, nv, v, true);
                     }
                 } else {
                     const int n = row_tile * TILE_ROWS + r;
@@ -698,14 +718,17 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_consta
                         const int m = m0 + j;
                         if (m >= p.M) break;
                         if (splitk) {
+                            // (sums added straight into the residual bring the bias with the first part of K; sums in
+                            // scratch get it from the finalize kernel)
+                            if (p.epilogue == 2 && split == 0 && p.bias) v[j] += __ldg(p.bias + n);
                             atomicAdd(p.accum + (size_t)m * p.accum_ld + n, v[j]);
                         } else if (p.epilogue == 0) {
-                            ((__nv_bfloat16*)p.out)[(size_t)m * p.ldc + n] = __float2bfloat16_rn(v[j]);
+                            ((__nv_bfloat16*)p.out)[(size_t)m * p.ldc + n] = __float2bfloat16_rn(finish_sum(p, n, v[j]));
                         } else if (p.epilogue == 1) {
-                            ((float*)p.out)[(size_t)m * p.ldc + n] = v[j];
+                            ((float*)p.out)[(size_t)m * p.ldc + n] = finish_sum(p, n, v[j]);
                         } else {
                             float* dst = (float*)p.out + (size_t)m * p.ldc + n;
-                            *dst = *dst + v[j];
+                            *dst = *dst + finish_sum(p, n, v[j]);
                         }
                     }
                 }
@@ -746,6 +769,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_consta
                 if (n >= p.N || m >= p.M) continue;
                 float v = 0.0f;
                 for (int s = 0; s < S; s++) v += recv[((size_t)s * RP + rl) * C + c];
+                v = finish_sum(p, n, v);
                 if (p.epilogue == 0) ((__nv_bfloat16*)p.out)[(size_t)m * p.ldc + n] = __float2bfloat16_rn(v);
                 else if (p.epilogue == 1) ((float*)p.out)[(size_t)m * p.ldc + n] = v;
                 else {
@@ -875,6 +899,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_rows, const __
         int li = 0;
         for (int u = blockIdx.x; u < units; u += gridDim.x, li++) {
             const int t = u / k_splits;
+            const bool u_first = u == t * k_splits;
             const int col_tile = t / p.row_tiles, row_tile = t - col_tile * p.row_tiles;
             const int acc = li & 1;
             const int m = row_tile * TILE_ROWS + r;
@@ -898,7 +923,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_rows, const __
                     for (int q = 0; q < 4; q++) {
                         const int n0 = col_tile * p.block_cols + c0 + q * 16;
                         if (!ok || m >= p.M || n0 >= p.N) continue;
-                        store_chunk_normal(p, m, n0, min(16, p.N - n0), reinterpret_cast<const float*>(u + q * 16));
+                        store_chunk_normal(p, m, n0, min(16, p.N - n0), reinterpret_cast<float*>(u + q * 16), u_first);
                     }
                 }
                 for (; c0 < p.block_cols; c0 += 16) {
@@ -906,7 +931,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_rows, const __
                     tmem_ld16(taddr_row + (uint32_t)c0, v);
                     const int n0 = col_tile * p.block_cols + c0;
                     if (!ok || m >= p.M || n0 >= p.N) continue;
-                    store_chunk_normal(p, m, n0, min(16, p.N - n0), v);
+                    store_chunk_normal(p, m, n0, min(16, p.N - n0), v, u_first);
                 }
             }
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -925,7 +950,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_rows, const __
 
 // Split-K finalize for the store epilogues: out = epilogue(accum), accum = 0.
 __global__ void gemm_tc_finalize_kernel(float* __restrict__ accum, int accum_ld, void* __restrict__ out, int ldc, int M,
-                                        int N, int epilogue, int act = 0) {
+                                        int N, int epilogue, int act = 0, const float* __restrict__ bias = nullptr) {
     pdl_launch_dependents();
     pdl_wait();
     const int n_out = epilogue == 3 ? N / 2 : N;
@@ -939,8 +964,9 @@ __global__ void gemm_tc_finalize_kernel(float* __restrict__ accum, int accum_ld,
         a[2 * j + 1] = 0.0f;
         ((__nv_bfloat16*)out)[(size_t)m * ldc + j] = __float2bfloat16_rn(gate_mul(g, u, act));
     } else {
-        const float c = a[j];
+        float c = a[j] + (bias ? bias[j] : 0.0f);
         a[j] = 0.0f;
+        if (act == 3) c = gelu_erf(c);
         if (epilogue == 0) ((__nv_bfloat16*)out)[(size_t)m * ldc + j] = __float2bfloat16_rn(c);
         else ((float*)out)[(size_t)m * ldc + j] = c;
     }
@@ -950,7 +976,7 @@ __global__ void gemm_tc_finalize_kernel(float* __restrict__ accum, int accum_ld,
 // of four and the rows 16-byte aligned.  At 64 tokens the one-element kernel took 11 us a call, a tenth of the step.
 template <int EPI>
 __global__ void gemm_tc_finalize4_kernel(float* __restrict__ accum, int accum_ld, void* __restrict__ out, int ldc, int M, int n_out,
-                                         int act = 0) {
+                                         int act = 0, const float* __restrict__ bias = nullptr) {
     pdl_launch_dependents();
     pdl_wait();
     const int groups = n_out >> 2;
@@ -970,6 +996,8 @@ __global__ void gemm_tc_finalize4_kernel(float* __restrict__ accum, int accum_ld
         const float4 x = a[0];
         a[0] = zero;
         r0 = x.x; r1 = x.y; r2 = x.z; r3 = x.w;
+        if (bias) { r0 += bias[j]; r1 += bias[j + 1]; r2 += bias[j + 2]; r3 += bias[j + 3]; }
+        if (act == 3) { r0 = gelu_erf(r0); r1 = gelu_erf(r1); r2 = gelu_erf(r2); r3 = gelu_erf(r3); }
     }
     if (EPI == 1) {
         *reinterpret_cast<float4*>((float*)out + (size_t)m * ldc + j) = make_float4(r0, r1, r2, r3);

@@ -170,6 +170,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_c
         int li = 0;
         for (int u = pair; u < units; u += n_pairs, li++) {
             const int t = u / k_splits;
+            const bool u_first = u == t * k_splits;
             const int col_tile = t / p.row_tiles, row_tile = t - col_tile * p.row_tiles;
             const int acc = li & 1;
             const int m = row_tile * 2 * TILE_ROWS + (int)rank * TILE_ROWS + r;
@@ -193,7 +194,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_c
                     for (int q = 0; q < 4; q++) {
                         const int n0 = col_tile * p.block_cols + c0 + q * 16;
                         if (!ok || m >= p.M || n0 >= p.N) continue;
-                        store_chunk_normal(p, m, n0, min(16, p.N - n0), reinterpret_cast<const float*>(u + q * 16));
+                        store_chunk_normal(p, m, n0, min(16, p.N - n0), reinterpret_cast<float*>(u + q * 16), u_first);
                     }
                 }
                 for (; c0 < p.block_cols; c0 += 16) {
@@ -201,7 +202,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_c
                     tmem_ld16(taddr_row + (uint32_t)c0, v);
                     const int n0 = col_tile * p.block_cols + c0;
                     if (!ok || m >= p.M || n0 >= p.N) continue;
-                    store_chunk_normal(p, m, n0, min(16, p.N - n0), v);
+                    store_chunk_normal(p, m, n0, min(16, p.N - n0), v, u_first);
                 }
             }
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");

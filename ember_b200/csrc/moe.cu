@@ -32,10 +32,11 @@ constexpr int MOE_BM = 32, MOE_BN = 64, MOE_BK = 16;
 // alone.  sigmoid 1: scores s = sigmoid(logit); the choice is by s + correction[e] (correction may be null), the
 // weights are the chosen experts' s times scale, divided by their sum first if renormalize.
 // sigmoid 2: scores s = softmax(logits) over all experts, otherwise as sigmoid 1.  groups > 0 (at most 32): the experts
-// form `groups` equal groups of neighbours, a group's score is its largest s + correction, and only experts of the
-// `keep` best groups (ties: the lower index) can be chosen.
+// form `groups` equal groups of neighbours, a group's score is its largest s + correction (group_top2: the sum of its two
+// largest, of its only one in groups of one), and only experts of the `keep` best groups (ties: the lower index) can be
+// chosen.  renorm_eps is added to the sum that renormalize divides by.
 struct RouteRule {
-    int sigmoid; const float* correction; float scale; int renormalize; int groups; int keep;
+    int sigmoid; const float* correction; float scale; int renormalize; int groups; int keep; int group_top2; float renorm_eps;
 };
 
 // One warp a token.  A lane holds experts lane, lane + 32, ... in z.
@@ -136,13 +137,23 @@ __device__ __forceinline__ void choose_experts(float (&z)[MOE_MAX_EXPERTS / 32],
             }
             float gbest = -INFINITY;
             for (int g = 0; g < rule.groups; g++) {
-                float b = -INFINITY;
+                float b = -INFINITY, second = -INFINITY;    // the lane's largest and its next
 #pragma unroll
                 for (int i = 0; i < MOE_MAX_EXPERTS / 32; i++) {
                     if (i >= ns) break;
-                    if (grp[i] == g) b = fmaxf(b, z[i]);
+                    if (grp[i] == g) { second = fmaxf(second, fminf(b, z[i])); b = fmaxf(b, z[i]); }
                 }
-                b = warp_max(b);
+                if (rule.group_top2 && per > 1) {           // the two largest of two pairs, lane by lane
+#pragma unroll
+                    for (int o = 16; o > 0; o >>= 1) {
+                        const float ob = __shfl_xor_sync(0xffffffffu, b, o), os = __shfl_xor_sync(0xffffffffu, second, o);
+                        second = fmaxf(fminf(b, ob), fmaxf(second, os));
+                        b = fmaxf(b, ob);
+                    }
+                    b += second;
+                } else {
+                    b = warp_max(b);
+                }
                 if (lane == g) gbest = b;
             }
             unsigned kept = 0u;
@@ -206,7 +217,7 @@ __device__ __forceinline__ void choose_experts(float (&z)[MOE_MAX_EXPERTS / 32],
         }
     }
     if (lane < top) {
-        if (rule.sigmoid) wgt[(size_t)t * top + lane] = (rule.renormalize ? mine / sum : mine) * rule.scale;
+        if (rule.sigmoid) wgt[(size_t)t * top + lane] = (rule.renormalize ? mine / (sum + rule.renorm_eps) : mine) * rule.scale;
         else wgt[(size_t)t * top + lane] = mine / sum;
     }
 }
@@ -596,20 +607,20 @@ using namespace ember;
 EMBER_API int ember_moe_tile_rows() { return MOE_BM; }
 
 EMBER_API int ember_moe_route(const float* logits, int T, int E, int top, int* sel, float* wgt, int sigmoid, const float* correction,
-                              float scale, int renormalize, int groups, int keep, void* stream) {
+                              float scale, int renormalize, int groups, int keep, int group_top2, float renorm_eps, void* stream) {
     if (T <= 0) return 0;
     if (E <= 0 || E > MOE_MAX_EXPERTS || top <= 0 || top > E || top > 32)
         return fail("moe_route: top %d of %d experts (at most 32 of %d)", top, E, MOE_MAX_EXPERTS);
     launch_kernel(moe_route_kernel, (unsigned)((T + 7) / 8), 256, 0, (cudaStream_t)stream, logits, E, top, sel, wgt, T,
-                  RouteRule{sigmoid, correction, scale, renormalize, groups, keep});
+                  RouteRule{sigmoid, correction, scale, renormalize, groups, keep, group_top2, renorm_eps});
     return check_launch("moe_route");
 }
 
 EMBER_API int ember_moe_router(const void* x, int x_dtype, const float* w, int T, int K, int E, int top, int* sel, float* wgt,
                                float* logits, int sigmoid, const float* correction, float scale, int renormalize, int groups, int keep,
-                               void* stream) {
+                               int group_top2, float renorm_eps, void* stream) {
     if (T <= 0) return 0;
-    const RouteRule rule{sigmoid, correction, scale, renormalize, groups, keep};
+    const RouteRule rule{sigmoid, correction, scale, renormalize, groups, keep, group_top2, renorm_eps};
     if (groups < 0 || groups > 32 || (groups > 0 && (!sigmoid || E % groups || keep < 1 || keep > groups || top > keep * (E / groups))))
         return fail("moe_router: %d groups of which %d are kept, for top %d of %d experts", groups, keep, top, E);
     if (E <= 0 || E > MOE_MAX_EXPERTS || top <= 0 || top > E || top > 32 || K <= 0)

@@ -90,13 +90,13 @@ __global__ void __launch_bounds__(256) whole_norm_store_kernel(WholeNormArgs p) 
 // The general form of whole_norm_store.  norm_mode 0: none; 1: one RMS norm over the whole query projection and one
 // over the whole key projection (weights of that size); 2: an RMS norm per head (weights of D, shared by the heads).
 // Then the first `rotary` elements of every query and key head turn (element i with i + rotary / 2) by the angle
-// position * inv_freq[i], and the query is multiplied by 1 + qt_coef * ln(floor((position + 1) / qt_every) + 1)
+// position * inv_freq[i], cosines and sines times `magnitude`, and the query is multiplied by 1 + qt_coef * ln(floor((position + 1) / qt_every) + 1)
 // (qt_every 0: not).  Queries out, keys and values into the token's page.
 struct HeadPrepareArgs {
     const float* qkv; int ld;          // [T, q | k | v] fp32
     const float* bias;                 // [q | k | v] or null
     int norm_mode; const float* q_w; const float* k_w; float eps;
-    const float* inv_freq; int rotary;
+    const float* inv_freq; int rotary; float magnitude;
     float qt_coef; int qt_every;
     int H, G, D, DV;
     const int* positions; const int* seq_of; const int* block_table;
@@ -159,6 +159,8 @@ __global__ void __launch_bounds__(256) head_prepare_store_kernel(HeadPrepareArgs
             const float other = normed(i + half);
             float sn, cs;
             sincosf((float)pos * p.inv_freq[d], &sn, &cs);
+            cs *= p.magnitude;
+            sn *= p.magnitude;
             write(i, (v * cs - other * sn) * mul);
             write(i + half, (other * cs + v * sn) * mul);
         } else {
@@ -200,6 +202,17 @@ __global__ void head_gate_apply_kernel(T* __restrict__ x, const float* __restric
     if (i >= n) return;
     const size_t th = i / DV;
     x[i] = from_float<T>(to_float(x[i]) * sigmoidf_(gate[(th / H) * (size_t)ld_gate + th % H]));
+}
+
+// x[t, i] *= sigmoid(gate[t, i]) for an attention result x [T, n]: a gate per element as a pass of its own, for the
+// attention kernels that do not take it.
+template <typename T>
+__global__ void element_gate_apply_kernel(T* __restrict__ x, const float* __restrict__ gate, int ld_gate, int n) {
+    pdl_launch_dependents();
+    pdl_wait();
+    T* row = x + (size_t)blockIdx.x * n;
+    const float* g = gate + (size_t)blockIdx.x * ld_gate;
+    for (int i = threadIdx.x; i < n; i += blockDim.x) row[i] = from_float<T>(to_float(row[i]) * sigmoidf_(g[i]));
 }
 
 // ------------------------------------------------------------------------------------- latents of a token
@@ -1046,7 +1059,7 @@ EMBER_API int ember_whole_norm_store(const float* qkv, int ld, const float* bias
 }
 
 EMBER_API int ember_head_prepare_store(const float* qkv, int ld, const float* bias, int norm_mode, const float* q_w, const float* k_w,
-                                       float eps, const float* inv_freq, int rotary, float qt_coef, int qt_every, int T_tokens, int H,
+                                       float eps, const float* inv_freq, int rotary, float magnitude, float qt_coef, int qt_every, int T_tokens, int H,
                                        int G, int D, int DV, const int* positions, const int* seq_of, const int* block_table,
                                        int max_blocks, int page, int num_pages, void* q_out, void* k_pool, void* v_pool, int dtype,
                                        int write_kv, int* err, void* stream) {
@@ -1055,7 +1068,7 @@ EMBER_API int ember_head_prepare_store(const float* qkv, int ld, const float* bi
     if (norm_mode < 0 || norm_mode > 2 || (norm_mode && (!q_w || !k_w))) return fail("head_prepare_store: norm mode %d", norm_mode);
     if (rotary < 0 || rotary > D || (rotary & 1) || (rotary && !inv_freq)) return fail("head_prepare_store: %d rotated elements of %d", rotary, D);
     if (qt_every < 0 || page <= 0 || max_blocks <= 0 || num_pages <= 0) return fail("head_prepare_store: bad geometry");
-    HeadPrepareArgs p{qkv, ld, bias, norm_mode, q_w, k_w, eps, inv_freq, rotary, qt_coef, qt_every, H, G, D, DV, positions, seq_of,
+    HeadPrepareArgs p{qkv, ld, bias, norm_mode, q_w, k_w, eps, inv_freq, rotary, magnitude, qt_coef, qt_every, H, G, D, DV, positions, seq_of,
                       block_table, max_blocks, page, num_pages, q_out, k_pool, v_pool, write_kv, err};
     const size_t smem = (size_t)(H + G) * sizeof(float);
     if (smem > 40 * 1024) return fail("head_prepare_store: %d heads are too many", H + G);
@@ -1076,6 +1089,16 @@ EMBER_API int ember_head_gate_apply(void* x, int dtype, const float* gate, int l
         launch_kernel(head_gate_apply_kernel<__nv_bfloat16>, (unsigned)((n + 255) / 256), 256, 0, st, (__nv_bfloat16*)x, gate, ld_gate, H, DV, n);
     else return fail("head_gate_apply: unsupported dtype %d", dtype);
     return check_launch("head_gate_apply");
+}
+
+EMBER_API int ember_element_gate_apply(void* x, int dtype, const float* gate, int ld_gate, int T_tokens, int n, void* stream) {
+    if (T_tokens <= 0) return 0;
+    if (n <= 0 || ld_gate < n) return fail("element_gate_apply: rows of %d, gate rows of %d", n, ld_gate);
+    cudaStream_t st = (cudaStream_t)stream;
+    if (dtype == EMBER_F32) launch_kernel(element_gate_apply_kernel<float>, T_tokens, 256, 0, st, (float*)x, gate, ld_gate, n);
+    else if (dtype == EMBER_BF16) launch_kernel(element_gate_apply_kernel<__nv_bfloat16>, T_tokens, 256, 0, st, (__nv_bfloat16*)x, gate, ld_gate, n);
+    else return fail("element_gate_apply: unsupported dtype %d", dtype);
+    return check_launch("element_gate_apply");
 }
 
 EMBER_API int ember_latent_prepare(const float* a, int ld, int q_col, int q_rank, int c_col, int kv_rank, int rot_dim,

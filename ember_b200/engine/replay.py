@@ -63,7 +63,7 @@ class TraceReplayer:
                                       f"({len(r.cache.live_requests())} requests are live)")
             if not r.reserve(rid, len(toks)):
                 raise ReplayError(
-                    f"step {step}: the cache pool ({r.cache.capacity_tokens()} tokens) has no pages for "
+                    f"step {step}: the cache pool ({r.cache.pool_tokens()} tokens) has no pages for "
                     f"{len(toks)} more tokens of {rid!r}; live requests hold {r.cache.used_pages()} pages")
             todo.append((rid, toks, want))
         out = None

@@ -27,6 +27,9 @@ class CausalLM:
         self.embedding_position = build_part("position", spec.embedding_position, spec.embedding_position_prefix)
         self.embedding_norm = (build_part("norm", spec.embedding_norm, spec.embedding_norm_prefix)
                                if spec.embedding_norm is not None else None)
+        self.embedding_term = (build_part("embedding_term", spec.embedding_term, spec.embedding_term_prefix)
+                               if spec.embedding_term is not None else None)
+        self.reentry = build_part("reentry", spec.reentry, spec.reentry_prefix) if spec.reentry is not None else None
         self.rt: Optional[Runtime] = None
         self._cache_subs = [tuple(b.cache_needs()) for b in self.blocks]      # sub-ids of each block's caches
 
@@ -38,8 +41,9 @@ class CausalLM:
             d.append(WeightDecl(s.head_name, (s.vocab_size, s.hidden_size), optional=s.head_optional))
         d += self.final_norm.weight_decls()
         d += self.embedding_position.weight_decls()
-        if self.embedding_norm is not None:
-            d += self.embedding_norm.weight_decls()
+        for part in (self.embedding_norm, self.embedding_term, self.reentry):
+            if part is not None:
+                d += part.weight_decls()
         for b in self.blocks:
             d += b.weight_decls()
         return d
@@ -65,8 +69,9 @@ class CausalLM:
             # logits scales them in the capping kernel instead, on the fp32 logits)
             self.final_norm.scale_output(float(s.logit_scale))
         self.embedding_position.load(store, rt)
-        if self.embedding_norm is not None:
-            self.embedding_norm.load(store, rt)
+        for part in (self.embedding_norm, self.embedding_term, self.reentry):
+            if part is not None:
+                part.load(store, rt)
         for b in self.blocks:
             b.load(store, rt)
         store.finish()
@@ -77,7 +82,7 @@ class CausalLM:
         """Whether decode steps may be captured into CUDA graphs: every part of every block must allow it."""
         return (all(getattr(b, "graph_safe", False) for b in self.blocks) and self.final_norm.graph_safe
                 and self.embedding_position.graph_safe
-                and (self.embedding_norm is None or self.embedding_norm.graph_safe))
+                and all(p is None or p.graph_safe for p in (self.embedding_norm, self.embedding_term, self.reentry)))
 
     # -------------------------------------------------------------------- cache
     @staticmethod
@@ -91,10 +96,13 @@ class CausalLM:
 
     def cache_needs(self) -> Dict[object, Optional[CacheNeed]]:
         """Need of every mixer of every layer that owns a cache (a layer that only reads another's owns none),
-        as the blocks report them."""
+        as the blocks report them; what the embedding's term keeps per request is known as a layer of number -1."""
         owners = {((e.cache_of if e.cache_of >= 0 else e.layer), e.instance) for e in self.spec.schedule}
-        return {self.cache_id(l, sub, inst): need for l, inst in sorted(owners)
-                for sub, need in self.blocks[l].cache_needs().items()}
+        needs = {self.cache_id(l, sub, inst): need for l, inst in sorted(owners)
+                 for sub, need in self.blocks[l].cache_needs().items()}
+        if self.embedding_term is not None:
+            needs.update({self.cache_id(-1, sub): need for sub, need in self.embedding_term.cache_needs().items()})
+        return needs
 
     def tile_requests(self):
         """Attention tile shapes the blocks' mixers will ask the step context for (sent with the step's upload)."""
@@ -114,8 +122,12 @@ class CausalLM:
         h = ctx.buf("model.residual", (ctx.max_tokens, copies * width), torch.float32)
         staged = copies > 1 or self.embedding_norm is not None
         e = ctx.buf("model.embedded", (ctx.max_tokens, width), torch.float32) if staged else h
-        ops.embed(ctx.tokens, self.embedding, e, err=ctx.err, stream=ctx.stream, prev_ids=ctx.prev_ids,
-                  scale=s.embedding_multiplier)
+        if self.embedding_term is not None:
+            self.embedding_term.embed(ctx, self.embedding, s.embedding_multiplier, e,
+                                      {sub: storage.layer(self.cache_id(-1, sub)) for sub in self.embedding_term.cache_needs()})
+        else:
+            ops.embed(ctx.tokens, self.embedding, e, err=ctx.err, stream=ctx.stream, prev_ids=ctx.prev_ids,
+                      scale=s.embedding_multiplier)
         self.embedding_position.on_embedding(ctx, e)          # nothing for rotary or absent encodings
         if self.embedding_norm is not None:
             n = h if copies == 1 else ctx.buf("model.embedded_normed", (ctx.max_tokens, width), torch.float32)
@@ -131,7 +143,11 @@ class CausalLM:
         if capture is not None:
             row = capture[0] if capture[0] >= 0 else ctx.T + capture[0]
             record(0)
+        if self.reentry is not None and not s.schedule[0].reentry:
+            self.reentry.keep(ctx, h)
         for i, e in enumerate(s.schedule):
+            if e.reentry:
+                self.reentry.forward(ctx, h, first=i == 0)
             owner = e.cache_of if e.cache_of >= 0 else e.layer
             block = self.blocks[e.layer]
             caches = {sub: storage.layer(self.cache_id(owner, sub, e.instance)) for sub in self._cache_subs[e.layer]}

@@ -19,6 +19,8 @@ EPI_STORE, EPI_STORE_F32, EPI_ADD_F32, EPI_SILU_MUL = 0, 1, 2, 3
 EPI_SUMS = 5      # tensor-core product of at most 128 tokens: the fp32 sums stay in the split-K scratch
 EPI_RELU_MUL = 6  # the gated epilogue with relu: relu(c[2j]) * c[2j + 1]
 EPI_GELU_MUL = 7  # ... with the tanh form of gelu: 0.5 g (1 + tanh(sqrt(2 / pi) (g + 0.044715 g^3))) * c[2j + 1]
+EPI_GELU = 8      # gelu(c + bias) in its exact form, 0.5 z (1 + erf(z / sqrt 2)), stored like EPI_STORE
+PLAIN_EPILOGUES = (EPI_STORE, EPI_STORE_F32, EPI_ADD_F32, EPI_GELU)      # those that take a bias in both products
 GATED_EPILOGUES = (EPI_SILU_MUL, EPI_RELU_MUL, EPI_GELU_MUL)
 GATED_EPILOGUE_OF = {"silu": EPI_SILU_MUL, "relu": EPI_RELU_MUL, "gelu_tanh": EPI_GELU_MUL}
 
@@ -105,6 +107,46 @@ def embed(tokens: torch.Tensor, table: torch.Tensor, out: torch.Tensor, err: Opt
     _call(lib, lib.ember_embed, _p(tokens), _p(prev_ids), c_int(prev_ids.numel() if prev_ids is not None else 0),
           _p(table), c_int(dtype_code(table.dtype)), _p(out), c_int(T), c_int(H), c_int(V), c_float(scale), _p(err),
           c_void_p(stream if stream is not None else current_stream_ptr()))
+
+
+def embed_bigram(tokens: torch.Tensor, table: torch.Tensor, bigram: torch.Tensor, out: torch.Tensor, buckets: int, mul_prev: int,
+                 mul_cur: int, positions: torch.Tensor, seq_of: torch.Tensor, query_start: torch.Tensor, slots: torch.Tensor,
+                 state: torch.Tensor, scale: float = 1.0, err: Optional[torch.Tensor] = None, stream: Optional[int] = None,
+                 prev_ids: Optional[torch.Tensor] = None) -> None:
+    """out[t] = scale * table[token] + bigram[(mul_prev * previous + mul_cur * token) mod buckets]; at position 0 the row
+    is number ``buckets``, the table's last.  A run's first token finds its previous one in ``state`` (int32 [slots, n], the
+    first element of its request's slot), and the run's last token is left there.  ``prev_ids`` as in ``embed``."""
+    for t, n in ((tokens, "tokens"), (positions, "positions"), (seq_of, "seq_of"), (query_start, "query_start"), (slots, "slots"),
+                 (state, "state")):
+        _check(t, n, torch.int32)
+    if prev_ids is not None:
+        _check(prev_ids, "prev_ids", torch.int32)
+    _check(table, "table")
+    _check(bigram, "bigram")
+    _check(out, "out", torch.float32)
+    T, (V, H) = tokens.numel(), table.shape
+    if tuple(bigram.shape) != (buckets + 1, H):
+        raise KernelError(f"embed_bigram: a table of {tuple(bigram.shape)} for {buckets} buckets of width {H}")
+    if out.shape[-1] != H or out.numel() < T * H or positions.numel() < T or seq_of.numel() < T or state.dim() != 2 or \
+            query_start.numel() != slots.numel() + 1:
+        raise KernelError(f"embed_bigram: the buffers do not fit {T} rows of width {H} in {slots.numel()} runs")
+    lib = _lib("elementwise")
+    _call(lib, lib.ember_embed_bigram, _p(tokens), _p(prev_ids), c_int(prev_ids.numel() if prev_ids is not None else 0),
+          _p(table), _p(bigram), c_int(dtype_code(table.dtype)), c_int(dtype_code(bigram.dtype)), _p(out), c_int(T), c_int(H), c_int(V), c_float(scale),
+          c_longlong(buckets), c_longlong(mul_prev), c_longlong(mul_cur), _p(positions), _p(seq_of), _p(query_start), _p(slots),
+          _p(state), c_int(state.stride(0)), _p(err), c_void_p(stream if stream is not None else current_stream_ptr()))
+
+
+def place_columns(x: torch.Tensor, out: torch.Tensor, T: int, col: int, col2: int = -1, stream: Optional[int] = None) -> None:
+    """out[t, col : col + H] = x[t] (and out[t, col2 : col2 + H] with ``col2`` >= 0), x fp32 [T, H], in ``out``'s type."""
+    _check(x, "x", torch.float32)
+    _check(out, "out")
+    H, ld = x.shape[-1], out.shape[-1]
+    if x.numel() < T * H or out.numel() < T * ld:
+        raise KernelError("place_columns: buffers do not fit the step")
+    lib = _lib("elementwise")
+    _call(lib, lib.ember_place_columns, _p(x), _p(out), c_int(dtype_code(out.dtype)), c_int(T), c_int(H), c_int(ld), c_int(col),
+          c_int(col2), c_void_p(stream if stream is not None else current_stream_ptr()))
 
 
 def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor, n_rows: int,
@@ -222,7 +264,7 @@ def gemm_simt(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, M: int, epilo
     if a.shape[-1] != K:
         raise KernelError(f"gemm: activations of width {a.shape[-1]} against weights {tuple(w.shape)}")
     n_out = N // 2 if epilogue in GATED_EPILOGUES else N
-    want = a.dtype if epilogue in (EPI_STORE,) + GATED_EPILOGUES else torch.float32
+    want = a.dtype if epilogue in (EPI_STORE, EPI_GELU) + GATED_EPILOGUES else torch.float32
     if out.dtype != want:
         raise KernelError(f"gemm: epilogue {epilogue} writes {want}, the output is {out.dtype}")
     if out.shape[-1] != n_out or out.numel() < M * n_out or a.numel() < M * K:
@@ -355,17 +397,19 @@ def _scratch(device, floats: int) -> torch.Tensor:
 
 
 def gemm_tc_usable(x: torch.Tensor, w: torch.Tensor, bias, epilogue: int) -> bool:
-    """Whether the tcgen05 product takes these operands: bf16 activations and weights, no bias,
-    K a multiple of 8 (TMA row pitch), an even N for the gated epilogue."""
-    if not TC_ENABLED or bias is not None or x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16:
+    """Whether the tcgen05 product takes these operands: bf16 activations and weights, K a multiple of 8 (TMA row
+    pitch), an even N and no bias for the gated epilogue."""
+    if not TC_ENABLED or (bias is not None and epilogue not in PLAIN_EPILOGUES) or x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16:
         return False
     n, k = w.shape
     return k % 8 == 0 and not (epilogue in GATED_EPILOGUES and n % 2)
 
 
 def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, M: int, epilogue: int = EPI_STORE,
-            err: Optional[torch.Tensor] = None, stream: Optional[int] = None, split_mode: int = 0) -> None:
-    """out (+)= a[:M] @ w.T on the tcgen05 tensor cores (bf16 in, fp32 accumulate).  With ``EPI_SUMS`` (``out`` None,
+            err: Optional[torch.Tensor] = None, stream: Optional[int] = None, split_mode: int = 0,
+            bias: Optional[torch.Tensor] = None) -> None:
+    """out (+)= a[:M] @ w.T (+ ``bias``, fp32 [N], in the plain epilogues) on the tcgen05 tensor cores (bf16 in, fp32
+    accumulate).  With ``EPI_SUMS`` (``out`` None,
     at most 128 tokens) the fp32 sums are left in the split-K scratch and returned as a view [M, N]: whoever reads
     them sets them back to zero (``qk_norm_rope_store_sums``).
     ``split_mode``: how split-K partial sums are combined (0 automatic, 1 atomics, 2 cluster); 3 runs
@@ -381,20 +425,24 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, M: int, epilogu
             raise KernelError(f"gemm: the sums of M={M} tokens stay in the scratch only for 1..128 tokens and without an output")
         scratch = _scratch(a.device, M * N)
         lib = _lib("gemm_tc")
-        _call(lib, lib.ember_gemm_tc, _p(a), _p(w), c_void_p(0), c_int(N), c_int(M), c_int(N), c_int(K), c_int(epilogue),
+        _call(lib, lib.ember_gemm_tc, _p(a), _p(w), c_void_p(0), c_int(N), c_int(M), c_int(N), c_int(K), c_int(epilogue), c_void_p(0),
               _p(scratch), c_longlong(scratch.numel()), c_int(_sms(a.device)), c_int(split_mode), _p(err),
               c_void_p(stream if stream is not None else current_stream_ptr()))
         return scratch[:M * N].view(M, N)
     _check(out, "out")
     n_out = N // 2 if epilogue in GATED_EPILOGUES else N
-    want = torch.bfloat16 if epilogue in (EPI_STORE,) + GATED_EPILOGUES else torch.float32
+    want = torch.bfloat16 if epilogue in (EPI_STORE, EPI_GELU) + GATED_EPILOGUES else torch.float32
     if out.dtype != want:
         raise KernelError(f"gemm: epilogue {epilogue} writes {want}, the output is {out.dtype}")
     if out.shape[-1] != n_out or out.numel() < M * n_out or a.numel() < M * K:
         raise KernelError(f"gemm: output {tuple(out.shape)} / input {tuple(a.shape)} do not fit M={M} N={n_out}")
+    if bias is not None:
+        _check(bias, "bias", torch.float32)
+        if bias.numel() != N or epilogue not in PLAIN_EPILOGUES:
+            raise KernelError(f"gemm: a bias of {bias.numel()} for N={N} under epilogue {epilogue}")
     scratch = _scratch(a.device, min(M, 128) * N) if M <= 128 else None
     lib = _lib("gemm_tc")
-    _call(lib, lib.ember_gemm_tc, _p(a), _p(w), _p(out), c_int(n_out), c_int(M), c_int(N), c_int(K), c_int(epilogue),
+    _call(lib, lib.ember_gemm_tc, _p(a), _p(w), _p(out), c_int(n_out), c_int(M), c_int(N), c_int(K), c_int(epilogue), _p(bias),
           _p(scratch), c_longlong(scratch.numel() if scratch is not None else 0), c_int(_sms(a.device)), c_int(split_mode),
           _p(err),
           c_void_p(stream if stream is not None else current_stream_ptr()))
@@ -404,7 +452,7 @@ def gemm_tc_qkv_usable(x: torch.Tensor, w: torch.Tensor, bias, M: int, n_heads: 
                        rotary: int) -> bool:
     """Whether the fused projection takes this step: bf16, no bias, heads of 128 rotated whole (or not at all),
     more than 128 tokens or at most 16 (the rule of ember_gemm_tc_qkv_supported)."""
-    if not gemm_tc_usable(x, w, bias, EPI_STORE):
+    if bias is not None or not gemm_tc_usable(x, w, bias, EPI_STORE):
         return False
     n, k = w.shape
     return (0 < M <= 16 or M > 128) and head_dim == 128 and rotary in (0, 128) and n == (n_heads + 2 * n_kv) * 128
@@ -508,13 +556,22 @@ def attention_fa_tile_queries(group: int) -> int:
     return 128 // group
 
 
+def _check_element_gate(gate, col: int, n: int) -> None:
+    if gate is not None:
+        _check(gate, "gate", torch.float32)
+        if gate.dim() != 2 or col < 0 or gate.shape[1] < col + n:
+            raise KernelError(f"attention: a gate of {tuple(gate.shape)} from column {col} for {n} elements a token")
+
+
 def attention_fa(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, out: torch.Tensor, n_heads: int,
                  n_kv: int, head_dim: int, tiles: torch.Tensor, n_tiles: int, block_table: torch.Tensor, page: int,
                  window: int, scale: float, err: Optional[torch.Tensor] = None, stream: Optional[int] = None,
-                 softcap: float = 0.0, chunk: int = 0) -> None:
+                 softcap: float = 0.0, chunk: int = 0, gate: Optional[torch.Tensor] = None, gate_col: int = 0) -> None:
     """bf16 causal attention of prompt portions on tcgen05 tensor cores (S and O in tensor memory).  ``softcap`` > 0: the
     scaled score becomes softcap * tanh(score / softcap); ``chunk`` > 0: position i sees j only if
-    floor(i / chunk) == floor(j / chunk)."""
+    floor(i / chunk) == floor(j / chunk); ``gate`` (fp32 [T, ..]): element i of a token's result is multiplied by
+    sigmoid(gate[t, gate_col + i])."""
+    _check_element_gate(gate, gate_col, n_heads * head_dim)
     _check(q, "q", torch.bfloat16)
     _check(out, "out", torch.bfloat16)
     _check(k_pool, "k_pool", torch.bfloat16)
@@ -527,6 +584,7 @@ def attention_fa(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, ou
     _call(lib, lib.ember_attention_fa, _p(q), _p(k_pool), _p(v_pool), _p(out), c_int(n_heads), c_int(n_kv), c_int(head_dim),
           _p(tiles), c_int(n_tiles), _p(block_table), c_int(block_table.shape[-1]), c_int(page), c_int(k_pool.shape[0]),
           c_int(window), c_float(scale), _p(err), c_float(softcap), c_int(chunk),
+          (_off(gate, gate_col) if gate is not None else c_void_p(0)), c_int(gate.shape[-1] if gate is not None else 0),
           c_void_p(stream if stream is not None else current_stream_ptr()))
 
 
@@ -534,12 +592,16 @@ def attention_tc(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, ou
                  n_heads: int, n_kv: int, head_dim: int, tiles: torch.Tensor, n_tiles: int, block_table: torch.Tensor,
                  page: int, window: int, scale: float, n_splits: int = 1, split_keys: int = 0,
                  part_o: Optional[torch.Tensor] = None, part_ml: Optional[torch.Tensor] = None,
-                 err: Optional[torch.Tensor] = None, stream: Optional[int] = None, softcap: float = 0.0, chunk: int = 0) -> None:
+                 err: Optional[torch.Tensor] = None, stream: Optional[int] = None, softcap: float = 0.0, chunk: int = 0,
+                 gate: Optional[torch.Tensor] = None, gate_col: int = 0) -> None:
     """bf16 attention over the paged cache on tensor cores (TMA-fed); ``softcap`` > 0 caps the scaled scores by a tanh,
-    ``chunk`` > 0 lets position i see j only if floor(i / chunk) == floor(j / chunk).  ``mode`` 0 takes tiles of
+    ``chunk`` > 0 lets position i see j only if floor(i / chunk) == floor(j / chunk), ``gate`` is the gate per element of
+    ``attention_fa``.  Splits are ranges of keys from key 0 on, under a chunk from the 64-key tile that holds the chunk's
+    first key.  ``mode`` 0 takes tiles of
     prompt portions, 1 takes single-token tiles and may split their key range: with ``part_o`` / ``part_ml`` the
     splits' partial results go through those buffers and a second kernel merges them; without them (at most 8
     splits) the splits of a tile are a thread-block cluster and are merged in shared memory."""
+    _check_element_gate(gate, gate_col, n_heads * head_dim)
     _check(q, "q", torch.bfloat16)
     _check(out, "out", torch.bfloat16)
     _check(k_pool, "k_pool", torch.bfloat16)
@@ -557,7 +619,8 @@ def attention_tc(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, ou
     _call(lib, lib.ember_attention_tc, _p(q), _p(k_pool), _p(v_pool), _p(out), c_int(mode), c_int(n_heads), c_int(n_kv),
           c_int(head_dim), _p(tiles), c_int(n_tiles), _p(block_table), c_int(block_table.shape[-1]), c_int(page),
           c_int(k_pool.shape[0]), c_int(window), c_float(scale), c_int(n_splits), c_int(split_keys), _p(part_o),
-          _p(part_ml), _p(err), c_float(softcap), c_int(chunk), c_void_p(stream if stream is not None else current_stream_ptr()))
+          _p(part_ml), _p(err), c_float(softcap), c_int(chunk), (_off(gate, gate_col) if gate is not None else c_void_p(0)),
+          c_int(gate.shape[-1] if gate is not None else 0), c_void_p(stream if stream is not None else current_stream_ptr()))
 
 
 # ------------------------------------------------ norms and gates around a sublayer (csrc/norm_gate.cu)
@@ -1058,16 +1121,27 @@ def head_gate_apply(x: torch.Tensor, gate: torch.Tensor, gate_col: int, T: int, 
           c_int(heads), c_int(vdim), _stream(stream))
 
 
+def element_gate_apply(x: torch.Tensor, gate: torch.Tensor, gate_col: int, T: int, n: int, stream: Optional[int] = None) -> None:
+    """x[t, i] *= sigmoid(gate[t, gate_col + i]) in place (x [T, n] bfloat16 or float32, gate fp32 logits)."""
+    _check(x, "x")
+    _check_element_gate(gate, gate_col, n)
+    if gate is None or x.numel() < T * n or gate.shape[0] < T:
+        raise KernelError("element_gate_apply: buffers do not fit the step")
+    lib = _lib("sink_attention")
+    _call(lib, lib.ember_element_gate_apply, _p(x), c_int(dtype_code(x.dtype)), _off(gate, gate_col), c_int(gate.shape[-1]), c_int(T),
+          c_int(n), _stream(stream))
+
+
 def head_prepare_store(qkv: torch.Tensor, bias: Optional[torch.Tensor], norm_mode: str, q_w: Optional[torch.Tensor],
                        k_w: Optional[torch.Tensor], eps: float, inv_freq: Optional[torch.Tensor], rotary: int, q_temp_coef: float,
                        q_temp_every: int, T: int, heads: int, kv_heads: int, dim: int, vdim: int, positions: torch.Tensor,
                        seq_of: torch.Tensor, block_table: torch.Tensor, page: int, k_pool: torch.Tensor, v_pool: torch.Tensor,
                        q_out: torch.Tensor, write_kv: bool = True, err: Optional[torch.Tensor] = None,
-                       stream: Optional[int] = None) -> None:
+                       stream: Optional[int] = None, magnitude: float = 1.0) -> None:
     """A token's q/k/v (``qkv`` fp32 [T, q | k | v], plus ``bias``) made ready for attention: an RMS norm of queries and
     keys (``norm_mode`` "none", "whole": over the whole projection with weights of that size, "head": per head with
     weights of ``dim`` shared by the heads), the rotation of the first ``rotary`` elements of every query and key head
-    (element i with i + rotary / 2, angle position * inv_freq[i]), the query times
+    (element i with i + rotary / 2, angle position * inv_freq[i], cosines and sines times ``magnitude``), the query times
     1 + q_temp_coef * ln(floor((position + 1) / q_temp_every) + 1) (``q_temp_every`` 0: not); queries to ``q_out``, keys and
     values into the token's page."""
     _check(qkv, "qkv", torch.float32)
@@ -1096,7 +1170,7 @@ def head_prepare_store(qkv: torch.Tensor, bias: Optional[torch.Tensor], norm_mod
         raise KernelError("head_prepare_store: buffers do not fit the step")
     lib = _lib("sink_attention")
     _call(lib, lib.ember_head_prepare_store, _p(qkv), c_int(qkv.shape[1]), _p(bias), c_int(modes[norm_mode]), _p(q_w), _p(k_w),
-          c_float(eps), _p(inv_freq), c_int(rotary), c_float(q_temp_coef), c_int(q_temp_every), c_int(T), c_int(heads), c_int(kv_heads),
+          c_float(eps), _p(inv_freq), c_int(rotary), c_float(magnitude), c_float(q_temp_coef), c_int(q_temp_every), c_int(T), c_int(heads), c_int(kv_heads),
           c_int(dim), c_int(vdim), _p(positions), _p(seq_of), _p(block_table), c_int(block_table.shape[-1]), c_int(page),
           c_int(k_pool.shape[0]), _p(q_out), _p(k_pool), _p(v_pool), c_int(dtype_code(q_out.dtype)), c_int(1 if write_kv else 0),
           _p(err), _stream(stream))
@@ -1272,14 +1346,18 @@ def moe_stream_usable(x: torch.Tensor, K: int) -> bool:
 
 
 def _route_rule(rule, experts: int):
-    """(sigmoid, correction pointer, scale, renormalize) of a routing rule: None is the softmax over the chosen logits;
+    """(sigmoid, correction pointer, scale, renormalize, ...) of a routing rule as the kernels take it: None is the softmax over the chosen logits;
     else (correction fp32 [experts] or None, scale, renormalize) for sigmoid scores."""
     if rule is None:
-        return c_int(0), c_void_p(0), c_float(1.0), c_int(0), c_int(0), c_int(0)
+        return c_int(0), c_void_p(0), c_float(1.0), c_int(0), c_int(0), c_int(0), c_int(0), c_float(0.0)
     correction, scale, renormalize = rule[:3]
     # longer rules: (..., scoring, groups, keep) with scoring "sigmoid" or "softmax" (over all experts) and the choice
-    # limited to the ``keep`` best of ``groups`` equal groups of neighbouring experts (groups 0: no limit)
-    scoring, groups, keep = (tuple(rule[3:]) + ("sigmoid", 0, 0)[len(rule) - 3:]) if len(rule) > 3 else ("sigmoid", 0, 0)
+    # limited to the ``keep`` best of ``groups`` equal groups of neighbouring experts (groups 0: no limit); then
+    # (..., group_score, renorm_eps) with a group scored by its largest score ("max") or the sum of its two largest ("top2")
+    defaults = ("sigmoid", 0, 0, "max", 0.0)
+    scoring, groups, keep, group_score, renorm_eps = tuple(rule[3:]) + defaults[len(rule) - 3:]
+    if group_score not in ("max", "top2"):
+        raise KernelError(f"routing: group score {group_score!r}")
     if scoring not in ("sigmoid", "softmax"):
         raise KernelError(f"routing: scoring {scoring!r}")
     if groups and (groups > 32 or experts % groups or not 1 <= keep <= groups):
@@ -1289,7 +1367,7 @@ def _route_rule(rule, experts: int):
         if correction.numel() != experts:
             raise KernelError(f"routing: a correction of {correction.numel()} for {experts} experts")
     return (c_int(1 if scoring == "sigmoid" else 2), _p(correction), c_float(scale), c_int(1 if renormalize else 0), c_int(groups),
-            c_int(keep))
+            c_int(keep), c_int(1 if group_score == "top2" else 0), c_float(renorm_eps))
 
 
 def moe_route(logits: torch.Tensor, T: int, top: int, sel: torch.Tensor, wgt: torch.Tensor, stream: Optional[int] = None,

@@ -23,7 +23,7 @@ from .registry import build_part, register_part
 
 
 def plan_decode_splits(n_tokens: int, max_context: int, window: int, num_kv_heads: int, head_dim: int, sms: int,
-                       cluster_splits: int, merge_kernel_us: float, cache_bytes_per_us: float):
+                       cluster_splits: int, merge_kernel_us: float, cache_bytes_per_us: float, chunk: int = 0):
     """How the key ranges of a decode step's single-token tiles are cut: ``(n_splits, split_keys, in_cluster)``.
 
     Splits are fixed ranges of ``split_keys`` keys (a multiple of 64) anchored at key 0 that cover ``max_context``;
@@ -31,8 +31,12 @@ def plan_decode_splits(n_tokens: int, max_context: int, window: int, num_kv_head
     of cache over the device's rate, stretched by idle SMs (blocks = tokens x key heads x splits against ``sms``)
     and by 4 % per further split.  ``in_cluster``: the splits of a tile are a thread-block cluster that merges in
     shared memory (at most ``cluster_splits``; 0 forbids it), chosen when the best such plan is estimated no slower
-    than the best plan of up to 16 splits plus what the merge kernel costs."""
+    than the best plan of up to 16 splits plus what the merge kernel costs.  ``chunk`` (instead of a window): a token sees
+    the keys of its own chunk, and its splits start at the 64-key tile that holds the chunk's first key, so none is empty
+    by design."""
     live = max_context if window <= 0 else min(max_context, window + 64)
+    if chunk > 0:
+        live = max_context = min(max_context, chunk + 63)
     blocks = max(1, n_tokens * num_kv_heads)
     stream_us = n_tokens * live * num_kv_heads * head_dim * 4 / cache_bytes_per_us         # keys and values, bf16
 
@@ -143,7 +147,7 @@ class Attention(Mixer):
                             s.qk_norm_eps, cos_sin, self.inv_freq if rotates and T <= 16 else None, ctx.positions,
                             ctx.seq_of, table, cache.page_tokens, cache.k, cache.v, q, write_kv=owns_cache, err=ctx.err,
                             stream=ctx.stream)
-        elif (self.SUMS_TO_HEADS and 16 < T <= 128 and ops.gemm_tc_usable(x, self.qkv.weight, self.qkv.bias, ops.EPI_STORE)
+        elif (self.SUMS_TO_HEADS and 16 < T <= 128 and self.qkv.bias is None and ops.gemm_tc_usable(x, self.qkv.weight, self.qkv.bias, ops.EPI_STORE)
               and ops.qk_norm_rope_store_sums_usable(s.head_dim, self.rotary if rotates else 0, self.qkv.n)):
             # 17 to 128 tokens: the product cuts K and adds its parts into a zeroed fp32 scratch; the head kernel
             # reads the sums there (and clears them) instead of a bf16 copy that a pass of its own would have to make
@@ -191,9 +195,12 @@ class Attention(Mixer):
             return [(tq, "multi"), (1, "single")] if single else [(tq, "all")]
         return [(ops.attention_tile_queries(s.group), "all")]
 
-    def attend(self, ctx, q: torch.Tensor, cache, table: torch.Tensor, out: torch.Tensor) -> None:
-        """out[t, h, :] = softmax over the visible keys of (q . k * scale) times v."""
+    def attend(self, ctx, q: torch.Tensor, cache, table: torch.Tensor, out: torch.Tensor, gate: Optional[torch.Tensor] = None,
+               gate_col: int = 0) -> None:
+        """out[t, h, :] = softmax over the visible keys of (q . k * scale) times v; with ``gate`` (fp32 logits, from column
+        ``gate_col`` on) element i of a token's result is multiplied by the sigmoid of its logit i."""
         s = self.spec
+        kw = dict(err=ctx.err, stream=ctx.stream, softcap=self.softcap, chunk=self.chunk, gate=gate, gate_col=gate_col)
         multi, single = self._tc_modes()
         if multi and ops.TC_ENABLED:
             tq = ops.attention_tc_tile_queries(s.group)
@@ -201,18 +208,18 @@ class Attention(Mixer):
             if not single:
                 tiles, n = ctx.attention_tiles(tq, "all")
                 ops.attention_tc(q, cache.k, cache.v, out, 0, *args, tiles, n, table, cache.page_tokens, s.window,
-                                 self.scale, err=ctx.err, stream=ctx.stream, softcap=self.softcap, chunk=self.chunk)
+                                 self.scale, **kw)
                 return
             if self._fa():
                 tiles, n = ctx.attention_tiles(ops.attention_fa_tile_queries(s.group), "multi")
                 if n:
                     ops.attention_fa(q, cache.k, cache.v, out, *args, tiles, n, table, cache.page_tokens, s.window,
-                                     self.scale, err=ctx.err, stream=ctx.stream, softcap=self.softcap, chunk=self.chunk)
+                                     self.scale, **kw)
             else:
                 tiles, n = ctx.attention_tiles(tq, "multi")
                 if n:
                     ops.attention_tc(q, cache.k, cache.v, out, 0, *args, tiles, n, table, cache.page_tokens, s.window,
-                                     self.scale, err=ctx.err, stream=ctx.stream, softcap=self.softcap, chunk=self.chunk)
+                                     self.scale, **kw)
             tiles, n = ctx.attention_tiles(1, "single")
             if n:
                 # Cut long key ranges only as far as it takes to keep the memory system busy: the kernel streams the
@@ -220,24 +227,24 @@ class Attention(Mixer):
                 # (partial results written and read, the merge kernel).  Measured at 16/8 heads, context 3,200, us a
                 # layer with 1 / 2 / 4 splits: 64 requests 122 / 130 / 134, 24 requests 52 / 60 / 58, 16 requests
                 # 40 / 37 / 41, 8 requests - / 22.6 / 22.5, one request 19 (2) / 12.8 (4) / 10.1 (8).  Splits are
-                # anchored at key 0, so with a window the early ones are empty.
+                # anchored at key 0 (with a window the early ones are empty) or, with chunks, at the chunk's first key.
                 # Up to 8 splits of a tile can be a thread-block cluster that merges in shared memory; more go
                 # through buffers and the merge kernel, which costs a step about MERGE_KERNEL_US a layer (batch 8,
                 # 3 splits: 1.895 -> 1.805 ms a step; one request at 3,072: 12 splits through buffers 1.351 ms, 8 in a
                 # cluster 1.305 ms; at 32,768 the 16 splits through buffers win, 28.5 against 42.9 us a layer).
                 n_splits, split_keys, in_cluster = plan_decode_splits(
-                    n, ctx.max_context, s.window or self.chunk, s.num_kv_heads, s.head_dim, ops.num_sms(q.device),
-                    ops.ATTENTION_CLUSTER_SPLITS if self.CLUSTER_MERGE else 0, self.MERGE_KERNEL_US, self.CACHE_BYTES_PER_US)
+                    n, ctx.max_context, s.window, s.num_kv_heads, s.head_dim, ops.num_sms(q.device),
+                    ops.ATTENTION_CLUSTER_SPLITS if self.CLUSTER_MERGE else 0, self.MERGE_KERNEL_US, self.CACHE_BYTES_PER_US,
+                    chunk=self.chunk)
                 part_o = part_ml = None
                 if n_splits > 1 and not in_cluster:
                     part_o = ctx.buf_dyn("attention.part_o", n * s.num_heads * n_splits * s.head_dim, torch.float32)
                     part_ml = ctx.buf_dyn("attention.part_ml", n * s.num_heads * n_splits * 2, torch.float32)
                 ops.attention_tc(q, cache.k, cache.v, out, 1, *args, tiles, n, table, cache.page_tokens, s.window,
-                                 self.scale, n_splits, split_keys, part_o, part_ml, err=ctx.err, stream=ctx.stream,
-                                 softcap=self.softcap, chunk=self.chunk)
+                                 self.scale, n_splits, split_keys, part_o, part_ml, **kw)
             return
-        if self.softcap > 0 or self.chunk > 0:
-            raise ops.KernelError("attention: the general kernel has no score cap and no chunks (the tensor-core kernels have)")
+        if self.softcap > 0 or self.chunk > 0 or gate is not None:
+            raise ops.KernelError("attention: the general kernel has no score cap, chunks or gate (the tensor-core kernels have)")
         tile_q = ops.attention_tile_queries(s.group)
         tiles, n_tiles = ctx.attention_tiles(tile_q, "all")
         # long key ranges of a small step are cut into fixed splits so that more SMs share them

@@ -15,6 +15,8 @@ Interfaces (what a new part must provide):
   ``forward(ctx, x[T, hidden], residual_f32[T, hidden], cache: LayerCache | None, owns_cache: bool)``;
   it *adds* its result to ``residual``.
 * ``FeedForward``:   ``forward(ctx, x[T, hidden], residual_f32[T, hidden])``; it adds its result.
+* ``EmbeddingTerm``: ``embed(ctx, table, scale, out_f32[T, hidden], cache)``: the embedded tokens with the term added.
+* ``Reentry``:       ``keep(ctx, h)`` and ``forward(ctx, h)``: what happens to the stream ahead of a pass of a loop.
 * ``Gate``:          ``forward(ctx, x[T, hidden], logits_f32[T, size])``.
 * ``Connection``:    ``read(ctx, streams_f32[T, copies * hidden], norm, out[T, hidden])`` and
   ``write(ctx, streams_f32, y_f32[T, hidden])``: how a sublayer reads from and writes to the copies of the residual stream.
@@ -53,7 +55,9 @@ class CacheNeed:
 
     kind "full":   pages holding every key/value of the request.
     kind "window": pages holding the last ``window`` keys; older pages are given back, except those that hold one of
-                   the first ``keep_first`` keys (a window that keeps the sequence's first tokens in sight).
+                   the first ``keep_first`` keys (a window that keeps the sequence's first tokens in sight).  With
+                   ``chunk`` instead of ``window``: pages holding the keys of the chunk of positions the next token falls
+                   into; those of chunks that have passed are given back.
     kind "state":  no pages; one slot of ``state_shape`` elements of ``state_dtype`` per request.
     Layers whose needs are equal share a group (one block table, one page pool per group).
     """
@@ -64,6 +68,7 @@ class CacheNeed:
     window: int = 0
     value_dim: int = 0            # size of a value head where it differs from a key head's (0: the same)
     keep_first: int = 0           # kind "window": the first tokens of a request whose pages are never given back
+    chunk: int = 0                # kind "window": keep the current chunk's keys instead of a window
     keys_only: bool = False       # one row per token and head (a latent that serves as key and value): no value pool
     state_shape: Tuple[int, ...] = ()
     state_dtype: str = "float32"
@@ -201,4 +206,32 @@ class FeedForward(Part):
     can_store = False
 
     def forward(self, ctx, x: torch.Tensor, residual: torch.Tensor) -> None:
+        raise NotImplementedError
+
+
+class EmbeddingTerm(Part):
+    """Something added to the embedded tokens that may depend on earlier tokens; ``cache_needs`` as a mixer's."""
+
+    family = "embedding_term"
+
+    def cache_needs(self) -> Dict[str, Optional[CacheNeed]]:
+        return {}
+
+    def embed(self, ctx, table: torch.Tensor, scale: float, out: torch.Tensor, caches) -> None:
+        """out[t] = scale * table[token t] + the term; ``caches``: sub-id -> ``LayerCache``."""
+        raise NotImplementedError
+
+
+class Reentry(Part):
+    """How the stream is mixed with the embedding's output ahead of a pass of a looped stretch of layers."""
+
+    family = "reentry"
+
+    def keep(self, ctx, h: torch.Tensor) -> None:
+        """Called with the embedding's output once a step (not if the step's first run re-enters: ``forward`` is then
+        called with ``first``)."""
+        raise NotImplementedError
+
+    def forward(self, ctx, h: torch.Tensor, first: bool = False) -> None:
+        """Replaces ``h``; ``first``: ``h`` is the embedding's output itself and ``keep`` has not been called."""
         raise NotImplementedError

@@ -303,7 +303,24 @@ class PostNormBlock(Arrangement):
             self._sublayer(ctx, h, ff, p["feed_forward_norm"], lambda x, y: ff.forward(ctx, x, y, **kw))
 
 
+class ParallelPreNormBlock(Arrangement):
+    """One norm whose output both sublayers read: x = norm(h); h += mixer(x) + feed_forward(x).  Both add into the
+    residual stream through the epilogue of their last product; a layer may have no feed-forward."""
+
+    ROLES = {"norm": "norm", "mixer": "mixer", "feed_forward": "feed_forward"}
+    OPTIONAL = frozenset({"feed_forward"})
+
+    def forward(self, ctx, h: torch.Tensor, caches, owns_cache: bool = True) -> None:
+        p = self.parts
+        x = ctx.buf("block.normed", (ctx.max_tokens, h.shape[-1]), self.rt.dtype)
+        p["norm"].forward(ctx, h, x, ctx.T)
+        p["mixer"].forward(ctx, x, h, self.cache_of(caches), owns_cache)
+        if "feed_forward" in p:
+            p["feed_forward"].forward(ctx, x, h)
+
+
 register_part("arrangement", "prenorm", PreNormBlock)
+register_part("arrangement", "parallel_prenorm", ParallelPreNormBlock)
 register_part("arrangement", "postnorm", PostNormBlock)
 register_part("arrangement", "connected_prenorm", ConnectedPreNormBlock)
 register_part("arrangement", "gated_sandwich", GatedSandwichBlock)

@@ -88,6 +88,45 @@ class GatedMLP(FeedForward):
         self.down(ctx, act, residual, ctx.T, ops.EPI_ADD_F32 if accumulate else ops.EPI_STORE_F32)
 
 
+class PlainMLP(FeedForward):
+    """Two matrices: down(gelu(up(x) + b) + b), the exact gelu; both biases and the activation are the products' epilogues."""
+
+    graph_safe = True
+    can_store = True
+
+    def __init__(self, spec, prefix: str = ""):
+        super().__init__(spec, prefix)
+        if spec.activation != "gelu":
+            raise ConfigError(f"feed-forward of two matrices: activation {spec.activation!r} is not supported (gelu)")
+        if min(spec.hidden_size, spec.intermediate_size) <= 0:
+            raise ConfigError("feed-forward: sizes must be positive")
+
+    def weight_decls(self) -> List[WeightDecl]:
+        s, p = self.spec, self.prefix
+        up, down = s.names
+        d = [WeightDecl(p + up, (s.intermediate_size, s.hidden_size)), WeightDecl(p + down, (s.hidden_size, s.intermediate_size))]
+        if s.bias:
+            d += [WeightDecl(p + up + s.bias_suffix, (s.intermediate_size,), init="zeros"),
+                  WeightDecl(p + down + s.bias_suffix, (s.hidden_size,), init="zeros")]
+        return d
+
+    def load(self, store, rt: Runtime) -> None:
+        s, p = self.spec, self.prefix
+        self.rt = rt
+        got = {d.name: store.take(d.name, d.shape) for d in self.weight_decls()}
+        if any(v is None for v in got.values()):
+            return
+        up, down = s.names
+        bias = lambda n: got[p + n + s.bias_suffix] if s.bias else None          # noqa: E731
+        self.up = Linear.from_host(got[p + up], rt, bias(up))
+        self.down = Linear.from_host(got[p + down], rt, bias(down))
+
+    def forward(self, ctx, x: torch.Tensor, residual: torch.Tensor, accumulate: bool = True) -> None:
+        act = ctx.buf("mlp.act", (ctx.max_tokens, self.spec.intermediate_size), self.rt.dtype)
+        self.up(ctx, x, act, ctx.T, ops.EPI_GELU)
+        self.down(ctx, act, residual, ctx.T, ops.EPI_ADD_F32 if accumulate else ops.EPI_STORE_F32)
+
+
 class RoutedMLP(FeedForward):
     """Mixture of experts: h += sum over the token's ``top`` experts of weight * W_down (g sigmoid(alpha g) (u + up_offset))
     with g = min(W_gate x, limit), u = clamp(W_up x, -limit, limit) (``limit`` 0: no clamps; alpha 1 and up_offset 0 then
@@ -110,7 +149,8 @@ class RoutedMLP(FeedForward):
     Tensors under the prefix: router, correction (if any), e<i>.gate, e<i>.up, e<i>.down.
 
     Scoring "softmax": s = softmax over all router outputs, otherwise as "sigmoid".  ``groups``: the outputs form equal
-    groups of neighbours, a group's score is its largest s + correction, and the choice is among the outputs of the
+    groups of neighbours, a group's score is its largest s + correction (``group_score`` "top2": the sum of its two
+    largest), and the choice is among the outputs of the
     ``keep_groups`` best groups.  ``identity``: the router has experts + identity outputs, the last ones experts without
     tensors whose output is the token's input itself (``forward(..., stream=)`` hands the fp32 input where the caller has
     it; else the product's input is used).  ``expert`` "square_relu": W_down relu(W_up h)^2, no gate matrix."""
@@ -133,6 +173,8 @@ class RoutedMLP(FeedForward):
             raise ConfigError(f"routed feed-forward: scoring {s.scoring!r} (softmax_top, sigmoid, softmax)")
         if s.scoring == "softmax_top" and (s.correction or s.renormalize or s.route_scale != 1.0 or s.groups):
             raise ConfigError("routed feed-forward: a correction, a scale, groups and renormalising belong to sigmoid or softmax scoring")
+        if s.group_score not in ("max", "top2") or s.renorm_eps < 0:
+            raise ConfigError(f"routed feed-forward: group score {s.group_score!r} (max, top2)")
         if s.identity < 0 or s.expert not in ("gated", "square_relu"):
             raise ConfigError(f"routed feed-forward: {s.identity} identity experts, expert {s.expert!r} (gated, square_relu)")
         self.outputs = s.experts + s.identity              # what the router chooses among
@@ -170,7 +212,7 @@ class RoutedMLP(FeedForward):
         self.rule = None
         if s.scoring != "softmax_top":
             self.rule = (rt.to_device(got[p + "correction"], torch.float32) if s.correction else None, float(s.route_scale),
-                         bool(s.renormalize), s.scoring, int(s.groups), int(s.keep_groups))
+                         bool(s.renormalize), s.scoring, int(s.groups), int(s.keep_groups), s.group_score, float(s.renorm_eps))
         down = torch.empty((s.experts, s.hidden_size, s.intermediate_size), dtype=wd, device=rt.device)
         if self.gated:
             gu = torch.empty((s.experts, s.intermediate_size, 2, s.hidden_size), dtype=wd, device=rt.device)
@@ -240,4 +282,5 @@ class RoutedMLP(FeedForward):
 
 
 register_part("feed_forward", "gated_mlp", GatedMLP)
+register_part("feed_forward", "mlp", PlainMLP)
 register_part("feed_forward", "routed_mlp", RoutedMLP)

@@ -8,8 +8,11 @@
   (each a parameter, off by default): an RMS norm per head with one weight for all heads; a short causal convolution on
   q, k, v straight after the projection (its last inputs are a per-request state beside the pages, sub-id "conv"); a
   rotation of queries and keys after the norm; a query temperature that grows with the logarithm of the position; a
-  tanh cap on the scaled scores; a chunked mask (i sees j only inside i's chunk of positions); a sigmoid gate per head on
-  the attention's output, computed from the mixer's input.
+  tanh cap on the scaled scores; a chunked mask (i sees j only inside i's chunk of positions, and the pages of chunks that
+  have passed go back); a sigmoid gate per head, or one per element, on the attention's output, computed from the
+  mixer's input.  A rotation in neighbouring pairs is the rotate-half form over rows of W_q and W_k put in another order
+  when they are loaded (the even elements of the rotated part, then the odd ones: the same order in queries and keys
+  leaves their products as they are), so the kernels know one layout.
 * "latent_attention": queries through a low-rank latent (c_q = RMSNorm(W_dq h), q = W_uq c_q, per head
   [head_dim unrotated | rot_dim rotated]) or, with ``q_rank`` 0, straight from the input (q = W_q h); the rotated parts
   turn in neighbouring pairs or in the rotate-half layout, with the position part's frequencies (stretched for long
@@ -27,7 +30,7 @@ norms, angles and sums are fp32 in both dtypes.
 """
 from __future__ import annotations
 
-from typing import List
+from typing import List, Optional
 
 import torch
 
@@ -94,9 +97,14 @@ class SinkAttention(_SinkSoftmax):
             raise ConfigError("sink attention: convolution taps (up to 64), chunk, temperature period and score cap must be >= 0")
         if s.chunk > 0 and s.window > 0:
             raise ConfigError("sink attention: a chunked mask and a window exclude one another")
+        if s.head_gate and s.element_gate:
+            raise ConfigError("sink attention: a gate per head and a gate per element exclude one another")
+        self.gate_cols = s.num_heads if s.head_gate else (s.num_heads * s.value_dim if s.element_gate else 0)
         self.q_dim, self.k_dim, self.v_dim = s.num_heads * s.head_dim, s.num_kv_heads * s.head_dim, s.num_kv_heads * s.value_dim
         self.channels = self.q_dim + self.k_dim + self.v_dim
         self.position = build_part("position", s.position)
+        self.magnitude = float(self.position.magnitude()) if hasattr(self.position, "magnitude") else 1.0
+        self.pairs_of = getattr(s.position, "rotary_dim", 0) if getattr(s.position, "layout", "half") == "interleaved" else 0
         # the general preparation kernel serves whatever the whole-projection one does not know
         self.general = (s.qk_norm == "head" or s.position.kind != "none" or s.q_temp_every > 0)
         # Causal softmax over keys and values of equal size (no sink, no window; a cap and chunks are parameters) is what
@@ -125,11 +133,21 @@ class SinkAttention(_SinkSoftmax):
         if s.conv_taps > 0:
             d += [WeightDecl(p + n + ".conv", (size, s.conv_taps), init="uniform", lo=-0.5, hi=0.5)
                   for n, size in (("q", self.q_dim), ("k", self.k_dim), ("v", self.v_dim))]
-        if s.head_gate:
-            d.append(WeightDecl(p + "g", (s.num_heads, s.hidden_size)))
+        if self.gate_cols:
+            d.append(WeightDecl(p + "g", (self.gate_cols, s.hidden_size)))
         if s.sink:
             d.append(WeightDecl(p + "sink", (s.num_heads,), init="uniform", lo=-1.0, hi=1.0))
         return d
+
+    def _half_order(self, t: Optional[torch.Tensor], heads: int) -> Optional[torch.Tensor]:
+        """The first dimension (``heads`` times head_dim) of a query or key tensor with the rotated part of every head in the
+        rotate-half order; as it is for other layouts."""
+        if t is None or not self.pairs_of:
+            return t
+        D, r = self.spec.head_dim, self.pairs_of
+        one = torch.cat([torch.arange(0, r, 2), torch.arange(1, r, 2), torch.arange(r, D)])
+        index = (torch.arange(heads)[:, None] * D + one[None, :]).reshape(-1)
+        return t.index_select(0, index.to(t.device))
 
     def load(self, store, rt: Runtime) -> None:
         s, p = self.spec, self.prefix
@@ -137,9 +155,13 @@ class SinkAttention(_SinkSoftmax):
         got = {d.name: store.take(d.name, d.shape) for d in self.weight_decls()}
         if any(v is None for v in got.values()):
             return
+        for n, heads in (("q", s.num_heads), ("k", s.num_kv_heads)):
+            for name in (n, n + ".b", n + ".conv", n + ".norm"):
+                if p + name in got:
+                    got[p + name] = self._half_order(got[p + name], 1 if name.endswith(".norm") and s.qk_norm == "head" else heads)
         wd = rt.weight_dtype(got[p + "q"].dtype)
-        # one product for q, k, v and, behind them, the per-head gate's logits (same input)
-        self.qkv = Linear(torch.cat([rt.to_device(got[p + n], wd) for n in ("q", "k", "v") + (("g",) if s.head_gate else ())], dim=0).contiguous())
+        # one product for q, k, v and, behind them, the gate's logits (same input)
+        self.qkv = Linear(torch.cat([rt.to_device(got[p + n], wd) for n in ("q", "k", "v") + (("g",) if self.gate_cols else ())], dim=0).contiguous())
         self.o = Linear.from_host(got[p + "o"], rt)
         f32 = lambda name: rt.to_device(got[p + name], torch.float32)          # noqa: E731
         self.bias = torch.cat([f32(n + ".b") for n in "qkv"]).contiguous() if s.bias else None
@@ -158,8 +180,8 @@ class SinkAttention(_SinkSoftmax):
 
     def cache_need(self) -> CacheNeed:
         s = self.spec
-        return CacheNeed(kind="window" if s.window > 0 else "full", num_kv_heads=s.num_kv_heads, head_dim=s.head_dim,
-                         window=s.window, value_dim=s.value_dim if s.value_dim != s.head_dim else 0,
+        return CacheNeed(kind="window" if s.window > 0 or s.chunk > 0 else "full", num_kv_heads=s.num_kv_heads, head_dim=s.head_dim,
+                         window=s.window, chunk=s.chunk, value_dim=s.value_dim if s.value_dim != s.head_dim else 0,
                          keep_first=s.keep_first if s.window > 0 else 0)
 
     def cache_needs(self):
@@ -202,19 +224,21 @@ class SinkAttention(_SinkSoftmax):
             ops.head_prepare_store(qkv, self.bias, s.qk_norm, self.q_norm_w, self.k_norm_w, s.qk_norm_eps,
                                    self.inv_freq if self.rotary else None, self.rotary, s.q_temp_coef, s.q_temp_every, T, H, G, D, V,
                                    ctx.positions, ctx.seq_of, table, cache.page_tokens, cache.k, cache.v, q, write_kv=owns_cache,
-                                   err=ctx.err, stream=ctx.stream)
+                                   err=ctx.err, stream=ctx.stream, magnitude=self.magnitude)
         else:
             ops.whole_norm_store(qkv, self.bias, self.q_norm_w, self.k_norm_w, s.qk_norm_eps, T, H, G, D, V, ctx.positions,
                                  ctx.seq_of, table, cache.page_tokens, cache.k, cache.v, q, write_kv=owns_cache, err=ctx.err,
                                  stream=ctx.stream)
         if self.dense is not None and getattr(self.dense, "rt", None) is not None and ops.TC_ENABLED:
-            self.dense.attend(ctx, q, cache, table, att)
+            self.dense.attend(ctx, q, cache, table, att, gate=proj if s.element_gate else None, gate_col=self.channels)
             if s.head_gate:
                 ops.head_gate_apply(att, proj, self.channels, T, H, V, stream=ctx.stream)
         else:
             self._attend(ctx, q, cache.k, cache.v, att, table, cache.page_tokens, H, G, D, V, s.window, s.keep_first, self.sink,
                          s.scale, chunk=s.chunk, softcap=s.softcap, head_gate=proj if s.head_gate else None,
                          head_gate_col=self.channels)
+            if s.element_gate:
+                ops.element_gate_apply(att, proj, self.channels, T, H * V, stream=ctx.stream)
         self.o(ctx, att, out, T, ops.EPI_ADD_F32 if accumulate else ops.EPI_STORE_F32)
 
 

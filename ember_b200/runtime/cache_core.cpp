@@ -6,7 +6,8 @@
 //
 // Pages: ids 0..n-1; a fresh pool hands out low ids first, afterwards the most recently freed page first.
 // Groups: kind 0 keeps all keys, kind 1 a window of them (pages wholly older than the window go back as soon
-// as no later query can see them; pages that hold one of the first `keep` keys never do), kind 2 is fixed-size
+// as no later query can see them; pages that hold one of the first `keep` keys never do) or, with a chunk, the keys of
+// the chunk of positions the next token falls into (chunks counted from position 0), kind 2 is fixed-size
 // state (no pages).  Every admitted request holds one
 // slot and one block table per group (-1 = page given back).
 #include <cstdint>
@@ -60,7 +61,7 @@ struct Pool {
 };
 
 struct Group {
-    int kind = 0, window = 0, keep = 0;
+    int kind = 0, window = 0, keep = 0, chunk = 0;
     Pool pool;
     bool paged() const { return kind != 2; }
 };
@@ -144,6 +145,14 @@ int ember_cache_set_keep(void* cv, int g, int keep) {
     return 0;
 }
 
+// Group g (kind 1) keeps the keys of the current chunk of `chunk` positions instead of a window of them.
+int ember_cache_set_chunk(void* cv, int g, int chunk) {
+    Core* c = (Core*)cv;
+    if (g < 0 || g >= (int)c->groups.size() || chunk < 0) return -1;
+    c->groups[g].chunk = chunk;
+    return 0;
+}
+
 // The pool of group g (for the queries above); null for a state group.
 void* ember_cache_pool(void* cv, int g) {
     Core* c = (Core*)cv;
@@ -214,7 +223,8 @@ int ember_cache_advance(void* cv, int h, long long tokens) {
         Group& grp = c->groups[g];
         if (grp.kind != 1) continue;
         // the next query is at position >= tokens and sees keys > position - window
-        long long first_key = tokens - grp.window + 1;
+        // (chunks: keys of its own chunk, and the earliest such query is at position `tokens`)
+        long long first_key = grp.chunk > 0 ? tokens - tokens % grp.chunk : tokens - grp.window + 1;
         if (first_key < 0) first_key = 0;
         const long long dead = first_key / c->page;
         auto& t = r->tables[g];

@@ -43,7 +43,8 @@ def test_spec_layers_and_cache_needs(name):
         else:
             a, r = m["left"], m["right"]
             n = needs[(i, "left")]
-            assert (n.kind, n.num_kv_heads, n.head_dim, n.value_dim or n.head_dim) == ("full", a["kv_heads"], a["dim"], a["vdim"])
+            assert (n.kind, n.num_kv_heads, n.head_dim, n.value_dim or n.head_dim) == ("window", a["kv_heads"], a["dim"], a["vdim"])
+            assert (n.chunk, n.window) == (a["mask"]["size"], 0)          # pages of chunks that have passed go back
             kv_bytes += 2 * a["kv_heads"] * (a["dim"] + a["vdim"])
             channels = a["heads"] * a["dim"] + a["kv_heads"] * (a["dim"] + a["vdim"])
             assert ((i, "left.conv") in needs) == (a["conv"] > 1)
