@@ -22,6 +22,7 @@ Other workloads of the same engine, one JSON line each (not part of the default 
     python bench.py --workload zufusun [--breakdown]   # Zufusun (two of eight experts a token) beside Qwen3 likewise
     python bench.py --workload fomanex [--breakdown]   # Fomanex beside Zufusun (its closest relative) and Qwen3 likewise
     python bench.py --workload pepapel [--breakdown]   # Pepapel beside Zufusun, Fadosun (its closest relatives) and Qwen3 likewise
+    python bench.py --workload filanex [--breakdown]   # Filanex beside Pepapel (its closest relative) and Qwen3 likewise
 """
 from __future__ import annotations
 
@@ -463,6 +464,32 @@ def workload_pepapel(args, pk) -> int:
                         others=[("zufusun", zufusun_config(n_layers)), ("fadosun", fadosun_config(n_layers))])
 
 
+def filanex_config(runs):
+    """``runs`` layer runs (6 or more) from two fewer listed layers: dense and expert feed-forwards in turn, attention inside
+    chunks of 2,048 (so that a decode step at a context of 1,024 reads as many keys as Qwen3's), 16 / 8 heads of 128, half
+    of each rotated, capped scores, a gate per element; the third and fourth layer run twice."""
+    from ember_b200.config import FilanexConfig
+    width, ff, vocab = QWEN3_1P7B["hidden_size"], QWEN3_1P7B["intermediate_size"], QWEN3_1P7B["vocab_size"]
+    mixer = {"heads": 16, "kv_heads": 8, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 50.0, "mask": {"size": 2048},
+             "rot": {"dims": 64, "base": 1e6, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    mlps = [{"kind": "dense", "ff": ff},
+            {"kind": "moe", "expert": {"ff": ff // 2}, "router": {"experts": 8, "top": 2, "groups": {"count": 4, "keep": 2}}}]
+    layers = [{"type": "attention", "mixer": mixer, "mlp": mlps[i % 2]} for i in range(runs - 2)]
+    return FilanexConfig.from_json({"architecture": "Filanex", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+                                    "embedding": {"bigram": {"buckets": 131071, "mul_prev": 7919, "mul_cur": 104729}},
+                                    "loop": {"start": 2, "stop": 4, "times": 2}, "layers": layers})
+
+
+def workload_filanex(args, pk) -> int:
+    """Filanex beside Pepapel (whose attention and experts are the like kernels) and Qwen3, all at the 1.7B width and
+    vocabulary and with as many layer runs (8 unless --layers says otherwise; random weights): the measurements of
+    ``--workload fadosun``."""
+    runs = max(args.layers or 8, 6)
+    return beside_qwen3(args, pk, "filanex", filanex_config(runs), runs,
+                        {"filanex_layers_listed": runs - 2, "loop": "layers 2 and 3 twice", "chunk": 2048, "experts": 8, "top": 2,
+                         "expert_ff": QWEN3_1P7B["intermediate_size"] // 2}, others=[("pepapel", pepapel_config(runs))])
+
+
 def beside_qwen3(args, pk, label, fcfg, n_layers, extra, others=()) -> int:
     """A design (``fcfg``) and Qwen3 at the 1.7B widths and ``n_layers`` layers, one after the other: prefill of 512 and
     2,048 tokens and decode steps at batch 8 and 64 from a context of 1,024, or with --breakdown the device time per
@@ -705,9 +732,9 @@ def main() -> int:
                     help="profiling aid: device time per kernel of three decode steps and one 2,048-token prefill step "
                          "(kernels serialised: EMBER_PDL=0 and no CUDA graphs are set by this flag)")
     ap.add_argument("--page-tokens", type=int, default=PAGE_TOKENS, choices=[16, 32, 64], help="tokens per cache page")
-    ap.add_argument("--workload", default="default", choices=["default", "serving-8b", "qwen3-32b", "fadosun", "zufusun", "fomanex", "pepapel"],
+    ap.add_argument("--workload", default="default", choices=["default", "serving-8b", "qwen3-32b", "fadosun", "zufusun", "fomanex", "pepapel", "filanex"],
                     help="default: the Qwen3-1.7B line; serving-8b and qwen3-32b are BASELINE's fourth "
-                         "and fifth configurations; fadosun, zufusun, fomanex, pepapel: that design beside Qwen3 at equal sizes (with "
+                         "and fifth configurations; fadosun, zufusun, fomanex, pepapel, filanex: that design beside Qwen3 at equal sizes (with "
                          "--breakdown also per kernel); one JSON line each")
     ap.add_argument("--prefill-tokens", type=int, default=PREFILL_TOKENS,
                     help="with --only-prefill: another prompt length (the reported line stays at 2,048)")
@@ -757,6 +784,8 @@ def main() -> int:
         return workload_fomanex(args, pk)
     if args.workload == "pepapel":
         return workload_pepapel(args, pk)
+    if args.workload == "filanex":
+        return workload_filanex(args, pk)
     if args.breakdown:
         return breakdown(cfg, n_layers, args.batch)
     if args.only_prefill:
