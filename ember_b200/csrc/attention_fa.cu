@@ -57,7 +57,7 @@ struct FaParams {
     int window;
     int chunk;                // > 0: a query sees a key only inside its own chunk of positions (chunks counted from position 0)
     float scale_log2;
-    float cap_over_scale, scale_over_cap;   // a cap on the scaled scores, cap * tanh(scale s / cap), applied to the raw scores as (cap / scale) tanh(s scale / cap); 0: no cap
+    float cap_log2, cap_arg, cap_z;      // a cap on the scaled scores, cap * tanh(scale s / cap): cap * log2(e), 2 log2(e) scale / cap, scale / cap
     const float* gate;        // logits of a gate per output element: row t, element head * 128 + d, or null
     int ld_gate;              // (a multiple of 4, rows 16-byte aligned)
     int n_tiles;
@@ -167,8 +167,58 @@ __device__ __forceinline__ float fa_ex2(float x) {
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
+__device__ __forceinline__ float fa_rcp(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+// A raw score, scaled and capped, in units of log2: cap tanh(z) log2(e) with tanh(z) = 1 - 2 / (e^(2z) + 1).  (The error is
+// a few 1e-7 of the cap; e^(2z) that overflows or vanishes gives the cap's ends.)
+__device__ __forceinline__ float fa_capped(const FaParams& p, float raw) {
+    return fmaf(-2.0f * p.cap_log2, fa_rcp(1.0f + fa_ex2(raw * p.cap_arg)), p.cap_log2);
+}
+// Packed fp32 pairs: one instruction for two lanes of arithmetic.
+__device__ __forceinline__ unsigned long long fa_pk2(float lo, float hi) {
+    unsigned long long r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "r"(__float_as_uint(lo)), "r"(__float_as_uint(hi)));
+    return r;
+}
+__device__ __forceinline__ unsigned long long fa_mul2(unsigned long long a, unsigned long long b) {
+    unsigned long long d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ unsigned long long fa_fma2(unsigned long long a, unsigned long long b, unsigned long long c) {
+    unsigned long long d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+// The same for two scores whose z = scale s / cap lies in [-1, 1], on the FMA pipes alone (two special functions an
+// element are what the form above costs): tanh(z) = z P(z^2), P the degree-6 fit of tanh(z) / z over z^2 in [0, 1] with
+// the smallest largest error (4e-8; found by iterated weighted least squares).
+__device__ __forceinline__ void fa_capped_small(const FaParams& p, float& s0, float& s1) {
+    const unsigned long long raw = fa_pk2(s0, s1), z = fa_mul2(raw, fa_pk2(p.cap_z, p.cap_z)), u = fa_mul2(z, z);
+    unsigned long long a = fa_pk2(1.0531364241614938e-3f, 1.0531364241614938e-3f);
+    a = fa_fma2(a, u, fa_pk2(-6.239818409085274e-3f, -6.239818409085274e-3f));
+    a = fa_fma2(a, u, fa_pk2(2.0331110805273056e-2f, 2.0331110805273056e-2f));
+    a = fa_fma2(a, u, fa_pk2(-5.347844585776329e-2f, -5.347844585776329e-2f));
+    a = fa_fma2(a, u, fa_pk2(0.13325709104537964f, 0.13325709104537964f));
+    a = fa_fma2(a, u, fa_pk2(-0.33332881331443787f, -0.33332881331443787f));
+    a = fa_fma2(a, u, fa_pk2(0.9999999403953552f, 0.9999999403953552f));
+    a = fa_mul2(a, fa_mul2(z, fa_pk2(p.cap_log2, p.cap_log2)));
+    uint32_t lo, hi;
+    asm("mov.b64 {%0, %1}, %2;" : "=r"(lo), "=r"(hi) : "l"(a));
+    s0 = __uint_as_float(lo);
+    s1 = __uint_as_float(hi);
+}
 __device__ __forceinline__ uint32_t fa_swz(int row, int chunk) { return (uint32_t)(row * 128 + ((chunk ^ (row & 7)) << 4)); }
 
+// CAP 0: no cap on the scores.  1: a cap of at most FA_PLAIN_CAP (in log2 units): exponents lie between its two ends, so
+// they are taken as they are, without a running maximum: e^cap and its sums stay far inside fp32's (and bf16's) range.
+// 2: a larger cap, with the running maximum.
+constexpr float FA_PLAIN_CAP = 88.0f;
+
+template <int CAP>
 __global__ void __launch_bounds__(FA_THREADS, 2)
 attention_fa_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, const FaParams p) {
     constexpr int Q_HALF = FA_ROWS * 128;                // 16 KiB: [128 rows][64 bf16]
@@ -376,9 +426,20 @@ attention_fa_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
             __syncwarp();
             if (lane == 0) fa_arrive(q_ready);
         }
+        if (p.gate && r < rows) {
+            const int rq = r / G, rg = r - rq * G;
+            const float* g = p.gate + (size_t)(row0 + rq) * p.ld_gate + (kvh * G + rg) * FA_D;
+#pragma unroll
+            for (int c = 0; c < FA_D; c += 32) asm volatile("prefetch.global.L2 [%0];" ::"l"(g + c));
+        }
         float m_ref = -INFINITY, l_run = 0.0f;      // reference maximum (exponent base) and denominator
         const uint32_t lane_base = (uint32_t)(quad * 32) << 16;
         bool ok = true;
+        // the first key this row sees, and the first that every row of the tile sees
+        const int last_q = pos0 + (rows - 1) / G;
+        int row_lo = lo, all_lo = lo;
+        if (p.window > 0) { row_lo = max(row_lo, qpos - p.window + 1); all_lo = max(all_lo, last_q - p.window + 1); }
+        if (p.chunk > 0) { row_lo = max(row_lo, qpos - qpos % p.chunk); all_lo = max(all_lo, last_q - last_q % p.chunk); }
         for (int j = 0; j < n_kt; j++) {
             const int k0 = k_begin + j * FA_KT;
             if (ok) ok = fa_wait(&s_full[j & 1], (uint32_t)(j >> 1) & 1u, abort_flag);
@@ -388,26 +449,38 @@ attention_fa_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
             fa_tmem_ld32_nowait(tmem_s0 + lane_base + (uint32_t)((j & 1) * FA_KT + 32), su + 32);
             fa_tmem_wait_ld();
             float* s = reinterpret_cast<float*>(su);
-            if (p.cap_over_scale > 0.0f) {
+            if (CAP) {
+                float a0 = 0.0f, a1 = 0.0f, a2 = 0.0f, a3 = 0.0f;
 #pragma unroll
-                for (int i = 0; i < FA_KT; i++) s[i] = p.cap_over_scale * tanhf(s[i] * p.scale_over_cap);
+                for (int i = 0; i < FA_KT; i += 4) {
+                    a0 = fmaxf(a0, fabsf(s[i]));
+                    a1 = fmaxf(a1, fabsf(s[i + 1]));
+                    a2 = fmaxf(a2, fabsf(s[i + 2]));
+                    a3 = fmaxf(a3, fabsf(s[i + 3]));
+                }
+                const bool small = fmaxf(fmaxf(a0, a1), fmaxf(a2, a3)) * p.cap_z <= 1.0f;
+                if (__all_sync(0xffffffffu, small)) {
+#pragma unroll
+                    for (int i = 0; i < FA_KT; i += 2) fa_capped_small(p, s[i], s[i + 1]);
+                } else {
+#pragma unroll
+                    for (int i = 0; i < FA_KT; i++) s[i] = fa_capped(p, s[i]);
+                }
             }
 
-            const bool interior = k0 >= lo && k0 + FA_KT <= hi && k0 + FA_KT - 1 <= pos0 &&
-                                  (p.window <= 0 || k0 > pos0 + (rows - 1) / G - p.window) &&
-                                  (p.chunk <= 0 || k0 >= (pos0 + (rows - 1) / G) - (pos0 + (rows - 1) / G) % p.chunk);
-            // the maximum is taken over the raw scores; the scale (> 0) is folded into the exponent below
+            const bool interior = k0 >= all_lo && k0 + FA_KT <= hi && k0 + FA_KT - 1 <= pos0;
+            // the maximum is taken over the raw scores; the scale (> 0) is folded into the exponent below (capped scores
+            // are scaled already)
+            const float to_log2 = CAP ? 1.0f : p.scale_log2;
             float tmax;
             if (!interior) {
 #pragma unroll
                 for (int i = 0; i < FA_KT; i++) {
                     const int key = k0 + i;
-                    const bool vis = key >= lo && key < hi && key <= qpos && (p.window <= 0 || key > qpos - p.window) &&
-                                     (p.chunk <= 0 || key >= qpos - qpos % p.chunk);
-                    s[i] = vis ? s[i] : -INFINITY;
+                    s[i] = key >= row_lo && key <= qpos ? s[i] : -INFINITY;
                 }
             }
-            {   // four independent chains instead of one of 64 dependent maxima
+            if (CAP != 1) {   // four independent chains instead of one of 64 dependent maxima
                 float t0 = s[0], t1 = s[1], t2 = s[2], t3 = s[3];
 #pragma unroll
                 for (int i = 4; i < FA_KT; i += 4) {
@@ -417,11 +490,13 @@ attention_fa_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
                     t3 = fmaxf(t3, s[i + 3]);
                 }
                 tmax = fmaxf(fmaxf(t0, t1), fmaxf(t2, t3));
+            } else {
+                tmax = -INFINITY;
             }
-            tmax *= p.scale_log2;
+            tmax *= to_log2;
             // raise the reference maximum only when the true one has outgrown it by more than 2^8
-            const bool raise = tmax > m_ref + 8.0f || (m_ref == -INFINITY && tmax > -INFINITY);
-            const bool warp_raise = __any_sync(0xffffffffu, raise);
+            const bool raise = CAP != 1 && (tmax > m_ref + 8.0f || (m_ref == -INFINITY && tmax > -INFINITY));
+            const bool warp_raise = CAP != 1 && __any_sync(0xffffffffu, raise);
             if (warp_raise && j > 0) {
                 // O is complete up to tile j - 1 once the previous second product has finished
                 if (ok) ok = fa_wait(pv_full, (uint32_t)(j - 1) & 1u, abort_flag);
@@ -447,8 +522,10 @@ attention_fa_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
             uint32_t packed[FA_KT / 2];
 #pragma unroll
             for (int i = 0; i < FA_KT / 2; i += 2) {
-                const float p0 = fa_ex2(fmaf(s[2 * i], p.scale_log2, neg_base)), p1 = fa_ex2(fmaf(s[2 * i + 1], p.scale_log2, neg_base));
-                const float p2 = fa_ex2(fmaf(s[2 * i + 2], p.scale_log2, neg_base)), p3 = fa_ex2(fmaf(s[2 * i + 3], p.scale_log2, neg_base));
+                const float p0 = fa_ex2(CAP == 1 ? s[2 * i] : fmaf(s[2 * i], to_log2, neg_base));
+                const float p1 = fa_ex2(CAP == 1 ? s[2 * i + 1] : fmaf(s[2 * i + 1], to_log2, neg_base));
+                const float p2 = fa_ex2(CAP == 1 ? s[2 * i + 2] : fmaf(s[2 * i + 2], to_log2, neg_base));
+                const float p3 = fa_ex2(CAP == 1 ? s[2 * i + 3] : fmaf(s[2 * i + 3], to_log2, neg_base));
                 sum0 += p0; sum1 += p1; sum2 += p2; sum3 += p3;
                 __nv_bfloat162 h2 = __floats2bfloat162_rn(p0, p1), h3 = __floats2bfloat162_rn(p2, p3);
                 packed[i] = *reinterpret_cast<uint32_t*>(&h2);
@@ -468,27 +545,50 @@ attention_fa_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
         // the wait in the loop above is safe, S_j being complete only after O += P V of tile j - 2)
         if (n_kt > 0 && ok) ok = fa_wait(o_done, 0, abort_flag);
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-        if (n_kt > 0) {
-            const float inv = l_run > 0.0f ? 1.0f / l_run : 0.0f;
+        const float inv = l_run > 0.0f ? 1.0f / l_run : 0.0f;
+        if (n_kt > 0 && p.gate) {
+            // The gate's logits and the results are rows of 512 and 256 bytes a (token, head): a warp turns its 32 rows in
+            // shared memory (queries, keys and values have all been read) so that its lanes walk along a row.
+            // Its logits have been on their way into the L2 since before the first tile.
+            ok = __all_sync(0xffffffffu, ok);
+            float* turn = reinterpret_cast<float*>(smem) + quad * 32 * (FA_D + 4);
+#pragma unroll
+            for (int c = 0; c < FA_D / 32; c++) {
+                uint32_t tu[32];
+                fa_tmem_ld32_nowait(tmem_o + lane_base + (uint32_t)(c * 32), tu);
+                fa_tmem_wait_ld();
+                if (ok) {
+#pragma unroll
+                    for (int e = 0; e < 32; e += 4)
+                        *reinterpret_cast<float4*>(turn + lane * (FA_D + 4) + c * 32 + e) =
+                            make_float4(__uint_as_float(tu[e]) * inv, __uint_as_float(tu[e + 1]) * inv, __uint_as_float(tu[e + 2]) * inv,
+                                        __uint_as_float(tu[e + 3]) * inv);
+                }
+            }
+            __syncwarp();
+            const int here = ok ? min(32, rows - quad * 32) : 0;
+#pragma unroll 8
+            for (int i = 0; i < here; i++) {
+                const int rr = quad * 32 + i, rq = rr / G, rg = rr - rq * G;
+                const size_t at = (size_t)(kvh * G + rg) * FA_D + 4 * lane;
+                const float4 g = __ldg(reinterpret_cast<const float4*>(p.gate + (size_t)(row0 + rq) * p.ld_gate + at));
+                const float4 v = *reinterpret_cast<const float4*>(turn + i * (FA_D + 4) + 4 * lane);
+                uint2 packed;
+                __nv_bfloat162 a = __floats2bfloat162_rn(v.x * __fdividef(1.0f, 1.0f + __expf(-g.x)), v.y * __fdividef(1.0f, 1.0f + __expf(-g.y)));
+                __nv_bfloat162 b = __floats2bfloat162_rn(v.z * __fdividef(1.0f, 1.0f + __expf(-g.z)), v.w * __fdividef(1.0f, 1.0f + __expf(-g.w)));
+                packed.x = *reinterpret_cast<uint32_t*>(&a);
+                packed.y = *reinterpret_cast<uint32_t*>(&b);
+                *reinterpret_cast<uint2*>(p.out + (size_t)(row0 + rq) * p.n_heads * FA_D + at) = packed;
+            }
+        } else if (n_kt > 0) {
             const int rq = r / G, rg = r - rq * G;
             __nv_bfloat16* dst = p.out + ((size_t)(row0 + rq) * p.n_heads + kvh * G + rg) * FA_D;
-            const float* gate = p.gate ? p.gate + (size_t)(row0 + rq) * p.ld_gate + (kvh * G + rg) * FA_D : nullptr;
 #pragma unroll
             for (int c = 0; c < FA_D / 32; c++) {
                 uint32_t tu[32];
                 fa_tmem_ld32_nowait(tmem_o + lane_base + (uint32_t)(c * 32), tu);
                 fa_tmem_wait_ld();
                 if (ok && r < rows) {
-                    if (gate) {
-#pragma unroll
-                        for (int e = 0; e < 32; e += 4) {
-                            const float4 gv = __ldg(reinterpret_cast<const float4*>(gate + c * 32 + e));
-                            tu[e] = __float_as_uint(__uint_as_float(tu[e]) / (1.0f + __expf(-gv.x)));
-                            tu[e + 1] = __float_as_uint(__uint_as_float(tu[e + 1]) / (1.0f + __expf(-gv.y)));
-                            tu[e + 2] = __float_as_uint(__uint_as_float(tu[e + 2]) / (1.0f + __expf(-gv.z)));
-                            tu[e + 3] = __float_as_uint(__uint_as_float(tu[e + 3]) / (1.0f + __expf(-gv.w)));
-                        }
-                    }
 #pragma unroll
                     for (int q4 = 0; q4 < 4; q4++) {
                         uint4 packed;
@@ -587,16 +687,22 @@ EMBER_API int ember_attention_fa(const void* q, const void* k_pool, const void* 
     p.q = (const __nv_bfloat16*)q; p.out = (__nv_bfloat16*)out; p.tiles = tiles; p.block_table = block_table;
     p.max_blocks = max_blocks; p.page = page; p.num_pages = num_pages; p.n_heads = n_heads; p.n_kv = n_kv;
     p.window = window; p.chunk = chunk < 0 ? 0 : chunk; p.scale_log2 = scale * FA_LOG2E;
-    p.cap_over_scale = (softcap > 0.0f && scale > 0.0f) ? softcap / scale : 0.0f;
-    p.scale_over_cap = softcap > 0.0f ? scale / softcap : 0.0f; p.gate = gate; p.ld_gate = ld_gate; p.n_tiles = n_tiles; p.err = err;
+    if (scale <= 0.0f) return fail("attention_fa: a score scale of %g (it must be positive)", scale);
+    p.cap_log2 = softcap * FA_LOG2E;
+    p.cap_z = softcap > 0.0f ? scale / softcap : 0.0f;
+    p.cap_arg = softcap > 0.0f ? 2.0f * FA_LOG2E * scale / softcap : 0.0f; p.gate = gate; p.ld_gate = ld_gate; p.n_tiles = n_tiles; p.err = err;
     const size_t smem = (size_t)2 * FA_ROWS * 128 + (size_t)(FA_K_STAGES + FA_V_STAGES) * 2 * FA_KT * 128 + 256;
-    static bool attr = false;
-    if (!attr) {
-        cudaError_t e = cudaFuncSetAttribute(attention_fa_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        if (e != cudaSuccess) return fail("attention_fa: shared memory %zu: %s", smem, cudaGetErrorString(e));
-        cudaFuncSetAttribute(attention_fa_kernel, cudaFuncAttributePreferredSharedMemoryCarveout, (int)cudaSharedmemCarveoutMaxShared);
-        attr = true;
-    }
-    launch_kernel(attention_fa_kernel, dim3(n_tiles, n_kv), dim3(FA_THREADS), smem, (cudaStream_t)stream, mk, mv, p);
-    return check_launch("attention_fa");
+    auto run = [&](auto kernel, bool& ready) -> int {
+        if (!ready) {
+            cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+            if (e != cudaSuccess) return fail("attention_fa: shared memory %zu: %s", smem, cudaGetErrorString(e));
+            cudaFuncSetAttribute(kernel, cudaFuncAttributePreferredSharedMemoryCarveout, (int)cudaSharedmemCarveoutMaxShared);
+            ready = true;
+        }
+        launch_kernel(kernel, dim3(n_tiles, n_kv), dim3(FA_THREADS), smem, (cudaStream_t)stream, mk, mv, p);
+        return check_launch("attention_fa");
+    };
+    static bool ready[3] = {false, false, false};
+    if (softcap <= 0.0f) return run(attention_fa_kernel<0>, ready[0]);
+    return p.cap_log2 <= FA_PLAIN_CAP ? run(attention_fa_kernel<1>, ready[1]) : run(attention_fa_kernel<2>, ready[2]);
 }

@@ -49,7 +49,7 @@ struct AttnTcParams {
     int window;
     int chunk;                // > 0: a query sees a key only inside its own chunk of positions (chunks counted from position 0)
     float scale_log2;         // softmax scale * log2(e)
-    float cap_log2, scale_over_cap;   // a cap on the scaled scores, cap * tanh(score / cap): cap * log2(e) and scale / cap (0: no cap)
+    float cap_log2, cap_arg;  // a cap on the scaled scores, cap * tanh(score / cap): cap * log2(e) and 2 log2(e) scale / cap (0: no cap)
     const float* gate;        // logits of a gate per output element: row t, element head * D + d, or null
     int ld_gate;
     int n_splits, split_keys;
@@ -60,13 +60,14 @@ struct AttnTcParams {
 
 __device__ __forceinline__ uint32_t s32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 
-// A raw score q . k as the exponent's argument in base 2: scaled, and capped where the layer has a cap.
+// A raw score q . k as the exponent's argument in base 2: scaled, and capped where the layer has a cap, with
+// tanh(z) = 1 - 2 / (e^(2z) + 1) (an error of a few 1e-7 of the cap).
 __device__ __forceinline__ float score_log2(const AttnTcParams& p, float raw) {
-    return p.cap_log2 > 0.0f ? p.cap_log2 * tanhf(raw * p.scale_over_cap) : raw * p.scale_log2;
+    return p.cap_log2 > 0.0f ? fmaf(-2.0f * p.cap_log2, __fdividef(1.0f, 1.0f + exp2f(fminf(raw * p.cap_arg, 120.0f))), p.cap_log2) : raw * p.scale_log2;
 }
 
 // A result element times the sigmoid of its gate's logit, where the layer has such a gate (`g` points at the row's logits).
-__device__ __forceinline__ float gated(const float* g, int i, float v) { return g ? v / (1.0f + __expf(-__ldg(g + i))) : v; }
+__device__ __forceinline__ float gated(const float* g, int i, float v) { return g ? v * __fdividef(1.0f, 1.0f + __expf(-__ldg(g + i))) : v; }
 
 __device__ __forceinline__ void ldsm_x4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
@@ -244,11 +245,21 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
     const int r_a = wrow + g8, r_b = wrow + g8 + 8;          // the two rows this thread holds
     const int qpos_a = pos0 + min(r_a, rows - 1) / G, qpos_b = pos0 + min(r_b, rows - 1) / G;
 
+    // the first key each of them sees
+    int lo_a = lo, lo_b = lo;
+    if (p.window > 0) { lo_a = max(lo_a, qpos_a - p.window + 1); lo_b = max(lo_b, qpos_b - p.window + 1); }
+    if (p.chunk > 0) { lo_a = max(lo_a, qpos_a - qpos_a % p.chunk); lo_b = max(lo_b, qpos_b - qpos_b % p.chunk); }
+
     float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.0f, l_b = 0.0f;
     float o[ND][4];
 #pragma unroll
     for (int j = 0; j < ND; j++) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.0f;
 
+    // ... and the first that every row of the warp sees
+    const int last_q = pos0 + min(wrow + 15, rows - 1) / G;
+    int all_lo = lo;
+    if (p.window > 0) all_lo = max(all_lo, last_q - p.window + 1);
+    if (p.chunk > 0) all_lo = max(all_lo, last_q - last_q % p.chunk);
     bool alive = true;
     for (int it = 0; it < n_kt && warp < 4; it++) {
         const int b = it % NSTAGE;
@@ -259,8 +270,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
             const int k0 = k_begin + it * KT;
             const int koff = DECODE ? warp * 16 : 0;                // this warp's keys inside the tile
             // in prefill mode a warp whose rows all lie before this key tile has nothing to do
-            const int warp_last_q = pos0 + min(wrow + 15, rows - 1) / G;
-            if (DECODE || (wrow < rows && k0 <= warp_last_q)) {
+            if (DECODE || (wrow < rows && k0 <= last_q)) {
                 float s[NKG][4];
 #pragma unroll
                 for (int j = 0; j < NKG; j++) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.0f;
@@ -284,9 +294,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
                 // no mask: only tiles at the causal diagonal and at range edges pay for the compares.
                 float tmax_a = -INFINITY, tmax_b = -INFINITY;
                 const int first_q = pos0 + min(wrow, rows - 1) / G;          // earliest query position of this warp
-                const bool interior = k0 + koff >= lo && k0 + koff + NKG * 8 <= hi && k0 + koff + NKG * 8 - 1 <= first_q &&
-                                      (p.window <= 0 || k0 + koff > warp_last_q - p.window) &&
-                                      (p.chunk <= 0 || k0 + koff >= warp_last_q - warp_last_q % p.chunk);
+                const bool interior = k0 + koff >= all_lo && k0 + koff + NKG * 8 <= hi && k0 + koff + NKG * 8 - 1 <= first_q;
                 if (interior) {
 #pragma unroll
                     for (int j = 0; j < NKG; j++) {
@@ -301,11 +309,8 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
 #pragma unroll
                         for (int e = 0; e < 2; e++) {
                             const int key = k0 + koff + j * 8 + 2 * t4 + e;
-                            const bool in = key >= lo && key < hi;
-                            const bool va = in && key <= qpos_a && (p.window <= 0 || key > qpos_a - p.window) &&
-                                            (p.chunk <= 0 || key >= qpos_a - qpos_a % p.chunk);
-                            const bool vb2 = in && key <= qpos_b && (p.window <= 0 || key > qpos_b - p.window) &&
-                                             (p.chunk <= 0 || key >= qpos_b - qpos_b % p.chunk);
+                            const bool va = key >= lo_a && key < hi && key <= qpos_a;
+                            const bool vb2 = key >= lo_b && key < hi && key <= qpos_b;
                             s[j][e] = va ? score_log2(p, s[j][e]) : -INFINITY;
                             s[j][2 + e] = vb2 ? score_log2(p, s[j][2 + e]) : -INFINITY;
                             tmax_a = fmaxf(tmax_a, s[j][e]);
@@ -631,7 +636,7 @@ EMBER_API int ember_attention_tc(const void* q, const void* k_pool, const void* 
     p.q = (const __nv_bfloat16*)q; p.out = (__nv_bfloat16*)out; p.part_o = part_o; p.part_ml = part_ml;
     p.tiles = tiles; p.block_table = block_table; p.max_blocks = max_blocks; p.page = page; p.num_pages = num_pages;
     p.n_heads = n_heads; p.n_kv = n_kv; p.window = window; p.chunk = chunk < 0 ? 0 : chunk; p.scale_log2 = scale * LOG2E;
-    p.cap_log2 = softcap * LOG2E; p.scale_over_cap = softcap > 0.0f ? scale / softcap : 0.0f;
+    p.cap_log2 = softcap * LOG2E; p.cap_arg = softcap > 0.0f ? 2.0f * LOG2E * scale / softcap : 0.0f;
     p.gate = gate; p.ld_gate = ld_gate;
     p.n_splits = n_splits; p.split_keys = split_keys; p.n_tiles = n_tiles; p.err = err;
     p.cluster_merge = cluster_merge ? 1 : 0;

@@ -112,7 +112,7 @@ class SinkAttention(_SinkSoftmax):
         # where they take the geometry, a bfloat16 step goes to them (``load`` decides, once the dtype and the page size
         # are known); a gate per head then is a pass of its own behind them
         self.dense = None
-        if (not s.sink and s.window == 0 and s.value_dim == s.head_dim
+        if (not s.sink and s.window == 0 and s.value_dim == s.head_dim and s.scale > 0
                 and s.head_dim % 2 == 0 and s.num_heads // s.num_kv_heads <= ops.ATTENTION_MAX_GROUP):
             from ..config.spec import AttentionSpec
             from .attention import Attention

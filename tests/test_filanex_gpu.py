@@ -310,7 +310,7 @@ def test_attention_alone(dtype, heads, kv, dim, vdim, hidden, softcap, chunk, ro
 @pytest.mark.parametrize("heads,kv,dim,softcap,chunk,rot", [
     (8, 1, 128, 25.0, 50, {"dims": 64, "base": 1e4, "scaling": YARN}), (4, 2, 64, 0.0, 64, {"dims": 64, "base": 500.0}),
     (2, 2, 128, 0.7, 7, {"dims": 16, "base": 1e6}), (16, 1, 64, 3.0, 300, {"dims": 32, "base": 1e4, "scaling": YARN}),
-    (12, 4, 128, 40.0, 0, {"dims": 128, "base": 1e4, "scaling": YARN}), (6, 2, 64, 5.0, 0, None)])
+    (12, 4, 128, 40.0, 0, {"dims": 128, "base": 1e4, "scaling": YARN}), (6, 2, 64, 5.0, 0, None), (4, 4, 128, 300.0, 90, None)])
 def test_layers_on_the_engines_dense_attention_kernels(dense, heads, kv, dim, softcap, chunk, rot, monkeypatch):
     """Keys and values of one size, 64 or 128: bfloat16 steps go to the kernels Qwen3's attention uses, which take the
     chunk, the cap and the gate per element (a group of three query heads a key head takes the mma.sync form for portions
