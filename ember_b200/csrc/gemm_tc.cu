@@ -203,18 +203,75 @@ static int launch_persistent(const void* A, const void* W, GemmTcParams p, int b
         return fail("gemm_tc: cuTensorMapEncodeTiled failed or is unavailable");
     static bool pattr = false;
     if (!pattr) {
-        cudaError_t e = cudaFuncSetAttribute(gemm_tc_persistent_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+        cudaError_t e = cudaFuncSetAttribute(gemm_tc_persistent_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
         if (e != cudaSuccess) return fail("gemm_tc: cannot raise the shared-memory limit: %s", cudaGetErrorString(e));
         pattr = true;
     }
     const int blocks = units < num_sms ? units : num_sms;
-    launch_kernel(gemm_tc_persistent_kernel, dim3(blocks), dim3(GEMM_THREADS), smem, st, map_rows, map_cols, p);
+    launch_kernel(gemm_tc_persistent_kernel<false>, dim3(blocks), dim3(GEMM_THREADS), smem, st, map_rows, map_cols, p);
     return check_launch("gemm_tc_persistent");
+}
+
+// The grouped form: the rows of every group against the group's own weights, one launch, nothing read by the host.
+static int launch_grouped(const void* A, const void* W, GemmTcParams p, int num_sms, cudaStream_t st) {
+    p.swapped = 0;
+    p.num_k_blocks = (p.K + TILE_K - 1) / TILE_K;
+    p.k_blocks_per_split = p.num_k_blocks;
+    p.cluster_splits = 1; p.rows_per = TILE_ROWS; p.accum = nullptr; p.accum_ld = 0; p.row_tiles = 0; p.total_tiles = 0;
+    // The tile width by the model of best_block_cols, with rows dealt evenly (half a row tile a group is lost to its end).
+    const double row_tiles = (double)p.M / TILE_ROWS + 0.5 * (p.groups < p.M ? p.groups : p.M);
+    int block_cols = 256;
+    double best = 1e30;
+    for (int bc = 256; bc >= 128; bc -= 16) {
+        const double waves = row_tiles * ((p.N + bc - 1) / bc) / num_sms;
+        const double cost = (waves < 1.0 ? 1.0 : waves + 0.5) * (bc + 40);
+        if (cost < best * 0.999) { best = cost; block_cols = bc; }
+    }
+    p.block_cols = block_cols;
+    int tc = 32;
+    while (tc < 2 * block_cols) tc <<= 1;
+    p.tmem_cols = tc;
+    const int stage_bytes = TILE_ROWS * TILE_K * 2 + ((block_cols * TILE_K * 2 + 1023) & ~1023);
+    int stages = (200 * 1024) / stage_bytes;
+    if (stages > MAX_STAGES) stages = MAX_STAGES;
+    if (stages < 2) stages = 2;
+    p.stages = stages;
+    const size_t smem = (size_t)stages * stage_bytes + 1024 + 256 + 2 * (MAX_GROUPS + 1) * sizeof(int);
+    CUtensorMap map_rows, map_cols;
+    if (!tensor_map(A, p.M, p.K, TILE_ROWS, &map_rows) || !tensor_map(W, p.groups * p.N, p.K, block_cols, &map_cols))
+        return fail("gemm_tc_grouped: cuTensorMapEncodeTiled failed or is unavailable");
+    static bool ready = false;
+    if (!ready) {
+        cudaError_t e = cudaFuncSetAttribute(gemm_tc_persistent_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+        if (e != cudaSuccess) return fail("gemm_tc_grouped: cannot raise the shared-memory limit: %s", cudaGetErrorString(e));
+        ready = true;
+    }
+    launch_kernel(gemm_tc_persistent_kernel<true>, dim3(num_sms), dim3(GEMM_THREADS), smem, st, map_rows, map_cols, p);
+    return check_launch("gemm_tc_grouped");
 }
 
 }  // namespace ember
 
 using namespace ember;
+
+// Groups of rows against weights of their own: rows [offsets[g], offsets[g + 1]) of A (offsets on the device, ascending, from
+// 0 to at most M) times W[g] [N, K], g < groups (at most 256), into the same rows of `out` under a storing or gated
+// epilogue.
+EMBER_API int ember_gemm_tc_grouped(const void* A, const void* W, void* out, int ldc, int M, int N, int K, int groups, const int* offsets,
+                                    int epilogue, int num_sms, int* err, void* stream) {
+    if (M <= 0 || N <= 0) return 0;
+    if (groups <= 0 || groups > MAX_GROUPS || !offsets) return fail("gemm_tc_grouped: %d groups (at most %d)", groups, MAX_GROUPS);
+    const bool gated = epilogue == 3 || epilogue == 6 || epilogue == 7;
+    if (K <= 0 || K % 8 || (gated && (N & 1)) || (epilogue != 0 && epilogue != 1 && !gated) || (long long)groups * N > 0x7fffffffll)
+        return fail("gemm_tc_grouped: sizes N=%d K=%d under epilogue %d are not taken", N, K, epilogue);
+    if ((((uintptr_t)A) & 15) || (((uintptr_t)W) & 15)) return fail("gemm_tc_grouped: operands must be 16-byte aligned");
+    if (num_sms <= 0) num_sms = 148;
+    GemmTcParams p = {};
+    p.M = M; p.N = N; p.K = K; p.act = epilogue == 6 ? 1 : (epilogue == 7 ? 2 : 0); p.bias = nullptr;
+    p.epilogue = gated ? 3 : epilogue; p.out = out; p.ldc = ldc; p.err = err;
+    p.group_offsets = offsets; p.groups = groups;
+    return launch_grouped(A, W, p, num_sms, (cudaStream_t)stream);
+}
 
 // Whether the tensor-core product takes these sizes (bf16 operands are the caller's business).
 EMBER_API int ember_gemm_tc_supported(int M, int N, int K, int epilogue) {

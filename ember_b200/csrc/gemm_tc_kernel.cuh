@@ -57,6 +57,8 @@ struct GemmTcParams {
     int row_tiles;        // persistent kernel: tiles along M, and their total number
     int total_tiles;
     int tmem_cols;
+    const int* group_offsets;      // grouped walk: the rows of group g are [group_offsets[g], group_offsets[g + 1]) ...
+    int groups;                    // ... and its weights rows g * N .. of W
     int* err;
     QkvEpilogue qkv;      // epilogue 4 only
 };
@@ -787,12 +789,18 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_consta
     }
 }
 
+constexpr int MAX_GROUPS = 256;
+
 // ------------------------------------------------------------------ persistent kernel (prefill)
 // Normal orientation only (accumulator rows are tokens).  One block per SM walks over output tiles
 // (tile t -> weight column tile t / row_tiles, token row tile t % row_tiles, so that blocks running at
 // the same time share weight tiles in L2).  Two accumulators live in tensor memory: while the four
 // epilogue warps drain and store tile i, the MMA warp already fills the other accumulator with tile
 // i + 1, and the TMA warp runs ahead through the ring of stages across tile borders.
+// GROUPED: the rows of A lie in groups (the tokens of each expert, one group after the other), every group against weights
+// of its own; the group borders are read on the device, a tile belongs to one group, and tiles walk a group's weight
+// columns before the next group's.  Rows of the next group that a tile's last rows bring along are computed and dropped.
+template <bool GROUPED>
 __global__ void __launch_bounds__(GEMM_THREADS, 1)
 gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_constant__ CUtensorMap map_cols,
                           const GemmTcParams p) {
@@ -812,8 +820,10 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_rows, const __
     const int n_kb = p.num_k_blocks;
     // With few tiles (a short prompt portion) the K range of the adding epilogue is cut: a unit is a tile and a part
     // of K, its sums are added at the L2 like any other, and every SM has work.
-    const int k_splits = (n_kb + p.k_blocks_per_split - 1) / p.k_blocks_per_split;
-    const int units = p.total_tiles * k_splits;
+    const int k_splits = GROUPED ? 1 : (n_kb + p.k_blocks_per_split - 1) / p.k_blocks_per_split;
+    int units = p.total_tiles * k_splits;
+    int* first_unit = reinterpret_cast<int*>(smem + (size_t)p.stages * stage_bytes + 256);      // grouped: [groups + 1], then
+    int* first_row = first_unit + MAX_GROUPS + 1;                                               // the groups' borders
 
     if (threadIdx.x == 0) {
         for (int s = 0; s < p.stages; s++) {
@@ -840,6 +850,41 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_rows, const __
     pdl_launch_dependents();
     pdl_wait();
 
+    if (GROUPED) {
+        for (int g = threadIdx.x; g <= p.groups; g += GEMM_THREADS) first_row[g] = p.group_offsets[g];
+        __syncthreads();
+        if (threadIdx.x == 0) {
+            const int col_tiles = (p.N + p.block_cols - 1) / p.block_cols;
+            int at = 0;
+            for (int g = 0; g < p.groups; g++) {
+                first_unit[g] = at;
+                at += (first_row[g + 1] - first_row[g] + TILE_ROWS - 1) / TILE_ROWS * col_tiles;
+            }
+            first_unit[p.groups] = at;
+        }
+        __syncthreads();
+        units = first_unit[p.groups];
+    }
+    // Where unit u's tile lies: its first row of A, the row behind its group's last, its first weight row (in W) and its
+    // first output column.  Units only grow along a walk, so the group is found by stepping on from the last one.
+    int cur_group = 0;
+    auto locate = [&](int u, int& row0, int& row_end, int& w_row, int& col0) {
+        if (GROUPED) {
+            while (u >= first_unit[cur_group + 1]) cur_group++;
+            const int a = first_row[cur_group];
+            row_end = first_row[cur_group + 1];
+            const int row_tiles = (row_end - a + TILE_ROWS - 1) / TILE_ROWS, t = u - first_unit[cur_group], c = t / row_tiles;
+            row0 = a + (t - c * row_tiles) * TILE_ROWS;
+            col0 = c * p.block_cols;
+            w_row = cur_group * p.N + col0;
+        } else {
+            const int t = u / k_splits, c = t / p.row_tiles;
+            row0 = (t - c * p.row_tiles) * TILE_ROWS;
+            row_end = p.M;
+            col0 = w_row = c * p.block_cols;
+        }
+    };
+
     if (warp == 0) {
         if (lane == 0) {
             int s = 0;
@@ -847,15 +892,16 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_rows, const __
             bool ok = true, wrapped = false;
             uint8_t* st = smem;
             for (int u = blockIdx.x; u < units && ok; u += gridDim.x) {
-                const int t = u / k_splits, kb0 = (u - t * k_splits) * p.k_blocks_per_split;
+                const int kb0 = (u % k_splits) * p.k_blocks_per_split;
                 const int kb1 = min(n_kb, kb0 + p.k_blocks_per_split);
-                const int col_tile = t / p.row_tiles, row_tile = t - col_tile * p.row_tiles;
+                int row0, row_end, w_row, col0;
+                locate(u, row0, row_end, w_row, col0);
                 for (int i = kb0; i < kb1; i++) {
                     if (wrapped) ok = mbar_wait(&empty_bar[s], phase ^ 1u, abort_flag);
                     if (!ok) break;
                     mbar_expect_tx(&full_bar[s], (uint32_t)(rows_bytes + cols_bytes));
-                    tma_load_2d(st, &map_rows, &full_bar[s], i * TILE_K, row_tile * TILE_ROWS);
-                    tma_load_2d(st + rows_bytes, &map_cols, &full_bar[s], i * TILE_K, col_tile * p.block_cols);
+                    tma_load_2d(st, &map_rows, &full_bar[s], i * TILE_K, row0);
+                    tma_load_2d(st + rows_bytes, &map_cols, &full_bar[s], i * TILE_K, w_row);
                     st += stage_bytes;
                     if (++s == p.stages) { s = 0; st = smem; phase ^= 1u; wrapped = true; }
                 }
@@ -898,18 +944,18 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_rows, const __
         bool ok = true;
         int li = 0;
         for (int u = blockIdx.x; u < units; u += gridDim.x, li++) {
-            const int t = u / k_splits;
-            const bool u_first = u == t * k_splits;
-            const int col_tile = t / p.row_tiles, row_tile = t - col_tile * p.row_tiles;
+            const bool u_first = u % k_splits == 0;
+            int row0, row_end, w_row, col0;
+            locate(u, row0, row_end, w_row, col0);
             const int acc = li & 1;
-            const int m = row_tile * TILE_ROWS + r;
+            const int m = row0 + r;
             QkvRow row;
-            if (p.epilogue == 4) qkv_row_prepare(p, m, ok && m < p.M, row);       // its loads travel during the wait
+            if (!GROUPED && p.epilogue == 4) qkv_row_prepare(p, m, ok && m < p.M, row);       // its loads travel during the wait
             if (ok) ok = mbar_wait(&tmem_full_bar[acc], (uint32_t)(li >> 1) & 1u, abort_flag);
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             const uint32_t taddr_row = tmem_d + ((uint32_t)(quad * 32) << 16) + (uint32_t)(acc * p.block_cols);
-            if (p.epilogue == 4) {
-                const int slot0 = col_tile * (p.block_cols >> 7);
+            if (!GROUPED && p.epilogue == 4) {
+                const int slot0 = col0 >> 7;
                 row.live = row.live && ok;
                 store_heads_normal(p, row, slot0, min(p.block_cols >> 7, (p.N >> 7) - slot0), taddr_row);
             } else {
@@ -921,16 +967,16 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_rows, const __
                     tmem_wait_ld();
 #pragma unroll
                     for (int q = 0; q < 4; q++) {
-                        const int n0 = col_tile * p.block_cols + c0 + q * 16;
-                        if (!ok || m >= p.M || n0 >= p.N) continue;
+                        const int n0 = col0 + c0 + q * 16;
+                        if (!ok || m >= row_end || n0 >= p.N) continue;
                         store_chunk_normal(p, m, n0, min(16, p.N - n0), reinterpret_cast<float*>(u + q * 16), u_first);
                     }
                 }
                 for (; c0 < p.block_cols; c0 += 16) {
                     float v[16];
                     tmem_ld16(taddr_row + (uint32_t)c0, v);
-                    const int n0 = col_tile * p.block_cols + c0;
-                    if (!ok || m >= p.M || n0 >= p.N) continue;
+                    const int n0 = col0 + c0;
+                    if (!ok || m >= row_end || n0 >= p.N) continue;
                     store_chunk_normal(p, m, n0, min(16, p.N - n0), v, u_first);
                 }
             }

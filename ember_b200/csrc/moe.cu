@@ -60,6 +60,63 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int E, int to
 
 // The router's product and the choice in one: logits[e] = sum_k x[t, k] w[e, k] with fp32 weights and sums.  A block
 // a token: its warps share the experts (four elements a lane and load), the first warp then chooses.
+// TB tokens a block (long steps: a weight element fetched once serves TB tokens; the first TB warps then choose).
+__device__ __forceinline__ void unpack4(const float* p, float (&f)[4]) {
+    const float4 v = *reinterpret_cast<const float4*>(p);
+    f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+}
+__device__ __forceinline__ void unpack4(const __nv_bfloat16* p, float (&f)[4]) {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    f[0] = __uint_as_float(v.x << 16); f[1] = __uint_as_float(v.x & 0xffff0000u);
+    f[2] = __uint_as_float(v.y << 16); f[3] = __uint_as_float(v.y & 0xffff0000u);
+}
+template <typename T, int TB>
+__global__ void __launch_bounds__(512) moe_router_many_kernel(const T* __restrict__ x, const float* __restrict__ w, int n_tokens, int K, int E, int top,
+                                                              int* __restrict__ sel, float* __restrict__ wgt, float* __restrict__ logits,
+                                                              RouteRule rule) {
+    __shared__ float zs[TB][MOE_MAX_EXPERTS];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t0 = blockIdx.x * TB, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+    const T* row[TB];
+#pragma unroll
+    for (int b = 0; b < TB; b++) row[b] = x + (size_t)min(t0 + b, n_tokens - 1) * K;
+    for (int e = warp; e < E; e += nw) {
+        const float* we = w + (size_t)e * K;
+        float s[TB][4] = {};                                 // the sums of the one-token kernel, in its order
+        for (int k = 4 * lane; k < K; k += 128) {
+            float wv[4];
+            unpack4(we + k, wv);
+#pragma unroll
+            for (int b = 0; b < TB; b++) {
+                float xv[4];
+                unpack4(row[b] + k, xv);
+#pragma unroll
+                for (int i = 0; i < 4; i++) s[b][i] = fmaf(xv[i], wv[i], s[b][i]);
+            }
+        }
+#pragma unroll
+        for (int b = 0; b < TB; b++) {
+            const float z = warp_sum((s[b][0] + s[b][1]) + (s[b][2] + s[b][3]));
+            if (lane == 0) {
+                zs[b][e] = z;
+                if (logits && t0 + b < n_tokens) logits[(size_t)(t0 + b) * E + e] = z;
+            }
+        }
+    }
+    __syncthreads();
+    for (int b = warp; b < TB; b += nw) {
+        if (t0 + b >= n_tokens) break;
+        float z[MOE_MAX_EXPERTS / 32];
+#pragma unroll
+        for (int i = 0; i < MOE_MAX_EXPERTS / 32; i++) {
+            const int e = lane + 32 * i;
+            z[i] = e < E ? zs[b][e] : -INFINITY;
+        }
+        choose_experts(z, E, top, sel, wgt, t0 + b, lane, rule);
+    }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(512) moe_router_kernel(const T* __restrict__ x, const float* __restrict__ w, int K, int E, int top,
                                                          int* __restrict__ sel, float* __restrict__ wgt, float* __restrict__ logits,
@@ -556,6 +613,19 @@ __global__ void moe_gather_kernel(const uint4* __restrict__ x, const int* __rest
     for (int i = threadIdx.x; i < row16; i += blockDim.x) dst[i] = src[i];
 }
 
+template <typename TO>
+__device__ __forceinline__ void store_quad(TO* dst, float a, float b, float c, float d);
+template <>
+__device__ __forceinline__ void store_quad<float>(float* dst, float a, float b, float c, float d) { *reinterpret_cast<float4*>(dst) = make_float4(a, b, c, d); }
+template <>
+__device__ __forceinline__ void store_quad<__nv_bfloat16>(__nv_bfloat16* dst, float a, float b, float c, float d) {
+    __nv_bfloat162 lo = __floats2bfloat162_rn(a, b), hi = __floats2bfloat162_rn(c, d);
+    uint2 u;
+    u.x = *reinterpret_cast<uint32_t*>(&lo);
+    u.y = *reinterpret_cast<uint32_t*>(&hi);
+    *reinterpret_cast<uint2*>(dst) = u;
+}
+
 // act[slot, j] = g sigmoid(alpha g) (u + 1), g = min(gu[slot, 2j], limit), u = clamp(gu[slot, 2j + 1], -limit, limit).
 template <typename TO>
 __global__ void moe_activation_kernel(const float2* __restrict__ gu, TO* __restrict__ act, size_t n, float limit, float alpha,
@@ -570,6 +640,26 @@ __global__ void moe_activation_kernel(const float2* __restrict__ gu, TO* __restr
     act[i] = from_float<TO>(g / (1.0f + expf(-alpha * g)) * (u + up_offset));
 }
 
+// The same, four outputs a thread (ff a multiple of four).
+template <typename TO>
+__global__ void moe_activation4_kernel(const float4* __restrict__ gu, TO* __restrict__ act, size_t n4, float limit, float alpha,
+                                       float up_offset, const float4* __restrict__ bias, int ff2) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= n4) return;
+    float o[4];
+#pragma unroll
+    for (int k = 0; k < 2; k++) {
+        float4 v = gu[2 * i + k];
+        if (bias) { const float4 b = bias[(2 * i + k) % ff2]; v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w; }
+        const float g0 = fminf(v.x, limit), u0 = fminf(fmaxf(v.y, -limit), limit), g1 = fminf(v.z, limit), u1 = fminf(fmaxf(v.w, -limit), limit);
+        o[2 * k] = g0 / (1.0f + expf(-alpha * g0)) * (u0 + up_offset);
+        o[2 * k + 1] = g1 / (1.0f + expf(-alpha * g1)) * (u1 + up_offset);
+    }
+    store_quad<TO>(act + 4 * i, o[0], o[1], o[2], o[3]);
+}
+
 // act[i] = relu(x[i])^2: the activation of an ungated expert whose product left fp32 sums.
 template <typename TO>
 __global__ void moe_square_relu_kernel(const float* __restrict__ x, TO* __restrict__ act, size_t n) {
@@ -579,6 +669,36 @@ __global__ void moe_square_relu_kernel(const float* __restrict__ x, TO* __restri
     if (i >= n) return;
     const float v = x[i];
     act[i] = from_float<TO>(v > 0.0f ? v * v : 0.0f);
+}
+
+template <typename TO>
+__global__ void moe_square_relu4_kernel(const float4* __restrict__ x, TO* __restrict__ act, size_t n4) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= n4) return;
+    const float4 v = x[i];
+    const float a = fmaxf(v.x, 0.0f), b = fmaxf(v.y, 0.0f), c = fmaxf(v.z, 0.0f), d = fmaxf(v.w, 0.0f);
+    store_quad<TO>(act + 4 * i, a * a, b * b, c * c, d * d);
+}
+
+// The weighted sum over a token's choices, four elements a thread (rows of a multiple of four elements, no identity
+// experts): out = (out +) sum over k, in order, of weight * y[slot].
+__global__ void moe_combine4_kernel(const float4* __restrict__ y, const float* __restrict__ wgt, const int* __restrict__ slot_of_pair,
+                                    int top, float4* __restrict__ out, int accumulate, int hidden4) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.y, i = blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= hidden4) return;
+    float4 s = make_float4(0.0f, 0.0f, 0.0f, 0.0f), o = s;
+    if (accumulate) o = out[(size_t)t * hidden4 + i];
+    for (int k = 0; k < top; k++) {
+        const float w = wgt[(size_t)t * top + k];
+        const float4 v = y[(size_t)slot_of_pair[(size_t)t * top + k] * hidden4 + i];
+        s.x = fmaf(w, v.x, s.x); s.y = fmaf(w, v.y, s.y); s.z = fmaf(w, v.z, s.z); s.w = fmaf(w, v.w, s.w);
+    }
+    if (accumulate) { s.x = o.x + s.x; s.y = o.y + s.y; s.z = o.z + s.z; s.w = o.w + s.w; }
+    out[(size_t)t * hidden4 + i] = s;
 }
 
 __global__ void moe_combine_kernel(const float* __restrict__ y, const float* __restrict__ wgt, const int* __restrict__ slot_of_pair,
@@ -627,6 +747,13 @@ EMBER_API int ember_moe_router(const void* x, int x_dtype, const float* w, int T
         return fail("moe_router: top %d of %d experts (at most 32 of %d), rows of %d", top, E, MOE_MAX_EXPERTS, K);
     cudaStream_t st = (cudaStream_t)stream;
     const unsigned threads = 32 * (E < 16 ? E : 16);          // a warp an expert, up to sixteen (eight experts: one round, as before)
+    if (T >= 1024 && K % 4 == 0 && ((((uintptr_t)x) | ((uintptr_t)w)) & 15) == 0 && (x_dtype == EMBER_F32 || x_dtype == EMBER_BF16)) {
+        constexpr int TB = 4;
+        const unsigned blocks = (T + TB - 1) / TB;
+        if (x_dtype == EMBER_F32) launch_kernel(moe_router_many_kernel<float, TB>, blocks, threads, 0, st, (const float*)x, w, T, K, E, top, sel, wgt, logits, rule);
+        else launch_kernel(moe_router_many_kernel<__nv_bfloat16, TB>, blocks, threads, 0, st, (const __nv_bfloat16*)x, w, T, K, E, top, sel, wgt, logits, rule);
+        return check_launch("moe_router_many");
+    }
     if (x_dtype == EMBER_F32) launch_kernel(moe_router_kernel<float>, T, threads, 0, st, (const float*)x, w, K, E, top, sel, wgt, logits, rule);
     else if (x_dtype == EMBER_BF16)
         launch_kernel(moe_router_kernel<__nv_bfloat16>, T, threads, 0, st, (const __nv_bfloat16*)x, w, K, E, top, sel, wgt, logits, rule);
@@ -726,6 +853,17 @@ EMBER_API int ember_moe_activation(const float* gu, void* act, int out_dtype, lo
     if (n <= 0) return 0;
     if (bias && ff <= 0) return fail("moe_activation: biases for rows of %d", ff);
     cudaStream_t st = (cudaStream_t)stream;
+    if (n % 4 == 0 && (!bias || ff % 4 == 0) && ((((uintptr_t)gu) | ((uintptr_t)act) | ((uintptr_t)bias)) & 15) == 0 &&
+        (out_dtype == EMBER_F32 || out_dtype == EMBER_BF16)) {
+        const unsigned blocks4 = (unsigned)((n / 4 + 255) / 256);
+        if (out_dtype == EMBER_F32)
+            launch_kernel(moe_activation4_kernel<float>, blocks4, 256, 0, st, (const float4*)gu, (float*)act, (size_t)(n / 4), limit, alpha, up_offset,
+                          (const float4*)bias, ff / 2);
+        else
+            launch_kernel(moe_activation4_kernel<__nv_bfloat16>, blocks4, 256, 0, st, (const float4*)gu, (__nv_bfloat16*)act, (size_t)(n / 4), limit, alpha,
+                          up_offset, (const float4*)bias, ff / 2);
+        return check_launch("moe_activation4");
+    }
     const unsigned blocks = (unsigned)((n + 255) / 256);
     if (out_dtype == EMBER_F32)
         launch_kernel(moe_activation_kernel<float>, blocks, 256, 0, st, (const float2*)gu, (float*)act, (size_t)n, limit, alpha, up_offset, (const float2*)bias, ff);
@@ -739,6 +877,12 @@ EMBER_API int ember_moe_activation(const float* gu, void* act, int out_dtype, lo
 EMBER_API int ember_moe_square_relu(const float* x, void* act, int out_dtype, long long n, void* stream) {
     if (n <= 0) return 0;
     cudaStream_t st = (cudaStream_t)stream;
+    if (n % 4 == 0 && ((((uintptr_t)x) | ((uintptr_t)act)) & 15) == 0 && (out_dtype == EMBER_F32 || out_dtype == EMBER_BF16)) {
+        const unsigned blocks4 = (unsigned)((n / 4 + 255) / 256);
+        if (out_dtype == EMBER_F32) launch_kernel(moe_square_relu4_kernel<float>, blocks4, 256, 0, st, (const float4*)x, (float*)act, (size_t)(n / 4));
+        else launch_kernel(moe_square_relu4_kernel<__nv_bfloat16>, blocks4, 256, 0, st, (const float4*)x, (__nv_bfloat16*)act, (size_t)(n / 4));
+        return check_launch("moe_square_relu4");
+    }
     const unsigned blocks = (unsigned)((n + 255) / 256);
     if (out_dtype == EMBER_F32) launch_kernel(moe_square_relu_kernel<float>, blocks, 256, 0, st, x, (float*)act, (size_t)n);
     else if (out_dtype == EMBER_BF16) launch_kernel(moe_square_relu_kernel<__nv_bfloat16>, blocks, 256, 0, st, x, (__nv_bfloat16*)act, (size_t)n);
@@ -750,6 +894,12 @@ EMBER_API int ember_moe_combine(const float* y, const float* wgt, const int* slo
                                 int hidden, const int* sel, int experts, const void* same, int same_dtype, void* stream) {
     if (T <= 0) return 0;
     if (sel && (!same || (same_dtype != EMBER_F32 && same_dtype != EMBER_BF16))) return fail("moe_combine: identity experts need the tokens' input rows");
+    if (!sel && hidden % 4 == 0 && ((((uintptr_t)y) | ((uintptr_t)out)) & 15) == 0 && T <= 65535) {
+        const int hidden4 = hidden / 4, threads = hidden4 >= 256 ? 256 : 128;
+        launch_kernel(moe_combine4_kernel, dim3((hidden4 + threads - 1) / threads, T), threads, 0, (cudaStream_t)stream, (const float4*)y, wgt,
+                      slot_of_pair, top, (float4*)out, accumulate, hidden4);
+        return check_launch("moe_combine4");
+    }
     launch_kernel(moe_combine_kernel, T, 256, 0, (cudaStream_t)stream, y, wgt, slot_of_pair, top, out, accumulate, hidden, sel, experts,
                   (const float*)(sel && same_dtype == EMBER_F32 ? same : nullptr),
                   (const __nv_bfloat16*)(sel && same_dtype == EMBER_BF16 ? same : nullptr));

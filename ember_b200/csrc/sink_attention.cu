@@ -106,9 +106,26 @@ struct HeadPrepareArgs {
     int* err;
 };
 
+// Four neighbouring elements in one store (16 bytes of floats, 8 of bfloat16).
 template <typename T>
+__device__ __forceinline__ void put4(T* dst, const float4& v);
+template <>
+__device__ __forceinline__ void put4<float>(float* dst, const float4& v) { *reinterpret_cast<float4*>(dst) = v; }
+template <>
+__device__ __forceinline__ void put4<__nv_bfloat16>(__nv_bfloat16* dst, const float4& v) {
+    __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    uint2 u;
+    u.x = *reinterpret_cast<uint32_t*>(&lo);
+    u.y = *reinterpret_cast<uint32_t*>(&hi);
+    *reinterpret_cast<uint2*>(dst) = u;
+}
+
+// A token's cosines and sines are made once, in shared memory, for all its heads.  W 4: sizes, half of the rotated part and
+// the rows are multiples of four elements, and a thread takes four neighbours at a time; W 1: any sizes.  Without a norm over
+// whole projections a token's heads may be shared out to gridDim.y blocks (a step of few tokens).
+template <typename T, int W>
 __global__ void __launch_bounds__(256) head_prepare_store_kernel(HeadPrepareArgs p) {
-    extern __shared__ float factor[];          // per-head norm factors: H for the queries, then G for the keys
+    extern __shared__ __align__(16) float factor[];          // cosines and sines [half] each, then per-head norm factors
     __shared__ float scratch[32];
     pdl_launch_dependents();
     pdl_wait();
@@ -117,78 +134,111 @@ __global__ void __launch_bounds__(256) head_prepare_store_kernel(HeadPrepareArgs
     const float* row = p.qkv + (size_t)t * p.ld;
     const float* b = p.bias;
     const bool kv = p.write_kv != 0;
+    const int half = p.rotary / 2, pos = p.positions[t];
+    float* cs = factor;
+    float* sn = factor + half;
+    float* hf = factor + 2 * half;
     auto val = [&](int i) { return row[i] + (b ? b[i] : 0.0f); };
+    auto val4 = [&](int i) {
+        float4 v = *reinterpret_cast<const float4*>(row + i);
+        if (b) { v.x += b[i]; v.y += b[i + 1]; v.z += b[i + 2]; v.w += b[i + 3]; }
+        return v;
+    };
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        float s, c;
+        sincosf((float)pos * p.inv_freq[i], &s, &c);
+        cs[i] = c * p.magnitude;
+        sn[i] = s * p.magnitude;
+    }
+    auto squares = [&](int from, int n, int first, int step) {
+        float ss = 0.0f;
+        if (W == 4) {
+            for (int i = 4 * first; i < n; i += 4 * step) {
+                const float4 v = val4(from + i);
+                ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+            }
+        } else {
+            for (int i = first; i < n; i += step) { const float v = val(from + i); ss = fmaf(v, v, ss); }
+        }
+        return ss;
+    };
     float rq = 1.0f, rk = 1.0f;
     if (p.norm_mode == 1) {
-        float ss = 0.0f;
-        for (int i = threadIdx.x; i < QN; i += blockDim.x) { const float v = val(i); ss = fmaf(v, v, ss); }
-        rq = 1.0f / sqrtf(block_sum(ss, scratch) / (float)QN + p.eps);
-        if (kv) {
-            ss = 0.0f;
-            for (int i = threadIdx.x; i < KN; i += blockDim.x) { const float v = val(QN + i); ss = fmaf(v, v, ss); }
-            rk = 1.0f / sqrtf(block_sum(ss, scratch) / (float)KN + p.eps);
-        }
+        rq = 1.0f / sqrtf(block_sum(squares(0, QN, threadIdx.x, blockDim.x), scratch) / (float)QN + p.eps);
+        if (kv) rk = 1.0f / sqrtf(block_sum(squares(QN, KN, threadIdx.x, blockDim.x), scratch) / (float)KN + p.eps);
     } else if (p.norm_mode == 2) {
         const int heads = p.H + (kv ? p.G : 0);
         for (int h = warp; h < heads; h += nw) {
-            float ss = 0.0f;
-            for (int d = lane; d < D; d += 32) { const float v = val(h * D + d); ss = fmaf(v, v, ss); }
-            ss = warp_sum(ss);
-            if (lane == 0) factor[h] = 1.0f / sqrtf(ss / (float)D + p.eps);
+            const float ss = warp_sum(squares(h * D, D, lane, 32));
+            if (lane == 0) hf[h] = 1.0f / sqrtf(ss / (float)D + p.eps);
         }
-        __syncthreads();
     }
-    const int pos = p.positions[t];
-    const int half = p.rotary / 2;
-    // element i of [q | k] (i < QN: a query element), normed and weighed
-    auto normed = [&](int i) {
-        const bool isq = i < QN;
-        const int j = isq ? i : i - QN;
-        float v = val(i);
-        if (p.norm_mode == 1) v *= (isq ? rq : rk) * (isq ? p.q_w[j] : p.k_w[j]);
-        else if (p.norm_mode == 2) v *= factor[i / D] * (isq ? p.q_w[j % D] : p.k_w[j % D]);
-        return v;
-    };
-    // element i of [q | k] after the rotation, handed to write(index, value); a rotated pair (i, i + half) is made by the
-    // thread that holds its first element, from one sine and one cosine
-    auto emit = [&](int i, float mul, auto&& write) {
-        const int d = i % D;
-        if (d >= half && d < p.rotary) return;
-        const float v = normed(i);
-        if (d < half) {
-            const float other = normed(i + half);
-            float sn, cs;
-            sincosf((float)pos * p.inv_freq[d], &sn, &cs);
-            cs *= p.magnitude;
-            sn *= p.magnitude;
-            write(i, (v * cs - other * sn) * mul);
-            write(i + half, (other * cs + v * sn) * mul);
-        } else {
-            write(i, v * mul);
-        }
-    };
+    __syncthreads();
     float temp = 1.0f;
     if (p.qt_every > 0) temp = 1.0f + p.qt_coef * logf((float)((pos + 1) / p.qt_every) + 1.0f);
     T* qo = (T*)p.q_out + (size_t)t * QN;
-    for (int i = threadIdx.x; i < QN; i += blockDim.x) emit(i, temp, [&](int j, float v) { qo[j] = from_float<T>(v); });
-    if (!kv) return;
-    const int seq = p.seq_of[t];
-    const int blk = p.block_table[(size_t)seq * p.max_blocks + pos / p.page];
-    if (blk < 0 || blk >= p.num_pages) {
-        if (threadIdx.x == 0 && p.err) atomicOr(p.err, EMBER_ERR_PAGE_RANGE);
-        return;
+    T* kp = nullptr;
+    T* vp = nullptr;
+    if (kv) {
+        const int blk = p.block_table[(size_t)p.seq_of[t] * p.max_blocks + pos / p.page];
+        if (blk < 0 || blk >= p.num_pages) {
+            if (threadIdx.x == 0 && p.err) atomicOr(p.err, EMBER_ERR_PAGE_RANGE);
+        } else {
+            const size_t first = (size_t)blk * p.G * p.page + pos % p.page;      // row of key head 0; heads are `page` rows apart
+            kp = (T*)p.k_pool + first * D;
+            vp = (T*)p.v_pool + first * p.DV;
+        }
     }
-    const int in_page = pos % p.page;
-    T* kp = (T*)p.k_pool;
-    T* vp = (T*)p.v_pool;
-    for (int i = threadIdx.x; i < KN; i += blockDim.x)
-        emit(QN + i, 1.0f, [&](int j, float v) {
-            const int g = (j - QN) / D, d = (j - QN) - g * D;
-            kp[(((size_t)blk * p.G + g) * p.page + in_page) * D + d] = from_float<T>(v);
-        });
-    for (int i = threadIdx.x; i < VN; i += blockDim.x) {
-        const int g = i / p.DV, d = i - g * p.DV;
-        vp[(((size_t)blk * p.G + g) * p.page + in_page) * p.DV + d] = from_float<T>(val(QN + KN + i));
+    // slots: the query heads, then the key heads, then the value heads; a thread's group is W elements of one head
+    const int dq = D / W, dv = p.DV / W, n_qk = (p.H + (kp ? p.G : 0)) * dq, n = n_qk + (vp ? p.G * dv : 0);
+    const int part = blockIdx.y * blockDim.x + threadIdx.x, stride = gridDim.y * blockDim.x;
+    for (int i = part; i < n; i += stride) {
+        if (i >= n_qk) {                                     // values pass as they are
+            const int g = (i - n_qk) / dv, d = ((i - n_qk) - g * dv) * W, at = QN + KN + g * p.DV + d;
+            T* dst = vp + (size_t)g * p.page * p.DV + d;
+            if (W == 4) put4<T>(dst, val4(at));
+            else *dst = from_float<T>(val(at));
+            continue;
+        }
+        const int h = i / dq, d = (i - h * dq) * W;
+        if (d >= half && d < p.rotary) continue;             // the thread with the pair's first element makes both
+        const bool isq = h < p.H;
+        T* dst = isq ? qo + h * D + d : kp + (size_t)(h - p.H) * p.page * D + d;
+        const float mul = isq ? temp : 1.0f;
+        float norm = 1.0f;
+        const float* w = nullptr;                            // the norm's weights of this head
+        if (p.norm_mode == 1) { norm = isq ? rq : rk; w = isq ? p.q_w + h * D : p.k_w + (h - p.H) * D; }
+        else if (p.norm_mode == 2) { norm = hf[h]; w = isq ? p.q_w : p.k_w; }
+        const int at = (isq ? h * D : QN + (h - p.H) * D) + d;
+        if (W == 4) {
+            auto normed = [&](int off) {
+                float4 v = val4(at + off);
+                if (w) {
+                    const float4 g = *reinterpret_cast<const float4*>(w + d + off);
+                    v.x *= norm * g.x; v.y *= norm * g.y; v.z *= norm * g.z; v.w *= norm * g.w;
+                }
+                return v;
+            };
+            const float4 v = normed(0);
+            if (d < half) {
+                const float4 o = normed(half), c = *reinterpret_cast<const float4*>(cs + d), s = *reinterpret_cast<const float4*>(sn + d);
+                put4<T>(dst, make_float4((v.x * c.x - o.x * s.x) * mul, (v.y * c.y - o.y * s.y) * mul, (v.z * c.z - o.z * s.z) * mul,
+                                         (v.w * c.w - o.w * s.w) * mul));
+                put4<T>(dst + half, make_float4((o.x * c.x + v.x * s.x) * mul, (o.y * c.y + v.y * s.y) * mul, (o.z * c.z + v.z * s.z) * mul,
+                                                (o.w * c.w + v.w * s.w) * mul));
+            } else {
+                put4<T>(dst, make_float4(v.x * mul, v.y * mul, v.z * mul, v.w * mul));
+            }
+        } else {
+            const float v = val(at) * (w ? norm * w[d] : 1.0f);
+            if (d < half) {
+                const float o = val(at + half) * (w ? norm * w[d + half] : 1.0f);
+                dst[0] = from_float<T>((v * cs[d] - o * sn[d]) * mul);
+                dst[half] = from_float<T>((o * cs[d] + v * sn[d]) * mul);
+            } else {
+                dst[0] = from_float<T>(v * mul);
+            }
+        }
     }
 }
 
@@ -1070,12 +1120,27 @@ EMBER_API int ember_head_prepare_store(const float* qkv, int ld, const float* bi
     if (qt_every < 0 || page <= 0 || max_blocks <= 0 || num_pages <= 0) return fail("head_prepare_store: bad geometry");
     HeadPrepareArgs p{qkv, ld, bias, norm_mode, q_w, k_w, eps, inv_freq, rotary, magnitude, qt_coef, qt_every, H, G, D, DV, positions, seq_of,
                       block_table, max_blocks, page, num_pages, q_out, k_pool, v_pool, write_kv, err};
-    const size_t smem = (size_t)(H + G) * sizeof(float);
-    if (smem > 40 * 1024) return fail("head_prepare_store: %d heads are too many", H + G);
+    const size_t smem = (size_t)(H + G + rotary) * sizeof(float);
+    if (smem > 40 * 1024) return fail("head_prepare_store: %d heads and %d rotated elements are too many", H + G, rotary);
     cudaStream_t st = (cudaStream_t)stream;
-    if (dtype == EMBER_F32) launch_kernel(head_prepare_store_kernel<float>, T_tokens, 256, smem, st, p);
-    else if (dtype == EMBER_BF16) launch_kernel(head_prepare_store_kernel<__nv_bfloat16>, T_tokens, 256, smem, st, p);
-    else return fail("head_prepare_store: unsupported dtype %d", dtype);
+    const uintptr_t bases = (uintptr_t)qkv | (uintptr_t)q_w | (uintptr_t)k_w | (uintptr_t)q_out | (uintptr_t)k_pool | (uintptr_t)v_pool;
+    const bool by4 = D % 4 == 0 && DV % 4 == 0 && rotary % 8 == 0 && ld % 4 == 0 && (bases & 15) == 0;
+    // few tokens: a token's heads are shared out so that about two blocks an SM have work
+    int parts = 1;
+    if (norm_mode != 1) {
+        const int groups = (H * D + G * (D + DV)) / (by4 ? 4 : 1);
+        while (parts < 8 && T_tokens * parts * 2 <= 296 && groups / (parts * 2) >= 256) parts *= 2;
+    }
+    const dim3 grid(T_tokens, parts);
+    if (dtype == EMBER_F32) {
+        if (by4) launch_kernel(head_prepare_store_kernel<float, 4>, grid, 256, smem, st, p);
+        else launch_kernel(head_prepare_store_kernel<float, 1>, grid, 256, smem, st, p);
+    } else if (dtype == EMBER_BF16) {
+        if (by4) launch_kernel(head_prepare_store_kernel<__nv_bfloat16, 4>, grid, 256, smem, st, p);
+        else launch_kernel(head_prepare_store_kernel<__nv_bfloat16, 1>, grid, 256, smem, st, p);
+    } else {
+        return fail("head_prepare_store: unsupported dtype %d", dtype);
+    }
     return check_launch("head_prepare_store");
 }
 

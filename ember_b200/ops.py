@@ -448,6 +448,27 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, M: int, epilogu
           c_void_p(stream if stream is not None else current_stream_ptr()))
 
 
+def gemm_tc_grouped(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, M: int, offsets: torch.Tensor, epilogue: int = EPI_STORE,
+                    err: Optional[torch.Tensor] = None, stream: Optional[int] = None) -> None:
+    """out[offsets[g] : offsets[g + 1]] = a[offsets[g] : offsets[g + 1]] @ w[g].T for every g, in one launch: ``w`` bfloat16
+    [groups, N, K], ``offsets`` int32 on the device (ascending from 0; rows from offsets[groups] on are not touched), ``M``
+    how many rows ``a`` has at most.  Storing and gated epilogues."""
+    _check(a, "a", torch.bfloat16)
+    _check(w, "w", torch.bfloat16)
+    _check(out, "out")
+    _check(offsets, "offsets", torch.int32)
+    if w.dim() != 3 or epilogue not in (EPI_STORE, EPI_STORE_F32) + GATED_EPILOGUES:
+        raise KernelError(f"gemm_tc_grouped: weights {tuple(w.shape)}, epilogue {epilogue}")
+    G, N, K = w.shape
+    n_out = N // 2 if epilogue in GATED_EPILOGUES else N
+    want = torch.float32 if epilogue == EPI_STORE_F32 else torch.bfloat16
+    if out.dtype != want or out.shape[-1] != n_out or out.numel() < M * n_out or a.shape[-1] != K or a.numel() < M * K or offsets.numel() < G + 1:
+        raise KernelError(f"gemm_tc_grouped: input {tuple(a.shape)}, weights {tuple(w.shape)}, output {tuple(out.shape)} {out.dtype}, M={M}")
+    lib = _lib("gemm_tc")
+    _call(lib, lib.ember_gemm_tc_grouped, _p(a), _p(w), _p(out), c_int(n_out), c_int(M), c_int(N), c_int(K), c_int(G), _p(offsets),
+          c_int(epilogue), c_int(_sms(a.device)), _p(err), c_void_p(stream if stream is not None else current_stream_ptr()))
+
+
 def gemm_tc_qkv_usable(x: torch.Tensor, w: torch.Tensor, bias, M: int, n_heads: int, n_kv: int, head_dim: int,
                        rotary: int) -> bool:
     """Whether the fused projection takes this step: bf16, no bias, heads of 128 rotated whole (or not at all),

@@ -142,10 +142,11 @@ class RoutedMLP(FeedForward):
     are read once per step however the tokens fall, and nothing comes back to the host (decode steps are captured
     into CUDA graphs like any other).
 
-    A bfloat16 step of more tokens than any captured step has (a prompt portion) takes the tensor cores instead: the
-    tokens' rows are gathered expert by expert, the host reads the experts' row counts (the step's one look at the
-    device) and every expert with rows runs the tcgen05 product on its slice, first gate/up into fp32, an element-wise
-    kernel for the clamped activation, then down; the weighted sum over a token's choices is the same kernel either way.
+    A bfloat16 step of a prompt portion's size takes the tensor cores instead: the tokens' rows are gathered expert by
+    expert, and one launch of the grouped tcgen05 product walks all experts' tiles (the experts' row ranges stay on the
+    device).  Where the activation is plain silu(gate) up it is that product's epilogue; a clamped one is an element-wise
+    kernel on fp32 sums.  A second grouped product is the way down; the weighted sum over a token's choices is the same
+    kernel either way.
     Tensors under the prefix: router, correction (if any), e<i>.gate, e<i>.up, e<i>.down.
 
     Scoring "softmax": s = softmax over all router outputs, otherwise as "sigmoid".  ``groups``: the outputs form equal
@@ -157,7 +158,7 @@ class RoutedMLP(FeedForward):
 
     graph_safe = True
     can_store = True
-    TC_MIN_TOKENS = 257          # more runs than a captured decode step can have: such a step is never inside a graph
+    TC_MIN_TOKENS = 257          # smaller steps stream the weights
     STREAM_MAX_TOKENS = 256      # up to here the products stream the weights past the few rows of a tile
 
     def __init__(self, spec, prefix: str = ""):
@@ -186,6 +187,7 @@ class RoutedMLP(FeedForward):
                               f"which {s.keep_groups} are kept for top {s.top}")
         self.gated = s.expert == "gated"
         self.limit = float(s.limit) if s.limit > 0 else float("inf")
+        self.plain_silu = self.gated and s.limit == 0 and s.alpha == 1.0 and s.up_offset == 0.0     # silu(gate) * up
 
     def weight_decls(self) -> List[WeightDecl]:
         s, p = self.spec, self.prefix
@@ -255,21 +257,17 @@ class RoutedMLP(FeedForward):
                                   ops.MOE_STREAM_ROWS if streaming else ops.MOE_TILE_ROWS, stream=ctx.stream, tiled=s.experts)
         if self._on_tensor_cores(ctx, x):
             xs = ctx.buf("routed_mlp.gathered", (mt * top, s.hidden_size), rt.dtype)
-            gu = ctx.buf("routed_mlp.gate_up", (mt * top, self.gate_up.shape[1]), torch.float32)
             ops.moe_gather(x, pair_of_slot, pairs, top, xs, stream=ctx.stream)
-            bounds = offsets.tolist()                      # the experts' row ranges: the host waits for the grouping here
-            for e in range(s.experts):
-                lo, n = bounds[e], bounds[e + 1] - bounds[e]
-                if n > 0:
-                    ops.gemm_tc(xs[lo:lo + n], self.gate_up[e], gu[lo:lo + n], n, ops.EPI_STORE_F32, err=ctx.err, stream=ctx.stream)
-            if self.gated:
-                ops.moe_activation(gu, act, pairs, self.limit, s.alpha, stream=ctx.stream, up_offset=s.up_offset)
+            if self.plain_silu:
+                ops.gemm_tc_grouped(xs, self.gate_up, act, pairs, offsets, ops.EPI_SILU_MUL, err=ctx.err, stream=ctx.stream)
             else:
-                ops.moe_square_relu(gu, act, pairs * s.intermediate_size, stream=ctx.stream)
-            for e in range(s.experts):
-                lo, n = bounds[e], bounds[e + 1] - bounds[e]
-                if n > 0:
-                    ops.gemm_tc(act[lo:lo + n], self.down[e], y[lo:lo + n], n, ops.EPI_STORE_F32, err=ctx.err, stream=ctx.stream)
+                gu = ctx.buf("routed_mlp.gate_up", (mt * top, self.gate_up.shape[1]), torch.float32)
+                ops.gemm_tc_grouped(xs, self.gate_up, gu, pairs, offsets, ops.EPI_STORE_F32, err=ctx.err, stream=ctx.stream)
+                if self.gated:
+                    ops.moe_activation(gu, act, pairs, self.limit, s.alpha, stream=ctx.stream, up_offset=s.up_offset)
+                else:
+                    ops.moe_square_relu(gu, act, pairs * s.intermediate_size, stream=ctx.stream)
+            ops.gemm_tc_grouped(act, self.down, y, pairs, offsets, ops.EPI_STORE_F32, err=ctx.err, stream=ctx.stream)
         else:
             ops.moe_gemm(x, self.gate_up, act, offsets, pair_of_slot, tiles, max_tiles, top, self.gated, self.limit, s.alpha,
                          stream=ctx.stream, streaming=streaming, up_offset=s.up_offset, square_relu=not self.gated)

@@ -549,3 +549,46 @@ def test_experts_of_prompt_portions_on_tensor_cores(dtype, tmp_path):
     steps = trace_portions(requests, sizes=(300, 2, 118))
     outputs, _ = replay(d, dtype, steps, 448, max_batch_tokens=512)
     assert_close(collect(steps, outputs), want, dtype, "experts on tensor cores")
+
+
+@pytest.mark.parametrize("N,K", [(96, 64), (512, 200), (1000, 1024), (2048, 512)])
+@pytest.mark.parametrize("counts", [(0, 1, 127, 128, 129, 0), (300,), (5, 700, 0, 0, 33, 256, 2, 64), tuple([3] * 200)])
+def test_grouped_products_in_one_launch(N, K, counts):
+    """Rows in groups against weights of their own: empty groups, groups of one row, of a tile exactly and of a row more, two
+    hundred groups; rows behind the last group stay as they are.  Stored in fp32 and bfloat16, and silu(gate) up."""
+    from ember_b200 import ops
+    g = torch.Generator().manual_seed(N + len(counts))
+    G, M = len(counts), sum(counts) + 7
+    a = torch.randn(M, K, generator=g).bfloat16().cuda()
+    w = (K ** -0.5 * torch.randn(G, N, K, generator=g)).bfloat16().cuda()
+    bounds = [0]
+    for c in counts:
+        bounds.append(bounds[-1] + c)
+    offsets = torch.tensor(bounds, dtype=torch.int32, device="cuda")
+    err = torch.zeros(1, dtype=torch.int32, device="cuda")
+    z = torch.cat([a[bounds[i]:bounds[i + 1]].double() @ w[i].double().T for i in range(G)])
+    for epi, want, dt, tol in ((ops.EPI_STORE_F32, z, torch.float32, 1e-5), (ops.EPI_STORE, z, torch.bfloat16, 5e-3),
+                               (ops.EPI_SILU_MUL, torch.nn.functional.silu(z[:, 0::2]) * z[:, 1::2], torch.bfloat16, 5e-3)):
+        out = torch.full((M, want.shape[1]), 7.0, dtype=dt, device="cuda")
+        ops.gemm_tc_grouped(a, w, out, M, offsets, epi, err=err)
+        assert _rel(out[:bounds[-1]].cpu(), want.cpu()) < tol, epi
+        assert float((out[bounds[-1]:].float() - 7.0).abs().max()) == 0.0
+    assert int(err.item()) == 0
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_the_router_of_long_steps_is_the_router_of_short_ones(dtype):
+    """From 1,024 tokens on a block routes four tokens: the same choices and weights, bit by bit, as in steps of 500."""
+    from ember_b200 import ops
+    T, E, K, top = 1303, 24, 132, 3
+    g = torch.Generator().manual_seed(4)
+    x, w = torch.randn(T, K, generator=g).to(dtype).cuda(), torch.randn(E, K, generator=g).cuda()
+    rule = (None, 1.0, True, "sigmoid", 6, 2, "top2", 1e-20)
+    outs = []
+    for pieces in ((T,), (500, 500, T - 1000)):
+        sel, wgt, at = torch.zeros(T * top, dtype=torch.int32, device="cuda"), torch.zeros(T * top, device="cuda"), 0
+        for n in pieces:
+            ops.moe_router(x[at:at + n].contiguous(), w, n, top, sel[at * top:], wgt[at * top:], rule=rule)
+            at += n
+        outs.append((sel.cpu(), wgt.cpu()))
+    assert torch.equal(outs[0][0], outs[1][0]) and torch.equal(outs[0][1], outs[1][1])
