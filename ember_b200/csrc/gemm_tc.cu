@@ -60,12 +60,16 @@ static bool tensor_map(const void* ptr, int rows, int K, int box_rows, CUtensorM
     return true;
 }
 
+// Whether a product's sums get a bias or an activation before they are stored (an instance of the kernels of its own).
+static bool finishes(const GemmTcParams& p) { return p.bias != nullptr || p.act == 3; }
+
 // How many pairs of blocks of the pair kernel the device runs at once (0: it cannot).
 static int pair_capacity(int num_sms) {
     static int max_pairs = -1;
     if (max_pairs < 0) {
         int n = 0;
-        if (cudaFuncSetAttribute(gemm_tc_pair_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) == cudaSuccess) {
+        if (cudaFuncSetAttribute(gemm_tc_pair_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) == cudaSuccess &&
+            cudaFuncSetAttribute(gemm_tc_pair_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) == cudaSuccess) {
             cudaLaunchConfig_t q = {};
             q.gridDim = dim3(2 * (num_sms / 2));
             q.blockDim = dim3(GEMM_THREADS);
@@ -74,7 +78,7 @@ static int pair_capacity(int num_sms) {
             a[0].id = cudaLaunchAttributeClusterDimension;
             a[0].val.clusterDim.x = 2; a[0].val.clusterDim.y = 1; a[0].val.clusterDim.z = 1;
             q.attrs = a; q.numAttrs = 1;
-            if (cudaOccupancyMaxActiveClusters(&n, gemm_tc_pair_kernel, &q) != cudaSuccess) { cudaGetLastError(); n = 0; }
+            if (cudaOccupancyMaxActiveClusters(&n, gemm_tc_pair_kernel<false>, &q) != cudaSuccess) { cudaGetLastError(); n = 0; }
         } else {
             cudaGetLastError();
         }
@@ -163,7 +167,8 @@ static int launch_pair(const void* A, const void* W, GemmTcParams p, int block_c
     attrs[1].id = cudaLaunchAttributeClusterDimension;
     attrs[1].val.clusterDim.x = 2; attrs[1].val.clusterDim.y = 1; attrs[1].val.clusterDim.z = 1;
     cfg.attrs = attrs; cfg.numAttrs = 2;
-    cudaLaunchKernelEx(&cfg, gemm_tc_pair_kernel, map_rows, map_cols, p);
+    if (finishes(p)) cudaLaunchKernelEx(&cfg, gemm_tc_pair_kernel<true>, map_rows, map_cols, p);
+    else cudaLaunchKernelEx(&cfg, gemm_tc_pair_kernel<false>, map_rows, map_cols, p);
     return check_launch("gemm_tc_pair");
 }
 
@@ -203,12 +208,14 @@ static int launch_persistent(const void* A, const void* W, GemmTcParams p, int b
         return fail("gemm_tc: cuTensorMapEncodeTiled failed or is unavailable");
     static bool pattr = false;
     if (!pattr) {
-        cudaError_t e = cudaFuncSetAttribute(gemm_tc_persistent_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+        cudaError_t e = cudaFuncSetAttribute(gemm_tc_persistent_kernel<false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(gemm_tc_persistent_kernel<false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
         if (e != cudaSuccess) return fail("gemm_tc: cannot raise the shared-memory limit: %s", cudaGetErrorString(e));
         pattr = true;
     }
     const int blocks = units < num_sms ? units : num_sms;
-    launch_kernel(gemm_tc_persistent_kernel<false>, dim3(blocks), dim3(GEMM_THREADS), smem, st, map_rows, map_cols, p);
+    if (finishes(p)) launch_kernel(gemm_tc_persistent_kernel<false, true>, dim3(blocks), dim3(GEMM_THREADS), smem, st, map_rows, map_cols, p);
+    else launch_kernel(gemm_tc_persistent_kernel<false, false>, dim3(blocks), dim3(GEMM_THREADS), smem, st, map_rows, map_cols, p);
     return check_launch("gemm_tc_persistent");
 }
 
@@ -242,11 +249,11 @@ static int launch_grouped(const void* A, const void* W, GemmTcParams p, int num_
         return fail("gemm_tc_grouped: cuTensorMapEncodeTiled failed or is unavailable");
     static bool ready = false;
     if (!ready) {
-        cudaError_t e = cudaFuncSetAttribute(gemm_tc_persistent_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+        cudaError_t e = cudaFuncSetAttribute(gemm_tc_persistent_kernel<true, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
         if (e != cudaSuccess) return fail("gemm_tc_grouped: cannot raise the shared-memory limit: %s", cudaGetErrorString(e));
         ready = true;
     }
-    launch_kernel(gemm_tc_persistent_kernel<true>, dim3(num_sms), dim3(GEMM_THREADS), smem, st, map_rows, map_cols, p);
+    launch_kernel(gemm_tc_persistent_kernel<true, false>, dim3(num_sms), dim3(GEMM_THREADS), smem, st, map_rows, map_cols, p);
     return check_launch("gemm_tc_grouped");
 }
 
@@ -441,9 +448,11 @@ EMBER_API int ember_gemm_tc(const void* A, const void* W, void* out, int ldc, in
 
     static bool attr_set = false;
     if (!attr_set) {
-        cudaError_t e = cudaFuncSetAttribute(gemm_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+        cudaError_t e = cudaFuncSetAttribute(gemm_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(gemm_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
         if (e != cudaSuccess) return fail("gemm_tc: cannot raise the shared-memory limit: %s", cudaGetErrorString(e));
-        cudaFuncSetAttribute(gemm_tc_kernel, cudaFuncAttributePreferredSharedMemoryCarveout, (int)cudaSharedmemCarveoutMaxShared);
+        cudaFuncSetAttribute(gemm_tc_kernel<false>, cudaFuncAttributePreferredSharedMemoryCarveout, (int)cudaSharedmemCarveoutMaxShared);
+        cudaFuncSetAttribute(gemm_tc_kernel<true>, cudaFuncAttributePreferredSharedMemoryCarveout, (int)cudaSharedmemCarveoutMaxShared);
         attr_set = true;
     }
     dim3 grid(row_tiles, col_tiles, splits);
@@ -464,7 +473,8 @@ EMBER_API int ember_gemm_tc(const void* A, const void* W, void* out, int ldc, in
         cfg.numAttrs = 2;
     }
     cfg.attrs = attrs;
-    cudaLaunchKernelEx(&cfg, gemm_tc_kernel, map_rows, map_cols, p);
+    if (finishes(p)) cudaLaunchKernelEx(&cfg, gemm_tc_kernel<true>, map_rows, map_cols, p);
+    else cudaLaunchKernelEx(&cfg, gemm_tc_kernel<false>, map_rows, map_cols, p);
     int rc = check_launch("gemm_tc");
     if (rc) return rc;
     if (splits > 1 && p.cluster_splits <= 1 && epilogue != 2 && !sums) {
@@ -526,9 +536,11 @@ static int launch_heads_swapped(const void* A, const void* W, GemmTcParams p, in
         return fail("gemm_tc: cuTensorMapEncodeTiled failed or is unavailable");
     static bool attr_set = false;
     if (!attr_set) {
-        cudaError_t e = cudaFuncSetAttribute(gemm_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+        cudaError_t e = cudaFuncSetAttribute(gemm_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(gemm_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
         if (e != cudaSuccess) return fail("gemm_tc: cannot raise the shared-memory limit: %s", cudaGetErrorString(e));
-        cudaFuncSetAttribute(gemm_tc_kernel, cudaFuncAttributePreferredSharedMemoryCarveout, (int)cudaSharedmemCarveoutMaxShared);
+        cudaFuncSetAttribute(gemm_tc_kernel<false>, cudaFuncAttributePreferredSharedMemoryCarveout, (int)cudaSharedmemCarveoutMaxShared);
+        cudaFuncSetAttribute(gemm_tc_kernel<true>, cudaFuncAttributePreferredSharedMemoryCarveout, (int)cudaSharedmemCarveoutMaxShared);
         attr_set = true;
     }
     cudaLaunchConfig_t cfg = {};
@@ -545,7 +557,7 @@ static int launch_heads_swapped(const void* A, const void* W, GemmTcParams p, in
     attrs[1].val.clusterDim.z = (unsigned)splits;
     cfg.attrs = attrs;
     cfg.numAttrs = 2;
-    cudaLaunchKernelEx(&cfg, gemm_tc_kernel, map_rows, map_cols, p);
+    cudaLaunchKernelEx(&cfg, gemm_tc_kernel<false>, map_rows, map_cols, p);
     return check_launch("gemm_tc_heads");
 }
 

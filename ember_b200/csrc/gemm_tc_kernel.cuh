@@ -152,7 +152,10 @@ __device__ __forceinline__ float gate_mul(float g, float u, int act) {
 
 __device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f)); }
 // A complete sum of output column n as the plain epilogues (0, 1, 2) want it: with its bias, through its activation.
+// FIN false: the kernels' instances for products without either, which pay nothing for them.
+template <bool FIN>
 __device__ __forceinline__ float finish_sum(const GemmTcParams& p, int n, float v) {
+    if (!FIN) return v;
     if (p.bias) v += __ldg(p.bias + n);
     return p.act == 3 ? gelu_erf(v) : v;
 }
@@ -161,13 +164,12 @@ __device__ __forceinline__ float finish_sum(const GemmTcParams& p, int n, float 
 // store bf16 / store fp32 / add into the fp32 residual / silu(gate) * up.
 __device__ __forceinline__ void store_finished_chunk(const GemmTcParams& p, int m, int n0, int nv, const float* v);
 // ``first``: these are the sums of the first part of K (the one that brings the bias).
+template <bool FIN>
 __device__ __forceinline__ void store_chunk_normal(const GemmTcParams& p, int m, int n0, int nv, float* v, bool first) {
-    if ((p.bias && first) || p.act == 3) {
-        if (p.epilogue != 3) {
+    if (FIN && ((p.bias && first) || p.act == 3)) {
 #pragma unroll
-            for (int j = 0; j < 16; j++)
-                if (j < nv) v[j] = finish_sum(p, n0 + j, v[j]);
-        }
+        for (int j = 0; j < 16; j++)
+            if (j < nv) v[j] = finish_sum<true>(p, n0 + j, v[j]);
     }
     store_finished_chunk(p, m, n0, nv, v);
 }
@@ -481,6 +483,7 @@ __device__ __forceinline__ void finish_heads_swapped(const GemmTcParams& p, cons
 }
 
 // ------------------------------------------------------------------------------------ kernel
+template <bool FIN>
 __global__ void __launch_bounds__(GEMM_THREADS, 1)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_constant__ CUtensorMap map_cols,
                const GemmTcParams p) {
@@ -663,9 +666,9 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_consta
                         const float other = __shfl_xor_sync(0xffffffffu, x, 1);             // gate rows are even, up rows odd
                         if ((lane & 1) == 0) reinterpret_cast<__nv_bfloat16*>(row)[r >> 1] = __float2bfloat16_rn(gate_mul(x, other, p.act));
                     } else if (p.epilogue == 0) {
-                        reinterpret_cast<__nv_bfloat16*>(row)[r] = __float2bfloat16_rn(finish_sum(p, row_tile * TILE_ROWS + r, x));
+                        reinterpret_cast<__nv_bfloat16*>(row)[r] = __float2bfloat16_rn(finish_sum<FIN>(p, row_tile * TILE_ROWS + r, x));
                     } else {
-                        reinterpret_cast<float*>(row)[r] = finish_sum(p, row_tile * TILE_ROWS + r, x);
+                        reinterpret_cast<float*>(row)[r] = finish_sum<FIN>(p, row_tile * TILE_ROWS + r, x);
                     }
                 };
                 // (64 columns a round trip to tensor memory, as the prefill epilogues read, gained nothing here)
@@ -698,7 +701,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_consta
                         float* dst = p.accum + (size_t)m * p.accum_ld + n0;
                         for (int j = 0; j < nv; j++) atomicAdd(dst + j, v[j]);
                     } else {
-                        store_chunk_normal(p, m, n0, nv, v, true);
+                        store_chunk_normal<FIN>(p, m, n0, nv, v, true);
                     }
                 } else {
                     const int n = row_tile * TILE_ROWS + r;
@@ -722,15 +725,15 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_consta
                         if (splitk) {
                             // (sums added straight into the residual bring the bias with the first part of K; sums in
                             // scratch get it from the finalize kernel)
-                            if (p.epilogue == 2 && split == 0 && p.bias) v[j] += __ldg(p.bias + n);
+                            if (FIN && p.epilogue == 2 && split == 0 && p.bias) v[j] += __ldg(p.bias + n);
                             atomicAdd(p.accum + (size_t)m * p.accum_ld + n, v[j]);
                         } else if (p.epilogue == 0) {
-                            ((__nv_bfloat16*)p.out)[(size_t)m * p.ldc + n] = __float2bfloat16_rn(finish_sum(p, n, v[j]));
+                            ((__nv_bfloat16*)p.out)[(size_t)m * p.ldc + n] = __float2bfloat16_rn(finish_sum<FIN>(p, n, v[j]));
                         } else if (p.epilogue == 1) {
-                            ((float*)p.out)[(size_t)m * p.ldc + n] = finish_sum(p, n, v[j]);
+                            ((float*)p.out)[(size_t)m * p.ldc + n] = finish_sum<FIN>(p, n, v[j]);
                         } else {
                             float* dst = (float*)p.out + (size_t)m * p.ldc + n;
-                            *dst = *dst + finish_sum(p, n, v[j]);
+                            *dst = *dst + finish_sum<FIN>(p, n, v[j]);
                         }
                     }
                 }
@@ -771,7 +774,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_consta
                 if (n >= p.N || m >= p.M) continue;
                 float v = 0.0f;
                 for (int s = 0; s < S; s++) v += recv[((size_t)s * RP + rl) * C + c];
-                v = finish_sum(p, n, v);
+                v = finish_sum<FIN>(p, n, v);
                 if (p.epilogue == 0) ((__nv_bfloat16*)p.out)[(size_t)m * p.ldc + n] = __float2bfloat16_rn(v);
                 else if (p.epilogue == 1) ((float*)p.out)[(size_t)m * p.ldc + n] = v;
                 else {
@@ -800,7 +803,7 @@ constexpr int MAX_GROUPS = 256;
 // GROUPED: the rows of A lie in groups (the tokens of each expert, one group after the other), every group against weights
 // of its own; the group borders are read on the device, a tile belongs to one group, and tiles walk a group's weight
 // columns before the next group's.  Rows of the next group that a tile's last rows bring along are computed and dropped.
-template <bool GROUPED>
+template <bool GROUPED, bool FIN>
 __global__ void __launch_bounds__(GEMM_THREADS, 1)
 gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_constant__ CUtensorMap map_cols,
                           const GemmTcParams p) {
@@ -969,7 +972,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_rows, const __
                     for (int q = 0; q < 4; q++) {
                         const int n0 = col0 + c0 + q * 16;
                         if (!ok || m >= row_end || n0 >= p.N) continue;
-                        store_chunk_normal(p, m, n0, min(16, p.N - n0), reinterpret_cast<float*>(u + q * 16), u_first);
+                        store_chunk_normal<FIN>(p, m, n0, min(16, p.N - n0), reinterpret_cast<float*>(u + q * 16), u_first);
                     }
                 }
                 for (; c0 < p.block_cols; c0 += 16) {
@@ -977,7 +980,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_rows, const __
                     tmem_ld16(taddr_row + (uint32_t)c0, v);
                     const int n0 = col0 + c0;
                     if (!ok || m >= row_end || n0 >= p.N) continue;
-                    store_chunk_normal(p, m, n0, min(16, p.N - n0), v, u_first);
+                    store_chunk_normal<FIN>(p, m, n0, min(16, p.N - n0), v, u_first);
                 }
             }
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");

@@ -58,6 +58,7 @@ __host__ __device__ __forceinline__ int pair_stage_bytes(int block_cols) {
 }
 
 // p.block_cols: weight rows per pair tile; p.row_tiles / p.total_tiles count pair tiles (256 tokens x block_cols).
+template <bool FIN>
 __global__ void __launch_bounds__(GEMM_THREADS, 1)
 gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_constant__ CUtensorMap map_cols,
                     const GemmTcParams p) {
@@ -194,7 +195,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_c
                     for (int q = 0; q < 4; q++) {
                         const int n0 = col_tile * p.block_cols + c0 + q * 16;
                         if (!ok || m >= p.M || n0 >= p.N) continue;
-                        store_chunk_normal(p, m, n0, min(16, p.N - n0), reinterpret_cast<float*>(u + q * 16), u_first);
+                        store_chunk_normal<FIN>(p, m, n0, min(16, p.N - n0), reinterpret_cast<float*>(u + q * 16), u_first);
                     }
                 }
                 for (; c0 < p.block_cols; c0 += 16) {
@@ -202,7 +203,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_c
                     tmem_ld16(taddr_row + (uint32_t)c0, v);
                     const int n0 = col_tile * p.block_cols + c0;
                     if (!ok || m >= p.M || n0 >= p.N) continue;
-                    store_chunk_normal(p, m, n0, min(16, p.N - n0), v, u_first);
+                    store_chunk_normal<FIN>(p, m, n0, min(16, p.N - n0), v, u_first);
                 }
             }
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");

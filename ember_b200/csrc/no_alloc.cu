@@ -32,7 +32,7 @@ int scratch_pointer(float** out) {
         e = cudaGetSymbolAddress((void**)&ptr, noalloc_scratch);
         if (e != cudaSuccess || !ptr)
             return ember::fail("gemm_tc_noalloc: cudaGetSymbolAddress failed on device %d: %s", dev, cudaGetErrorString(e));
-        e = cudaFuncSetAttribute(ember::gemm_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+        e = cudaFuncSetAttribute(ember::gemm_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
         if (e != cudaSuccess)
             return ember::fail("gemm_tc_noalloc: cannot raise the shared-memory limit: %s", cudaGetErrorString(e));
         scratch_of_device[dev] = ptr;
@@ -129,7 +129,7 @@ EMBER_API int ember_gemm_tc_noalloc(const void* A, const void* W, void* out, int
         return fail("gemm_tc_noalloc: cuTensorMapEncodeTiled failed or is unavailable");
 
     dim3 grid(row_tiles, 1, splits);
-    gemm_tc_kernel<<<grid, GEMM_THREADS, smem, st>>>(map_rows, map_cols, p);
+    gemm_tc_kernel<false><<<grid, GEMM_THREADS, smem, st>>>(map_rows, map_cols, p);
     if (int rc = check_launch("gemm_tc_noalloc")) return rc;
     if (splits > 1 && epilogue != 2) {
         const size_t total = (size_t)M * (epilogue == 3 ? N / 2 : N);
