@@ -73,7 +73,7 @@ FILANEX = {
         "architecture": "Filanex", "vocab": 512, "width": 256, "norm": {"eps": 1e-6}, "loop": {"start": 2, "stop": 3, "times": 1},
         "layers": [
             _layer(_attention(8, 1, 128, 128, 0.0884, 25.0, 256, _rot(64, 10000.0, (4.0, 256, 32.0, 1.0))), _moe(256, 8, 2, (4, 2))),
-            _layer(_attention(4, 2, 128, 128, 0.0884, 50.0, 100, _rot(128, 50000.0, (8.0, 1024, 32.0, 1.0))), _dense(512)),
+            _layer(_attention(6, 2, 128, 128, 0.09, 50.0, 100, _rot(128, 50000.0, (8.0, 1024, 32.0, 1.0))), _dense(512)),
             _layer(_attention(2, 1, 64, 128, 0.125, 30.0, 77, _rot(16, 10000.0)), _dense(384)),
         ]}),
     # every layer once: no loop, and the embedding's key is there without a bigram

@@ -165,13 +165,13 @@ def test_plain_rotation_turns_neighbours_with_stretched_frequencies():
     y = plain.rotate_pairs(x, {"dims": 4, "base": 100.0})
     assert abs(float(y[2, 0, 2]) - math.cos(2 * 0.1)) < 1e-12 and abs(float(y[2, 0, 3]) - math.sin(0.2)) < 1e-12
     assert float(y[2, 0, 0]) == 0.0 and float(y[1, 0, 5]) == 9.0
-    # 16 elements, base 10000, made for 512 positions: dim(32) = 16 ln(512 / 64 pi) / (2 ln 10000) = 0.81.. -> lo 0,
-    # dim(1) = 16 ln(512 / 2 pi) / (2 ln 10000) = 3.82.. -> hi 4: pair 0 keeps its frequency, pairs from 4 on are divided
-    f, mag = plain.frequencies({"dims": 16, "base": 10000.0, "scaling": {"factor": 4.0, "original": 512, "fast": 32.0, "slow": 1.0}}, torch.float64)
+    # 16 elements, base 10000, made for 1000 positions: dim(32) = 16 ln(1000 / 64 pi) / (2 ln 10000) = 1.39.. -> lo 1,
+    # dim(1) = 16 ln(1000 / 2 pi) / (2 ln 10000) = 4.40.. -> hi 5: pairs 0 and 1 keep their frequency, from 5 on it is divided
+    f, mag = plain.frequencies({"dims": 16, "base": 10000.0, "scaling": {"factor": 8.0, "original": 1000, "fast": 32.0, "slow": 1.0}}, torch.float64)
     plain_f, one = plain.frequencies({"dims": 16, "base": 10000.0}, torch.float64)
     ratio = (f / plain_f).tolist()
-    assert ratio[0] == 1.0 and all(abs(r - 0.25) < 1e-12 for r in ratio[4:]) and abs(ratio[2] - (0.5 / 4 + 0.5)) < 1e-12
-    assert one == 1.0 and abs(mag - (0.1 * math.log(4.0) + 1.0)) < 1e-12
+    assert ratio[:2] == [1.0, 1.0] and all(abs(r - 0.125) < 1e-12 for r in ratio[5:]) and abs(ratio[3] - (0.5 / 8 + 0.5)) < 1e-12
+    assert one == 1.0 and abs(mag - (0.1 * math.log(8.0) + 1.0)) < 1e-12
 
 
 def test_plain_mask_counts_chunks_from_the_start():

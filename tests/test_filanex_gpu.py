@@ -134,7 +134,7 @@ def test_a_long_prompt_then_decoding(dtype, dirs, plain_logits):
 
 
 def test_a_request_longer_than_the_pool(dirs, plain_logits):
-    """Every layer of this model works in chunks: a pool of 192 tokens serves a request of 500, because the pages of chunks
+    """Every layer of this model works in chunks: a pool of 384 tokens serves a request of 700, because the pages of chunks
     that have passed come back while it runs."""
     requests = make_requests("c", (700,), seed=19)
     steps = trace_portions(requests, sizes=(64, 30, 1, 1, 50))
@@ -333,8 +333,6 @@ def test_single_tokens_over_split_keys_in_a_chunk(chunk, at, merge, monkeypatch)
     """A decoded token whose chunk is cut into key splits that start where the chunk does (inside a tile of 64 keys), merged
     in a cluster or through buffers; the gate joins behind the merge."""
     from ember_b200 import ops
-    from ember_b200.config import AttentionSpec
-    from ember_b200.parts.attention import Attention
     heads, kv, dim, page = 4, 2, 128, 16
     g = torch.Generator().manual_seed(at)
     n = at + 1
@@ -366,7 +364,6 @@ def test_single_tokens_over_split_keys_in_a_chunk(chunk, at, merge, monkeypatch)
     want = plain.capped_attention(q.double(), k.double(), v.double(), 0.3, mask, 9.0)
     want = want * torch.sigmoid(gate[:, 24:].double()).reshape(1, heads, dim)
     assert _rel(out.cpu(), want) < 1e-2
-    assert AttentionSpec and Attention                                        # (the part that plans these splits)
 
 
 def test_the_gate_the_cap_and_the_stretching_are_there():
