@@ -2,7 +2,7 @@
 from .spec import (AttentionSpec, BigramEmbeddingSpec, ConcatReentrySpec, ConfigError, DynamicTanhSpec, HyperConnectionSpec, TimeMixSpec, GatedDeltaSpec, GatedLinearAttentionSpec, GatedMLPSpec, LatentAttentionSpec,
                    LayerNormSpec, LayerSpec, MatrixMemorySpec, MLPSpec, ModelSpec, NoPositionSpec, ParallelMixerSpec, PartSpec,
                    RMSNormSpec, RotarySpec, RoutedMLPSpec, ScheduleEntry, SigmoidAttentionSpec, SigmoidGateSpec,
-                   SinkAttentionSpec, StateSpaceSpec, default_schedule)
+                   SelectiveScanSpec, SinkAttentionSpec, StateSpaceSpec, default_schedule)
 from .registry import (config_from_dict, load_config, load_model_spec, register_architecture,
                        registered_architectures, resolve_architecture)
 from .qwen3 import Qwen3Config
@@ -11,6 +11,7 @@ from .zufusun import ZufusunConfig
 from .fomanex import FomanexConfig
 from .pepapel import PepapelConfig
 from .filanex import FilanexConfig
+from .malusun import MalusunConfig
 
 __all__ = [
     "AttentionSpec", "ConfigError", "GatedMLPSpec", "LayerSpec", "ModelSpec", "NoPositionSpec", "PartSpec",
@@ -20,4 +21,5 @@ __all__ = [
     "SigmoidAttentionSpec", "SigmoidGateSpec", "StateSpaceSpec", "ZufusunConfig", "GatedLinearAttentionSpec",
     "LatentAttentionSpec", "RoutedMLPSpec", "SinkAttentionSpec", "FomanexConfig", "DynamicTanhSpec", "HyperConnectionSpec",
     "TimeMixSpec", "PepapelConfig", "FilanexConfig", "BigramEmbeddingSpec", "ConcatReentrySpec", "MLPSpec",
+    "MalusunConfig", "SelectiveScanSpec",
 ]

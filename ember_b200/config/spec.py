@@ -30,13 +30,14 @@ class PartSpec:
 # ----------------------------------------------------------------------------- norms
 @dataclass(frozen=True)
 class RMSNormSpec(PartSpec):
-    """out = weight * (x * rsqrt(mean(x^2) + eps)); plain weight (not 1 + weight).  The tensor is named prefix +
-    ``weight_suffix``."""
+    """out = (weight_offset + weight) * (x * rsqrt(mean(x^2) + eps)); ``weight_offset`` 0: the stored weight as it is,
+    1: weights stored around zero.  The tensor is named prefix + ``weight_suffix``."""
 
     kind: ClassVar[str] = "rmsnorm"
     size: int = 0
     eps: float = 1e-6
     weight_suffix: str = "weight"
+    weight_offset: float = 0.0
 
 
 @dataclass(frozen=True)
@@ -160,7 +161,11 @@ class SinkAttentionSpec(PartSpec):
     (score <- softcap * tanh(score / softcap) after the scale); ``chunk`` > 0 (position i sees j <= i only if
     floor(i / chunk) == floor(j / chunk), chunks counted from the sequence's start); ``head_gate`` (head h's output is
     multiplied by sigmoid(W_g x)_h, tensor ``g`` [heads, hidden]); ``element_gate`` (the concatenated heads are multiplied
-    element by element by sigmoid(W_g x), tensor ``g`` [heads value_dim, hidden])."""
+    element by element by sigmoid(W_g x), tensor ``g`` [heads value_dim, hidden]); ``sink`` with ``fixed_sink`` (every
+    head's sink is that number: no tensor); ``slope_span`` > 0 (slope_h * (i - j) is taken off the score, after the cap,
+    with slope_h = 2^(-slope_span (h + 1) / num_heads)); ``value_mix`` "source" (the layer's values, before they are cached,
+    are left for later layers of the step) or "mix" (v <- (1 - lambda) v + lambda v_source with the values a "source" layer
+    before left for the same token and lambda the stored scalar ``vmix``; the mixed values are cached), "" for neither."""
 
     kind: ClassVar[str] = "sink_attention"
     hidden_size: int = 0
@@ -183,6 +188,9 @@ class SinkAttentionSpec(PartSpec):
     chunk: int = 0
     head_gate: bool = False
     element_gate: bool = False
+    fixed_sink: Optional[float] = None
+    slope_span: float = 0.0
+    value_mix: str = ""
 
 
 @dataclass(frozen=True)
@@ -303,6 +311,21 @@ class StateSpaceSpec(PartSpec):
 
 
 @dataclass(frozen=True)
+class SelectiveScanSpec(PartSpec):
+    """Selective scan with a diagonal state per channel (Mamba): W_in h = [x | z], both of size ``inner``; x passes a short
+    causal convolution (``conv`` [inner, conv_taps], bias ``conv.b``) and silu; W_x x = [low | B | C] of sizes ``dt_rank``,
+    ``state_size``, ``state_size``; dt = softplus(W_dt low + dt.b), one per channel; S[c, n] <- exp(-dt_c exp(A_log[c, n])) S[c, n]
+    + dt_c x_c B_n; y_c = sum_n S[c, n] C_n + D_c x_c; W_o (y silu(z)).  Tensors: in, conv, conv.b, x, dt, dt.b, A_log, D, o."""
+
+    kind: ClassVar[str] = "mamba1"
+    hidden_size: int = 0
+    inner: int = 0
+    state_size: int = 0
+    dt_rank: int = 0
+    conv_taps: int = 4
+
+
+@dataclass(frozen=True)
 class ParallelMixerSpec(PartSpec):
     """Two mixers that read the same input; the result is left_scale * left + right_scale * right.  ``branch_norm``:
     each result is first RMS-normed over the model width with a weight of its own (tensors ``left_norm_name`` and
@@ -356,7 +379,8 @@ class GatedMLPSpec(PartSpec):
 
 @dataclass(frozen=True)
 class MLPSpec(PartSpec):
-    """down( act(up(x)) ), one matrix up and one down; act is "gelu" (0.5 z (1 + erf(z / sqrt 2))).  ``names``: the two
+    """down( act(up(x)) ), one matrix up and one down; act is "gelu" (0.5 z (1 + erf(z / sqrt 2))) or "square_relu"
+    (max(z, 0)^2).  ``names``: the two
     tensors' names under the prefix (up, down); ``bias``: both have biases, named like the matrices with ``bias_suffix``
     behind."""
 
@@ -406,6 +430,11 @@ class RoutedMLPSpec(PartSpec):
     identity: int = 0
     # ``expert`` "gated" as above, or "square_relu": W_down relu(W_up h)^2, tensors e<i>.up and e<i>.down only.
     expert: str = "gated"
+    # ``weigh`` "output": sum of weight * expert(h); "input": sum of expert(weight * h) (gated experts).
+    weigh: str = "output"
+    # ``shared_size`` > 0: one more expert of that size (silu(gate) up, tensors shared.gate, shared.up, shared.down) runs for
+    # every token, unweighted, and is added.
+    shared_size: int = 0
 
 
 # --------------------------------------------------------- what is added to the embedded tokens

@@ -61,7 +61,7 @@ static bool tensor_map(const void* ptr, int rows, int K, int box_rows, CUtensorM
 }
 
 // Whether a product's sums get a bias or an activation before they are stored (an instance of the kernels of its own).
-static bool finishes(const GemmTcParams& p) { return p.bias != nullptr || p.act == 3; }
+static bool finishes(const GemmTcParams& p) { return p.bias != nullptr || p.act >= 3; }
 
 // How many pairs of blocks of the pair kernel the device runs at once (0: it cannot).
 static int pair_capacity(int num_sms) {
@@ -296,15 +296,15 @@ EMBER_API long long ember_gemm_tc_scratch_floats(int max_tokens_swapped, int N) 
 
 // C = A . W^T with the fused epilogue.  `scratch` is a zero-filled fp32 buffer of at least
 // min(M, 128) * N floats (used only when the K range is split; it is left zeroed).
-// Epilogue 8 stores gelu(sum + bias) in bf16 (the exact form, by erf).  `bias` (fp32 [N] or null) joins the sums of
+// Epilogue 8 stores gelu(sum + bias) in bf16 (the exact form, by erf), epilogue 9 max(sum + bias, 0)^2.  `bias` (fp32 [N] or null) joins the sums of
 // epilogues 0, 1, 2 and 8.  Epilogue 5 (at most 128 tokens): the fp32 sums are left in `scratch` as [M, N] for a consumer that reads them and
 // sets them back to zero (`out` is not used); it saves the pass that rounds, stores and clears.
 EMBER_API int ember_gemm_tc(const void* A, const void* W, void* out, int ldc, int M, int N, int K, int epilogue, const float* bias,
                             float* scratch, long long scratch_floats, int num_sms, int split_mode, int* err, void* stream) {
     if (M <= 0 || N <= 0) return 0;
-    const int act = epilogue == 6 ? 1 : (epilogue == 7 ? 2 : (epilogue == 8 ? 3 : 0));      // epilogues 6, 7: the gated epilogue with relu, with gelu (tanh form)
+    const int act = epilogue == 6 ? 1 : (epilogue == 7 ? 2 : (epilogue == 8 ? 3 : (epilogue == 9 ? 4 : 0)));      // epilogues 6, 7: the gated epilogue with relu, with gelu (tanh form)
     if (epilogue == 6 || epilogue == 7) epilogue = 3;
-    if (epilogue == 8) epilogue = 0;
+    if (epilogue == 8 || epilogue == 9) epilogue = 0;
     if (bias && (epilogue == 3 || epilogue == 5)) return fail("gemm_tc: the gated epilogue and sums left in scratch take no bias");
     const bool sums = epilogue == 5;
     if (sums) {

@@ -46,7 +46,7 @@ struct GemmTcParams {
     int num_k_blocks;     // ceil(K / TILE_K)
     int k_blocks_per_split;
     int epilogue;         // 0 store bf16, 1 store fp32, 2 add fp32, 3 act(gate)*up -> bf16
-    int act;              // epilogue 3: 0 silu, 1 relu, 2 gelu (tanh form); epilogue 0: 0 none, 3 gelu (exact, by erf)
+    int act;              // epilogue 3: 0 silu, 1 relu, 2 gelu (tanh form); epilogue 0: 0 none, 3 gelu (exact, by erf), 4 max(x, 0)^2
     const float* bias;    // [N] added to the sums of epilogues 0, 1 and 2 (once, whatever the parts of K), or null
     void* out;
     int ldc;
@@ -151,13 +151,18 @@ __device__ __forceinline__ float gate_mul(float g, float u, int act) {
 }
 
 __device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f)); }
+// The activations of the plain epilogue: 3 gelu (exact), 4 relu squared, others none.
+__device__ __forceinline__ float plain_activation(float z, int act) {
+    if (act == 4) { z = fmaxf(z, 0.0f); return z * z; }
+    return act == 3 ? gelu_erf(z) : z;
+}
 // A complete sum of output column n as the plain epilogues (0, 1, 2) want it: with its bias, through its activation.
 // FIN false: the kernels' instances for products without either, which pay nothing for them.
 template <bool FIN>
 __device__ __forceinline__ float finish_sum(const GemmTcParams& p, int n, float v) {
     if (!FIN) return v;
     if (p.bias) v += __ldg(p.bias + n);
-    return p.act == 3 ? gelu_erf(v) : v;
+    return plain_activation(v, p.act);
 }
 
 // Fused epilogue of 16 consecutive output columns of one token row (normal orientation):
@@ -166,7 +171,7 @@ __device__ __forceinline__ void store_finished_chunk(const GemmTcParams& p, int 
 // ``first``: these are the sums of the first part of K (the one that brings the bias).
 template <bool FIN>
 __device__ __forceinline__ void store_chunk_normal(const GemmTcParams& p, int m, int n0, int nv, float* v, bool first) {
-    if (FIN && ((p.bias && first) || p.act == 3)) {
+    if (FIN && ((p.bias && first) || p.act >= 3)) {
 #pragma unroll
         for (int j = 0; j < 16; j++)
             if (j < nv) v[j] = finish_sum<true>(p, n0 + j, v[j]);
@@ -1015,7 +1020,7 @@ __global__ void gemm_tc_finalize_kernel(float* __restrict__ accum, int accum_ld,
     } else {
         float c = a[j] + (bias ? bias[j] : 0.0f);
         a[j] = 0.0f;
-        if (act == 3) c = gelu_erf(c);
+        c = plain_activation(c, act);
         if (epilogue == 0) ((__nv_bfloat16*)out)[(size_t)m * ldc + j] = __float2bfloat16_rn(c);
         else ((float*)out)[(size_t)m * ldc + j] = c;
     }
@@ -1046,7 +1051,7 @@ __global__ void gemm_tc_finalize4_kernel(float* __restrict__ accum, int accum_ld
         a[0] = zero;
         r0 = x.x; r1 = x.y; r2 = x.z; r3 = x.w;
         if (bias) { r0 += bias[j]; r1 += bias[j + 1]; r2 += bias[j + 2]; r3 += bias[j + 3]; }
-        if (act == 3) { r0 = gelu_erf(r0); r1 = gelu_erf(r1); r2 = gelu_erf(r2); r3 = gelu_erf(r3); }
+        if (act >= 3) { r0 = plain_activation(r0, act); r1 = plain_activation(r1, act); r2 = plain_activation(r2, act); r3 = plain_activation(r3, act); }
     }
     if (EPI == 1) {
         *reinterpret_cast<float4*>((float*)out + (size_t)m * ldc + j) = make_float4(r0, r1, r2, r3);

@@ -9,6 +9,8 @@
 //             f = g sigmoid(alpha g) (u + 1);
 //   down:     y[slot] = W_down[e] act[slot]  (fp32);
 //   combine:  out[token] = sum over its choices, in order, of weight * y[slot]  (stored, or added to what is there).
+// A router may weigh an expert's input instead of its output: gate_up then multiplies its sums by the pair's weight (or the
+// gathered rows are multiplied) and combine adds the rows as they are.
 // Both products come in two forms: tiles of 32 slots x 64 outputs through shared memory (any sizes, any step), and,
 // for steps of few tokens, a streaming form in which a block keeps its (at most 16) rows in shared memory and every
 // warp streams whole weight rows past them in 16-byte pieces, so an expert's weights are read once at the rate of
@@ -332,8 +334,10 @@ struct MoeGemmArgs {
     int N, K;
     float limit, alpha, up_offset;      // (limit may be +inf: no clamps)
     int act;                            // ungated product: 0 stores the sums, 1 stores relu(sum)^2
+    const float* in_w;                  // gated product: a weight per pair that multiplies the expert's input (its gate and up sums), or null
 };
 
+__device__ __forceinline__ float slot_weight(const MoeGemmArgs& p, int slot) { return p.in_w ? p.in_w[p.pair_of_slot[slot]] : 1.0f; }
 __device__ __forceinline__ float plain_act(float v, int act) { return act == 1 ? (v > 0.0f ? v * v : 0.0f) : v; }
 
 // GATED: N counts interleaved (gate, up) rows, the output has N / 2 columns.
@@ -388,12 +392,13 @@ __global__ void __launch_bounds__(256) moe_gemm_kernel(MoeGemmArgs p) {
         if (r >= rows) continue;
         TO* o = (TO*)p.out + (size_t)(row0 + r) * p.ld_o;
         if (GATED) {
+            const float wi = slot_weight(p, row0 + r);
 #pragma unroll
             for (int j = 0; j < 4; j += 2) {
                 const int n = n0 + tx * 4 + j;
                 if (n >= p.N) continue;
-                const float g = fminf(acc[i][j], p.limit);
-                const float u = fminf(fmaxf(acc[i][j + 1], -p.limit), p.limit);
+                const float g = fminf(acc[i][j] * wi, p.limit);
+                const float u = fminf(fmaxf(acc[i][j + 1] * wi, -p.limit), p.limit);
                 o[n >> 1] = from_float<TO>(g / (1.0f + expf(-p.alpha * g)) * (u + p.up_offset));
             }
         } else {
@@ -466,7 +471,8 @@ __device__ __forceinline__ void moe_stream_rows(const MoeGemmArgs& p, const uint
         if (lane < rows) {
             TO* o = (TO*)p.out + (size_t)(row0 + lane) * p.ld_o;
             if (GATED) {
-                const float g = fminf(v0, p.limit), u = fminf(fmaxf(v1, -p.limit), p.limit);
+                const float wi = slot_weight(p, row0 + lane);
+                const float g = fminf(v0 * wi, p.limit), u = fminf(fmaxf(v1 * wi, -p.limit), p.limit);
                 o[pr] = from_float<TO>(g / (1.0f + expf(-p.alpha * g)) * (u + p.up_offset));
             } else {
                 o[n0] = from_float<TO>(plain_act(v0, p.act));
@@ -593,7 +599,8 @@ __global__ void __launch_bounds__(MT_WARPS * 32) moe_stream_tc_kernel(MoeGemmArg
                 if (GATED) {
                     const float up = __shfl_xor_sync(0xffffffffu, v, 4);     // the odd row beside this even one
                     if ((g & 1) == 0 && n < p.N && slot < rows) {
-                        const float gt = fminf(v, p.limit), u = fminf(fmaxf(up, -p.limit), p.limit);
+                        const float wi = slot_weight(p, row0 + slot);
+                        const float gt = fminf(v * wi, p.limit), u = fminf(fmaxf(up * wi, -p.limit), p.limit);
                         ((TO*)p.out)[(size_t)(row0 + slot) * p.ld_o + (n >> 1)] = from_float<TO>(gt / (1.0f + expf(-p.alpha * gt)) * (u + p.up_offset));
                     }
                 } else if (n < p.N && slot < rows) {
@@ -611,6 +618,27 @@ __global__ void moe_gather_kernel(const uint4* __restrict__ x, const int* __rest
     const uint4* src = x + (size_t)(pair_of_slot[slot] / top) * row16;
     uint4* dst = xs + (size_t)slot * row16;
     for (int i = threadIdx.x; i < row16; i += blockDim.x) dst[i] = src[i];
+}
+
+// The same for bfloat16 rows, each times its pair's weight (the weight on an expert's input).
+__global__ void moe_gather_weighted_kernel(const uint4* __restrict__ x, const int* __restrict__ pair_of_slot, const float* __restrict__ wgt,
+                                           int top, uint4* __restrict__ xs, int row16) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int slot = blockIdx.x, pair = pair_of_slot[slot];
+    const float w = wgt[pair];
+    const uint4* src = x + (size_t)(pair / top) * row16;
+    uint4* dst = xs + (size_t)slot * row16;
+    for (int i = threadIdx.x; i < row16; i += blockDim.x) {
+        const uint4 v = src[i];
+        float f[8];
+        Piece<__nv_bfloat16>::unpack(v, f);
+        uint4 o;
+        __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&o);
+#pragma unroll
+        for (int k = 0; k < 4; k++) h[k] = __floats2bfloat162_rn(f[2 * k] * w, f[2 * k + 1] * w);
+        dst[i] = o;
+    }
 }
 
 template <typename TO>
@@ -693,7 +721,7 @@ __global__ void moe_combine4_kernel(const float4* __restrict__ y, const float* _
     float4 s = make_float4(0.0f, 0.0f, 0.0f, 0.0f), o = s;
     if (accumulate) o = out[(size_t)t * hidden4 + i];
     for (int k = 0; k < top; k++) {
-        const float w = wgt[(size_t)t * top + k];
+        const float w = wgt ? wgt[(size_t)t * top + k] : 1.0f;
         const float4 v = y[(size_t)slot_of_pair[(size_t)t * top + k] * hidden4 + i];
         s.x = fmaf(w, v.x, s.x); s.y = fmaf(w, v.y, s.y); s.z = fmaf(w, v.z, s.z); s.w = fmaf(w, v.w, s.w);
     }
@@ -714,7 +742,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const float* __r
             const bool same = sel && sel[(size_t)t * top + k] >= experts;
             const float v = same ? (same_f ? same_f[(size_t)t * hidden + i] : to_float(same_h[(size_t)t * hidden + i]))
                                  : y[(size_t)slot_of_pair[(size_t)t * top + k] * hidden + i];
-            s = fmaf(wgt[(size_t)t * top + k], v, s);
+            s = fmaf(wgt ? wgt[(size_t)t * top + k] : 1.0f, v, s);
         }
         out[(size_t)t * hidden + i] = accumulate ? out[(size_t)t * hidden + i] + s : s;
     }
@@ -774,10 +802,11 @@ EMBER_API int ember_moe_group(const int* sel, int n_pairs, int E, int* offsets, 
 EMBER_API int ember_moe_gemm(const void* x, int x_dtype, int ld_x, const void* w, int w_dtype, long long w_expert, void* out,
                              int out_dtype, int ld_o, const int* offsets, const int* pair_of_slot, const int* n_tiles,
                              const int* tile_expert, const int* tile_row0, int max_tiles, int top, int N, int K, int gated,
-                             float limit, float alpha, float up_offset, int act, void* stream) {
+                             float limit, float alpha, float up_offset, int act, const float* in_w, void* stream) {
     if (max_tiles <= 0) return 0;
     if (N <= 0 || K <= 0 || (gated && (N & 1))) return fail("moe_gemm: N=%d K=%d", N, K);
-    MoeGemmArgs p{x, ld_x, w, w_expert, out, ld_o, offsets, pair_of_slot, n_tiles, tile_expert, tile_row0, top, N, K, limit, alpha, up_offset, act};
+    if (in_w && !gated) return fail("moe_gemm: weights on the input belong to the gated product");
+    MoeGemmArgs p{x, ld_x, w, w_expert, out, ld_o, offsets, pair_of_slot, n_tiles, tile_expert, tile_row0, top, N, K, limit, alpha, up_offset, act, in_w};
     dim3 grid(max_tiles, (N + MOE_BN - 1) / MOE_BN);
     cudaStream_t st = (cudaStream_t)stream;
     const int key = x_dtype * 100 + w_dtype * 10 + out_dtype;       // F32 = 0, BF16 = 1
@@ -801,14 +830,15 @@ EMBER_API int ember_moe_stream_rows() { return MS_ROWS; }
 EMBER_API int ember_moe_stream(const void* x, int x_dtype, int ld_x, const void* w, int w_dtype, long long w_expert, void* out,
                                int out_dtype, int ld_o, const int* offsets, const int* pair_of_slot, const int* n_tiles,
                                const int* tile_expert, const int* tile_row0, int max_tiles, int top, int N, int K, int gated,
-                               float limit, float alpha, float up_offset, int act, void* stream) {
+                               float limit, float alpha, float up_offset, int act, const float* in_w, void* stream) {
     if (max_tiles <= 0) return 0;
     if (N <= 0 || K <= 0 || (gated && (N & 1))) return fail("moe_stream: N=%d K=%d", N, K);
+    if (in_w && !gated) return fail("moe_stream: weights on the input belong to the gated product");
     const int elem = x_dtype == EMBER_F32 ? 4 : 2;
     if (((size_t)K * elem) % 16 || ((size_t)ld_x * elem) % 16) return fail("moe_stream: rows of %d elements are no multiple of 16 bytes", K);
     const size_t smem = (size_t)MS_ROWS * K * elem;
     if (smem > 200 * 1024) return fail("moe_stream: %d rows of %d do not fit in shared memory", MS_ROWS, K);
-    MoeGemmArgs p{x, ld_x, w, w_expert, out, ld_o, offsets, pair_of_slot, n_tiles, tile_expert, tile_row0, top, N, K, limit, alpha, up_offset, act};
+    MoeGemmArgs p{x, ld_x, w, w_expert, out, ld_o, offsets, pair_of_slot, n_tiles, tile_expert, tile_row0, top, N, K, limit, alpha, up_offset, act, in_w};
     cudaStream_t st = (cudaStream_t)stream;
     const int key = x_dtype * 100 + w_dtype * 10 + out_dtype;       // F32 = 0, BF16 = 1
     static int tc_on = -1;
@@ -841,9 +871,14 @@ EMBER_API int ember_moe_stream(const void* x, int x_dtype, int ld_x, const void*
     return fail("moe_stream: unsupported dtypes %d", key);
 }
 
-EMBER_API int ember_moe_gather(const void* x, const int* pair_of_slot, int n_pairs, int top, void* xs, int row_bytes, void* stream) {
+EMBER_API int ember_moe_gather(const void* x, const int* pair_of_slot, int n_pairs, int top, void* xs, int row_bytes,
+                               const float* wgt, void* stream) {
     if (n_pairs <= 0) return 0;
     if (row_bytes <= 0 || row_bytes % 16) return fail("moe_gather: rows of %d bytes (a multiple of 16)", row_bytes);
+    if (wgt) {                                                // bfloat16 rows times their pairs' weights
+        launch_kernel(moe_gather_weighted_kernel, n_pairs, 128, 0, (cudaStream_t)stream, (const uint4*)x, pair_of_slot, wgt, top, (uint4*)xs, row_bytes / 16);
+        return check_launch("moe_gather_weighted");
+    }
     launch_kernel(moe_gather_kernel, n_pairs, 128, 0, (cudaStream_t)stream, (const uint4*)x, pair_of_slot, top, (uint4*)xs, row_bytes / 16);
     return check_launch("moe_gather");
 }

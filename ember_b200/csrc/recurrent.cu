@@ -21,13 +21,15 @@ __device__ __forceinline__ float logsigmoidf_(float x) { return fminf(x, 0.0f) -
 
 // ------------------------------------------------------------------------------- short causal convolution + silu
 // out[t, c] = silu(bias[c] + sum_j taps[c, j] * in(t - (n - 1 - j), c)) (or, silu = 0, the sum itself); inputs before the run come from the
-// request's carried inputs carry[slot][j][c] (j = 0 the oldest of n - 1), zeros for a new request.
+// request's carried inputs carry[slot][j][c] (j = 0 the oldest of n - 1), zeros for a new request.  `rounded` (or null) gets the
+// same rows in bfloat16, for a product behind the convolution.
 constexpr int CONV_MAX_TAPS = 8;  // taps the kernel keeps in registers; longer filters read them from memory
 
 __global__ void conv_silu_kernel(const float* __restrict__ x, int ldx, int c0, const float* __restrict__ taps,
                                  const float* __restrict__ bias, int n, const float* __restrict__ carry, long long carry_stride,
                                  const int* __restrict__ seq_of, const int* __restrict__ query_start,
-                                 const int* __restrict__ slots, float* __restrict__ out, int C, int silu, int T, int tt) {
+                                 const int* __restrict__ slots, float* __restrict__ out, __nv_bfloat16* __restrict__ rounded, int C,
+                                 int silu, int T, int tt) {
     pdl_launch_dependents();
     pdl_wait();
     const int t0 = blockIdx.y * tt,          // a block walks tt tokens: its taps and bias are read once for all of them
@@ -56,7 +58,9 @@ __global__ void conv_silu_kernel(const float* __restrict__ x, int ldx, int c0, c
                 acc = fmaf(taps[(size_t)c * n + j], v, acc);
             }
         }
-        out[(size_t)t * C + c] = silu ? acc / (1.0f + expf(-acc)) : acc;
+        const float y = silu ? acc / (1.0f + expf(-acc)) : acc;
+        out[(size_t)t * C + c] = y;
+        if (rounded) rounded[(size_t)t * C + c] = __float2bfloat16_rn(y);
     }
 }
 
@@ -860,7 +864,7 @@ using namespace ember;
 
 EMBER_API int ember_conv_silu(const float* x, int ldx, int c0, const float* taps, const float* bias, int n, float* carry,
                               long long carry_stride, const int* seq_of, const int* query_start, const int* slots, float* out,
-                              int T, int S, int C, int silu, void* stream) {
+                              void* rounded, int T, int S, int C, int silu, void* stream) {
     if (T <= 0 || S <= 0) return 0;
     if (C <= 0 || n < 1 || n > 64 || ldx < c0 + C) return fail("conv_silu: %d channels from column %d in rows of %d, %d taps", C, c0, ldx, n);
     if (T > 65535 || S > 65535) return fail("conv_silu: %d tokens in %d runs are too many for one launch", T, S);
@@ -868,7 +872,7 @@ EMBER_API int ember_conv_silu(const float* x, int ldx, int c0, const float* taps
     const unsigned bx = (unsigned)((C + 127) / 128);
     const int tt = T >= 1024 ? 8 : 1;          // prompt portions: eight tokens a block; small steps keep a block a token
     launch_kernel(conv_silu_kernel, dim3(bx, (T + tt - 1) / tt), 128, 0, st, x, ldx, c0, taps, bias, n, (const float*)carry,
-                  carry_stride, seq_of, query_start, slots, out, C, silu, T, tt);
+                  carry_stride, seq_of, query_start, slots, out, (__nv_bfloat16*)rounded, C, silu, T, tt);
     if (n > 1)
         launch_kernel(conv_carry_kernel, dim3(bx, S), 128, 0, st, x, ldx, c0, n, carry, carry_stride, query_start, slots, C);
     return check_launch("conv_silu");

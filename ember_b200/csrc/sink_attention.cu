@@ -10,6 +10,7 @@
 //     up-projection of the attended latent; fp32 multiply-adds in general, mma.sync tiles for bfloat16 weights;
 //   * sink_attention:    o = sum_j w_j v_j with w = softmax over the visible keys and one more term exp(sink[h]) in the
 //     denominator that has no key and no value; visible: j <= i and (no window, or i - j < window, or j < keep_first).
+//     Optionally a linear bias slope[h] * (i - j) is taken off the scores.
 //     Keys have D elements, values DV; with no value pool a value is the first DV elements of the key row (the
 //     latent serves as both).  Any number of query heads per key head.
 //
@@ -91,7 +92,8 @@ __global__ void __launch_bounds__(256) whole_norm_store_kernel(WholeNormArgs p) 
 // over the whole key projection (weights of that size); 2: an RMS norm per head (weights of D, shared by the heads).
 // Then the first `rotary` elements of every query and key head turn (element i with i + rotary / 2) by the angle
 // position * inv_freq[i], cosines and sines times `magnitude`, and the query is multiplied by 1 + qt_coef * ln(floor((position + 1) / qt_every) + 1)
-// (qt_every 0: not).  Queries out, keys and values into the token's page.
+// (qt_every 0: not).  Queries out, keys and values into the token's page.  Values may be handed from layer to layer: a
+// source leaves its (biased) values in mix_out, fp32; a layer with mix_in stores (1 - lambda) v + lambda v_source instead of v.
 struct HeadPrepareArgs {
     const float* qkv; int ld;          // [T, q | k | v] fp32
     const float* bias;                 // [q | k | v] or null
@@ -104,6 +106,8 @@ struct HeadPrepareArgs {
     void* q_out; void* k_pool; void* v_pool;
     int write_kv;
     int* err;
+    float* mix_out;                    // [T, G DV] or null
+    const float* mix_in; const float* lambda;   // [T, G DV] and one number, or null
 };
 
 // Four neighbouring elements in one store (16 bytes of floats, 8 of bfloat16).
@@ -192,12 +196,27 @@ __global__ void __launch_bounds__(256) head_prepare_store_kernel(HeadPrepareArgs
     // slots: the query heads, then the key heads, then the value heads; a thread's group is W elements of one head
     const int dq = D / W, dv = p.DV / W, n_qk = (p.H + (kp ? p.G : 0)) * dq, n = n_qk + (vp ? p.G * dv : 0);
     const int part = blockIdx.y * blockDim.x + threadIdx.x, stride = gridDim.y * blockDim.x;
+    const float lam = p.mix_in ? *p.lambda : 0.0f;
     for (int i = part; i < n; i += stride) {
         if (i >= n_qk) {                                     // values pass as they are
             const int g = (i - n_qk) / dv, d = ((i - n_qk) - g * dv) * W, at = QN + KN + g * p.DV + d;
             T* dst = vp + (size_t)g * p.page * p.DV + d;
-            if (W == 4) put4<T>(dst, val4(at));
-            else *dst = from_float<T>(val(at));
+            const size_t mi = (size_t)t * VN + g * p.DV + d;
+            if (W == 4) {
+                float4 v = val4(at);
+                if (p.mix_out) *reinterpret_cast<float4*>(p.mix_out + mi) = v;
+                if (p.mix_in) {
+                    const float4 s = *reinterpret_cast<const float4*>(p.mix_in + mi);
+                    v.x = (1.0f - lam) * v.x + lam * s.x; v.y = (1.0f - lam) * v.y + lam * s.y;
+                    v.z = (1.0f - lam) * v.z + lam * s.z; v.w = (1.0f - lam) * v.w + lam * s.w;
+                }
+                put4<T>(dst, v);
+            } else {
+                float v = val(at);
+                if (p.mix_out) p.mix_out[mi] = v;
+                if (p.mix_in) v = (1.0f - lam) * v + lam * p.mix_in[mi];
+                *dst = from_float<T>(v);
+            }
             continue;
         }
         const int h = i / dq, d = (i - h * dq) * W;
@@ -450,6 +469,7 @@ struct SinkAttnParams {
     int chunk;            // > 0: position i sees j only if i / chunk == j / chunk (chunks counted from position 0 of the sequence)
     float softcap;        // > 0: score <- softcap * tanh(score / softcap), after the scale
     const float* head_gate; int ld_gate;   // [T, ld_gate] logits, one per head: the head's output is multiplied by its sigmoid; or null
+    const float* slopes;  // [H] or null: slopes[h] * (query position - key position) is taken off the (capped) score
 };
 
 // First key a tile starting at position pos0 can see, and whether key `key` is visible from position qpos.
@@ -516,6 +536,13 @@ sink_attention_kernel(SinkAttnParams p) {
         l[i] = 0.0f;
 #pragma unroll
         for (int c = 0; c < NC; c++) acc[i][c] = 0.0f;
+    }
+
+    float slope[SA_ROWS_PER_WARP];
+#pragma unroll
+    for (int i = 0; i < SA_ROWS_PER_WARP; i++) {
+        const int r = warp + i * SA_WARPS;
+        slope[i] = p.slopes && r < rows ? p.slopes[head0 + r % nh] : 0.0f;
     }
 
     const int* bt = p.block_table + (size_t)seq * p.max_blocks;
@@ -587,7 +614,7 @@ sink_attention_kernel(SinkAttnParams p) {
                 if (r >= rows) continue;  // uniform per warp
                 const int qpos = pos0 + r / nh;
                 const bool visible = key >= a && key < b && key_visible(p, key, qpos);
-                const float sv = visible ? capped_score(p, sc[i]) : -INFINITY;
+                const float sv = visible ? capped_score(p, sc[i]) - slope[i] * (float)(qpos - key) : -INFINITY;
                 const float m_new = fmaxf(m[i], warp_max(sv));
                 if (m_new == -INFINITY) continue;  // nothing visible so far (uniform per warp)
                 const float corr = expf(m[i] - m_new);
@@ -856,6 +883,7 @@ __global__ void __launch_bounds__(256, 1) shared_row_attention_tc_kernel(SinkAtt
     const int rA = wr * 16 + g, rB = rA + 8;                   // the thread's two rows
     const int qposA = pos0 + rA / nh, qposB = pos0 + rB / nh;
     const bool liveA = rA < rows, liveB = rB < rows;
+    const float slopeA = p.slopes && liveA ? p.slopes[head0 + rA % nh] : 0.0f, slopeB = p.slopes && liveB ? p.slopes[head0 + rB % nh] : 0.0f;
     const int half = narrow ? DV / 8 : DV / 2, col0 = wc * half;      // the warp's value columns
 
     float mA = -INFINITY, mB = -INFINITY, lA = 0.0f, lB = 0.0f;
@@ -954,8 +982,8 @@ __global__ void __launch_bounds__(256, 1) shared_row_attention_tc_kernel(SinkAtt
                     const bool in = key >= a && key < b;
                     const bool vA = liveA && in && key_visible(p, key, qposA);
                     const bool vB = liveB && in && key_visible(p, key, qposB);
-                    sc[nt][e] = vA ? capped_score(p, sc[nt][e]) : -INFINITY;
-                    sc[nt][2 + e] = vB ? capped_score(p, sc[nt][2 + e]) : -INFINITY;
+                    sc[nt][e] = vA ? capped_score(p, sc[nt][e]) - slopeA * (float)(qposA - key) : -INFINITY;
+                    sc[nt][2 + e] = vB ? capped_score(p, sc[nt][2 + e]) - slopeB * (float)(qposB - key) : -INFINITY;
                     tmA = fmaxf(tmA, sc[nt][e]);
                     tmB = fmaxf(tmB, sc[nt][2 + e]);
                 }
@@ -1112,18 +1140,20 @@ EMBER_API int ember_head_prepare_store(const float* qkv, int ld, const float* bi
                                        float eps, const float* inv_freq, int rotary, float magnitude, float qt_coef, int qt_every, int T_tokens, int H,
                                        int G, int D, int DV, const int* positions, const int* seq_of, const int* block_table,
                                        int max_blocks, int page, int num_pages, void* q_out, void* k_pool, void* v_pool, int dtype,
-                                       int write_kv, int* err, void* stream) {
+                                       int write_kv, int* err, float* mix_out, const float* mix_in, const float* lambda, void* stream) {
     if (T_tokens <= 0) return 0;
+    if ((mix_in && !lambda) || ((mix_in || mix_out) && !write_kv)) return fail("head_prepare_store: values blend with a factor and go to pages");
     if (H <= 0 || G <= 0 || D <= 0 || DV <= 0 || ld < H * D + G * (D + DV)) return fail("head_prepare_store: %d/%d heads of %d / %d in rows of %d", H, G, D, DV, ld);
     if (norm_mode < 0 || norm_mode > 2 || (norm_mode && (!q_w || !k_w))) return fail("head_prepare_store: norm mode %d", norm_mode);
     if (rotary < 0 || rotary > D || (rotary & 1) || (rotary && !inv_freq)) return fail("head_prepare_store: %d rotated elements of %d", rotary, D);
     if (qt_every < 0 || page <= 0 || max_blocks <= 0 || num_pages <= 0) return fail("head_prepare_store: bad geometry");
     HeadPrepareArgs p{qkv, ld, bias, norm_mode, q_w, k_w, eps, inv_freq, rotary, magnitude, qt_coef, qt_every, H, G, D, DV, positions, seq_of,
-                      block_table, max_blocks, page, num_pages, q_out, k_pool, v_pool, write_kv, err};
+                      block_table, max_blocks, page, num_pages, q_out, k_pool, v_pool, write_kv, err, mix_out, mix_in, lambda};
     const size_t smem = (size_t)(H + G + rotary) * sizeof(float);
     if (smem > 40 * 1024) return fail("head_prepare_store: %d heads and %d rotated elements are too many", H + G, rotary);
     cudaStream_t st = (cudaStream_t)stream;
-    const uintptr_t bases = (uintptr_t)qkv | (uintptr_t)q_w | (uintptr_t)k_w | (uintptr_t)q_out | (uintptr_t)k_pool | (uintptr_t)v_pool;
+    const uintptr_t bases = (uintptr_t)qkv | (uintptr_t)q_w | (uintptr_t)k_w | (uintptr_t)q_out | (uintptr_t)k_pool | (uintptr_t)v_pool |
+                            (uintptr_t)mix_out | (uintptr_t)mix_in;
     const bool by4 = D % 4 == 0 && DV % 4 == 0 && rotary % 8 == 0 && ld % 4 == 0 && (bases & 15) == 0;
     // few tokens: a token's heads are shared out so that about two blocks an SM have work
     int parts = 1;
@@ -1230,7 +1260,7 @@ EMBER_API int ember_sink_attention(const void* q, const void* k_pool, const void
                                    int T_tokens, int H, int G, int D, int DV, const int* tiles, int n_tiles, int tile_q,
                                    const int* block_table, int max_blocks, int page, int num_pages, int window,
                                    int keep_first, const float* sink, float scale, int n_splits, int split_keys,
-                                   float* part_o, float* part_ml, int* err, int key_chunk, float softcap, const float* head_gate, int ld_gate, void* stream) {
+                                   float* part_o, float* part_ml, int* err, int key_chunk, float softcap, const float* head_gate, int ld_gate, const float* slopes, void* stream) {
     if (n_tiles <= 0 || T_tokens <= 0) return 0;
     if (D <= 0 || DV <= 0 || DV > 512 || (!v_pool && DV > D)) return fail("sink_attention: heads of %d / %d are not taken", D, DV);
     if (H <= 0 || G <= 0 || H % G) return fail("sink_attention: %d heads do not divide into %d groups", H, G);
@@ -1247,7 +1277,7 @@ EMBER_API int ember_sink_attention(const void* q, const void* k_pool, const void
     p.H = H; p.G = G; p.D = D; p.DV = DV; p.head_chunk = chunk; p.window = window; p.keep_first = keep_first; p.scale = scale;
     p.n_splits = n_splits; p.split_keys = split_keys; p.err = err;
     if (key_chunk < 0 || softcap < 0.0f || (head_gate && ld_gate < H)) return fail("sink_attention: chunk %d, score cap %g, gate rows of %d", key_chunk, softcap, ld_gate);
-    p.chunk = key_chunk; p.softcap = softcap; p.head_gate = head_gate; p.ld_gate = ld_gate;
+    p.chunk = key_chunk; p.softcap = softcap; p.head_gate = head_gate; p.ld_gate = ld_gate; p.slopes = slopes;
     cudaStream_t st = (cudaStream_t)stream;
     if (dtype == EMBER_F32) return launch_sink_attention<float, float>(p, n_tiles, T_tokens, st);
     if (dtype == EMBER_BF16)
@@ -1264,7 +1294,7 @@ EMBER_API int ember_shared_row_attention_tc_head_chunk(int group) { return group
 EMBER_API int ember_shared_row_attention_tc(const void* q, const void* k_pool, const void* v_pool, void* out, int out_f32, int T_tokens, int H, int G, int D,
                                             int DV, const int* tiles, int n_tiles, int tile_q, const int* block_table, int max_blocks,
                                             int page, int num_pages, int window, int keep_first, const float* sink, float scale,
-                                            int n_splits, int split_keys, float* part_o, float* part_ml, int* err, int key_chunk, float softcap, const float* head_gate, int ld_gate, void* stream) {
+                                            int n_splits, int split_keys, float* part_o, float* part_ml, int* err, int key_chunk, float softcap, const float* head_gate, int ld_gate, const float* slopes, void* stream) {
     if (n_tiles <= 0 || T_tokens <= 0) return 0;
     if (D <= 0 || DV <= 0 || (D & 15) || (DV & 15) || (!v_pool && DV > D) || DV > 512) return fail("shared_row_attention_tc: rows of %d / %d are not taken", D, DV);
     if (H <= 0 || G <= 0 || H % G) return fail("shared_row_attention_tc: %d heads do not divide into %d groups", H, G);
@@ -1280,7 +1310,7 @@ EMBER_API int ember_shared_row_attention_tc(const void* q, const void* k_pool, c
     p.H = H; p.G = G; p.D = D; p.DV = DV; p.head_chunk = chunk; p.window = window; p.keep_first = keep_first; p.scale = scale;
     p.n_splits = n_splits; p.split_keys = split_keys; p.err = err;
     if (key_chunk < 0 || softcap < 0.0f || (head_gate && ld_gate < H)) return fail("sink_attention: chunk %d, score cap %g, gate rows of %d", key_chunk, softcap, ld_gate);
-    p.chunk = key_chunk; p.softcap = softcap; p.head_gate = head_gate; p.ld_gate = ld_gate;
+    p.chunk = key_chunk; p.softcap = softcap; p.head_gate = head_gate; p.ld_gate = ld_gate; p.slopes = slopes;
     cudaStream_t st = (cudaStream_t)stream;
     return out_f32 ? launch_shared_row_tc<float>(p, n_tiles, T_tokens, st) : launch_shared_row_tc<__nv_bfloat16>(p, n_tiles, T_tokens, st);
 }

@@ -20,7 +20,8 @@ EPI_SUMS = 5      # tensor-core product of at most 128 tokens: the fp32 sums sta
 EPI_RELU_MUL = 6  # the gated epilogue with relu: relu(c[2j]) * c[2j + 1]
 EPI_GELU_MUL = 7  # ... with the tanh form of gelu: 0.5 g (1 + tanh(sqrt(2 / pi) (g + 0.044715 g^3))) * c[2j + 1]
 EPI_GELU = 8      # gelu(c + bias) in its exact form, 0.5 z (1 + erf(z / sqrt 2)), stored like EPI_STORE
-PLAIN_EPILOGUES = (EPI_STORE, EPI_STORE_F32, EPI_ADD_F32, EPI_GELU)      # those that take a bias in both products
+EPI_SQUARE_RELU = 9      # max(c + bias, 0)^2, stored like EPI_STORE
+PLAIN_EPILOGUES = (EPI_STORE, EPI_STORE_F32, EPI_ADD_F32, EPI_GELU, EPI_SQUARE_RELU)      # those that take a bias in both products
 GATED_EPILOGUES = (EPI_SILU_MUL, EPI_RELU_MUL, EPI_GELU_MUL)
 GATED_EPILOGUE_OF = {"silu": EPI_SILU_MUL, "relu": EPI_RELU_MUL, "gelu_tanh": EPI_GELU_MUL}
 
@@ -264,7 +265,7 @@ def gemm_simt(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, M: int, epilo
     if a.shape[-1] != K:
         raise KernelError(f"gemm: activations of width {a.shape[-1]} against weights {tuple(w.shape)}")
     n_out = N // 2 if epilogue in GATED_EPILOGUES else N
-    want = a.dtype if epilogue in (EPI_STORE, EPI_GELU) + GATED_EPILOGUES else torch.float32
+    want = a.dtype if epilogue in (EPI_STORE, EPI_GELU, EPI_SQUARE_RELU) + GATED_EPILOGUES else torch.float32
     if out.dtype != want:
         raise KernelError(f"gemm: epilogue {epilogue} writes {want}, the output is {out.dtype}")
     if out.shape[-1] != n_out or out.numel() < M * n_out or a.numel() < M * K:
@@ -431,7 +432,7 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, M: int, epilogu
         return scratch[:M * N].view(M, N)
     _check(out, "out")
     n_out = N // 2 if epilogue in GATED_EPILOGUES else N
-    want = torch.bfloat16 if epilogue in (EPI_STORE, EPI_GELU) + GATED_EPILOGUES else torch.float32
+    want = torch.bfloat16 if epilogue in (EPI_STORE, EPI_GELU, EPI_SQUARE_RELU) + GATED_EPILOGUES else torch.float32
     if out.dtype != want:
         raise KernelError(f"gemm: epilogue {epilogue} writes {want}, the output is {out.dtype}")
     if out.shape[-1] != n_out or out.numel() < M * n_out or a.numel() < M * K:
@@ -905,11 +906,15 @@ def _check_runs(query_start: torch.Tensor, slots: torch.Tensor, S: int) -> None:
 
 def conv_silu(x: torch.Tensor, col: int, taps: torch.Tensor, bias: Optional[torch.Tensor], carry: torch.Tensor,
               carry_col: int, seq_of: torch.Tensor, query_start: torch.Tensor, slots: torch.Tensor, out: torch.Tensor,
-              T: int, S: int, stream: Optional[int] = None, silu: bool = True) -> None:
+              T: int, S: int, stream: Optional[int] = None, silu: bool = True, rounded: Optional[torch.Tensor] = None) -> None:
     """Short causal convolution per channel + silu (``silu`` False: the convolution alone) over the step's runs.  ``x`` fp32 [T, ld]: channels are its
     columns col .. col + C; ``taps`` fp32 [C, n] (the last column meets the current token); ``carry`` fp32
     [slots, row]: a request's last n - 1 inputs live at columns carry_col .. carry_col + (n - 1) C of its row and
-    are replaced by this step's."""
+    are replaced by this step's.  ``rounded`` (bfloat16, like ``out``) also receives the rows."""
+    if rounded is not None:
+        _check(rounded, "rounded", torch.bfloat16)
+        if rounded.numel() < T * taps.shape[0]:
+            raise KernelError("conv_silu: the rounded rows do not fit")
     for t, n in ((x, "x"), (taps, "taps"), (carry, "carry"), (out, "out")):
         _check(t, n, torch.float32)
     _check(seq_of, "seq_of", torch.int32)
@@ -920,8 +925,8 @@ def conv_silu(x: torch.Tensor, col: int, taps: torch.Tensor, bias: Optional[torc
         raise KernelError(f"conv_silu: {C} channels x {n} taps from column {col} of {tuple(x.shape)}, carry {tuple(carry.shape)}")
     lib = _lib("recurrent")
     _call(lib, lib.ember_conv_silu, _p(x), c_int(x.shape[1]), c_int(col), _p(taps), _p(bias), c_int(n), _off(carry, carry_col),
-          c_longlong(carry.shape[1]), _p(seq_of), _p(query_start), _p(slots), _p(out), c_int(T), c_int(S), c_int(C),
-          c_int(1 if silu else 0), _stream(stream))
+          c_longlong(carry.shape[1]), _p(seq_of), _p(query_start), _p(slots), _p(out), _p(rounded), c_int(T), c_int(S),
+          c_int(C), c_int(1 if silu else 0), _stream(stream))
 
 
 def delta_scan(conv: torch.Tensor, beta: torch.Tensor, beta_col: int, a: torch.Tensor, a_col: int, dt_bias: torch.Tensor,
@@ -982,6 +987,32 @@ def ssm_scan(conv: torch.Tensor, dt: torch.Tensor, dt_col: int, dt_bias: torch.T
     _call(lib, lib.ember_ssm_scan, _p(conv), c_int(conv.shape[1]), _off(dt, dt_col), c_int(dt.shape[1]), _p(dt_bias), _p(A_log),
           _p(skip), _p(state), c_longlong(state.shape[1]), _p(out), _p(query_start), _p(slots), c_int(T), c_int(S), c_int(heads),
           c_int(groups), c_int(n_state), c_int(vdim), _stream(stream))
+
+
+SELECTIVE_MAX_STATES = 256       # states a channel the selective scan takes
+
+
+def selective_scan(x: torch.Tensor, dt: torch.Tensor, bc: torch.Tensor, bc_col: int, z: torch.Tensor, z_col: int, dt_bias: torch.Tensor,
+                   a: torch.Tensor, skip: torch.Tensor, state: torch.Tensor, out: torch.Tensor, query_start: torch.Tensor,
+                   slots: torch.Tensor, T: int, S: int, stream: Optional[int] = None) -> None:
+    """Selective scan with a diagonal state per channel over the step's runs (csrc/selective_scan.cu).  ``x`` fp32 [T, inner]
+    (after convolution and silu), ``dt`` fp32 [T, inner] raw steps (softplus of them plus ``dt_bias`` is taken here), ``bc`` fp32
+    with B and C behind one another from column ``bc_col`` on, ``z`` fp32 with the gate from column ``z_col`` on, ``a`` fp32
+    [inner, states] = -exp(A_log) log2(e), ``skip`` [inner]; a request's state is the first inner * states floats of its row
+    of ``state``.  out [T, inner] (fp32 or bfloat16) = (S C + skip x) silu(z)."""
+    for t, n in ((x, "x"), (dt, "dt"), (bc, "bc"), (z, "z"), (dt_bias, "dt_bias"), (a, "a"), (skip, "skip"), (state, "state")):
+        _check(t, n, torch.float32)
+    _check(out, "out")
+    _check_runs(query_start, slots, S)
+    inner, N = a.shape
+    if x.shape[-1] != inner or dt.shape[-1] != inner or z.shape[-1] < z_col + inner or bc.shape[-1] < bc_col + 2 * N or \
+            min(x.shape[0], dt.shape[0], z.shape[0], bc.shape[0]) < T or dt_bias.numel() != inner or skip.numel() != inner or \
+            out.shape[-1] != inner or out.numel() < T * inner or state.dim() != 2 or state.shape[1] < inner * N:
+        raise KernelError(f"selective_scan: buffers do not fit {inner} channels of {N} states")
+    lib = _lib("selective_scan")
+    _call(lib, lib.ember_selective_scan, _p(x), c_int(x.shape[-1]), _p(dt), c_int(dt.shape[-1]), _off(bc, bc_col), c_int(bc.shape[-1]),
+          _off(z, z_col), c_int(z.shape[-1]), _p(dt_bias), _p(a), _p(skip), _p(state), c_longlong(state.shape[1]), _p(out),
+          c_int(dtype_code(out.dtype)), _p(query_start), _p(slots), c_int(T), c_int(S), c_int(inner), c_int(N), _stream(stream))
 
 
 def token_shift(x: torch.Tensor, mu: torch.Tensor, carry: torch.Tensor, carry_col: int, seq_of: torch.Tensor,
@@ -1131,6 +1162,13 @@ def _check_head_gate(head_gate, T: int, heads: int, col: int = 0) -> None:
             raise KernelError(f"attention: a head gate of {tuple(head_gate.shape)} from column {col} for {T} tokens of {heads} heads")
 
 
+def _check_slopes(slopes, heads: int) -> None:
+    if slopes is not None:
+        _check(slopes, "slopes", torch.float32)
+        if slopes.numel() != heads:
+            raise KernelError(f"attention: {slopes.numel()} distance slopes for {heads} heads")
+
+
 def head_gate_apply(x: torch.Tensor, gate: torch.Tensor, gate_col: int, T: int, heads: int, vdim: int, stream: Optional[int] = None) -> None:
     """x[t, h, :] *= sigmoid(gate[t, gate_col + h]) in place (x [T, heads vdim] bfloat16 or float32, gate fp32 logits)."""
     _check(x, "x")
@@ -1158,13 +1196,15 @@ def head_prepare_store(qkv: torch.Tensor, bias: Optional[torch.Tensor], norm_mod
                        q_temp_every: int, T: int, heads: int, kv_heads: int, dim: int, vdim: int, positions: torch.Tensor,
                        seq_of: torch.Tensor, block_table: torch.Tensor, page: int, k_pool: torch.Tensor, v_pool: torch.Tensor,
                        q_out: torch.Tensor, write_kv: bool = True, err: Optional[torch.Tensor] = None,
-                       stream: Optional[int] = None, magnitude: float = 1.0) -> None:
+                       stream: Optional[int] = None, magnitude: float = 1.0, mix_out: Optional[torch.Tensor] = None,
+                       mix_in: Optional[torch.Tensor] = None, mix_factor: Optional[torch.Tensor] = None) -> None:
     """A token's q/k/v (``qkv`` fp32 [T, q | k | v], plus ``bias``) made ready for attention: an RMS norm of queries and
     keys (``norm_mode`` "none", "whole": over the whole projection with weights of that size, "head": per head with
     weights of ``dim`` shared by the heads), the rotation of the first ``rotary`` elements of every query and key head
     (element i with i + rotary / 2, angle position * inv_freq[i], cosines and sines times ``magnitude``), the query times
     1 + q_temp_coef * ln(floor((position + 1) / q_temp_every) + 1) (``q_temp_every`` 0: not); queries to ``q_out``, keys and
-    values into the token's page."""
+    values into the token's page.  ``mix_out`` (fp32 [T, kv_heads vdim]) also receives the values; with ``mix_in`` (the same
+    shape) and ``mix_factor`` (fp32, one number f) the page gets (1 - f) v + f mix_in instead of v."""
     _check(qkv, "qkv", torch.float32)
     modes = {"none": 0, "whole": 1, "head": 2}
     if norm_mode not in modes:
@@ -1180,6 +1220,13 @@ def head_prepare_store(qkv: torch.Tensor, bias: Optional[torch.Tensor], norm_mod
         raise KernelError("head_prepare_store: a norm needs its weights")
     if rotary and inv_freq is None:
         raise KernelError("head_prepare_store: a rotation needs its frequencies")
+    for t, n in ((mix_out, "mix_out"), (mix_in, "mix_in")):
+        if t is not None:
+            _check(t, n, torch.float32)
+            if t.numel() < T * kv_heads * vdim or t.shape[-1] != kv_heads * vdim:
+                raise KernelError(f"head_prepare_store: {n} {tuple(t.shape)} does not hold the values of {T} tokens")
+    if mix_in is not None:
+        _check(mix_factor, "mix_factor", torch.float32)
     _check(positions, "positions", torch.int32)
     _check(seq_of, "seq_of", torch.int32)
     _check(block_table, "block_table", torch.int32)
@@ -1194,7 +1241,7 @@ def head_prepare_store(qkv: torch.Tensor, bias: Optional[torch.Tensor], norm_mod
           c_float(eps), _p(inv_freq), c_int(rotary), c_float(magnitude), c_float(q_temp_coef), c_int(q_temp_every), c_int(T), c_int(heads), c_int(kv_heads),
           c_int(dim), c_int(vdim), _p(positions), _p(seq_of), _p(block_table), c_int(block_table.shape[-1]), c_int(page),
           c_int(k_pool.shape[0]), _p(q_out), _p(k_pool), _p(v_pool), c_int(dtype_code(q_out.dtype)), c_int(1 if write_kv else 0),
-          _p(err), _stream(stream))
+          _p(err), _p(mix_out), _p(mix_in), _p(mix_factor if mix_in is not None else None), _stream(stream))
 
 
 def whole_norm_store(qkv: torch.Tensor, bias: Optional[torch.Tensor], q_w: Optional[torch.Tensor], k_w: Optional[torch.Tensor],
@@ -1311,14 +1358,17 @@ def sink_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: Optional[torch
                    page: int, window: int, keep_first: int, sink: Optional[torch.Tensor], scale: float, n_splits: int = 1,
                    split_keys: int = 0, part_o: Optional[torch.Tensor] = None, part_ml: Optional[torch.Tensor] = None,
                    err: Optional[torch.Tensor] = None, stream: Optional[int] = None, chunk: int = 0,
-                   softcap: float = 0.0, head_gate: Optional[torch.Tensor] = None, head_gate_col: int = 0) -> None:
+                   softcap: float = 0.0, head_gate: Optional[torch.Tensor] = None, head_gate_col: int = 0,
+                   slopes: Optional[torch.Tensor] = None) -> None:
     """out[t, h] = sum_j w_j v_j over the visible keys j <= t (under a window: t - j < window or j < keep_first), w the
     softmax of scale * q . k_j whose denominator also holds exp(sink[h]).  Keys [.., dim], values [.., vdim]; without
     ``v_pool`` a value is the first ``vdim`` elements of the key row.  ``out`` is q's dtype or float32.  ``chunk`` > 0:
     j is visible only if floor(t / chunk) == floor(j / chunk) (positions, counted from the sequence's start);
     ``softcap`` > 0: the scaled score becomes softcap * tanh(score / softcap); ``head_gate`` (fp32 [T, >= heads] logits):
-    head h's output is multiplied by sigmoid(head_gate[t, head_gate_col + h])."""
+    head h's output is multiplied by sigmoid(head_gate[t, head_gate_col + h]); ``slopes`` (fp32 [heads]): slopes[h] * (t - j)
+    is taken off the score after the cap."""
     _check_head_gate(head_gate, T, heads, head_gate_col)
+    _check_slopes(slopes, heads)
     _check(q, "q")
     _check(k_pool, "k_pool", q.dtype)
     if v_pool is not None:
@@ -1346,7 +1396,7 @@ def sink_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: Optional[torch
           c_int(n_tiles), c_int(tile_q), _p(block_table), c_int(block_table.shape[-1]), c_int(page), c_int(k_pool.shape[0]),
           c_int(window), c_int(keep_first), _p(sink), c_float(scale), c_int(n_splits), c_int(split_keys), _p(part_o), _p(part_ml),
           _p(err), c_int(chunk), c_float(softcap), (_off(head_gate, head_gate_col) if head_gate is not None else _p(None)), c_int(head_gate.shape[-1] if head_gate is not None else 0),
-          _stream(stream))
+          _p(slopes), _stream(stream))
 
 
 # --------------------------------------------------------------------- routed feed-forward (csrc/moe.cu)
@@ -1428,7 +1478,8 @@ def moe_group(sel: torch.Tensor, n_pairs: int, experts: int, offsets: torch.Tens
 
 def moe_gemm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, offsets: torch.Tensor, pair_of_slot: torch.Tensor,
              tiles: torch.Tensor, max_tiles: int, top: int, gated: bool, limit: float = 0.0, alpha: float = 1.0,
-             stream: Optional[int] = None, streaming: bool = False, up_offset: float = 1.0, square_relu: bool = False) -> None:
+             stream: Optional[int] = None, streaming: bool = False, up_offset: float = 1.0, square_relu: bool = False,
+             in_weights: Optional[torch.Tensor] = None) -> None:
     """The product of every slot's row with its expert's matrix (``w`` [experts, N, K]).  ``top`` > 0: a slot's row of
     ``x`` is its token's (x [tokens, K], gathered through the pairs); 0: x has a row per slot.  ``gated``: w's rows are
     interleaved (gate, up) and out[slot, j] = g sigmoid(alpha g) (u + up_offset) with g = min(gate, limit),
@@ -1437,6 +1488,10 @@ def moe_gemm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, offsets: torch
     lists of 16-row tiles (``moe_group`` with ``MOE_STREAM_ROWS``), else the form for 32-row tiles."""
     _check(x, "x")
     _check(w, "w", x.dtype)
+    if in_weights is not None:                               # fp32, one per pair: multiplies the expert's input
+        _check(in_weights, "in_weights", torch.float32)
+        if not gated:
+            raise KernelError("moe_gemm: weights on the input belong to the gated product")
     if gated and square_relu:
         raise KernelError("moe_gemm: relu^2 is the activation of an ungated product")
     _check(out, "out", x.dtype if (gated or square_relu) else torch.float32)
@@ -1448,17 +1503,18 @@ def moe_gemm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, offsets: torch
     _call(lib, lib.ember_moe_stream if streaming else lib.ember_moe_gemm, _p(x), c_int(dtype_code(x.dtype)), c_int(K), _p(w), c_int(dtype_code(w.dtype)), c_longlong(N * K),
           _p(out), c_int(dtype_code(out.dtype)), c_int(n_out), _p(offsets), _p(pair_of_slot), _off(tiles, 0), _off(tiles, 1),
           _off(tiles, 1 + max_tiles), c_int(max_tiles), c_int(top), c_int(N), c_int(K), c_int(1 if gated else 0), c_float(limit),
-          c_float(alpha), c_float(up_offset), c_int(1 if square_relu else 0), _stream(stream))
+          c_float(alpha), c_float(up_offset), c_int(1 if square_relu else 0), _p(in_weights), _stream(stream))
 
 
-def moe_combine(y: torch.Tensor, wgt: torch.Tensor, slot_of_pair: torch.Tensor, T: int, top: int, out: torch.Tensor,
+def moe_combine(y: torch.Tensor, wgt: Optional[torch.Tensor], slot_of_pair: torch.Tensor, T: int, top: int, out: torch.Tensor,
                 accumulate: bool = False, stream: Optional[int] = None, sel: Optional[torch.Tensor] = None, experts: int = 0,
                 same: Optional[torch.Tensor] = None) -> None:
     """out[t] (+)= sum over the token's choices, in order, of wgt[t, k] * y[slot of (t, k)]; all fp32.  With ``sel``
     (the choices) a choice from ``experts`` on is an identity expert, whose output is the token's row of ``same``
     (fp32 or bfloat16 [T, hidden]) instead of a row of y."""
     _check(y, "y", torch.float32)
-    _check(wgt, "wgt", torch.float32)
+    if wgt is not None:                                      # (None: every weight is one)
+        _check(wgt, "wgt", torch.float32)
     _check(out, "out", torch.float32)
     _check(slot_of_pair, "slot_of_pair", torch.int32)
     hidden = out.shape[-1]
@@ -1475,8 +1531,14 @@ def moe_combine(y: torch.Tensor, wgt: torch.Tensor, slot_of_pair: torch.Tensor, 
           c_int(dtype_code(same.dtype) if sel is not None else 0), _stream(stream))
 
 
-def moe_gather(x: torch.Tensor, pair_of_slot: torch.Tensor, n_pairs: int, top: int, xs: torch.Tensor, stream: Optional[int] = None) -> None:
-    """xs[slot] = x[token of the slot's pair]: every expert's rows side by side (rows of a multiple of 16 bytes)."""
+def moe_gather(x: torch.Tensor, pair_of_slot: torch.Tensor, n_pairs: int, top: int, xs: torch.Tensor, stream: Optional[int] = None,
+               weights: Optional[torch.Tensor] = None) -> None:
+    """xs[slot] = x[token of the slot's pair]: every expert's rows side by side (rows of a multiple of 16 bytes); with
+    ``weights`` (fp32, one per pair; bfloat16 rows) each row times its pair's weight."""
+    if weights is not None:
+        _check(weights, "weights", torch.float32)
+        if x.dtype != torch.bfloat16 or weights.numel() < n_pairs:
+            raise KernelError("moe_gather: weighted rows are bfloat16, with a weight for every pair")
     _check(x, "x")
     _check(xs, "xs", x.dtype)
     _check(pair_of_slot, "pair_of_slot", torch.int32)
@@ -1484,7 +1546,7 @@ def moe_gather(x: torch.Tensor, pair_of_slot: torch.Tensor, n_pairs: int, top: i
     if xs.shape[-1] != x.shape[-1] or xs.numel() < n_pairs * x.shape[-1] or pair_of_slot.numel() < n_pairs:
         raise KernelError("moe_gather: buffers do not fit the step")
     lib = _lib("moe")
-    _call(lib, lib.ember_moe_gather, _p(x), _p(pair_of_slot), c_int(n_pairs), c_int(top), _p(xs), c_int(row), _stream(stream))
+    _call(lib, lib.ember_moe_gather, _p(x), _p(pair_of_slot), c_int(n_pairs), c_int(top), _p(xs), c_int(row), _p(weights), _stream(stream))
 
 
 def moe_activation(gu: torch.Tensor, act: torch.Tensor, rows: int, limit: float, alpha: float, stream: Optional[int] = None,
@@ -1555,9 +1617,11 @@ def shared_row_attention_tc(q: torch.Tensor, k_pool: torch.Tensor, v_pool: Optio
                             window: int, keep_first: int, sink: Optional[torch.Tensor], scale: float, n_splits: int = 1,
                             split_keys: int = 0, part_o: Optional[torch.Tensor] = None, part_ml: Optional[torch.Tensor] = None,
                             err: Optional[torch.Tensor] = None, stream: Optional[int] = None, chunk: int = 0,
-                   softcap: float = 0.0, head_gate: Optional[torch.Tensor] = None, head_gate_col: int = 0) -> None:
+                   softcap: float = 0.0, head_gate: Optional[torch.Tensor] = None, head_gate_col: int = 0,
+                   slopes: Optional[torch.Tensor] = None) -> None:
     """``sink_attention`` on the tensor cores (bfloat16 queries, keys, values; scores, weights and sums fp32)."""
     _check_head_gate(head_gate, T, heads, head_gate_col)
+    _check_slopes(slopes, heads)
     _check(q, "q", torch.bfloat16)
     _check(k_pool, "k_pool", torch.bfloat16)
     if v_pool is not None:
@@ -1584,4 +1648,4 @@ def shared_row_attention_tc(q: torch.Tensor, k_pool: torch.Tensor, v_pool: Optio
           c_int(heads), c_int(kv_heads), c_int(dim), c_int(vdim), _p(tiles), c_int(n_tiles), c_int(tile_q), _p(block_table),
           c_int(block_table.shape[-1]), c_int(page), c_int(k_pool.shape[0]), c_int(window), c_int(keep_first), _p(sink),
           c_float(scale), c_int(n_splits), c_int(split_keys), _p(part_o), _p(part_ml), _p(err), c_int(chunk), c_float(softcap),
-          (_off(head_gate, head_gate_col) if head_gate is not None else _p(None)), c_int(head_gate.shape[-1] if head_gate is not None else 0), _stream(stream))
+          (_off(head_gate, head_gate_col) if head_gate is not None else _p(None)), c_int(head_gate.shape[-1] if head_gate is not None else 0), _p(slopes), _stream(stream))

@@ -14,7 +14,7 @@ from typing import List, Optional
 import torch
 
 from .. import ops
-from ..config.spec import ConfigError
+from ..config.spec import ConfigError, GatedMLPSpec
 from .base import FeedForward, Runtime, WeightDecl
 from .linear import Linear
 from .registry import register_part
@@ -89,15 +89,18 @@ class GatedMLP(FeedForward):
 
 
 class PlainMLP(FeedForward):
-    """Two matrices: down(gelu(up(x) + b) + b), the exact gelu; both biases and the activation are the products' epilogues."""
+    """Two matrices: down(act(up(x) + b) + b), act the exact gelu or relu squared; biases and activation are the products'
+    epilogues."""
+
+    EPILOGUE_OF = {"gelu": ops.EPI_GELU, "square_relu": ops.EPI_SQUARE_RELU}
 
     graph_safe = True
     can_store = True
 
     def __init__(self, spec, prefix: str = ""):
         super().__init__(spec, prefix)
-        if spec.activation != "gelu":
-            raise ConfigError(f"feed-forward of two matrices: activation {spec.activation!r} is not supported (gelu)")
+        if spec.activation not in self.EPILOGUE_OF:
+            raise ConfigError(f"feed-forward of two matrices: activation {spec.activation!r} is not supported ({', '.join(self.EPILOGUE_OF)})")
         if min(spec.hidden_size, spec.intermediate_size) <= 0:
             raise ConfigError("feed-forward: sizes must be positive")
 
@@ -123,7 +126,7 @@ class PlainMLP(FeedForward):
 
     def forward(self, ctx, x: torch.Tensor, residual: torch.Tensor, accumulate: bool = True) -> None:
         act = ctx.buf("mlp.act", (ctx.max_tokens, self.spec.intermediate_size), self.rt.dtype)
-        self.up(ctx, x, act, ctx.T, ops.EPI_GELU)
+        self.up(ctx, x, act, ctx.T, self.EPILOGUE_OF[self.spec.activation])
         self.down(ctx, act, residual, ctx.T, ops.EPI_ADD_F32 if accumulate else ops.EPI_STORE_F32)
 
 
@@ -154,7 +157,10 @@ class RoutedMLP(FeedForward):
     largest), and the choice is among the outputs of the
     ``keep_groups`` best groups.  ``identity``: the router has experts + identity outputs, the last ones experts without
     tensors whose output is the token's input itself (``forward(..., stream=)`` hands the fp32 input where the caller has
-    it; else the product's input is used).  ``expert`` "square_relu": W_down relu(W_up h)^2, no gate matrix."""
+    it; else the product's input is used).  ``expert`` "square_relu": W_down relu(W_up h)^2, no gate matrix.  ``weigh`` "input": an
+    expert reads weight * h and the results are added as they are (the weight enters as a factor of the gate and up sums, or
+    of the gathered rows).  ``shared_size``: one more gated expert (tensors shared.gate, shared.up, shared.down) that every token
+    uses, unweighted."""
 
     graph_safe = True
     can_store = True
@@ -186,6 +192,12 @@ class RoutedMLP(FeedForward):
             raise ConfigError(f"routed feed-forward: {self.outputs} router outputs in {s.groups} groups (at most 32, equal) of "
                               f"which {s.keep_groups} are kept for top {s.top}")
         self.gated = s.expert == "gated"
+        if s.weigh not in ("output", "input") or (s.weigh == "input" and (not self.gated or s.identity)):
+            raise ConfigError(f"routed feed-forward: weights on the {s.weigh!r} (output, or input with gated experts alone)")
+        if s.shared_size < 0:
+            raise ConfigError(f"routed feed-forward: a shared expert of {s.shared_size}")
+        self.shared = GatedMLP(GatedMLPSpec(hidden_size=s.hidden_size, intermediate_size=s.shared_size, names=("gate", "up", "down")),
+                               prefix + "shared.") if s.shared_size else None
         self.limit = float(s.limit) if s.limit > 0 else float("inf")
         self.plain_silu = self.gated and s.limit == 0 and s.alpha == 1.0 and s.up_offset == 0.0     # silu(gate) * up
 
@@ -199,12 +211,17 @@ class RoutedMLP(FeedForward):
                 d.append(WeightDecl(f"{p}e{e}.gate", (s.intermediate_size, s.hidden_size)))
             d += [WeightDecl(f"{p}e{e}.up", (s.intermediate_size, s.hidden_size)),
                   WeightDecl(f"{p}e{e}.down", (s.hidden_size, s.intermediate_size))]
-        return d
+        return d + (self.shared.weight_decls() if self.shared else [])
 
     def load(self, store, rt: Runtime) -> None:
         s, p = self.spec, self.prefix
         self.rt = rt
-        got = {d.name: store.take(d.name, d.shape) for d in self.weight_decls()}
+        if self.shared:
+            self.shared.load(store, rt)
+        mine = self.weight_decls()
+        if self.shared:
+            mine = mine[:-len(self.shared.weight_decls())]
+        got = {d.name: store.take(d.name, d.shape) for d in mine}
         if any(v is None for v in got.values()):
             return
         wd = rt.weight_dtype(got[f"{p}e0.up"].dtype)
@@ -250,14 +267,18 @@ class RoutedMLP(FeedForward):
         tiles = ctx.buf("routed_mlp.tiles", (1 + 2 * ops.moe_max_tiles(mt * top, E, ops.MOE_STREAM_ROWS),), torch.int32)
         act = ctx.buf("routed_mlp.act", (mt * top, s.intermediate_size), rt.dtype)
         y = ctx.buf("routed_mlp.down", (mt * top, s.hidden_size), torch.float32)
+        if self.shared:
+            self.shared.forward(ctx, x, residual, accumulate=accumulate)
+            accumulate = True
         ops.moe_router(x, self.router, T, top, sel, wgt, stream=ctx.stream, rule=self.rule)
+        in_wgt, wgt = (wgt, None) if s.weigh == "input" else (None, wgt)
         streaming = (T <= self.STREAM_MAX_TOKENS and ops.moe_stream_usable(x, s.hidden_size)
                      and ops.moe_stream_usable(x, s.intermediate_size))
         max_tiles = ops.moe_group(sel, pairs, E, offsets, pair_of_slot, slot_of_pair, tiles,
                                   ops.MOE_STREAM_ROWS if streaming else ops.MOE_TILE_ROWS, stream=ctx.stream, tiled=s.experts)
         if self._on_tensor_cores(ctx, x):
             xs = ctx.buf("routed_mlp.gathered", (mt * top, s.hidden_size), rt.dtype)
-            ops.moe_gather(x, pair_of_slot, pairs, top, xs, stream=ctx.stream)
+            ops.moe_gather(x, pair_of_slot, pairs, top, xs, stream=ctx.stream, weights=in_wgt)
             if self.plain_silu:
                 ops.gemm_tc_grouped(xs, self.gate_up, act, pairs, offsets, ops.EPI_SILU_MUL, err=ctx.err, stream=ctx.stream)
             else:
@@ -270,7 +291,7 @@ class RoutedMLP(FeedForward):
             ops.gemm_tc_grouped(act, self.down, y, pairs, offsets, ops.EPI_STORE_F32, err=ctx.err, stream=ctx.stream)
         else:
             ops.moe_gemm(x, self.gate_up, act, offsets, pair_of_slot, tiles, max_tiles, top, self.gated, self.limit, s.alpha,
-                         stream=ctx.stream, streaming=streaming, up_offset=s.up_offset, square_relu=not self.gated)
+                         stream=ctx.stream, streaming=streaming, up_offset=s.up_offset, square_relu=not self.gated, in_weights=in_wgt)
             ops.moe_gemm(act, self.down, y, offsets, pair_of_slot, tiles, max_tiles, 0, False, stream=ctx.stream, streaming=streaming)
         if s.identity:
             ops.moe_combine(y, wgt, slot_of_pair, T, top, residual, accumulate=accumulate, stream=ctx.stream, sel=sel,

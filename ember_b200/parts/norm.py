@@ -1,7 +1,8 @@
 """Norms.  RMSNorm: out = weight * (x * rsqrt(mean(x^2) + eps)), statistics in fp32.
 
 Formula: src/backend/cpu/cpu_backend.cpp:34-39 (the weight multiplies after the scaling; it
-is the plain weight, not 1 + weight).
+is the plain weight there).  A design that stores its weights around zero gives ``weight_offset`` 1: the
+sum is made once, in fp32, when the weights are loaded.
 """
 from __future__ import annotations
 
@@ -21,11 +22,17 @@ class RMSNorm(Norm):
         return self.prefix + getattr(self.spec, "weight_suffix", "weight")
 
     def weight_decls(self) -> List[WeightDecl]:
-        return [WeightDecl(self._name(), (self.spec.size,), init="norm")]
+        # (the random weights of a norm are near one, those of an offset norm near zero)
+        return [WeightDecl(self._name(), (self.spec.size,), init="zeros" if self._offset() else "norm")]
+
+    def _offset(self) -> float:
+        return float(getattr(self.spec, "weight_offset", 0.0))
 
     def load(self, store, rt: Runtime) -> None:
         w = store.take(self._name(), (self.spec.size,))
         self.weight = rt.to_device(w, torch.float32) if w is not None else None
+        if self.weight is not None and self._offset():
+            self.weight = self.weight + self._offset()
 
     def scale_output(self, scale: float) -> None:
         if self.weight is not None:

@@ -5,7 +5,8 @@
 * "mamba2":        selective state space with a scalar decay per head,
 * "gla":           linear attention with a decay per head and key channel (no convolution, no delta correction),
 * "wkv":           time mixing: blends with the previous token's input, a data-dependent decay per head and key channel,
-                   a read-out of the state before its update plus a bonus for the current token.
+                   a read-out of the state before its update plus a bonus for the current token,
+* "mamba1":        selective scan with a diagonal state per channel (a step, a B and a C per token).
 
 All of them project their input with one fused product whose fp32 result the recurrence kernel reads in place (column
 offsets, no copies), run the same kernels for prompt portions and single tokens (a block walks its run's tokens in
@@ -423,6 +424,74 @@ class TimeMix(_StateMixer):
         self._out(ctx, y, out, accumulate)
 
 
+# ---------------------------------------------------------------------------------------------- mamba1
+class SelectiveScan(_StateMixer):
+    """W_in h = [x | z]; x passes a short causal convolution (with bias) and silu; W_x x = [low | B | C];
+    dt = softplus(W_dt low + dt.b), one per channel; per channel c and state n
+
+        S[c, n] <- exp(-dt_c exp(A_log[c, n])) S[c, n] + dt_c x_c B_n;  y_c = sum_n S[c, n] C_n + D_c x_c
+
+    then y * silu(z) and the output product.  The products read bfloat16 operands on the bfloat16 path and leave fp32; steps,
+    decays, B, C and the state are fp32.  The step's projection reads ``low`` where the product before it left it.  The
+    state row of a request holds S [inner, states] and, behind it, the convolution's last inputs.  Tensors under the
+    prefix: in, conv, conv.b, x, dt, dt.b, A_log, D, o."""
+
+    def __init__(self, spec, prefix: str = ""):
+        super().__init__(spec, prefix)
+        s = spec
+        if min(s.hidden_size, s.inner, s.state_size, s.dt_rank, s.conv_taps) <= 0:
+            raise ConfigError("mamba1: sizes must be positive")
+        if s.state_size > ops.SELECTIVE_MAX_STATES or s.conv_taps > 64:
+            raise ConfigError(f"mamba1: {s.state_size} states a channel (at most {ops.SELECTIVE_MAX_STATES}), {s.conv_taps} taps (at most 64)")
+
+    def state_floats(self) -> int:
+        s = self.spec
+        return s.inner * s.state_size + (s.conv_taps - 1) * s.inner
+
+    def weight_decls(self) -> List[WeightDecl]:
+        s, p = self.spec, self.prefix
+        return [WeightDecl(p + "in", (2 * s.inner, s.hidden_size)),
+                WeightDecl(p + "conv", (s.inner, s.conv_taps), init="uniform", lo=-0.5, hi=0.5),
+                WeightDecl(p + "conv.b", (s.inner,), init="zeros"),
+                WeightDecl(p + "x", (s.dt_rank + 2 * s.state_size, s.inner)), WeightDecl(p + "dt", (s.inner, s.dt_rank)),
+                WeightDecl(p + "dt.b", (s.inner,), init="uniform", lo=-5.0, hi=-1.0),
+                WeightDecl(p + "A_log", (s.inner, s.state_size), init="uniform", lo=0.0, hi=2.5),
+                WeightDecl(p + "D", (s.inner,), init="norm"), WeightDecl(p + "o", (s.hidden_size, s.inner))]
+
+    def load(self, store, rt: Runtime) -> None:
+        s, p = self.spec, self.prefix
+        self.rt = rt
+        w = self._take_all(store)
+        if w is None:
+            return
+        self.in_proj, self.x_proj, self.o = (Linear.from_host(w[p + n], rt) for n in ("in", "x", "o"))
+        # (the step's product is the per-head one with a single head: it reads fp32 columns of the product before it)
+        self.dt_w = rt.to_device(w[p + "dt"], rt.dtype).view(1, s.inner, s.dt_rank)
+        self.taps, self.conv_bias, self.dt_bias, self.skip = (rt.to_device(w[p + n], torch.float32) for n in ("conv", "conv.b", "dt.b", "D"))
+        # decays are powers of two: -exp(A_log) log2(e), made in double precision and rounded once
+        self.a = rt.to_device((-torch.exp(w[p + "A_log"].double()) * 1.4426950408889634).float(), torch.float32)
+
+    def forward(self, ctx, x, out, cache, owns_cache: bool = True, accumulate: bool = True) -> None:
+        s, rt, T, mt = self.spec, self.rt, ctx.T, ctx.max_tokens
+        inner, N, R = s.inner, s.state_size, s.dt_rank
+        proj = ctx.buf("mamba1.proj", (mt, 2 * inner), torch.float32)
+        conv = ctx.buf("mamba1.conv", (mt, inner), torch.float32)
+        half = rt.dtype != torch.float32 and self.x_proj.weight.dtype == rt.dtype
+        conv_r = ctx.buf("mamba1.conv_rounded", (mt, inner), rt.dtype) if half else conv
+        low = ctx.buf("mamba1.low", (mt, R + 2 * N), torch.float32)
+        dt = ctx.buf("mamba1.dt", (mt, inner), torch.float32)
+        y = ctx.buf("mamba1.gated", (mt, inner), rt.dtype)
+        self.in_proj(ctx, x, proj, T, ops.EPI_STORE_F32)
+        ops.conv_silu(proj, 0, self.taps, self.conv_bias, cache.state, inner * N, ctx.seq_of, ctx.query_start, ctx.state_slots,
+                      conv, T, ctx.S, stream=ctx.stream, rounded=conv_r if half else None)
+        self.x_proj(ctx, conv_r, low, T, ops.EPI_STORE_F32)
+        ops.head_gemm(low, R, 0, self.dt_w, dt, inner, 0, T, stream=ctx.stream)
+        ops.selective_scan(conv, dt, low, R, proj, inner, self.dt_bias, self.a, self.skip, cache.state, y, ctx.query_start,
+                           ctx.state_slots, T, ctx.S, stream=ctx.stream)
+        self._out(ctx, y, out, accumulate)
+
+
+register_part("mixer", "mamba1", SelectiveScan)
 register_part("mixer", "wkv", TimeMix)
 register_part("mixer", "gla", GatedLinearAttention)
 register_part("mixer", "channel_delta", GatedDelta)

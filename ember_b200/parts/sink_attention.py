@@ -10,7 +10,8 @@
   rotation of queries and keys after the norm; a query temperature that grows with the logarithm of the position; a
   tanh cap on the scaled scores; a chunked mask (i sees j only inside i's chunk of positions, and the pages of chunks that
   have passed go back); a sigmoid gate per head, or one per element, on the attention's output, computed from the
-  mixer's input.  A rotation in neighbouring pairs is the rotate-half form over rows of W_q and W_k put in another order
+  mixer's input; a sink that is one fixed number for all heads; a distance bias slope_h (i - j) taken off the scores;
+  values blended with those of an earlier layer of the step for the same token (a layer is the source or blends).  A rotation in neighbouring pairs is the rotate-half form over rows of W_q and W_k put in another order
   when they are loaded (the even elements of the rotated part, then the odd ones: the same order in queries and keys
   leaves their products as they are), so the kernels know one layout.
 * "latent_attention": queries through a low-rank latent (c_q = RMSNorm(W_dq h), q = W_uq c_q, per head
@@ -56,7 +57,7 @@ class _SinkSoftmax(Mixer):
     TC_MIN_TOKENS = int(__import__("os").environ.get("EMBER_SINK_TC_MIN_TOKENS", "1"))
 
     def _attend(self, ctx, q, k_pool, v_pool, out, table, page, heads, kv_heads, dim, vdim, window, keep_first, sink, scale,
-                chunk: int = 0, softcap: float = 0.0, head_gate=None, head_gate_col: int = 0):
+                chunk: int = 0, softcap: float = 0.0, head_gate=None, head_gate_col: int = 0, slopes=None):
         on_tc = ctx.T >= self.TC_MIN_TOKENS and ops.shared_row_attention_tc_usable(q, v_pool, dim, vdim)
         tile_q = (ops.shared_row_attention_tc_tile_queries if on_tc else ops.sink_attention_tile_queries)(heads // kv_heads)
         tiles, n_tiles = ctx.attention_tiles(tile_q, "all")
@@ -73,12 +74,12 @@ class _SinkSoftmax(Mixer):
             ops.shared_row_attention_tc(q, k_pool, v_pool, out, ctx.T, heads, kv_heads, dim, vdim, tiles, n_tiles, tile_q, table,
                                         page, window, keep_first, sink, scale, n_splits, self.SPLIT_KEYS, part_o, part_ml,
                                         err=ctx.err, stream=ctx.stream, chunk=chunk, softcap=softcap, head_gate=head_gate,
-                                        head_gate_col=head_gate_col)
+                                        head_gate_col=head_gate_col, slopes=slopes)
         else:
             ops.sink_attention(q, k_pool, v_pool, out, ctx.T, heads, kv_heads, dim, vdim, tiles, n_tiles, tile_q, table, page,
                                window, keep_first, sink, scale, n_splits, self.SPLIT_KEYS, part_o, part_ml, err=ctx.err,
                                stream=ctx.stream, chunk=chunk, softcap=softcap, head_gate=head_gate,
-                                        head_gate_col=head_gate_col)
+                                        head_gate_col=head_gate_col, slopes=slopes)
 
 
 class SinkAttention(_SinkSoftmax):
@@ -97,6 +98,9 @@ class SinkAttention(_SinkSoftmax):
             raise ConfigError("sink attention: convolution taps (up to 64), chunk, temperature period and score cap must be >= 0")
         if s.chunk > 0 and s.window > 0:
             raise ConfigError("sink attention: a chunked mask and a window exclude one another")
+        if s.value_mix not in ("", "source", "mix") or s.slope_span < 0 or (s.fixed_sink is not None and not s.sink):
+            raise ConfigError(f"sink attention: value mix {s.value_mix!r} (source, mix or none), slope span {s.slope_span}, a fixed "
+                              "sink needs the sink")
         if s.head_gate and s.element_gate:
             raise ConfigError("sink attention: a gate per head and a gate per element exclude one another")
         self.gate_cols = s.num_heads if s.head_gate else (s.num_heads * s.value_dim if s.element_gate else 0)
@@ -106,18 +110,21 @@ class SinkAttention(_SinkSoftmax):
         self.magnitude = float(self.position.magnitude()) if hasattr(self.position, "magnitude") else 1.0
         self.pairs_of = getattr(s.position, "rotary_dim", 0) if getattr(s.position, "layout", "half") == "interleaved" else 0
         # the general preparation kernel serves whatever the whole-projection one does not know
-        self.general = (s.qk_norm == "head" or s.position.kind != "none" or s.q_temp_every > 0)
-        # Causal softmax over keys and values of equal size (no sink, no window; a cap and chunks are parameters) is what
+        self.general = (s.qk_norm == "head" or s.position.kind != "none" or s.q_temp_every > 0 or bool(s.value_mix)
+                        or s.slope_span > 0)
+        # Causal softmax over keys and values of equal size (no sink, no kept first tokens, no distance bias; a window, a
+        # cap and chunks are parameters) is what
         # the engine's TMA-fed kernels compute (tcgen05 for prompt portions, mma.sync with key splits for single tokens):
         # where they take the geometry, a bfloat16 step goes to them (``load`` decides, once the dtype and the page size
         # are known); a gate per head then is a pass of its own behind them
         self.dense = None
-        if (not s.sink and s.window == 0 and s.value_dim == s.head_dim and s.scale > 0
+        if (not s.sink and (s.window == 0 or s.keep_first == 0) and s.slope_span == 0 and s.value_dim == s.head_dim and s.scale > 0
                 and s.head_dim % 2 == 0 and s.num_heads // s.num_kv_heads <= ops.ATTENTION_MAX_GROUP):
             from ..config.spec import AttentionSpec
             from .attention import Attention
             self.dense = Attention(AttentionSpec(hidden_size=s.hidden_size, num_heads=s.num_heads, num_kv_heads=s.num_kv_heads,
-                                                 head_dim=s.head_dim, softmax_scale=s.scale, softcap=s.softcap, chunk=s.chunk))
+                                                 head_dim=s.head_dim, window=s.window, softmax_scale=s.scale, softcap=s.softcap,
+                                                 chunk=s.chunk))
 
     def weight_decls(self) -> List[WeightDecl]:
         s, p = self.spec, self.prefix
@@ -135,8 +142,10 @@ class SinkAttention(_SinkSoftmax):
                   for n, size in (("q", self.q_dim), ("k", self.k_dim), ("v", self.v_dim))]
         if self.gate_cols:
             d.append(WeightDecl(p + "g", (self.gate_cols, s.hidden_size)))
-        if s.sink:
+        if s.sink and s.fixed_sink is None:
             d.append(WeightDecl(p + "sink", (s.num_heads,), init="uniform", lo=-1.0, hi=1.0))
+        if s.value_mix == "mix":
+            d.append(WeightDecl(p + "vmix", (), init="uniform", lo=0.2, hi=0.8))
         return d
 
     def _half_order(self, t: Optional[torch.Tensor], heads: int) -> Optional[torch.Tensor]:
@@ -167,7 +176,15 @@ class SinkAttention(_SinkSoftmax):
         self.bias = torch.cat([f32(n + ".b") for n in "qkv"]).contiguous() if s.bias else None
         self.q_norm_w = f32("q.norm") if s.qk_norm != "none" else None
         self.k_norm_w = f32("k.norm") if s.qk_norm != "none" else None
-        self.sink = f32("sink") if s.sink else None
+        self.sink = f32("sink") if s.sink and s.fixed_sink is None else None
+        if s.fixed_sink is not None:
+            self.sink = torch.full((s.num_heads,), float(s.fixed_sink), dtype=torch.float32, device=rt.device)
+        self.slopes = None
+        if s.slope_span > 0:
+            self.slopes = torch.tensor([2.0 ** (-s.slope_span * (h + 1) / s.num_heads) for h in range(s.num_heads)], dtype=torch.float32, device=rt.device)
+        self.mix_factor = f32("vmix").reshape(1) if s.value_mix == "mix" else None
+        if s.value_mix == "source":
+            store.allow_unused(p + "vmix")             # (a source layer may carry a factor that nothing reads)
         self.taps = torch.cat([f32(n + ".conv") for n in "qkv"], dim=0).contiguous() if s.conv_taps > 0 else None
         self.inv_freq, self.rotary = self.position.rotary_table(rt)
         if self.dense is not None:
@@ -175,6 +192,19 @@ class SinkAttention(_SinkSoftmax):
             multi, single = self.dense._tc_modes()
             if not (self.DENSE_KERNELS and single and (multi or self.dense._fa())):
                 self.dense = None
+
+    def _values(self, ctx) -> dict:
+        """The step's buffer of the source layer's values, as the preparation kernel writes or reads it."""
+        s = self.spec
+        if not s.value_mix:
+            return {}
+        if s.value_mix == "mix" and "sink_attention.values" not in ctx.memo:
+            raise ops.KernelError("attention blends values, and no layer before it in this step left any")
+        values = ctx.buf("sink_attention.values", (ctx.max_tokens, self.v_dim), torch.float32)
+        if s.value_mix == "source":
+            ctx.memo["sink_attention.values"] = True
+            return {"mix_out": values}
+        return {"mix_in": values, "mix_factor": self.mix_factor}
 
     DENSE_KERNELS = True        # tests switch it off to run such layers on this file's own kernels
 
@@ -224,7 +254,7 @@ class SinkAttention(_SinkSoftmax):
             ops.head_prepare_store(qkv, self.bias, s.qk_norm, self.q_norm_w, self.k_norm_w, s.qk_norm_eps,
                                    self.inv_freq if self.rotary else None, self.rotary, s.q_temp_coef, s.q_temp_every, T, H, G, D, V,
                                    ctx.positions, ctx.seq_of, table, cache.page_tokens, cache.k, cache.v, q, write_kv=owns_cache,
-                                   err=ctx.err, stream=ctx.stream, magnitude=self.magnitude)
+                                   err=ctx.err, stream=ctx.stream, magnitude=self.magnitude, **self._values(ctx))
         else:
             ops.whole_norm_store(qkv, self.bias, self.q_norm_w, self.k_norm_w, s.qk_norm_eps, T, H, G, D, V, ctx.positions,
                                  ctx.seq_of, table, cache.page_tokens, cache.k, cache.v, q, write_kv=owns_cache, err=ctx.err,
@@ -236,7 +266,7 @@ class SinkAttention(_SinkSoftmax):
         else:
             self._attend(ctx, q, cache.k, cache.v, att, table, cache.page_tokens, H, G, D, V, s.window, s.keep_first, self.sink,
                          s.scale, chunk=s.chunk, softcap=s.softcap, head_gate=proj if s.head_gate else None,
-                         head_gate_col=self.channels)
+                         head_gate_col=self.channels, slopes=self.slopes)
             if s.element_gate:
                 ops.element_gate_apply(att, proj, self.channels, T, H * V, stream=ctx.stream)
         self.o(ctx, att, out, T, ops.EPI_ADD_F32 if accumulate else ops.EPI_STORE_F32)
