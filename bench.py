@@ -23,6 +23,7 @@ Other workloads of the same engine, one JSON line each (not part of the default 
     python bench.py --workload fomanex [--breakdown]   # Fomanex beside Zufusun (its closest relative) and Qwen3 likewise
     python bench.py --workload pepapel [--breakdown]   # Pepapel beside Zufusun, Fadosun (its closest relatives) and Qwen3 likewise
     python bench.py --workload filanex [--breakdown]   # Filanex beside Pepapel (its closest relative) and Qwen3 likewise
+    python bench.py --workload malusun [--breakdown]   # Malusun beside Zufusun and Fadosun (its closest relatives) and Qwen3 likewise
 """
 from __future__ import annotations
 
@@ -490,6 +491,39 @@ def workload_filanex(args, pk) -> int:
                          "expert_ff": QWEN3_1P7B["intermediate_size"] // 2}, others=[("pepapel", pepapel_config(runs))])
 
 
+MALUSUN_MIXERS = [
+    ("mamba1", {"inner": 4096, "state": 16, "dt_rank": 128, "conv": 4}),
+    ("attention", {"heads": 16, "kv_heads": 8, "dim": 128, "vdim": 128, "scale": 0.0884, "mask": {"size": 1024},
+                   "rot": {"dims": 64, "base": 1e6}, "v_mix": True}),
+    ("mamba1", {"inner": 4096, "state": 16, "dt_rank": 128, "conv": 4}),
+    ("attention_2", {"heads": 16, "kv_heads": 8, "dim": 128, "vdim": 128, "scale": 0.0884, "mask": {"size": 1024}, "v_mix": True}),
+]
+
+
+def malusun_config(n_layers):
+    """``n_layers`` layers: selective scans (4,096 channels of 16 states) and attention in windows of 1,024 (16/8 heads of 128;
+    rotated, then with distance slopes and the fixed sink, all blending values) in turn; the first feed-forward is dense and of
+    Qwen3's size, the others' one of eight experts of half that size a token and a shared one of that size."""
+    from ember_b200.config import MalusunConfig
+    width, ff, vocab = QWEN3_1P7B["hidden_size"], QWEN3_1P7B["intermediate_size"], QWEN3_1P7B["vocab_size"]
+    moe = {"kind": "moe", "expert": {"ff": ff // 2}, "router": {"experts": 8, "top": 1}, "shared": {"ff": ff // 2}}
+    layers = [{"type": MALUSUN_MIXERS[i % 4][0], "mixer": MALUSUN_MIXERS[i % 4][1], "mlp": moe if i else {"kind": "dense", "ff": ff}}
+              for i in range(n_layers)]
+    return MalusunConfig.from_json({"architecture": "Malusun", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+                                    "embedding": {"scale": 45.25}, "layers": layers})
+
+
+def workload_malusun(args, pk) -> int:
+    """Malusun beside Zufusun (whose windowed attention with a sink and experts are the like kernels), Fadosun (whose state
+    space, convolution and layers between two norms are) and Qwen3, all at the 1.7B width and vocabulary and with as many
+    layers (8 unless --layers says otherwise; random weights): the measurements of ``--workload fadosun``."""
+    n_layers = args.layers or 8
+    return beside_qwen3(args, pk, "malusun", malusun_config(n_layers), n_layers,
+                        {"malusun_layers": [k for k, _ in MALUSUN_MIXERS], "window": 1024, "experts": 8, "top": 1, "shared": 1,
+                         "expert_ff": QWEN3_1P7B["intermediate_size"] // 2},
+                        others=[("zufusun", zufusun_config(n_layers)), ("fadosun", fadosun_config(n_layers))])
+
+
 def beside_qwen3(args, pk, label, fcfg, n_layers, extra, others=()) -> int:
     """A design (``fcfg``) and Qwen3 at the 1.7B widths and ``n_layers`` layers, one after the other: prefill of 512 and
     2,048 tokens and decode steps at batch 8 and 64 from a context of 1,024, or with --breakdown the device time per
@@ -732,9 +766,9 @@ def main() -> int:
                     help="profiling aid: device time per kernel of three decode steps and one 2,048-token prefill step "
                          "(kernels serialised: EMBER_PDL=0 and no CUDA graphs are set by this flag)")
     ap.add_argument("--page-tokens", type=int, default=PAGE_TOKENS, choices=[16, 32, 64], help="tokens per cache page")
-    ap.add_argument("--workload", default="default", choices=["default", "serving-8b", "qwen3-32b", "fadosun", "zufusun", "fomanex", "pepapel", "filanex"],
+    ap.add_argument("--workload", default="default", choices=["default", "serving-8b", "qwen3-32b", "fadosun", "zufusun", "fomanex", "pepapel", "filanex", "malusun"],
                     help="default: the Qwen3-1.7B line; serving-8b and qwen3-32b are BASELINE's fourth "
-                         "and fifth configurations; fadosun, zufusun, fomanex, pepapel, filanex: that design beside Qwen3 at equal sizes (with "
+                         "and fifth configurations; fadosun, zufusun, fomanex, pepapel, filanex, malusun: that design beside Qwen3 at equal sizes (with "
                          "--breakdown also per kernel); one JSON line each")
     ap.add_argument("--prefill-tokens", type=int, default=PREFILL_TOKENS,
                     help="with --only-prefill: another prompt length (the reported line stays at 2,048)")
@@ -786,6 +820,8 @@ def main() -> int:
         return workload_pepapel(args, pk)
     if args.workload == "filanex":
         return workload_filanex(args, pk)
+    if args.workload == "malusun":
+        return workload_malusun(args, pk)
     if args.breakdown:
         return breakdown(cfg, n_layers, args.batch)
     if args.only_prefill:
