@@ -60,6 +60,9 @@ struct FaParams {
     float cap_log2, cap_arg, cap_z;      // a cap on the scaled scores, cap * tanh(scale s / cap): cap * log2(e), 2 log2(e) scale / cap, scale / cap
     const float* gate;        // logits of a gate per output element: row t, element head * 128 + d, or null
     int ld_gate;              // (a multiple of 4, rows 16-byte aligned)
+    const float* slopes;      // [n_heads] or null: slopes[h] * (query position - key position) is taken off the (capped) score
+    const float* sink;        // [n_heads] or null: exp(sink[h]) joins the denominator, without key and value
+    float raw_per_slope;      // what a slope of 1 is in the units of the scores as they come: 1 / scale, or log2(e) behind a cap
     int n_tiles;
     int* err;
 };
@@ -216,9 +219,11 @@ __device__ __forceinline__ uint32_t fa_swz(int row, int chunk) { return (uint32_
 // CAP 0: no cap on the scores.  1: a cap of at most FA_PLAIN_CAP (in log2 units): exponents lie between its two ends, so
 // they are taken as they are, without a running maximum: e^cap and its sums stay far inside fp32's (and bf16's) range.
 // 2: a larger cap, with the running maximum.
+// BIAS: slopes and a sink may be there.  The bias of a key is slope (key - query position): its part that differs inside a
+// tile is added to the scores, the rest (one number a row and tile) enters where the exponents are formed.
 constexpr float FA_PLAIN_CAP = 88.0f;
 
-template <int CAP>
+template <int CAP, bool BIAS>
 __global__ void __launch_bounds__(FA_THREADS, 2)
 attention_fa_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, const FaParams p) {
     constexpr int Q_HALF = FA_ROWS * 128;                // 16 KiB: [128 rows][64 bf16]
@@ -440,6 +445,8 @@ attention_fa_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
         int row_lo = lo, all_lo = lo;
         if (p.window > 0) { row_lo = max(row_lo, qpos - p.window + 1); all_lo = max(all_lo, last_q - p.window + 1); }
         if (p.chunk > 0) { row_lo = max(row_lo, qpos - qpos % p.chunk); all_lo = max(all_lo, last_q - last_q % p.chunk); }
+        const int head = kvh * G + min(r, rows - 1) % G;
+        const float slope = BIAS && p.slopes ? p.slopes[head] * p.raw_per_slope : 0.0f;
         for (int j = 0; j < n_kt; j++) {
             const int k0 = k_begin + j * FA_KT;
             if (ok) ok = fa_wait(&s_full[j & 1], (uint32_t)(j >> 1) & 1u, abort_flag);
@@ -468,6 +475,10 @@ attention_fa_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
                 }
             }
 
+            if (BIAS) {
+#pragma unroll
+                for (int i = 0; i < FA_KT; i++) s[i] = fmaf(slope, (float)i, s[i]);
+            }
             const bool interior = k0 >= all_lo && k0 + FA_KT <= hi && k0 + FA_KT - 1 <= pos0;
             // the maximum is taken over the raw scores; the scale (> 0) is folded into the exponent below (capped scores
             // are scaled already)
@@ -493,7 +504,8 @@ attention_fa_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
             } else {
                 tmax = -INFINITY;
             }
-            tmax *= to_log2;
+            const float tile_bias = BIAS ? slope * (float)(k0 - qpos) * to_log2 : 0.0f;
+            tmax = BIAS ? fmaf(tmax, to_log2, tile_bias) : tmax * to_log2;
             // raise the reference maximum only when the true one has outgrown it by more than 2^8
             const bool raise = CAP != 1 && (tmax > m_ref + 8.0f || (m_ref == -INFINITY && tmax > -INFINITY));
             const bool warp_raise = CAP != 1 && __any_sync(0xffffffffu, raise);
@@ -517,7 +529,7 @@ attention_fa_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
                 l_run *= m_ref == -INFINITY ? 0.0f : exp2f(m_ref - tmax);
                 m_ref = tmax;
             }
-            const float neg_base = m_ref == -INFINITY ? 0.0f : -m_ref;
+            const float neg_base = (m_ref == -INFINITY ? 0.0f : -m_ref) + tile_bias;
             float sum0 = 0.0f, sum1 = 0.0f, sum2 = 0.0f, sum3 = 0.0f;
             uint32_t packed[FA_KT / 2];
 #pragma unroll
@@ -545,6 +557,7 @@ attention_fa_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
         // the wait in the loop above is safe, S_j being complete only after O += P V of tile j - 2)
         if (n_kt > 0 && ok) ok = fa_wait(o_done, 0, abort_flag);
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+        if (BIAS && p.sink) l_run += fa_ex2(fmaf(p.sink[head], FA_LOG2E, m_ref == -INFINITY ? 0.0f : -m_ref));
         const float inv = l_run > 0.0f ? 1.0f / l_run : 0.0f;
         if (n_kt > 0 && p.gate) {
             // The gate's logits and the results are rows of 512 and 256 bytes a (token, head): a warp turns its 32 rows in
@@ -672,7 +685,7 @@ EMBER_API int ember_attention_fa_tile_queries(int group) { return group >= 1 && 
 EMBER_API int ember_attention_fa(const void* q, const void* k_pool, const void* v_pool, void* out, int n_heads, int n_kv,
                                  int D, const int* tiles, int n_tiles, const int* block_table, int max_blocks, int page,
                                  int num_pages, int window, float scale, int* err, float softcap, int chunk, const float* gate, int ld_gate,
-                                 void* stream) {
+                                 const float* slopes, const float* sink, void* stream) {
     if (n_tiles <= 0) return 0;
     if (gate && ((((uintptr_t)gate) & 15) || ld_gate < n_heads * FA_D || (ld_gate & 3))) return fail("attention_fa: gate rows of %d", ld_gate);
     if (n_heads <= 0 || n_kv <= 0 || n_heads % n_kv) return fail("attention_fa: bad head counts %d/%d", n_heads, n_kv);
@@ -691,6 +704,7 @@ EMBER_API int ember_attention_fa(const void* q, const void* k_pool, const void* 
     p.cap_log2 = softcap * FA_LOG2E;
     p.cap_z = softcap > 0.0f ? scale / softcap : 0.0f;
     p.cap_arg = softcap > 0.0f ? 2.0f * FA_LOG2E * scale / softcap : 0.0f; p.gate = gate; p.ld_gate = ld_gate; p.n_tiles = n_tiles; p.err = err;
+    p.slopes = slopes; p.sink = sink; p.raw_per_slope = softcap > 0.0f ? FA_LOG2E : 1.0f / scale;
     const size_t smem = (size_t)2 * FA_ROWS * 128 + (size_t)(FA_K_STAGES + FA_V_STAGES) * 2 * FA_KT * 128 + 256;
     auto run = [&](auto kernel, bool& ready) -> int {
         if (!ready) {
@@ -702,7 +716,8 @@ EMBER_API int ember_attention_fa(const void* q, const void* k_pool, const void* 
         launch_kernel(kernel, dim3(n_tiles, n_kv), dim3(FA_THREADS), smem, (cudaStream_t)stream, mk, mv, p);
         return check_launch("attention_fa");
     };
-    static bool ready[3] = {false, false, false};
-    if (softcap <= 0.0f) return run(attention_fa_kernel<0>, ready[0]);
-    return p.cap_log2 <= FA_PLAIN_CAP ? run(attention_fa_kernel<1>, ready[1]) : run(attention_fa_kernel<2>, ready[2]);
+    static bool ready[5] = {false, false, false, false, false};
+    if (slopes || sink) return softcap <= 0.0f ? run(attention_fa_kernel<0, true>, ready[3]) : run(attention_fa_kernel<2, true>, ready[4]);
+    if (softcap <= 0.0f) return run(attention_fa_kernel<0, false>, ready[0]);
+    return p.cap_log2 <= FA_PLAIN_CAP ? run(attention_fa_kernel<1, false>, ready[1]) : run(attention_fa_kernel<2, false>, ready[2]);
 }

@@ -52,6 +52,8 @@ struct AttnTcParams {
     float cap_log2, cap_arg;  // a cap on the scaled scores, cap * tanh(score / cap): cap * log2(e) and 2 log2(e) scale / cap (0: no cap)
     const float* gate;        // logits of a gate per output element: row t, element head * D + d, or null
     int ld_gate;
+    const float* slopes;      // [n_heads] or null: slopes[h] * (query position - key position) is taken off the (capped) score
+    const float* sink;        // [n_heads] or null: exp(sink[h]) joins the denominator once, without key and value
     int n_splits, split_keys;
     int n_tiles;
     int cluster_merge;        // the splits of a tile are a thread-block cluster and are merged in its first block's shared memory
@@ -116,11 +118,20 @@ __device__ __forceinline__ void atc_st_cluster(uint32_t addr, float v) {
 __device__ __forceinline__ void atc_cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
 __device__ __forceinline__ void atc_cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
 
+// The sink joins a row's merged sums (maximum M in log2 units, denominator L): what the row's sums are multiplied by.
+__device__ __forceinline__ float with_sink(const float* sink, int head, float M, float L) {
+    if (!sink) return L > 0.0f ? 1.0f / L : 0.0f;
+    const float sk = sink[head] * LOG2E, top = fmaxf(M, sk);
+    const float keep = M == -INFINITY ? 0.0f : exp2f(M - top), total = L * keep + exp2f(sk - top);
+    return total > 0.0f ? keep / total : 0.0f;
+}
+
 // Byte offset of (row, 16-byte chunk) inside a [rows][64 bf16] half-tile with the 128-byte swizzle.
 __device__ __forceinline__ uint32_t swz(int row, int chunk) { return (uint32_t)(row * 128 + ((chunk ^ (row & 7)) << 4)); }
 
-// HALVES = head_dim / 64.  DECODE: warps split the keys of a tile; else warps split the rows.
-template <int HALVES, bool DECODE>
+// HALVES = head_dim / 64.  DECODE: warps split the keys of a tile; else warps split the rows.  BIAS: slopes and a sink may
+// be there.
+template <int HALVES, bool DECODE, bool BIAS>
 __global__ void __launch_bounds__(ATC_THREADS)
 attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                     const AttnTcParams p) {
@@ -250,6 +261,9 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
     if (p.window > 0) { lo_a = max(lo_a, qpos_a - p.window + 1); lo_b = max(lo_b, qpos_b - p.window + 1); }
     if (p.chunk > 0) { lo_a = max(lo_a, qpos_a - qpos_a % p.chunk); lo_b = max(lo_b, qpos_b - qpos_b % p.chunk); }
 
+    const int head_a = kvh * G + min(r_a, rows - 1) % G, head_b = kvh * G + min(r_b, rows - 1) % G;
+    const float slope_a = BIAS && p.slopes ? p.slopes[head_a] * LOG2E : 0.0f, slope_b = BIAS && p.slopes ? p.slopes[head_b] * LOG2E : 0.0f;
+
     float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.0f, l_b = 0.0f;
     float o[ND][4];
 #pragma unroll
@@ -299,7 +313,13 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
 #pragma unroll
                     for (int j = 0; j < NKG; j++) {
 #pragma unroll
-                        for (int e = 0; e < 4; e++) s[j][e] = score_log2(p, s[j][e]);
+                        for (int e = 0; e < 4; e++) {
+                            s[j][e] = score_log2(p, s[j][e]);
+                            if (BIAS) {
+                                const int key = k0 + koff + j * 8 + 2 * t4 + (e & 1);
+                                s[j][e] = fmaf(e < 2 ? slope_a : slope_b, (float)(key - (e < 2 ? qpos_a : qpos_b)), s[j][e]);
+                            }
+                        }
                         tmax_a = fmaxf(tmax_a, fmaxf(s[j][0], s[j][1]));
                         tmax_b = fmaxf(tmax_b, fmaxf(s[j][2], s[j][3]));
                     }
@@ -313,6 +333,10 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
                             const bool vb2 = key >= lo_b && key < hi && key <= qpos_b;
                             s[j][e] = va ? score_log2(p, s[j][e]) : -INFINITY;
                             s[j][2 + e] = vb2 ? score_log2(p, s[j][2 + e]) : -INFINITY;
+                            if (BIAS) {
+                                if (va) s[j][e] = fmaf(slope_a, (float)(key - qpos_a), s[j][e]);
+                                if (vb2) s[j][2 + e] = fmaf(slope_b, (float)(key - qpos_b), s[j][2 + e]);
+                            }
                             tmax_a = fmaxf(tmax_a, s[j][e]);
                             tmax_b = fmaxf(tmax_b, s[j][2 + e]);
                         }
@@ -377,7 +401,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
 
     if (!DECODE) {
         // ---- rows are private to a warp: normalise and store
-        const float inv_a = l_a > 0.0f ? 1.0f / l_a : 0.0f, inv_b = l_b > 0.0f ? 1.0f / l_b : 0.0f;
+        const float inv_a = with_sink(BIAS ? p.sink : nullptr, head_a, m_a, l_a), inv_b = with_sink(BIAS ? p.sink : nullptr, head_b, m_b, l_b);
         if (r_a < rows) {
             const int qi = r_a / G, g = r_a - qi * G;
             __nv_bfloat16* dst = p.out + ((size_t)(row0 + qi) * p.n_heads + kvh * G + g) * D;
@@ -437,7 +461,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
         // nq == 1: row r is head r of the group
         if (p.n_splits <= 1) {
             p.out[((size_t)row0 * p.n_heads + kvh * G + r) * D + d] =
-                __float2bfloat16_rn(gated(gate_row, r * D + d, L > 0.0f ? acc / L : 0.0f));
+                __float2bfloat16_rn(gated(gate_row, r * D + d, BIAS ? acc * with_sink(p.sink, kvh * G + r, M, L) : (L > 0.0f ? acc / L : 0.0f)));
         } else if (merge_in_cluster) {
             atc_st_cluster(recv_o0 + (uint32_t)((split * rows + r) * D + d) * 4u, acc);
             if (d == 0) {
@@ -473,7 +497,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
                 acc = fmaf(ro[((size_t)sp * rows + r) * D + d], f, acc);
             }
             p.out[((size_t)row0 * p.n_heads + kvh * G + r) * D + d] =
-                __float2bfloat16_rn(gated(gate_row, r * D + d, L > 0.0f ? acc * (1.0f / L) : 0.0f));
+                __float2bfloat16_rn(gated(gate_row, r * D + d, acc * with_sink(BIAS ? p.sink : nullptr, kvh * G + r, M, L)));
         }
     }
 }
@@ -484,7 +508,8 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
 // dependent loads before, which is what the kernel's time was at batch 1 with 13 splits).
 __global__ void attention_tc_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                             __nv_bfloat16* __restrict__ out, const int* __restrict__ tiles,
-                                            int n_heads, int n_splits, int D, const float* __restrict__ gate, int ld_gate) {
+                                            int n_heads, int n_splits, int D, const float* __restrict__ gate, int ld_gate,
+                                            const float* __restrict__ sink) {
     extern __shared__ float w_s[];                                         // [n_splits] weights, then 1 / L
     float& inv_s = w_s[n_splits];
     pdl_launch_dependents();
@@ -520,7 +545,7 @@ __global__ void attention_tc_combine_kernel(const float* __restrict__ part_o, co
             }
             for (int i = 0; i < 32 && s0 + i < n_splits; i++) L += __shfl_sync(0xffffffffu, l, i);   // ascending
         }
-        if (threadIdx.x == 0) inv_s = L > 0.0f ? 1.0f / L : 0.0f;
+        if (threadIdx.x == 0) inv_s = with_sink(sink, head, M * LOG2E, L);
     }
     __syncthreads();
     const float inv = inv_s;
@@ -612,7 +637,7 @@ EMBER_API int ember_attention_tc(const void* q, const void* k_pool, const void* 
                                  int n_heads, int n_kv, int D, const int* tiles, int n_tiles,
                                  const int* block_table, int max_blocks, int page, int num_pages, int window,
                                  float scale, int n_splits, int split_keys, float* part_o, float* part_ml,
-                                 int* err, float softcap, int chunk, const float* gate, int ld_gate, void* stream) {
+                                 int* err, float softcap, int chunk, const float* gate, int ld_gate, const float* slopes, const float* sink, void* stream) {
     if (n_tiles <= 0) return 0;
     if (gate && ld_gate < n_heads * D) return fail("attention_tc: gate rows of %d", ld_gate);
     if (softcap < 0.0f) return fail("attention_tc: a score cap of %g", softcap);
@@ -637,7 +662,7 @@ EMBER_API int ember_attention_tc(const void* q, const void* k_pool, const void* 
     p.tiles = tiles; p.block_table = block_table; p.max_blocks = max_blocks; p.page = page; p.num_pages = num_pages;
     p.n_heads = n_heads; p.n_kv = n_kv; p.window = window; p.chunk = chunk < 0 ? 0 : chunk; p.scale_log2 = scale * LOG2E;
     p.cap_log2 = softcap * LOG2E; p.cap_arg = softcap > 0.0f ? 2.0f * LOG2E * scale / softcap : 0.0f;
-    p.gate = gate; p.ld_gate = ld_gate;
+    p.gate = gate; p.ld_gate = ld_gate; p.slopes = slopes; p.sink = sink;
     p.n_splits = n_splits; p.split_keys = split_keys; p.n_tiles = n_tiles; p.err = err;
     p.cluster_merge = cluster_merge ? 1 : 0;
     cudaStream_t st = (cudaStream_t)stream;
@@ -670,13 +695,16 @@ EMBER_API int ember_attention_tc(const void* q, const void* k_pool, const void* 
         return check_launch("attention_tc (cluster)");
     };
     int rc;
-    if (D == 128) rc = mode == 1 ? run(attention_tc_kernel<2, true>) : run(attention_tc_kernel<2, false>);
-    else rc = mode == 1 ? run(attention_tc_kernel<1, true>) : run(attention_tc_kernel<1, false>);
+    if (slopes || sink) {
+        if (D == 128) rc = mode == 1 ? run(attention_tc_kernel<2, true, true>) : run(attention_tc_kernel<2, false, true>);
+        else rc = mode == 1 ? run(attention_tc_kernel<1, true, true>) : run(attention_tc_kernel<1, false, true>);
+    } else if (D == 128) rc = mode == 1 ? run(attention_tc_kernel<2, true, false>) : run(attention_tc_kernel<2, false, false>);
+    else rc = mode == 1 ? run(attention_tc_kernel<1, true, false>) : run(attention_tc_kernel<1, false, false>);
     if (rc) return rc;
     if (n_splits > 1 && !cluster_merge) {
         launch_kernel(attention_tc_combine_kernel, (unsigned)((size_t)n_tiles * n_heads), D, (size_t)(n_splits + 1) * sizeof(float), st,
                       (const float*)part_o,
-                      (const float*)part_ml, (__nv_bfloat16*)out, tiles, n_heads, n_splits, D, gate, ld_gate);
+                      (const float*)part_ml, (__nv_bfloat16*)out, tiles, n_heads, n_splits, D, gate, ld_gate, sink);
         return check_launch("attention_tc_combine");
     }
     return 0;

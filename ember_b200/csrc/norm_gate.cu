@@ -2,6 +2,7 @@
 //   layer_norm        out[r] = (x - mean) / sqrt(var + eps) * w + b      (var = mean of squared deviations)
 //   gated_norm_add    residual[r] += norm(y[r] * sigmoid(gate_logits[r])) for a layer norm or an RMS norm; the new
 //                     residual row can also be left rounded to bfloat16 (for a sublayer that reads the stream itself)
+//   norm_add_norm     residual[r] += rms_norm(y[r]), and the RMS norm of the new row for whoever reads it next
 //   scaled_add_norm   residual[r] = norm(alpha * residual[r] + y[r] + bias): the norm *after* the sum (a post-norm layer), in place,
 //                     with the same optional bfloat16 copy of the new rows
 //   pair_norm_sum     out[r] (+)= wa * a[r] / rms(a[r]) + wb * b[r] / rms(b[r]): two branches, each RMS-normed over the row
@@ -82,6 +83,75 @@ gated_norm_add_kernel(const float* __restrict__ y, const float* __restrict__ gat
         const float r = residual[base + i] + ((row[i] - mean) * rstd * w[i] + (b ? b[i] : 0.0f));
         residual[base + i] = r;
         if (rounded) rounded[base + i] = __float2bfloat16_rn(r);      // what the next sublayer's products read
+    }
+}
+
+// ---------------------------------------------------------------- norm, add to the stream, norm of what comes next
+// residual[r] += y[r] / rms(y[r]) * w; out[r] = residual[r] / rms(residual[r]) * w2: the norm behind a sublayer and the one
+// ahead of the next in one pass over the stream.  W elements a thread and load.
+template <int W>
+__device__ __forceinline__ void row_load(const float* p, float (&v)[W]) {
+    if (W == 4) {
+        const float4 f = *reinterpret_cast<const float4*>(p);
+        v[0] = f.x; v[W > 1 ? 1 : 0] = f.y; v[W > 2 ? 2 : 0] = f.z; v[W > 3 ? 3 : 0] = f.w;
+    } else v[0] = *p;
+}
+template <int W>
+__device__ __forceinline__ void row_store(float* p, const float (&v)[W]) {
+    if (W == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[W > 1 ? 1 : 0], v[W > 2 ? 2 : 0], v[W > 3 ? 3 : 0]);
+    else *p = v[0];
+}
+template <int W>
+__device__ __forceinline__ void row_store(__nv_bfloat16* p, const float (&v)[W]) {
+    if (W == 4) {
+        __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[W > 1 ? 1 : 0]), hi = __floats2bfloat162_rn(v[W > 2 ? 2 : 0], v[W > 3 ? 3 : 0]);
+        uint2 u;
+        u.x = *reinterpret_cast<uint32_t*>(&lo);
+        u.y = *reinterpret_cast<uint32_t*>(&hi);
+        *reinterpret_cast<uint2*>(p) = u;
+    } else p[0] = __float2bfloat16_rn(v[0]);
+}
+
+template <typename TO, int W>
+__global__ void __launch_bounds__(ROW_THREADS)
+norm_add_norm_kernel(const float* __restrict__ y, const float* __restrict__ w, float eps, float* __restrict__ residual,
+                     const float* __restrict__ w2, float eps2, TO* __restrict__ out, int H) {
+    extern __shared__ __align__(16) float row[];          // H floats: y, then the new row of the stream
+    __shared__ float scratch[32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t base = (size_t)blockIdx.x * H;
+    float ss = 0.0f;
+    for (int i = threadIdx.x * W; i < H; i += ROW_THREADS * W) {
+        float v[W];
+        row_load<W>(y + base + i, v);
+        row_store<W>(row + i, v);
+#pragma unroll
+        for (int k = 0; k < W; k++) ss = fmaf(v[k], v[k], ss);
+    }
+    const float r1 = 1.0f / sqrtf(block_sum(ss, scratch) / (float)H + eps);
+    ss = 0.0f;
+    for (int i = threadIdx.x * W; i < H; i += ROW_THREADS * W) {
+        float v[W], h[W], g[W];
+        row_load<W>(row + i, v);
+        row_load<W>(residual + base + i, h);
+        row_load<W>(w + i, g);
+#pragma unroll
+        for (int k = 0; k < W; k++) {
+            h[k] += v[k] * r1 * g[k];
+            ss = fmaf(h[k], h[k], ss);
+        }
+        row_store<W>(residual + base + i, h);
+        row_store<W>(row + i, h);
+    }
+    const float r2 = 1.0f / sqrtf(block_sum(ss, scratch) / (float)H + eps2);
+    for (int i = threadIdx.x * W; i < H; i += ROW_THREADS * W) {
+        float h[W], g[W];
+        row_load<W>(row + i, h);
+        row_load<W>(w2 + i, g);
+#pragma unroll
+        for (int k = 0; k < W; k++) h[k] = h[k] * r2 * g[k];
+        row_store<W>(out + base + i, h);
     }
 }
 
@@ -434,6 +504,26 @@ EMBER_API int ember_gated_norm_add(const float* y, const float* gate, const floa
     if (centred) launch_kernel(gated_norm_add_kernel<true>, n_rows, ROW_THREADS, smem, st, y, gate, gate_bias, w, b, eps, residual, (__nv_bfloat16*)rounded, H);
     else launch_kernel(gated_norm_add_kernel<false>, n_rows, ROW_THREADS, smem, st, y, gate, gate_bias, w, b, eps, residual, (__nv_bfloat16*)rounded, H);
     return check_launch("gated_norm_add");
+}
+
+EMBER_API int ember_norm_add_norm(const float* y, const float* w, float eps, float* residual, const float* w2, float eps2, void* out,
+                                  int out_dtype, int n_rows, int H, void* stream) {
+    if (n_rows <= 0) return 0;
+    if (H <= 0 || (size_t)H * 4 > 200 * 1024) return fail("norm_add_norm: width %d is not taken", H);
+    const size_t smem = (size_t)H * sizeof(float);
+    const bool by4 = H % 4 == 0 && ((((uintptr_t)y) | ((uintptr_t)w) | ((uintptr_t)residual) | ((uintptr_t)w2) | ((uintptr_t)out)) & 15) == 0;
+    auto run = [&](auto kernel, auto* o) -> int {
+        if (smem > 48 * 1024) {
+            cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+            if (e != cudaSuccess) return fail("norm_add_norm: shared memory %zu: %s", smem, cudaGetErrorString(e));
+        }
+        launch_kernel(kernel, n_rows, ROW_THREADS, smem, (cudaStream_t)stream, y, w, eps, residual, w2, eps2, o, H);
+        return check_launch("norm_add_norm");
+    };
+    if (out_dtype == EMBER_F32) return by4 ? run(norm_add_norm_kernel<float, 4>, (float*)out) : run(norm_add_norm_kernel<float, 1>, (float*)out);
+    if (out_dtype == EMBER_BF16)
+        return by4 ? run(norm_add_norm_kernel<__nv_bfloat16, 4>, (__nv_bfloat16*)out) : run(norm_add_norm_kernel<__nv_bfloat16, 1>, (__nv_bfloat16*)out);
+    return fail("norm_add_norm: unsupported dtype %d", out_dtype);
 }
 
 EMBER_API int ember_scaled_add_norm(const float* y, const float* y_bias, float alpha, const float* w, const float* b, float eps,

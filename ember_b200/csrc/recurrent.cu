@@ -64,6 +64,82 @@ __global__ void conv_silu_kernel(const float* __restrict__ x, int ldx, int c0, c
     }
 }
 
+// The same for few taps: the last NT - 1 inputs of W neighbouring channels roll through registers, so an input is read once
+// however many taps look at it; at the start of a block or of a run they come from the rows before or from what was carried.
+// Steps of single tokens (`single`) also leave the carried inputs as conv_carry_kernel would.
+template <int NT, int W>
+__global__ void __launch_bounds__(128) conv_roll_kernel(const float* __restrict__ x, int ldx, int c0, const float* __restrict__ taps,
+                                                        const float* __restrict__ bias, float* __restrict__ carry, long long carry_stride,
+                                                        const int* __restrict__ seq_of, const int* __restrict__ query_start,
+                                                        const int* __restrict__ slots, float* __restrict__ out,
+                                                        __nv_bfloat16* __restrict__ rounded, int C, int silu, int T, int tt, int single) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int c = (blockIdx.x * blockDim.x + threadIdx.x) * W, t0 = blockIdx.y * tt, t1 = min(t0 + tt, T);
+    if (c >= C) return;
+    auto load = [&](const float* p, float (&v)[W]) {
+        if (W == 4) {
+            const float4 f = *reinterpret_cast<const float4*>(p);
+            v[0] = f.x; v[W > 1 ? 1 : 0] = f.y; v[W > 2 ? 2 : 0] = f.z; v[W > 3 ? 3 : 0] = f.w;
+        } else v[0] = *p;
+    };
+    auto store = [&](float* p, const float (&v)[W]) {
+        if (W == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[W > 1 ? 1 : 0], v[W > 2 ? 2 : 0], v[W > 3 ? 3 : 0]);
+        else *p = v[0];
+    };
+    float w[NT][W], b[W], h[NT][W];                      // h[j]: the input NT - 1 - j tokens back
+#pragma unroll
+    for (int k = 0; k < W; k++) {
+        b[k] = bias ? bias[c + k] : 0.0f;
+#pragma unroll
+        for (int j = 0; j < NT; j++) w[j][k] = taps[(size_t)(c + k) * NT + j];
+    }
+    int s = seq_of[t0], first = query_start[s], next = query_start[s + 1];
+    float ahead[W];
+    load(x + (size_t)t0 * ldx + c0 + c, ahead);
+    for (int t = t0; t < t1; t++) {
+        if (t >= next) { s = seq_of[t]; first = query_start[s]; next = query_start[s + 1]; }
+        if (t == t0 || t == first) {
+            const float* cs = carry + (size_t)slots[s] * carry_stride + c;
+#pragma unroll
+            for (int j = 0; j < NT - 1; j++) {
+                const int src = t - (NT - 1 - j);
+                load(src >= first ? x + (size_t)src * ldx + c0 + c : cs + (size_t)(NT - 1 + src - first) * C, h[j]);
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < W; k++) h[NT - 1][k] = ahead[k];
+        if (t + 1 < t1) load(x + (size_t)(t + 1) * ldx + c0 + c, ahead);
+        float y[W];
+#pragma unroll
+        for (int k = 0; k < W; k++) {
+            float acc = b[k];
+#pragma unroll
+            for (int j = 0; j < NT; j++) acc = fmaf(w[j][k], h[j][k], acc);
+            y[k] = silu ? acc / (1.0f + expf(-acc)) : acc;
+        }
+        store(out + (size_t)t * C + c, y);
+        if (rounded) {
+            if (W == 4) {
+                __nv_bfloat162 lo = __floats2bfloat162_rn(y[0], y[W > 1 ? 1 : 0]), hi = __floats2bfloat162_rn(y[W > 2 ? 2 : 0], y[W > 3 ? 3 : 0]);
+                uint2 u;
+                u.x = *reinterpret_cast<uint32_t*>(&lo);
+                u.y = *reinterpret_cast<uint32_t*>(&hi);
+                *reinterpret_cast<uint2*>(rounded + (size_t)t * C + c) = u;
+            } else rounded[(size_t)t * C + c] = __float2bfloat16_rn(y[0]);
+        }
+#pragma unroll
+        for (int j = 0; j < NT - 1; j++)
+#pragma unroll
+            for (int k = 0; k < W; k++) h[j][k] = h[j + 1][k];
+        if (single) {
+            float* cs = carry + (size_t)slots[s] * carry_stride + c;
+#pragma unroll
+            for (int j = 0; j < NT - 1; j++) store(cs + (size_t)j * C, h[j]);
+        }
+    }
+}
+
 // After the convolution: the request's last n - 1 inputs (from the run, or shifted down from what was carried).
 __global__ void conv_carry_kernel(const float* __restrict__ x, int ldx, int c0, int n, float* __restrict__ carry,
                                   long long carry_stride, const int* __restrict__ query_start, const int* __restrict__ slots, int C) {
@@ -870,6 +946,21 @@ EMBER_API int ember_conv_silu(const float* x, int ldx, int c0, const float* taps
     if (T > 65535 || S > 65535) return fail("conv_silu: %d tokens in %d runs are too many for one launch", T, S);
     cudaStream_t st = (cudaStream_t)stream;
     const unsigned bx = (unsigned)((C + 127) / 128);
+    if (n >= 2 && n <= 4) {
+        const uintptr_t bases = (uintptr_t)x | (uintptr_t)carry | (uintptr_t)out | (uintptr_t)rounded;
+        const bool by4 = C % 4 == 0 && ldx % 4 == 0 && c0 % 4 == 0 && carry_stride % 4 == 0 && (bases & 15) == 0;
+        const int single = T == S ? 1 : 0, rt = T >= 1024 ? 16 : (T >= 256 ? 4 : 1), cols = by4 ? C / 4 : C;
+        const dim3 grid((cols + 127) / 128, (T + rt - 1) / rt);
+        auto run = [&](auto kernel) {
+            launch_kernel(kernel, grid, 128, 0, st, x, ldx, c0, taps, bias, carry, carry_stride, seq_of, query_start, slots, out,
+                          (__nv_bfloat16*)rounded, C, silu, T, rt, single);
+        };
+        if (n == 2) { if (by4) run(conv_roll_kernel<2, 4>); else run(conv_roll_kernel<2, 1>); }
+        else if (n == 3) { if (by4) run(conv_roll_kernel<3, 4>); else run(conv_roll_kernel<3, 1>); }
+        else { if (by4) run(conv_roll_kernel<4, 4>); else run(conv_roll_kernel<4, 1>); }
+        if (!single) launch_kernel(conv_carry_kernel, dim3(bx, S), 128, 0, st, x, ldx, c0, n, carry, carry_stride, query_start, slots, C);
+        return check_launch("conv_roll");
+    }
     const int tt = T >= 1024 ? 8 : 1;          // prompt portions: eight tokens a block; small steps keep a block a token
     launch_kernel(conv_silu_kernel, dim3(bx, (T + tt - 1) / tt), 128, 0, st, x, ldx, c0, taps, bias, n, (const float*)carry,
                   carry_stride, seq_of, query_start, slots, out, (__nv_bfloat16*)rounded, C, silu, T, tt);

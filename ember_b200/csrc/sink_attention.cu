@@ -6,7 +6,7 @@
 //     rotated shared key part behind it into the token's single cache row [c | k_rot];
 //   * rotate_pairs:      rotation of neighbouring pairs (2i, 2i + 1) of a slice of every head, fp32 in, cache type out;
 //   * head_gemm:         out[t, h, :] = W[h] x[t, h, :] for every head (a product per head, weights [H, N, K]), with an
-//     optional sigmoid gate on the result: folds a head's key up-projection into its query and takes a head's value
+//     optional bias, softplus and sigmoid gate on the result: folds a head's key up-projection into its query and takes a head's value
 //     up-projection of the attended latent; fp32 multiply-adds in general, mma.sync tiles for bfloat16 weights;
 //   * sink_attention:    o = sum_j w_j v_j with w = softmax over the visible keys and one more term exp(sink[h]) in the
 //     denominator that has no key and no value; visible: j <= i and (no window, or i - j < window, or j < keep_first).
@@ -384,7 +384,21 @@ struct HeadGemmArgs {
     void* out; int ld_o, o_head, o_col;
     const float* gate; int ld_g, g_col;  // gate[t, g_col + h N + n] or null
     int T, H, N, K;
+    const float* bias; int softplus;     // bias [H N] or null joins the sum; then softplus of it (before a gate)
 };
+
+__device__ __forceinline__ float head_gemm_finish(const HeadGemmArgs& p, int t, int h, int n, float v) {
+    if (p.bias) v += p.bias[(size_t)h * p.N + n];
+    if (p.softplus) v = v > 20.0f ? v : log1pf(expf(v));
+    if (p.gate) v *= sigmoidf_(p.gate[(size_t)t * p.ld_g + p.g_col + (size_t)h * p.N + n]);
+    return v;
+}
+template <typename T>
+__device__ __forceinline__ void put2(T* dst, float a, float b);
+template <>
+__device__ __forceinline__ void put2<float>(float* dst, float a, float b) { *reinterpret_cast<float2*>(dst) = make_float2(a, b); }
+template <>
+__device__ __forceinline__ void put2<__nv_bfloat16>(__nv_bfloat16* dst, float a, float b) { *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(a, b); }
 
 template <typename TW, typename TO>
 __global__ void __launch_bounds__(256) head_gemm_kernel(HeadGemmArgs p) {
@@ -430,9 +444,7 @@ __global__ void __launch_bounds__(256) head_gemm_kernel(HeadGemmArgs p) {
         for (int j = 0; j < 4; j++) {
             const int n = n0 + tx * 4 + j;
             if (n >= p.N) continue;
-            float v = acc[i][j];
-            if (p.gate) v *= sigmoidf_(p.gate[(size_t)t * p.ld_g + p.g_col + (size_t)h * p.N + n]);
-            ((TO*)p.out)[(size_t)t * p.ld_o + (size_t)h * p.o_head + p.o_col + n] = from_float<TO>(v);
+            ((TO*)p.out)[(size_t)t * p.ld_o + (size_t)h * p.o_head + p.o_col + n] = from_float<TO>(head_gemm_finish(p, t, h, n, acc[i][j]));
         }
     }
 }
@@ -773,9 +785,10 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     return *reinterpret_cast<const uint32_t*>(&v);
 }
 
-// The per-head product on the tensor cores: tiles of 64 tokens x 64 outputs, K in steps of 32, four warps of 16 rows; x is
-// rounded to bfloat16 as it enters shared memory (the weights are bfloat16), sums are fp32.
-constexpr int HT_BM = 64, HT_BN = 64, HT_BK = 32, HT_LD = HT_BK + 8;
+// The per-head product on the tensor cores: tiles of 64 tokens x 64 outputs, K up to 128 at a time (one trip to memory and
+// one barrier for the ranks that are usual), four warps of 16 rows; x is rounded to bfloat16 as it enters shared memory
+// (the weights are bfloat16), sums are fp32.
+constexpr int HT_BM = 64, HT_BN = 64, HT_BK = 128, HT_LD = HT_BK + 8;
 
 template <typename TO>
 __global__ void __launch_bounds__(128) head_gemm_tc_kernel(HeadGemmArgs p) {
@@ -790,8 +803,10 @@ __global__ void __launch_bounds__(128) head_gemm_tc_kernel(HeadGemmArgs p) {
 #pragma unroll
     for (int i = 0; i < 8; i++) { acc[i][0] = 0.0f; acc[i][1] = 0.0f; acc[i][2] = 0.0f; acc[i][3] = 0.0f; }
     for (int k0 = 0; k0 < p.K; k0 += HT_BK) {
+        const int kc = min(HT_BK, (p.K - k0 + 15) & ~15);      // (columns up to a multiple of 16 are filled with zeros)
+#pragma unroll 8
         for (int idx = threadIdx.x; idx < HT_BM * (HT_BK / 4); idx += 128) {
-            const int r = idx / (HT_BK / 4), c = (idx - r * (HT_BK / 4)) * 4;
+            const int r = idx / (HT_BK / 4), c = (idx % (HT_BK / 4)) * 4;
             float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
             if (m0 + r < p.T && k0 + c < p.K)
                 v = *reinterpret_cast<const float4*>(p.x + (size_t)(m0 + r) * p.ld_x + (size_t)h * p.x_head + p.x_col + k0 + c);
@@ -800,15 +815,15 @@ __global__ void __launch_bounds__(128) head_gemm_tc_kernel(HeadGemmArgs p) {
             packed.y = pack_bf16(v.z, v.w);
             *reinterpret_cast<uint2*>(As + r * HT_LD + c) = packed;
         }
+#pragma unroll 8
         for (int idx = threadIdx.x; idx < HT_BN * (HT_BK / 8); idx += 128) {
-            const int r = idx / (HT_BK / 8), c = (idx - r * (HT_BK / 8)) * 8;
+            const int r = idx / (HT_BK / 8), c = (idx % (HT_BK / 8)) * 8;
             uint4 v = make_uint4(0u, 0u, 0u, 0u);
             if (n0 + r < p.N && k0 + c < p.K) v = *reinterpret_cast<const uint4*>(w + (size_t)(n0 + r) * p.K + k0 + c);
             *reinterpret_cast<uint4*>(Bs + r * HT_LD + c) = v;
         }
         __syncthreads();
-#pragma unroll
-        for (int kk = 0; kk < HT_BK; kk += 16) {
+        for (int kk = 0; kk < kc; kk += 16) {
             uint32_t af[4];
             ldmatrix_x4(af, As + (warp * 16 + (lane & 15)) * HT_LD + kk + (lane >> 4) * 8);
 #pragma unroll
@@ -821,15 +836,22 @@ __global__ void __launch_bounds__(128) head_gemm_tc_kernel(HeadGemmArgs p) {
         }
         __syncthreads();
     }
+    const bool pairs = ((p.ld_o | p.o_head | p.o_col) & 1) == 0;      // a thread's two neighbouring outputs in one store
 #pragma unroll
     for (int nt = 0; nt < 8; nt++)
 #pragma unroll
-        for (int e = 0; e < 4; e++) {
-            const int row = m0 + warp * 16 + g + (e >> 1) * 8, n = n0 + nt * 8 + 2 * t + (e & 1);
+        for (int half = 0; half < 2; half++) {
+            const int row = m0 + warp * 16 + g + half * 8, n = n0 + nt * 8 + 2 * t;
             if (row >= p.T || n >= p.N) continue;
-            float v = acc[nt][e];
-            if (p.gate) v *= sigmoidf_(p.gate[(size_t)row * p.ld_g + p.g_col + (size_t)h * p.N + n]);
-            ((TO*)p.out)[(size_t)row * p.ld_o + (size_t)h * p.o_head + p.o_col + n] = from_float<TO>(v);
+            const bool two = n + 1 < p.N;
+            const float v0 = head_gemm_finish(p, row, h, n, acc[nt][2 * half]);
+            const float v1 = two ? head_gemm_finish(p, row, h, n + 1, acc[nt][2 * half + 1]) : 0.0f;
+            TO* dst = (TO*)p.out + (size_t)row * p.ld_o + (size_t)h * p.o_head + p.o_col + n;
+            if (two && pairs) put2<TO>(dst, v0, v1);
+            else {
+                dst[0] = from_float<TO>(v0);
+                if (two) dst[1] = from_float<TO>(v1);
+            }
         }
 }
 
@@ -1233,13 +1255,14 @@ EMBER_API int ember_rotate_pairs(const float* in, int ld_in, int in_head, int in
 
 EMBER_API int ember_head_gemm(const float* x, int ld_x, int x_head, int x_col, const void* w, int w_dtype, void* out, int out_dtype,
                               int ld_o, int o_head, int o_col, const float* gate, int ld_g, int g_col, int T, int H, int N, int K,
-                              void* stream) {
+                              const float* bias, int softplus, void* stream) {
     if (T <= 0) return 0;
     if (H <= 0 || N <= 0 || K <= 0 || H > 65535) return fail("head_gemm: %d heads of %d x %d", H, N, K);
-    HeadGemmArgs p{x, ld_x, x_head, x_col, w, out, ld_o, o_head, o_col, gate, ld_g, g_col, T, H, N, K};
+    HeadGemmArgs p{x, ld_x, x_head, x_col, w, out, ld_o, o_head, o_col, gate, ld_g, g_col, T, H, N, K, bias, softplus};
     cudaStream_t st = (cudaStream_t)stream;
     // bfloat16 weights with rows of whole 16-byte pieces (and x rows of whole float4s): the tensor-core form
-    if (w_dtype == EMBER_BF16 && K % 8 == 0 && ld_x % 4 == 0 && x_head % 4 == 0 && x_col % 4 == 0 && head_gemm_on_tensor_cores()) {
+    if (w_dtype == EMBER_BF16 && K % 8 == 0 && ld_x % 4 == 0 && x_head % 4 == 0 && x_col % 4 == 0 && (((uintptr_t)x) & 15) == 0 && (((uintptr_t)w) & 15) == 0 && (((uintptr_t)out) & 7) == 0 &&
+        head_gemm_on_tensor_cores()) {
         dim3 tgrid((T + HT_BM - 1) / HT_BM, (N + HT_BN - 1) / HT_BN, H);
         if (out_dtype == EMBER_BF16) launch_kernel(head_gemm_tc_kernel<__nv_bfloat16>, tgrid, 128, 0, st, p);
         else launch_kernel(head_gemm_tc_kernel<float>, tgrid, 128, 0, st, p);

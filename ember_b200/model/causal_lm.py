@@ -152,6 +152,10 @@ class CausalLM:
             block = self.blocks[e.layer]
             caches = {sub: storage.layer(self.cache_id(owner, sub, e.instance)) for sub in self._cache_subs[e.layer]}
             ctx.memo["schedule.index"] = i            # (a block may leave something for the run right after it)
+            after = s.schedule[i + 1] if i + 1 < len(s.schedule) else None
+            # the norm the next run begins with, for a block that can make it while it adds to the stream
+            ctx.memo["block.next_norm"] = (getattr(self.blocks[after.layer], "leading_norm", None)
+                                           if after is not None and not after.reentry and copies == 1 else None)
             block.forward(ctx, h, caches, owns_cache=(owner == e.layer))
             if capture is not None:
                 record(i + 1)

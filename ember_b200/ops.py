@@ -588,12 +588,16 @@ def _check_element_gate(gate, col: int, n: int) -> None:
 def attention_fa(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, out: torch.Tensor, n_heads: int,
                  n_kv: int, head_dim: int, tiles: torch.Tensor, n_tiles: int, block_table: torch.Tensor, page: int,
                  window: int, scale: float, err: Optional[torch.Tensor] = None, stream: Optional[int] = None,
-                 softcap: float = 0.0, chunk: int = 0, gate: Optional[torch.Tensor] = None, gate_col: int = 0) -> None:
+                 softcap: float = 0.0, chunk: int = 0, gate: Optional[torch.Tensor] = None, gate_col: int = 0,
+                 slopes: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None) -> None:
     """bf16 causal attention of prompt portions on tcgen05 tensor cores (S and O in tensor memory).  ``softcap`` > 0: the
     scaled score becomes softcap * tanh(score / softcap); ``chunk`` > 0: position i sees j only if
     floor(i / chunk) == floor(j / chunk); ``gate`` (fp32 [T, ..]): element i of a token's result is multiplied by
-    sigmoid(gate[t, gate_col + i])."""
+    sigmoid(gate[t, gate_col + i]); ``slopes`` (fp32 [n_heads]): slopes[h] * (i - j) is taken off the score after the cap;
+    ``sink`` (fp32 [n_heads]): exp(sink[h]) joins the softmax's denominator."""
     _check_element_gate(gate, gate_col, n_heads * head_dim)
+    _check_slopes(slopes, n_heads)
+    _check_slopes(sink, n_heads)
     _check(q, "q", torch.bfloat16)
     _check(out, "out", torch.bfloat16)
     _check(k_pool, "k_pool", torch.bfloat16)
@@ -607,7 +611,7 @@ def attention_fa(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, ou
           _p(tiles), c_int(n_tiles), _p(block_table), c_int(block_table.shape[-1]), c_int(page), c_int(k_pool.shape[0]),
           c_int(window), c_float(scale), _p(err), c_float(softcap), c_int(chunk),
           (_off(gate, gate_col) if gate is not None else c_void_p(0)), c_int(gate.shape[-1] if gate is not None else 0),
-          c_void_p(stream if stream is not None else current_stream_ptr()))
+          _p(slopes), _p(sink), c_void_p(stream if stream is not None else current_stream_ptr()))
 
 
 def attention_tc(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, out: torch.Tensor, mode: int,
@@ -615,15 +619,18 @@ def attention_tc(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, ou
                  page: int, window: int, scale: float, n_splits: int = 1, split_keys: int = 0,
                  part_o: Optional[torch.Tensor] = None, part_ml: Optional[torch.Tensor] = None,
                  err: Optional[torch.Tensor] = None, stream: Optional[int] = None, softcap: float = 0.0, chunk: int = 0,
-                 gate: Optional[torch.Tensor] = None, gate_col: int = 0) -> None:
+                 gate: Optional[torch.Tensor] = None, gate_col: int = 0, slopes: Optional[torch.Tensor] = None,
+                 sink: Optional[torch.Tensor] = None) -> None:
     """bf16 attention over the paged cache on tensor cores (TMA-fed); ``softcap`` > 0 caps the scaled scores by a tanh,
-    ``chunk`` > 0 lets position i see j only if floor(i / chunk) == floor(j / chunk), ``gate`` is the gate per element of
-    ``attention_fa``.  Splits are ranges of keys from key 0 on, under a chunk from the 64-key tile that holds the chunk's
+    ``chunk`` > 0 lets position i see j only if floor(i / chunk) == floor(j / chunk), ``gate``, ``slopes`` and
+    ``sink`` are those of ``attention_fa``.  Splits are ranges of keys from key 0 on, under a chunk from the 64-key tile that holds the chunk's
     first key.  ``mode`` 0 takes tiles of
     prompt portions, 1 takes single-token tiles and may split their key range: with ``part_o`` / ``part_ml`` the
     splits' partial results go through those buffers and a second kernel merges them; without them (at most 8
     splits) the splits of a tile are a thread-block cluster and are merged in shared memory."""
     _check_element_gate(gate, gate_col, n_heads * head_dim)
+    _check_slopes(slopes, n_heads)
+    _check_slopes(sink, n_heads)
     _check(q, "q", torch.bfloat16)
     _check(out, "out", torch.bfloat16)
     _check(k_pool, "k_pool", torch.bfloat16)
@@ -642,7 +649,8 @@ def attention_tc(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, ou
           c_int(head_dim), _p(tiles), c_int(n_tiles), _p(block_table), c_int(block_table.shape[-1]), c_int(page),
           c_int(k_pool.shape[0]), c_int(window), c_float(scale), c_int(n_splits), c_int(split_keys), _p(part_o),
           _p(part_ml), _p(err), c_float(softcap), c_int(chunk), (_off(gate, gate_col) if gate is not None else c_void_p(0)),
-          c_int(gate.shape[-1] if gate is not None else 0), c_void_p(stream if stream is not None else current_stream_ptr()))
+          c_int(gate.shape[-1] if gate is not None else 0), _p(slopes), _p(sink),
+          c_void_p(stream if stream is not None else current_stream_ptr()))
 
 
 # ------------------------------------------------ norms and gates around a sublayer (csrc/norm_gate.cu)
@@ -696,6 +704,22 @@ def gated_norm_add(y: torch.Tensor, gate_logits: Optional[torch.Tensor], weight:
             raise KernelError("gated_norm_add: the rounded copy does not fit the rows")
     _call(lib, lib.ember_gated_norm_add, _p(y), _p(gate_logits), _p(gate_bias), _p(weight), _p(bias), c_float(eps), c_int(1 if centred else 0),
           _p(residual), _p(rounded), c_int(n_rows), c_int(H), _stream(stream))
+
+
+def norm_add_norm(y: torch.Tensor, weight: torch.Tensor, eps: float, residual: torch.Tensor, next_weight: torch.Tensor, next_eps: float,
+                  out: torch.Tensor, n_rows: int, stream: Optional[int] = None) -> None:
+    """residual[r] += rms_norm(y[r]) and out[r] = rms_norm(residual[r]) of the new rows, each norm with its weight and eps, in
+    one kernel; fp32 (``out`` may be bfloat16)."""
+    for t, n in ((y, "y"), (weight, "weight"), (residual, "residual"), (next_weight, "next_weight")):
+        _check(t, n, torch.float32)
+    _check(out, "out")
+    H = residual.shape[-1]
+    if any(t.shape[-1] != H or t.numel() < n_rows * H for t in (y, out)) or weight.numel() != H or next_weight.numel() != H or \
+            residual.numel() < n_rows * H:
+        raise KernelError(f"norm_add_norm: rows of {H}, y {tuple(y.shape)}, out {tuple(out.shape)}")
+    lib = _lib("norm_gate")
+    _call(lib, lib.ember_norm_add_norm, _p(y), _p(weight), c_float(eps), _p(residual), _p(next_weight), c_float(next_eps), _p(out),
+          c_int(dtype_code(out.dtype)), c_int(n_rows), c_int(H), _stream(stream))
 
 
 def scaled_add_norm(y: torch.Tensor, y_bias: Optional[torch.Tensor], alpha: float, weight: torch.Tensor, bias: Optional[torch.Tensor],
@@ -992,26 +1016,26 @@ def ssm_scan(conv: torch.Tensor, dt: torch.Tensor, dt_col: int, dt_bias: torch.T
 SELECTIVE_MAX_STATES = 256       # states a channel the selective scan takes
 
 
-def selective_scan(x: torch.Tensor, dt: torch.Tensor, bc: torch.Tensor, bc_col: int, z: torch.Tensor, z_col: int, dt_bias: torch.Tensor,
+def selective_scan(x: torch.Tensor, dt: torch.Tensor, bc: torch.Tensor, bc_col: int, z: torch.Tensor, z_col: int,
                    a: torch.Tensor, skip: torch.Tensor, state: torch.Tensor, out: torch.Tensor, query_start: torch.Tensor,
                    slots: torch.Tensor, T: int, S: int, stream: Optional[int] = None) -> None:
     """Selective scan with a diagonal state per channel over the step's runs (csrc/selective_scan.cu).  ``x`` fp32 [T, inner]
-    (after convolution and silu), ``dt`` fp32 [T, inner] raw steps (softplus of them plus ``dt_bias`` is taken here), ``bc`` fp32
+    (after convolution and silu), ``dt`` fp32 [T, inner] the steps, ``bc`` fp32
     with B and C behind one another from column ``bc_col`` on, ``z`` fp32 with the gate from column ``z_col`` on, ``a`` fp32
     [inner, states] = -exp(A_log) log2(e), ``skip`` [inner]; a request's state is the first inner * states floats of its row
     of ``state``.  out [T, inner] (fp32 or bfloat16) = (S C + skip x) silu(z)."""
-    for t, n in ((x, "x"), (dt, "dt"), (bc, "bc"), (z, "z"), (dt_bias, "dt_bias"), (a, "a"), (skip, "skip"), (state, "state")):
+    for t, n in ((x, "x"), (dt, "dt"), (bc, "bc"), (z, "z"), (a, "a"), (skip, "skip"), (state, "state")):
         _check(t, n, torch.float32)
     _check(out, "out")
     _check_runs(query_start, slots, S)
     inner, N = a.shape
     if x.shape[-1] != inner or dt.shape[-1] != inner or z.shape[-1] < z_col + inner or bc.shape[-1] < bc_col + 2 * N or \
-            min(x.shape[0], dt.shape[0], z.shape[0], bc.shape[0]) < T or dt_bias.numel() != inner or skip.numel() != inner or \
+            min(x.shape[0], dt.shape[0], z.shape[0], bc.shape[0]) < T or skip.numel() != inner or \
             out.shape[-1] != inner or out.numel() < T * inner or state.dim() != 2 or state.shape[1] < inner * N:
         raise KernelError(f"selective_scan: buffers do not fit {inner} channels of {N} states")
     lib = _lib("selective_scan")
     _call(lib, lib.ember_selective_scan, _p(x), c_int(x.shape[-1]), _p(dt), c_int(dt.shape[-1]), _off(bc, bc_col), c_int(bc.shape[-1]),
-          _off(z, z_col), c_int(z.shape[-1]), _p(dt_bias), _p(a), _p(skip), _p(state), c_longlong(state.shape[1]), _p(out),
+          _off(z, z_col), c_int(z.shape[-1]), _p(a), _p(skip), _p(state), c_longlong(state.shape[1]), _p(out),
           c_int(dtype_code(out.dtype)), _p(query_start), _p(slots), c_int(T), c_int(S), c_int(inner), c_int(N), _stream(stream))
 
 
@@ -1166,7 +1190,7 @@ def _check_slopes(slopes, heads: int) -> None:
     if slopes is not None:
         _check(slopes, "slopes", torch.float32)
         if slopes.numel() != heads:
-            raise KernelError(f"attention: {slopes.numel()} distance slopes for {heads} heads")
+            raise KernelError(f"attention: {slopes.numel()} distance slopes or sinks for {heads} heads")
 
 
 def head_gate_apply(x: torch.Tensor, gate: torch.Tensor, gate_col: int, T: int, heads: int, vdim: int, stream: Optional[int] = None) -> None:
@@ -1334,9 +1358,15 @@ def rotate_pairs(x: torch.Tensor, x_head: int, x_col: int, out: torch.Tensor, ou
 
 
 def head_gemm(x: torch.Tensor, x_head: int, x_col: int, w: torch.Tensor, out: torch.Tensor, out_head: int, out_col: int, T: int,
-              gate: Optional[torch.Tensor] = None, gate_col: int = 0, stream: Optional[int] = None) -> None:
+              gate: Optional[torch.Tensor] = None, gate_col: int = 0, stream: Optional[int] = None, bias: Optional[torch.Tensor] = None,
+              softplus: bool = False) -> None:
     """out[t, h, out_col + n] = sum_k x[t, h, x_col + k] * w[h, n, k], a product per head (``w`` [heads, N, K]); with
-    ``gate`` (fp32 rows) the result is multiplied by sigmoid(gate[t, gate_col + h N + n]).  x fp32 2-D."""
+    ``gate`` (fp32 rows) the result is multiplied by sigmoid(gate[t, gate_col + h N + n]).  x fp32 2-D.  ``bias`` (fp32
+    [heads N]) joins the sum, and ``softplus`` is taken of it, before the gate."""
+    if bias is not None:
+        _check(bias, "bias", torch.float32)
+        if bias.numel() != w.shape[0] * w.shape[1]:
+            raise KernelError(f"head_gemm: a bias of {bias.numel()} for {tuple(w.shape)}")
     _check(x, "x", torch.float32)
     _check(w, "w")
     _check(out, "out")
@@ -1350,7 +1380,8 @@ def head_gemm(x: torch.Tensor, x_head: int, x_col: int, w: torch.Tensor, out: to
     lib = _lib("sink_attention")
     _call(lib, lib.ember_head_gemm, _p(x), c_int(x.shape[1]), c_int(x_head), c_int(x_col), _p(w), c_int(dtype_code(w.dtype)), _p(out),
           c_int(dtype_code(out.dtype)), c_int(out.shape[1]), c_int(out_head), c_int(out_col), _p(gate),
-          c_int(gate.shape[1] if gate is not None else 0), c_int(gate_col), c_int(T), c_int(H), c_int(N), c_int(K), _stream(stream))
+          c_int(gate.shape[1] if gate is not None else 0), c_int(gate_col), c_int(T), c_int(H), c_int(N), c_int(K), _p(bias),
+          c_int(1 if softplus else 0), _stream(stream))
 
 
 def sink_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: Optional[torch.Tensor], out: torch.Tensor, T: int, heads: int,

@@ -196,11 +196,13 @@ class Attention(Mixer):
         return [(ops.attention_tile_queries(s.group), "all")]
 
     def attend(self, ctx, q: torch.Tensor, cache, table: torch.Tensor, out: torch.Tensor, gate: Optional[torch.Tensor] = None,
-               gate_col: int = 0) -> None:
+               gate_col: int = 0, slopes: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None) -> None:
         """out[t, h, :] = softmax over the visible keys of (q . k * scale) times v; with ``gate`` (fp32 logits, from column
-        ``gate_col`` on) element i of a token's result is multiplied by the sigmoid of its logit i."""
+        ``gate_col`` on) element i of a token's result is multiplied by the sigmoid of its logit i; with ``slopes`` (fp32, one a
+        head) slope * (i - j) is taken off the scores, with ``sink`` exp(sink) joins the denominators."""
         s = self.spec
-        kw = dict(err=ctx.err, stream=ctx.stream, softcap=self.softcap, chunk=self.chunk, gate=gate, gate_col=gate_col)
+        kw = dict(err=ctx.err, stream=ctx.stream, softcap=self.softcap, chunk=self.chunk, gate=gate, gate_col=gate_col,
+                  slopes=slopes, sink=sink)
         multi, single = self._tc_modes()
         if multi and ops.TC_ENABLED:
             tq = ops.attention_tc_tile_queries(s.group)
@@ -243,8 +245,8 @@ class Attention(Mixer):
                 ops.attention_tc(q, cache.k, cache.v, out, 1, *args, tiles, n, table, cache.page_tokens, s.window,
                                  self.scale, n_splits, split_keys, part_o, part_ml, **kw)
             return
-        if self.softcap > 0 or self.chunk > 0 or gate is not None:
-            raise ops.KernelError("attention: the general kernel has no score cap, chunks or gate (the tensor-core kernels have)")
+        if self.softcap > 0 or self.chunk > 0 or any(t is not None for t in (gate, slopes, sink)):
+            raise ops.KernelError("attention: the general kernel has no score cap, chunks, gate, slopes or sink (the tensor-core kernels have)")
         tile_q = ops.attention_tile_queries(s.group)
         tiles, n_tiles = ctx.attention_tiles(tile_q, "all")
         # long key ranges of a small step are cut into fixed splits so that more SMs share them

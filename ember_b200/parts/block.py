@@ -19,6 +19,7 @@ import torch
 from .. import ops
 from ..config.spec import ConfigError
 from .base import CacheNeed, Runtime, WeightDecl
+from .norm import RMSNorm
 from .registry import build_part, register_part
 
 
@@ -121,7 +122,11 @@ class GatedSandwichBlock(Arrangement):
     The input norms may be left out as well: the sublayer then reads the residual stream itself,
     ``h += norm_out(sublayer(h))``.  On the float32 path that is the stream's own buffer; on the bfloat16 path it is the
     stream rounded once, which the ``gated_add`` before it leaves beside the new residual rows (the first sublayer of
-    a step, or one that follows another arrangement, rounds the stream in a kernel of its own)."""
+    a step, or one that follows another arrangement, rounds the stream in a kernel of its own).
+
+    Without a gate, and with RMS norms on both sides, the output norm, the addition and the *next* sublayer's input norm
+    are one kernel (``add_then_norm``): the feed-forward's of this layer, and the mixer's of the layer that runs next, which
+    the model names in ``ctx.memo["block.next_norm"]`` and which finds its normed rows in the blocks' common buffer."""
 
     ROLES = {"mixer_norm": "norm", "mixer": "mixer", "mixer_gate": "gate", "mixer_out_norm": "norm",
              "feed_forward_norm": "norm", "feed_forward": "feed_forward", "feed_forward_gate": "gate",
@@ -150,12 +155,20 @@ class GatedSandwichBlock(Arrangement):
             ops.round_rows(h, r, ctx.T * h.shape[-1], stream=ctx.stream)
         return r, r
 
-    def _sublayer(self, ctx, h, x, norm_in, run, gate, norm_out, can_store: bool) -> None:
+    @property
+    def leading_norm(self):
+        """The norm the layer begins with (None if its mixer reads the stream itself)."""
+        return self.parts.get("mixer_norm")
+
+    def _sublayer(self, ctx, h, x, norm_in, run, gate, norm_out, can_store: bool, normed: bool = False, norm_next=None) -> bool:
+        """``normed``: x already holds the normed rows.  Returns whether x was left holding ``norm_next`` of the new stream."""
         T, hidden = ctx.T, h.shape[-1]
         y = ctx.buf("block.sublayer", (ctx.max_tokens, hidden), torch.float32)
         rounded = None
+        normed_x = x
         if norm_in is not None:
-            norm_in.forward(ctx, h, x, T)
+            if not normed:
+                norm_in.forward(ctx, h, x, T)
         else:
             x, rounded = self._stream(ctx, h)
         if not can_store:
@@ -165,12 +178,16 @@ class GatedSandwichBlock(Arrangement):
         if gate is not None:
             logits = ctx.buf("block.gate", (ctx.max_tokens, hidden), torch.float32)
             gate.forward(ctx, x, logits)
+        if gate is None and rounded is None and isinstance(norm_out, RMSNorm) and isinstance(norm_next, RMSNorm):
+            norm_out.add_then_norm(ctx, y, h, T, norm_next, normed_x)
+            return True
         if rounded is not None:
             norm_out.gated_add(ctx, y, logits, h, T, gate_bias=getattr(gate, "bias", None), rounded=rounded)
             ctx.memo["block.stream_rounded.at"] = ctx.memo.get("schedule.index")
             ctx.memo["block.stream_rounded.of"] = h.data_ptr()
         else:
             norm_out.gated_add(ctx, y, logits, h, T, gate_bias=getattr(gate, "bias", None))
+        return False
 
     def forward(self, ctx, h: torch.Tensor, caches, owns_cache: bool = True) -> None:
         p = self.parts
@@ -178,14 +195,18 @@ class GatedSandwichBlock(Arrangement):
         mixer = p["mixer"]
         store = bool(getattr(mixer, "can_store", False))
         kw = {"accumulate": False} if store else {}
-        self._sublayer(ctx, h, x, p.get("mixer_norm"), lambda x, y: mixer.forward(ctx, x, y, self.cache_of(caches), owns_cache, **kw),
-                       p.get("mixer_gate"), p["mixer_out_norm"], store)
-        ff = p.get("feed_forward")
+        ff, next_layer = p.get("feed_forward"), ctx.memo.get("block.next_norm")
+        left = ctx.memo.pop("block.normed.for", None) == (ctx.memo.get("schedule.index"), h.data_ptr())
+        left = self._sublayer(ctx, h, x, p.get("mixer_norm"), lambda x, y: mixer.forward(ctx, x, y, self.cache_of(caches), owns_cache, **kw),
+                              p.get("mixer_gate"), p["mixer_out_norm"], store, normed=left,
+                              norm_next=p.get("feed_forward_norm") if ff is not None else next_layer)
         if ff is not None:
             store = bool(getattr(ff, "can_store", False))
-            kw = {"accumulate": False} if store else {}
-            self._sublayer(ctx, h, x, p.get("feed_forward_norm"), lambda x, y: ff.forward(ctx, x, y, **kw),
-                           p.get("feed_forward_gate"), p["feed_forward_out_norm"], store)
+            kwf = {"accumulate": False} if store else {}
+            left = self._sublayer(ctx, h, x, p.get("feed_forward_norm"), lambda x, y: ff.forward(ctx, x, y, **kwf),
+                                  p.get("feed_forward_gate"), p["feed_forward_out_norm"], store, normed=left, norm_next=next_layer)
+        if left:
+            ctx.memo["block.normed.for"] = (ctx.memo["schedule.index"] + 1, h.data_ptr())
 
 
 class ConnectedPreNormBlock(Arrangement):

@@ -48,6 +48,10 @@ class RMSNorm(Norm):
         ops.gated_norm_add(y, gate_logits, self.weight, None, self.spec.eps, False, residual, n_rows, gate_bias=gate_bias,
                            rounded=rounded, stream=ctx.stream)
 
+    def add_then_norm(self, ctx, y: torch.Tensor, residual: torch.Tensor, n_rows: int, after: "RMSNorm", out: torch.Tensor) -> None:
+        """residual += norm(y), and ``out`` = the norm ``after`` of the new rows, in one kernel."""
+        ops.norm_add_norm(y, self.weight, self.spec.eps, residual, after.weight, after.spec.eps, out, n_rows, stream=ctx.stream)
+
     def scaled_add(self, ctx, y: torch.Tensor, residual: torch.Tensor, n_rows: int, alpha: float,
                    y_bias: Optional[torch.Tensor] = None, rounded: Optional[torch.Tensor] = None) -> None:
         """residual = norm(alpha * residual + y + y_bias) in one kernel, in place: the norm after the residual sum;

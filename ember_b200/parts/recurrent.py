@@ -432,7 +432,8 @@ class SelectiveScan(_StateMixer):
         S[c, n] <- exp(-dt_c exp(A_log[c, n])) S[c, n] + dt_c x_c B_n;  y_c = sum_n S[c, n] C_n + D_c x_c
 
     then y * silu(z) and the output product.  The products read bfloat16 operands on the bfloat16 path and leave fp32; steps,
-    decays, B, C and the state are fp32.  The step's projection reads ``low`` where the product before it left it.  The
+    decays, B, C and the state are fp32.  The step's projection reads ``low`` where the product before it left it, and adds
+    the bias and takes the softplus where it stores.  The
     state row of a request holds S [inner, states] and, behind it, the convolution's last inputs.  Tensors under the
     prefix: in, conv, conv.b, x, dt, dt.b, A_log, D, o."""
 
@@ -485,8 +486,8 @@ class SelectiveScan(_StateMixer):
         ops.conv_silu(proj, 0, self.taps, self.conv_bias, cache.state, inner * N, ctx.seq_of, ctx.query_start, ctx.state_slots,
                       conv, T, ctx.S, stream=ctx.stream, rounded=conv_r if half else None)
         self.x_proj(ctx, conv_r, low, T, ops.EPI_STORE_F32)
-        ops.head_gemm(low, R, 0, self.dt_w, dt, inner, 0, T, stream=ctx.stream)
-        ops.selective_scan(conv, dt, low, R, proj, inner, self.dt_bias, self.a, self.skip, cache.state, y, ctx.query_start,
+        ops.head_gemm(low, R, 0, self.dt_w, dt, inner, 0, T, stream=ctx.stream, bias=self.dt_bias, softplus=True)
+        ops.selective_scan(conv, dt, low, R, proj, inner, self.a, self.skip, cache.state, y, ctx.query_start,
                            ctx.state_slots, T, ctx.S, stream=ctx.stream)
         self._out(ctx, y, out, accumulate)
 

@@ -112,13 +112,13 @@ class SinkAttention(_SinkSoftmax):
         # the general preparation kernel serves whatever the whole-projection one does not know
         self.general = (s.qk_norm == "head" or s.position.kind != "none" or s.q_temp_every > 0 or bool(s.value_mix)
                         or s.slope_span > 0)
-        # Causal softmax over keys and values of equal size (no sink, no kept first tokens, no distance bias; a window, a
-        # cap and chunks are parameters) is what
+        # Causal softmax over keys and values of equal size (no kept first tokens; a window, a cap, chunks, distance slopes
+        # and the sink are parameters) is what
         # the engine's TMA-fed kernels compute (tcgen05 for prompt portions, mma.sync with key splits for single tokens):
         # where they take the geometry, a bfloat16 step goes to them (``load`` decides, once the dtype and the page size
         # are known); a gate per head then is a pass of its own behind them
         self.dense = None
-        if (not s.sink and (s.window == 0 or s.keep_first == 0) and s.slope_span == 0 and s.value_dim == s.head_dim and s.scale > 0
+        if ((s.window == 0 or s.keep_first == 0) and s.value_dim == s.head_dim and s.scale > 0
                 and s.head_dim % 2 == 0 and s.num_heads // s.num_kv_heads <= ops.ATTENTION_MAX_GROUP):
             from ..config.spec import AttentionSpec
             from .attention import Attention
@@ -260,7 +260,8 @@ class SinkAttention(_SinkSoftmax):
                                  ctx.seq_of, table, cache.page_tokens, cache.k, cache.v, q, write_kv=owns_cache, err=ctx.err,
                                  stream=ctx.stream)
         if self.dense is not None and getattr(self.dense, "rt", None) is not None and ops.TC_ENABLED:
-            self.dense.attend(ctx, q, cache, table, att, gate=proj if s.element_gate else None, gate_col=self.channels)
+            self.dense.attend(ctx, q, cache, table, att, gate=proj if s.element_gate else None, gate_col=self.channels,
+                              slopes=self.slopes, sink=self.sink)
             if s.head_gate:
                 ops.head_gate_apply(att, proj, self.channels, T, H, V, stream=ctx.stream)
         else:
