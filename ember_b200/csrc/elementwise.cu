@@ -97,6 +97,15 @@ __global__ void place_columns_kernel(const float* __restrict__ x, TO* __restrict
     }
 }
 
+// out[t, i] = x[t, i] for i < n: some columns of fp32 rows as rows of their own.
+template <typename TO>
+__global__ void round_columns_kernel(const float* __restrict__ x, int ldx, TO* __restrict__ out, int n, size_t total) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i < total) out[i] = from_float<TO>(x[i / n * ldx + i % n]);
+}
+
 // -------------------------------------------------------------------------------- RMSNorm
 // out[r, i] = w[i] * (x[row(r), i] * (1 / sqrt(mean(x^2) + eps))), statistics in fp32.
 // `rows` (nullable) gathers input rows: the final norm runs only on the rows whose logits
@@ -514,6 +523,17 @@ EMBER_API int ember_embed_bigram(const int* tokens, const int* prev_ids, int n_p
         else run(embed_bigram_kernel<__nv_bfloat16, __nv_bfloat16>, (const __nv_bfloat16*)table);
     }
     return check_launch("embed_bigram");
+}
+
+EMBER_API int ember_round_columns(const float* x, int ldx, void* out, int out_dtype, int T, int n, void* stream) {
+    if (T <= 0) return 0;
+    if (n <= 0 || n > ldx) return fail("round_columns: %d columns of rows of %d", n, ldx);
+    const size_t total = (size_t)T * n;
+    const unsigned blocks = (unsigned)((total + 255) / 256);
+    if (out_dtype == EMBER_F32) launch_kernel(round_columns_kernel<float>, blocks, 256, 0, (cudaStream_t)stream, x, ldx, (float*)out, n, total);
+    else if (out_dtype == EMBER_BF16) launch_kernel(round_columns_kernel<__nv_bfloat16>, blocks, 256, 0, (cudaStream_t)stream, x, ldx, (__nv_bfloat16*)out, n, total);
+    else return fail("round_columns: unsupported output dtype %d", out_dtype);
+    return check_launch("round_columns");
 }
 
 EMBER_API int ember_place_columns(const float* x, void* out, int out_dtype, int T, int H, int ld, int col, int col2, void* stream) {

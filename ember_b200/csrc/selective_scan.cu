@@ -6,12 +6,18 @@
 // and out = y * silu(z).  Everything is fp32 (`out` may be bfloat16: it is the operand of the next product).  The decay is
 // taken as 2^(dt a) with a = -exp(A_log) log2(e) made once when the weights are loaded.
 //
-// A step's tokens are S runs (query_start [S + 1]); run s belongs to state slot slots[s], whose row holds S as [inner, N].
-// A block walks one run for CB channels: LPC neighbouring lanes share a channel, each with NS of its states in registers,
-// so the loop over tokens has no exchange between lanes at all: a lane leaves its partial of sum_n S C in shared memory
-// and the pass that finishes a chunk of CT tokens adds the LPC partials in lane order.  While a chunk is computed the next
-// one's inputs travel into registers.  A prompt portion and a single decoded token are the same code (CT 16 and 1), so
-// the state after a step does not depend on how the tokens were cut into steps.
+// A step's tokens are S runs (query_start [S + 1]); run s belongs to state slot slots[s], whose row holds S as [N, inner]
+// (neighbouring channels side by side, like every other operand).  A block walks one run for 32 channels: a lane is a
+// channel, and the block's NW warps share its states, NS each, in registers.  A token's B and C are then the same address for
+// a whole warp, the loop over tokens has no exchange between threads at all, and a warp leaves its partials of sum_n S C in
+// shared memory for the pass that finishes a chunk of CT tokens, which adds the warps' partials in order.  (With neighbouring
+// lanes sharing a channel the B and C reads were four shared-memory wavefronts a warp and token and bounded the kernel.)
+// States go two by two through packed fp32 arithmetic.  As many warps again bring the inputs, by cp.async into a ring of
+// chunks some way ahead (what a block has in flight is what keeps the memory busy: with one chunk in flight the kernel waited
+// for it), and finish the chunk before (sums, gate, store) while a chunk is computed: one barrier a chunk.
+// A step whose runs are single tokens takes a kernel of its own, a thread a channel with all its states.
+#include <type_traits>
+
 #include "common.cuh"
 
 EMBER_DEFINE_LAST_ERROR
@@ -24,47 +30,43 @@ __device__ __forceinline__ float exp2_approx(float x) {
     return y;
 }
 
-constexpr int SS_THREADS = 128;
+constexpr int SS_CHUNK = 32;          // tokens a chunk
+constexpr int SS_RING = 5;            // chunks of inputs in shared memory: one being finished, one computed, the rest on their way
 
 struct SelectiveArgs {
     const float* x; int ld_x;                  // [T, inner] after convolution and silu
     const float* dt; int ld_dt;                // [T, inner] steps
     const float* bc; int ld_bc;                // [T, B (N) | C (N)]
     const float* z; int ld_z;                  // [T, inner] gate
-    const float* a; const float* skip;         // [inner, N], [inner]
-    float* state; long long state_stride;      // [slot][inner][N]
+    const float* a; const float* skip;         // [N, inner], [inner]
+    float* state; long long state_stride;      // [slot][N][inner]
     void* out;                                 // [T, inner]
     const int* query_start; const int* slots;
     int inner, N;
-    int vec;                                   // states of a lane lie on vector boundaries in global memory
+    int by16;                                  // rows of x, dt and z can be copied 16 bytes at a time
 };
 
-// NS neighbouring floats: the widest vectors NS allows.
-template <int NS>
-__device__ __forceinline__ void read_row(const float* p, float (&v)[NS]) {
-    if (NS % 4 == 0) {
-#pragma unroll
-        for (int i = 0; i < NS / 4; i++) {
-            const float4 f = reinterpret_cast<const float4*>(p)[i];
-            v[4 * i] = f.x; v[4 * i + 1] = f.y; v[4 * i + 2] = f.z; v[4 * i + 3] = f.w;
-        }
-    } else {
-#pragma unroll
-        for (int i = 0; i < NS / 2; i++) {
-            const float2 f = reinterpret_cast<const float2*>(p)[i];
-            v[2 * i] = f.x; v[2 * i + 1] = f.y;
-        }
-    }
+// Packed fp32 pairs.
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pk2(float lo, float hi) {
+    f32x2 r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "r"(__float_as_uint(lo)), "r"(__float_as_uint(hi)));
+    return r;
 }
-template <int NS>
-__device__ __forceinline__ void write_row(float* p, const float (&v)[NS]) {
-    if (NS % 4 == 0) {
-#pragma unroll
-        for (int i = 0; i < NS / 4; i++) reinterpret_cast<float4*>(p)[i] = make_float4(v[4 * i], v[4 * i + 1], v[4 * i + 2], v[4 * i + 3]);
-    } else {
-#pragma unroll
-        for (int i = 0; i < NS / 2; i++) reinterpret_cast<float2*>(p)[i] = make_float2(v[2 * i], v[2 * i + 1]);
-    }
+__device__ __forceinline__ float2 up2(f32x2 v) {
+    uint32_t lo, hi;
+    asm("mov.b64 {%0, %1}, %2;" : "=r"(lo), "=r"(hi) : "l"(v));
+    return make_float2(__uint_as_float(lo), __uint_as_float(hi));
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+    f32x2 d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+    f32x2 d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
 }
 // z sigmoid(z); the bfloat16 form with the fast exponential and division.
 template <typename TO>
@@ -74,156 +76,228 @@ __device__ __forceinline__ float silu_<float>(float z) { return z / (1.0f + expf
 template <>
 __device__ __forceinline__ float silu_<__nv_bfloat16>(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
 
-template <int LPC, int NS, int CT, typename TO>
-__global__ void __launch_bounds__(SS_THREADS) selective_scan_kernel(SelectiveArgs p) {
-    constexpr int CB = SS_THREADS / LPC, NP = LPC * NS;            // channels a block, states a channel (with padding)
-    constexpr int EPT = (CT * CB + SS_THREADS - 1) / SS_THREADS;   // (token, channel) elements of a chunk a thread stages
-    constexpr int BPT = (2 * CT * NP + SS_THREADS - 1) / SS_THREADS;
-    constexpr bool EVEN = CT * CB % SS_THREADS == 0;               // every thread has EPT elements, all of one channel
-    static_assert(NS % 2 == 0, "a lane's states are read in pairs or fours");
+__device__ __forceinline__ void copy16(void* dst, const void* src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void copy4(void* dst, const void* src) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+
+// NW warps compute, NW warps feed them and finish what they leave.
+template <int NW, int NS, int CT, int RING, typename TO>
+__global__ void __launch_bounds__(64 * NW) selective_scan_kernel(SelectiveArgs p) {
+    constexpr int THREADS = 32 * NW, NP = NW * NS, N2 = NS / 2;    // states a channel (with padding); pairs a thread
+    constexpr int TILE = CT * 32;                                  // a chunk's elements of x, of dt and of z
+    static_assert(NS % 2 == 0 && CT % NW == 0 && RING >= 4, "states go two by two, tokens are shared out evenly");
     extern __shared__ __align__(16) float smem[];
-    float2* du = reinterpret_cast<float2*>(smem);      // 2 x [CT][CB] (step, step times input)
-    float* bs = smem + 4 * CT * CB;                    // 2 x [CT][NP] pairs (B, C)
-    float* yp = bs + 4 * CT * NP;                      // [CT][SS_THREADS] partial read-outs
+    float* xs = smem;                                  // RING x [x | dt | z] x [CT][32]
+    float* bs = xs + RING * 3 * TILE;                  // RING x [CT][NP / 2] (B, B, C, C) of two states
+    float* yp = bs + RING * CT * NP * 2;               // 2 x [CT][NW][32] partial read-outs
     pdl_launch_dependents();
-    pdl_wait();
-    const int s = blockIdx.y, c0 = blockIdx.x * CB, inner = p.inner, N = p.N;
-    const int cl = threadIdx.x / LPC, l = threadIdx.x % LPC, c = c0 + cl, n0 = l * NS;
-    const int first = p.query_start[s], end = p.query_start[s + 1];
-    float* S = p.state + (size_t)p.slots[s] * p.state_stride + (size_t)c * N + n0;
-    const float* A = p.a + (size_t)c * N + n0;
-    // what this thread stages and finishes: tokens threadIdx.x / CB, + SS_THREADS / CB, ... of a chunk, all of channel ec
-    const int ec = c0 + threadIdx.x % CB, et = threadIdx.x / CB;
-    const bool mine = ec < inner && (EVEN || threadIdx.x < CT * CB);
-    const float skip = mine ? p.skip[ec] : 0.0f;
-    const float* px = p.x + ec;
-    const float* pd = p.dt + ec;
-    const float* pz = p.z + ec;
-
-    float fx[EPT], fd[EPT], fz[EPT], fb[BPT], gx[EPT], gz[EPT];
-    auto fetch = [&](int t0) {                 // the chunk from t0 on: into registers
-#pragma unroll
-        for (int e = 0; e < EPT; e++) {
-            const int t = t0 + et + e * (SS_THREADS / CB);
-            const bool in = mine && t < end;
-            fx[e] = in ? px[(size_t)t * p.ld_x] : 0.0f;
-            fd[e] = in ? pd[(size_t)t * p.ld_dt] : 0.0f;
-            fz[e] = in ? pz[(size_t)t * p.ld_z] : 0.0f;
-        }
-#pragma unroll
-        for (int e = 0; e < BPT; e++) {
-            const int i = threadIdx.x + e * SS_THREADS, t = t0 + i / (2 * NP), w = i % (2 * NP), n = w % NP;
-            const bool in = (2 * CT * NP % SS_THREADS == 0 || i < 2 * CT * NP) && t < end && n < N;
-            fb[e] = in ? p.bc[(size_t)t * p.ld_bc + (w < NP ? 0 : N) + n] : 0.0f;
-        }
-    };
-    auto stage = [&](int buf) {                // and from there into shared memory
-#pragma unroll
-        for (int e = 0; e < EPT; e++) {
-            gx[e] = fx[e];
-            gz[e] = fz[e];
-            if (EVEN || threadIdx.x < CT * CB) du[buf * CT * CB + threadIdx.x + e * SS_THREADS] = make_float2(fd[e], fd[e] * fx[e]);
-        }
-#pragma unroll
-        for (int e = 0; e < BPT; e++) {
-            const int i = threadIdx.x + e * SS_THREADS, w = i % (2 * NP);
-            if (2 * CT * NP % SS_THREADS == 0 || i < 2 * CT * NP) bs[(buf * CT + i / (2 * NP)) * 2 * NP + (w % NP) * 2 + w / NP] = fb[e];
-        }
-    };
-
-    fetch(first);
-    float st[NS], a[NS];
-    const bool whole = p.vec && c < inner && n0 + NS <= N;
-    if (whole) {
-        read_row<NS>(S, st);
-        read_row<NS>(A, a);
-    } else {
-#pragma unroll
-        for (int i = 0; i < NS; i++) {
-            const bool in = c < inner && n0 + i < N;
-            st[i] = in ? S[i] : 0.0f;
-            a[i] = in ? A[i] : 0.0f;           // (a padded state decays by 1 and gets B = 0: it stays zero)
-        }
-    }
-    stage(0);
+    const int s = blockIdx.y, inner = p.inner, N = p.N;
+    const int lane = threadIdx.x & 31, c0 = blockIdx.x * 32, c = c0 + lane;
+    const bool feeds = threadIdx.x >= THREADS;
+    const int warp = (threadIdx.x >> 5) - (feeds ? NW : 0), tid = threadIdx.x - (feeds ? THREADS : 0);
+    for (int i = threadIdx.x; i < RING * CT * NP * 2; i += 2 * THREADS) bs[i] = 0.0f;      // (B and C of padded states stay zero)
     __syncthreads();
-    int cur = 0;
-    for (int t0 = first; t0 < end; t0 += CT, cur ^= 1) {
-        const bool more = t0 + CT < end;
-        if (more) fetch(t0 + CT);
-        const int n_tok = min(CT, end - t0);
-        const float2* dc = du + cur * CT * CB + cl;
-        const float* bc = bs + (cur * CT * NP + n0) * 2;
-        auto token = [&](int tt) {
-            const float2 d = dc[tt * CB];
-            float pair[2 * NS];                // B and C in turn
-            read_row<2 * NS>(bc + tt * 2 * NP, pair);
-            float acc = 0.0f;
+    pdl_wait();
+    const int first = p.query_start[s], end = p.query_start[s + 1];
+    const int chunks = (end - first + CT - 1) / CT;
+    const bool live = c < inner;
+    if (feeds) {
+        const float skip = live ? p.skip[c] : 0.0f;
+        auto issue = [&](int i) {              // the inputs of chunk i on their way
+            const int t0 = first + i * CT, n_tok = min(CT, end - t0);
+            if (n_tok > 0) {
+                float* xd = xs + (i % RING) * 3 * TILE;
+                if (p.by16) {
 #pragma unroll
-            for (int i = 0; i < NS; i++) {
-                st[i] = fmaf(exp2_approx(d.x * a[i]), st[i], d.y * pair[2 * i]);
-                acc = fmaf(st[i], pair[2 * i + 1], acc);
+                    for (int e = tid; e < 3 * CT * 8; e += THREADS) {
+                        const int which = e / (CT * 8), r = e % (CT * 8), tt = r / 8, ch = c0 + (r % 8) * 4;
+                        const float* base = which == 0 ? p.x : (which == 1 ? p.dt : p.z);
+                        const int ld = which == 0 ? p.ld_x : (which == 1 ? p.ld_dt : p.ld_z);
+                        if (tt < n_tok && ch < inner) copy16(xd + which * TILE + r * 4, base + (size_t)(t0 + tt) * ld + ch);
+                    }
+                } else {
+                    for (int e = tid; e < 3 * TILE; e += THREADS) {
+                        const int which = e / TILE, r = e % TILE, tt = r / 32;
+                        const float* base = which == 0 ? p.x : (which == 1 ? p.dt : p.z);
+                        const int ld = which == 0 ? p.ld_x : (which == 1 ? p.ld_dt : p.ld_z);
+                        if (tt < n_tok && live) copy4(xd + which * TILE + r, base + (size_t)(t0 + tt) * ld + c);
+                    }
+                }
+                float* bd = bs + (i % RING) * CT * NP * 2;
+#pragma unroll 4
+                for (int e = tid; e < CT * 2 * NP; e += THREADS) {
+                    const int tt = e / (2 * NP), w = e % (2 * NP), n = w % NP;
+                    if (tt < n_tok && n < N)
+                        copy4(bd + tt * 2 * NP + (n >> 1) * 4 + (n & 1) + (w < NP ? 0 : 2), p.bc + (size_t)(t0 + tt) * p.ld_bc + (w < NP ? 0 : N) + n);
+                }
             }
-            yp[tt * SS_THREADS + threadIdx.x] = acc;
+            asm volatile("cp.async.commit_group;" ::: "memory");
+        };
+        auto finish = [&](int i) {             // chunk i: its partials, gate, store
+            const int t0 = first + i * CT, n_tok = min(CT, end - t0);
+            const float* xd = xs + (i % RING) * 3 * TILE + lane;
+            const float* yc = yp + (i & 1) * CT * THREADS + lane;
+#pragma unroll
+            for (int tt = warp; tt < CT; tt += NW) {
+                if (live && tt < n_tok) {
+                    const float* part = yc + tt * THREADS;
+                    float y0 = 0.0f, y1 = 0.0f;
+#pragma unroll
+                    for (int k = 0; k < NW; k += 2) { y0 += part[k * 32]; y1 += part[(k + 1) * 32]; }
+                    const float y = fmaf(skip, xd[tt * 32], y0 + y1);
+                    ((TO*)p.out)[(size_t)(t0 + tt) * inner + c] = from_float<TO>(y * silu_<TO>(xd[2 * TILE + tt * 32]));
+                }
+            }
+        };
+        for (int i = 0; i < RING - 2; i++) issue(i);
+        asm volatile("cp.async.wait_group %0;" ::"n"(RING - 3) : "memory");          // chunk 0 is there
+        __syncthreads();
+        for (int i = 0; i < chunks; i++) {
+            issue(i + RING - 2);               // (into the place of chunk i - 2, which has been finished)
+            if (i > 0) finish(i - 1);
+            asm volatile("cp.async.wait_group %0;" ::"n"(RING - 3) : "memory");      // chunk i + 1 is there
+            __syncthreads();
+        }
+        finish(chunks - 1);
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        return;
+    }
+    const int n0 = warp * NS;
+    float* S = p.state + (size_t)p.slots[s] * p.state_stride + c;
+    const float* A = p.a + c;
+    f32x2 st[N2], a[N2];
+#pragma unroll
+    for (int i = 0; i < N2; i++) {             // (a padded state decays by 1 and gets B = 0: it stays zero)
+        const int n = n0 + 2 * i;
+        const bool in0 = live && n < N, in1 = live && n + 1 < N;
+        st[i] = pk2(in0 ? S[(size_t)n * inner] : 0.0f, in1 ? S[(size_t)(n + 1) * inner] : 0.0f);
+        a[i] = pk2(in0 ? A[(size_t)n * inner] : 0.0f, in1 ? A[(size_t)(n + 1) * inner] : 0.0f);
+    }
+    __syncthreads();
+    for (int i = 0; i < chunks; i++) {
+        const int n_tok = min(CT, end - first - i * CT);
+        const float* xc = xs + (i % RING) * 3 * TILE + lane;
+        const float4* bc = reinterpret_cast<const float4*>(bs + (i % RING) * CT * 2 * NP + 2 * n0);
+        float* yc = yp + (i & 1) * CT * THREADS + warp * 32 + lane;
+        // a group of tokens: first everything that does not depend on the state (their operands, decays and inputs), then the
+        // chain through the state, then the stores (one between two tokens would keep the next one's operands from being
+        // fetched ahead of it)
+        auto group = [&](auto size, int g0) {
+            constexpr int GR = decltype(size)::value;
+            f32x2 decay[GR][N2], in[GR][N2], out[GR][N2];
+#pragma unroll
+            for (int k = 0; k < GR; k++) {
+                const float d = xc[TILE + (g0 + k) * 32], u = d * xc[(g0 + k) * 32];
+                const f32x2 dd = pk2(d, d), uu = pk2(u, u);
+#pragma unroll
+                for (int j = 0; j < N2; j++) {
+                    const float4 v = bc[(g0 + k) * (NP / 2) + j];                // the same address for the whole warp
+                    const float2 e = up2(mul2(dd, a[j]));
+                    decay[k][j] = pk2(exp2_approx(e.x), exp2_approx(e.y));
+                    in[k][j] = mul2(uu, pk2(v.x, v.y));
+                    out[k][j] = pk2(v.z, v.w);
+                }
+            }
+            float y[GR];
+#pragma unroll
+            for (int k = 0; k < GR; k++) {
+                f32x2 acc;
+#pragma unroll
+                for (int j = 0; j < N2; j++) {
+                    st[j] = fma2(decay[k][j], st[j], in[k][j]);
+                    acc = j == 0 ? mul2(st[j], out[k][j]) : fma2(st[j], out[k][j], acc);
+                }
+                const float2 r = up2(acc);
+                y[k] = r.x + r.y;
+            }
+#pragma unroll
+            for (int k = 0; k < GR; k++) yc[(g0 + k) * THREADS] = y[k];
         };
         if (n_tok == CT) {
-#pragma unroll 16
-            for (int tt = 0; tt < CT; tt++) token(tt);
+            constexpr int GR = NS > 8 ? 2 : (NS > 4 ? 4 : 8);
+            for (int g0 = 0; g0 < CT; g0 += GR) group(std::integral_constant<int, GR>{}, g0);
         } else {
-            for (int tt = 0; tt < n_tok; tt++) token(tt);
+            for (int tt = 0; tt < n_tok; tt++) group(std::integral_constant<int, 1>{}, tt);
         }
-        __syncthreads();
-#pragma unroll
-        for (int e = 0; e < EPT; e++) {
-            const int tt = et + e * (SS_THREADS / CB);
-            if (mine && tt < n_tok) {
-                const float* part = yp + tt * SS_THREADS + (threadIdx.x % CB) * LPC;
-                float y = 0.0f;
-#pragma unroll
-                for (int k = 0; k < LPC / 4; k++) {
-                    const float4 f = reinterpret_cast<const float4*>(part)[k];
-                    y += f.x; y += f.y; y += f.z; y += f.w;
-                }
-                y = fmaf(skip, gx[e], y);
-                ((TO*)p.out)[(size_t)(t0 + tt) * inner + ec] = from_float<TO>(y * silu_<TO>(gz[e]));
-            }
-        }
-        if (more) stage(cur ^ 1);
         __syncthreads();
     }
-    if (whole) write_row<NS>(S, st);
-    else {
 #pragma unroll
-        for (int i = 0; i < NS; i++)
-            if (c < inner && n0 + i < N) S[i] = st[i];
+    for (int i = 0; i < N2; i++) {
+        const int n = n0 + 2 * i;
+        const float2 v = up2(st[i]);
+        if (live && n < N) S[(size_t)n * inner] = v.x;
+        if (live && n + 1 < N) S[(size_t)(n + 1) * inner] = v.y;
     }
 }
 
-template <int LPC, int NS, int CT, typename TO>
+// One token a run: a thread takes a channel with all its states, ST of them in flight at a time.
+constexpr int SS_STEP_THREADS = 128;
+template <int ST, typename TO>
+__global__ void __launch_bounds__(SS_STEP_THREADS) selective_step_kernel(SelectiveArgs p) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int s = blockIdx.y, inner = p.inner, N = p.N, c = blockIdx.x * SS_STEP_THREADS + threadIdx.x;
+    if (c >= inner) return;
+    const int t = p.query_start[s];
+    float* S = p.state + (size_t)p.slots[s] * p.state_stride + c;
+    const float* A = p.a + c;
+    const float* bc = p.bc + (size_t)t * p.ld_bc;
+    const float x = p.x[(size_t)t * p.ld_x + c], d = p.dt[(size_t)t * p.ld_dt + c], z = p.z[(size_t)t * p.ld_z + c], skip = p.skip[c];
+    const float u = d * x;
+    float y0 = 0.0f, y1 = 0.0f;
+    for (int n0 = 0; n0 < N; n0 += ST) {
+        float st[ST], a[ST];
+#pragma unroll
+        for (int i = 0; i < ST; i++) {
+            const bool in = n0 + i < N;
+            st[i] = in ? S[(size_t)(n0 + i) * inner] : 0.0f;
+            a[i] = in ? A[(size_t)(n0 + i) * inner] : 0.0f;
+        }
+#pragma unroll
+        for (int i = 0; i < ST; i++) {
+            const bool in = n0 + i < N;
+            st[i] = fmaf(exp2_approx(d * a[i]), st[i], u * (in ? bc[n0 + i] : 0.0f));
+            float& y = i & 1 ? y1 : y0;
+            y = fmaf(st[i], in ? bc[N + n0 + i] : 0.0f, y);
+            if (in) S[(size_t)(n0 + i) * inner] = st[i];
+        }
+    }
+    ((TO*)p.out)[(size_t)t * inner + c] = from_float<TO>(fmaf(skip, x, y0 + y1) * silu_<TO>(z));
+}
+
+template <int NW, int NS, int CT, typename TO, int RING = SS_RING>
 int launch_selective(const SelectiveArgs& p, int S, cudaStream_t st) {
-    constexpr int CB = SS_THREADS / LPC, NP = LPC * NS;
-    const size_t smem = (size_t)(4 * CT * CB + 4 * CT * NP + CT * SS_THREADS) * sizeof(float);
+    const size_t smem = (size_t)(RING * 3 * CT * 32 + RING * 2 * CT * NW * NS + 2 * CT * NW * 32) * sizeof(float);
     if (smem > 48 * 1024) {
-        cudaError_t e = cudaFuncSetAttribute(selective_scan_kernel<LPC, NS, CT, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(selective_scan_kernel<NW, NS, CT, RING, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return fail("selective_scan: shared memory %zu: %s", smem, cudaGetErrorString(e));
     }
-    SelectiveArgs q = p;
-    constexpr int VW = NS % 4 == 0 ? 4 : 2;
-    q.vec = p.N % VW == 0 && p.state_stride % VW == 0 && ((((uintptr_t)p.state) | ((uintptr_t)p.a)) & 15) == 0;
-    launch_kernel(selective_scan_kernel<LPC, NS, CT, TO>, dim3((p.inner + CB - 1) / CB, S), SS_THREADS, smem, st, q);
+    launch_kernel(selective_scan_kernel<NW, NS, CT, RING, TO>, dim3((p.inner + 31) / 32, S), 64 * NW, smem, st, p);
     return check_launch("selective_scan");
 }
 
-// Lanes a channel and states a lane by the number of states.
-template <int CT, typename TO>
-int pick_selective(const SelectiveArgs& p, int S, cudaStream_t st) {
+// Computing warps a block and states a thread by the number of states.  Sixteen states: eight warps of two states while every
+// block has an SM for itself (2,048 tokens of 4,096 channels: 98 us against 115), four warps of four, with fewer reads of
+// shared memory a state, when blocks share SMs (four runs of 512 tokens: 80 us against 102; 8,192 channels: 150 against 187).
+template <typename TO>
+int pick_selective(const SelectiveArgs& p, int S, bool single, cudaStream_t st) {
     const int N = p.N;
-    if (N <= 8) return launch_selective<4, 2, CT, TO>(p, S, st);
-    if (N <= 16) return launch_selective<8, 2, CT, TO>(p, S, st);
-    if (N <= 32) return launch_selective<8, 4, CT, TO>(p, S, st);
-    if (N <= 64) return launch_selective<16, 4, CT, TO>(p, S, st);
-    if (N <= 128) return launch_selective<32, 4, CT, TO>(p, S, st);
-    return launch_selective<32, 8, CT, TO>(p, S, st);
+    if (single) {
+        const dim3 grid((p.inner + SS_STEP_THREADS - 1) / SS_STEP_THREADS, S);
+        if (N <= 8) launch_kernel(selective_step_kernel<8, TO>, grid, SS_STEP_THREADS, 0, st, p);
+        else launch_kernel(selective_step_kernel<16, TO>, grid, SS_STEP_THREADS, 0, st, p);
+        return check_launch("selective_step");
+    }
+    if (N <= 8) return launch_selective<4, 2, SS_CHUNK, TO>(p, S, st);
+    if (N <= 16 && (long long)S * ((p.inner + 31) / 32) <= 148) return launch_selective<8, 2, SS_CHUNK, TO>(p, S, st);
+    if (N <= 16) return launch_selective<4, 4, SS_CHUNK, TO>(p, S, st);
+    if (N <= 32) return launch_selective<8, 4, SS_CHUNK, TO>(p, S, st);
+    if (N <= 64) return launch_selective<8, 8, SS_CHUNK, TO>(p, S, st);
+    if (N <= 128) return launch_selective<8, 16, 16, TO, 4>(p, S, st);
+    return launch_selective<16, 16, 16, TO, 4>(p, S, st);
 }
 
 }  // namespace ember
@@ -243,9 +317,10 @@ EMBER_API int ember_selective_scan(const float* x, int ld_x, const float* dt, in
         return fail("selective_scan: rows of %d / %d / %d / %d, state rows of %lld do not hold %d channels of %d states", ld_x, ld_dt, ld_z, ld_bc, state_stride, inner, N);
     if (S > 65535) return fail("selective_scan: %d runs are too many for one launch", S);
     SelectiveArgs p{x, ld_x, dt, ld_dt, bc, ld_bc, z, ld_z, a, skip, state, state_stride, out, query_start, slots, inner, N, 0};
+    p.by16 = inner % 4 == 0 && ld_x % 4 == 0 && ld_dt % 4 == 0 && ld_z % 4 == 0 && ((((uintptr_t)x) | ((uintptr_t)dt) | ((uintptr_t)z)) & 15) == 0;
     cudaStream_t st = (cudaStream_t)stream;
     const bool single = T == S;
-    if (out_dtype == EMBER_F32) return single ? pick_selective<1, float>(p, S, st) : pick_selective<16, float>(p, S, st);
-    if (out_dtype == EMBER_BF16) return single ? pick_selective<1, __nv_bfloat16>(p, S, st) : pick_selective<16, __nv_bfloat16>(p, S, st);
+    if (out_dtype == EMBER_F32) return pick_selective<float>(p, S, single, st);
+    if (out_dtype == EMBER_BF16) return pick_selective<__nv_bfloat16>(p, S, single, st);
     return fail("selective_scan: unsupported output dtype %d", out_dtype);
 }

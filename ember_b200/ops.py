@@ -21,7 +21,8 @@ EPI_RELU_MUL = 6  # the gated epilogue with relu: relu(c[2j]) * c[2j + 1]
 EPI_GELU_MUL = 7  # ... with the tanh form of gelu: 0.5 g (1 + tanh(sqrt(2 / pi) (g + 0.044715 g^3))) * c[2j + 1]
 EPI_GELU = 8      # gelu(c + bias) in its exact form, 0.5 z (1 + erf(z / sqrt 2)), stored like EPI_STORE
 EPI_SQUARE_RELU = 9      # max(c + bias, 0)^2, stored like EPI_STORE
-PLAIN_EPILOGUES = (EPI_STORE, EPI_STORE_F32, EPI_ADD_F32, EPI_GELU, EPI_SQUARE_RELU)      # those that take a bias in both products
+EPI_SOFTPLUS_F32 = 10    # log(1 + e^(c + bias)), stored in fp32
+PLAIN_EPILOGUES = (EPI_STORE, EPI_STORE_F32, EPI_ADD_F32, EPI_GELU, EPI_SQUARE_RELU, EPI_SOFTPLUS_F32)      # those that take a bias in both products
 GATED_EPILOGUES = (EPI_SILU_MUL, EPI_RELU_MUL, EPI_GELU_MUL)
 GATED_EPILOGUE_OF = {"silu": EPI_SILU_MUL, "relu": EPI_RELU_MUL, "gelu_tanh": EPI_GELU_MUL}
 
@@ -136,6 +137,18 @@ def embed_bigram(tokens: torch.Tensor, table: torch.Tensor, bigram: torch.Tensor
           _p(table), _p(bigram), c_int(dtype_code(table.dtype)), c_int(dtype_code(bigram.dtype)), _p(out), c_int(T), c_int(H), c_int(V), c_float(scale),
           c_longlong(buckets), c_longlong(mul_prev), c_longlong(mul_cur), _p(positions), _p(seq_of), _p(query_start), _p(slots),
           _p(state), c_int(state.stride(0)), _p(err), c_void_p(stream if stream is not None else current_stream_ptr()))
+
+
+def round_columns(x: torch.Tensor, col: int, n: int, out: torch.Tensor, T: int, stream: Optional[int] = None) -> None:
+    """out[t, :n] = x[t, col : col + n] in out's type (x fp32 [T, ld], out [T, n]): columns of one product made the operand of
+    another."""
+    _check(x, "x", torch.float32)
+    _check(out, "out")
+    if x.dim() != 2 or x.shape[0] < T or col < 0 or col + n > x.shape[1] or out.shape[-1] != n or out.numel() < T * n:
+        raise KernelError(f"round_columns: {n} columns from {col} of {tuple(x.shape)} into {tuple(out.shape)}")
+    lib = _lib("elementwise")
+    _call(lib, lib.ember_round_columns, _off(x, col), c_int(x.shape[1]), _p(out), c_int(dtype_code(out.dtype)), c_int(T), c_int(n),
+          _stream(stream))
 
 
 def place_columns(x: torch.Tensor, out: torch.Tensor, T: int, col: int, col2: int = -1, stream: Optional[int] = None) -> None:
@@ -1022,13 +1035,13 @@ def selective_scan(x: torch.Tensor, dt: torch.Tensor, bc: torch.Tensor, bc_col: 
     """Selective scan with a diagonal state per channel over the step's runs (csrc/selective_scan.cu).  ``x`` fp32 [T, inner]
     (after convolution and silu), ``dt`` fp32 [T, inner] the steps, ``bc`` fp32
     with B and C behind one another from column ``bc_col`` on, ``z`` fp32 with the gate from column ``z_col`` on, ``a`` fp32
-    [inner, states] = -exp(A_log) log2(e), ``skip`` [inner]; a request's state is the first inner * states floats of its row
-    of ``state``.  out [T, inner] (fp32 or bfloat16) = (S C + skip x) silu(z)."""
+    [states, inner] = -exp(A_log) log2(e), ``skip`` [inner]; a request's state, [states, inner], is the first inner * states
+    floats of its row of ``state``.  out [T, inner] (fp32 or bfloat16) = (S C + skip x) silu(z)."""
     for t, n in ((x, "x"), (dt, "dt"), (bc, "bc"), (z, "z"), (a, "a"), (skip, "skip"), (state, "state")):
         _check(t, n, torch.float32)
     _check(out, "out")
     _check_runs(query_start, slots, S)
-    inner, N = a.shape
+    N, inner = a.shape
     if x.shape[-1] != inner or dt.shape[-1] != inner or z.shape[-1] < z_col + inner or bc.shape[-1] < bc_col + 2 * N or \
             min(x.shape[0], dt.shape[0], z.shape[0], bc.shape[0]) < T or skip.numel() != inner or \
             out.shape[-1] != inner or out.numel() < T * inner or state.dim() != 2 or state.shape[1] < inner * N:
