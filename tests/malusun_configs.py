@@ -43,7 +43,7 @@ MALUSUN = {
     # widths the tensor-core kernels take; the first layer that blends values is the second one, a layer in between keeps its
     # own; windows of 33 and 50 on pages of 16; a scan of sixteen states; 64-wide heads in the last layers (in bfloat16 they
     # run on the kernels Qwen3's attention uses)
-    "a": dict(seed=3, json={
+    "a": dict(seed=20, json={
         "architecture": "Malusun", "vocab": 320, "width": 128, "norm": {"eps": 1e-6}, "embedding": {"scale": 8.0},
         "layers": [
             _layer("mamba1", _mamba(256, 16, 8, 4), _moe(48, 6, 2, 64)),

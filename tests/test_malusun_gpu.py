@@ -525,7 +525,7 @@ ROUTED_CASES = [
     (64, 40, 6, 2, 32), (100, 30, 3, 3, 50), (96, 24, 5, 1, 0), (128, 256, 48, 4, 128), (64, 50, 8, 1, 64), (64, 16, 1, 1, 8), (72, 20, 64, 6, 0)]
 
 
-def _routed(hidden, ff, experts, top, shared, seed, spread=4.0):
+def _routed(hidden, ff, experts, top, shared, seed, spread=1.0):
     from ember_b200.config import RoutedMLPSpec
     spec = RoutedMLPSpec(hidden_size=hidden, intermediate_size=ff, experts=experts, top=top, limit=0.0, alpha=1.0, up_offset=0.0,
                          scoring="sigmoid", weigh="input", shared_size=shared)
@@ -554,7 +554,7 @@ def test_routed_feed_forward_alone(dtype, hidden, ff, experts, top, shared):
         chosen, weights = plain.route(x.double(), W, "f.", top)
         at_output = sum(weights[:, i:i + 1] * torch.cat([plain.expert(x[t:t + 1].double(), W, f"f.e{int(chosen[t, i])}.") for t in range(90)])
                         for i in range(top))
-        assert _rel(at_output, want - (plain.expert(x.double(), W, "f.shared.") if shared else 0)) > 0.05
+        assert _rel(at_output, want - (plain.expert(x.double(), W, "f.shared.") if shared else 0)) > 0.03
     got, _, _ = _run_feed_forward(spec, w, x, dtype)
     errs = sorted(_rel(got[t], want[t]) for t in range(90))
     # a token whose choice is a close call may fall the other way in bfloat16 (the router reads the rounded input)
