@@ -11,7 +11,6 @@
 //   2 add into an fp32 matrix (residual) 3 silu(c[2j]) * c[2j+1] over interleaved gate/up rows
 //   6 relu(c[2j]) * c[2j+1] likewise     7 gelu(c[2j]) * c[2j+1], gelu in its tanh form
 //   8 gelu(c) in its exact form (erf), stored in the activation dtype     9 max(c, 0)^2 likewise
-//   10 softplus(c), stored in fp32
 // An optional fp32 bias[N] is added before the epilogue.
 #include "common.cuh"
 
@@ -76,8 +75,7 @@ gemm_simt_kernel(const TA* __restrict__ A, int lda, const TW* __restrict__ W, in
                 if (EPI == 8) c = 0.5f * c * (1.0f + erff(c * 0.7071067811865476f));
                 if (EPI == 9) { c = fmaxf(c, 0.0f); c *= c; }
                 ((TA*)Cv)[(size_t)m * ldc + n] = from_float<TA>(c);
-            } else if (EPI == 1 || EPI == 10) {
-                if (EPI == 10) c = c > 20.0f ? c : log1pf(expf(c));
+            } else if (EPI == 1) {
                 ((float*)Cv)[(size_t)m * ldc + n] = c;
             } else if (EPI == 2) {
                 float* p = (float*)Cv + (size_t)m * ldc + n;
@@ -109,7 +107,6 @@ int launch(const void* A, int lda, const void* W, int ldw, const float* bias, vo
         case 7: launch_kernel(gemm_simt_kernel<TA, TW, 7>, grid, 256, 0, st, a, lda, w, ldw, bias, C, ldc, M, N, K); break;
         case 8: launch_kernel(gemm_simt_kernel<TA, TW, 8>, grid, 256, 0, st, a, lda, w, ldw, bias, C, ldc, M, N, K); break;
         case 9: launch_kernel(gemm_simt_kernel<TA, TW, 9>, grid, 256, 0, st, a, lda, w, ldw, bias, C, ldc, M, N, K); break;
-        case 10: launch_kernel(gemm_simt_kernel<TA, TW, 10>, grid, 256, 0, st, a, lda, w, ldw, bias, C, ldc, M, N, K); break;
         default: return fail("gemm: unknown epilogue %d", epi);
     }
     return check_launch("gemm_simt");

@@ -296,17 +296,15 @@ EMBER_API long long ember_gemm_tc_scratch_floats(int max_tokens_swapped, int N) 
 
 // C = A . W^T with the fused epilogue.  `scratch` is a zero-filled fp32 buffer of at least
 // min(M, 128) * N floats (used only when the K range is split; it is left zeroed).
-// Epilogue 8 stores gelu(sum + bias) in bf16 (the exact form, by erf), epilogue 9 max(sum + bias, 0)^2, epilogue 10
-// softplus(sum + bias) in fp32.  `bias` (fp32 [N] or null) joins the sums of
+// Epilogue 8 stores gelu(sum + bias) in bf16 (the exact form, by erf), epilogue 9 max(sum + bias, 0)^2.  `bias` (fp32 [N] or null) joins the sums of
 // epilogues 0, 1, 2 and 8.  Epilogue 5 (at most 128 tokens): the fp32 sums are left in `scratch` as [M, N] for a consumer that reads them and
 // sets them back to zero (`out` is not used); it saves the pass that rounds, stores and clears.
 EMBER_API int ember_gemm_tc(const void* A, const void* W, void* out, int ldc, int M, int N, int K, int epilogue, const float* bias,
                             float* scratch, long long scratch_floats, int num_sms, int split_mode, int* err, void* stream) {
     if (M <= 0 || N <= 0) return 0;
-    const int act = epilogue == 6 ? 1 : (epilogue == 7 ? 2 : (epilogue == 8 ? 3 : (epilogue == 9 ? 4 : (epilogue == 10 ? 5 : 0))));      // epilogues 6, 7: the gated epilogue with relu, with gelu (tanh form)
+    const int act = epilogue == 6 ? 1 : (epilogue == 7 ? 2 : (epilogue == 8 ? 3 : (epilogue == 9 ? 4 : 0)));      // epilogues 6, 7: the gated epilogue with relu, with gelu (tanh form)
     if (epilogue == 6 || epilogue == 7) epilogue = 3;
     if (epilogue == 8 || epilogue == 9) epilogue = 0;
-    if (epilogue == 10) epilogue = 1;
     if (bias && (epilogue == 3 || epilogue == 5)) return fail("gemm_tc: the gated epilogue and sums left in scratch take no bias");
     const bool sums = epilogue == 5;
     if (sums) {
@@ -486,7 +484,7 @@ EMBER_API int ember_gemm_tc(const void* A, const void* W, void* out, int ldc, in
         if (by4) {
             const unsigned blocks = (unsigned)((total / 4 + 255) / 256);
             if (epilogue == 3) launch_kernel(gemm_tc_finalize4_kernel<3>, blocks, 256, 0, st, p.accum, p.accum_ld, out, ldc, M, n_out, act, (const float*)nullptr);
-            else if (epilogue == 1) launch_kernel(gemm_tc_finalize4_kernel<1>, blocks, 256, 0, st, p.accum, p.accum_ld, out, ldc, M, n_out, act, bias);
+            else if (epilogue == 1) launch_kernel(gemm_tc_finalize4_kernel<1>, blocks, 256, 0, st, p.accum, p.accum_ld, out, ldc, M, n_out, 0, bias);
             else launch_kernel(gemm_tc_finalize4_kernel<0>, blocks, 256, 0, st, p.accum, p.accum_ld, out, ldc, M, n_out, act, bias);
         } else {
             launch_kernel(gemm_tc_finalize_kernel, (unsigned)((total + 255) / 256), 256, 0, st, p.accum, p.accum_ld, out, ldc, M, N, epilogue, act, bias);

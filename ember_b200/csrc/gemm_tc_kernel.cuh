@@ -46,7 +46,7 @@ struct GemmTcParams {
     int num_k_blocks;     // ceil(K / TILE_K)
     int k_blocks_per_split;
     int epilogue;         // 0 store bf16, 1 store fp32, 2 add fp32, 3 act(gate)*up -> bf16
-    int act;              // epilogue 3: 0 silu, 1 relu, 2 gelu (tanh form); epilogues 0, 1: 0 none, 3 gelu (exact, by erf), 4 max(x, 0)^2, 5 softplus
+    int act;              // epilogue 3: 0 silu, 1 relu, 2 gelu (tanh form); epilogue 0: 0 none, 3 gelu (exact, by erf), 4 max(x, 0)^2
     const float* bias;    // [N] added to the sums of epilogues 0, 1 and 2 (once, whatever the parts of K), or null
     void* out;
     int ldc;
@@ -151,16 +151,9 @@ __device__ __forceinline__ float gate_mul(float g, float u, int act) {
 }
 
 __device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f)); }
-// softplus(z) = log(1 + e^z): the logarithm's series where e^z is small (the fast logarithm has no relative precision near 1).
-__device__ __forceinline__ float softplus_fast(float z) {
-    const float e = __expf(z);
-    const float series = e * fmaf(e, fmaf(e, fmaf(e, fmaf(e, 0.2f, -0.25f), 1.0f / 3.0f), -0.5f), 1.0f);
-    return z > 20.0f ? z : (e < 0.0625f ? series : __logf(1.0f + e));
-}
-// The activations of the plain epilogue: 3 gelu (exact), 4 relu squared, 5 softplus, others none.
+// The activations of the plain epilogue: 3 gelu (exact), 4 relu squared, others none.
 __device__ __forceinline__ float plain_activation(float z, int act) {
     if (act == 4) { z = fmaxf(z, 0.0f); return z * z; }
-    if (act == 5) return softplus_fast(z);
     return act == 3 ? gelu_erf(z) : z;
 }
 // A complete sum of output column n as the plain epilogues (0, 1, 2) want it: with its bias, through its activation.

@@ -1,5 +1,5 @@
-// Selective scan with a diagonal state per channel (Mamba) over a ragged batch.  Per channel c and state n, with a step dt
-// per token and channel and one B and one C row per token:
+// Selective scan with a diagonal state per channel (Mamba) over a ragged batch.  Per channel c and state n, with
+// dt = softplus(raw step + bias) per token and channel and one B and one C row per token:
 //
 //     S[c, n] <- exp(-dt_c exp(A_log[c, n])) S[c, n] + dt_c x_c B_n;   y_c = sum_n S[c, n] C_n + D_c x_c
 //
@@ -35,10 +35,10 @@ constexpr int SS_RING = 5;            // chunks of inputs in shared memory: one 
 
 struct SelectiveArgs {
     const float* x; int ld_x;                  // [T, inner] after convolution and silu
-    const float* dt; int ld_dt;                // [T, inner] steps
+    const float* dt; int ld_dt;                // [T, inner] raw steps
     const float* bc; int ld_bc;                // [T, B (N) | C (N)]
     const float* z; int ld_z;                  // [T, inner] gate
-    const float* a; const float* skip;         // [N, inner], [inner]
+    const float* dt_bias; const float* a; const float* skip;      // [inner], [N, inner], [inner]
     float* state; long long state_stride;      // [slot][N][inner]
     void* out;                                 // [T, inner]
     const int* query_start; const int* slots;
@@ -67,6 +67,18 @@ __device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
     f32x2 d;
     asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
     return d;
+}
+// softplus(z) = log(1 + e^z).  The bfloat16 form takes the logarithm's series where e^z is small (the fast logarithm has no
+// relative precision near 1): an error of a few 1e-6.
+template <typename TO>
+__device__ __forceinline__ float softplus_(float z);
+template <>
+__device__ __forceinline__ float softplus_<float>(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
+template <>
+__device__ __forceinline__ float softplus_<__nv_bfloat16>(float z) {
+    const float e = __expf(z);
+    const float series = e * fmaf(e, fmaf(e, fmaf(e, fmaf(e, 0.2f, -0.25f), 1.0f / 3.0f), -0.5f), 1.0f);
+    return z > 20.0f ? z : (e < 0.0625f ? series : __logf(1.0f + e));
 }
 // z sigmoid(z); the bfloat16 form with the fast exponential and division.
 template <typename TO>
@@ -136,6 +148,16 @@ __global__ void __launch_bounds__(64 * NW) selective_scan_kernel(SelectiveArgs p
             }
             asm volatile("cp.async.commit_group;" ::: "memory");
         };
+        const float dt_bias = live ? p.dt_bias[c] : 0.0f;
+        auto arrived = [&](int i) {            // chunk i is there: raw steps become steps
+            asm volatile("cp.async.wait_group %0;" ::"n"(RING - 3) : "memory");
+            asm volatile("bar.sync 1, %0;" ::"n"(THREADS) : "memory");      // (pieces that other feeding threads copied)
+            if (i < chunks) {
+                float* xd = xs + (i % RING) * 3 * TILE + TILE + lane;
+#pragma unroll
+                for (int tt = warp; tt < CT; tt += NW) xd[tt * 32] = softplus_<TO>(xd[tt * 32] + dt_bias);
+            }
+        };
         auto finish = [&](int i) {             // chunk i: its partials, gate, store
             const int t0 = first + i * CT, n_tok = min(CT, end - t0);
             const float* xd = xs + (i % RING) * 3 * TILE + lane;
@@ -153,12 +175,12 @@ __global__ void __launch_bounds__(64 * NW) selective_scan_kernel(SelectiveArgs p
             }
         };
         for (int i = 0; i < RING - 2; i++) issue(i);
-        asm volatile("cp.async.wait_group %0;" ::"n"(RING - 3) : "memory");          // chunk 0 is there
+        arrived(0);
         __syncthreads();
         for (int i = 0; i < chunks; i++) {
             issue(i + RING - 2);               // (into the place of chunk i - 2, which has been finished)
             if (i > 0) finish(i - 1);
-            asm volatile("cp.async.wait_group %0;" ::"n"(RING - 3) : "memory");      // chunk i + 1 is there
+            arrived(i + 1);
             __syncthreads();
         }
         finish(chunks - 1);
@@ -245,7 +267,7 @@ __global__ void __launch_bounds__(SS_STEP_THREADS) selective_step_kernel(Selecti
     float* S = p.state + (size_t)p.slots[s] * p.state_stride + c;
     const float* A = p.a + c;
     const float* bc = p.bc + (size_t)t * p.ld_bc;
-    const float x = p.x[(size_t)t * p.ld_x + c], d = p.dt[(size_t)t * p.ld_dt + c], z = p.z[(size_t)t * p.ld_z + c], skip = p.skip[c];
+    const float x = p.x[(size_t)t * p.ld_x + c], d = softplus_<TO>(p.dt[(size_t)t * p.ld_dt + c] + p.dt_bias[c]), z = p.z[(size_t)t * p.ld_z + c], skip = p.skip[c];
     const float u = d * x;
     float y0 = 0.0f, y1 = 0.0f;
     for (int n0 = 0; n0 < N; n0 += ST) {
@@ -308,7 +330,7 @@ EMBER_API int ember_selective_scan_max_states() { return 256; }
 
 // T == S (every run is one token): the form with chunks of one token.
 EMBER_API int ember_selective_scan(const float* x, int ld_x, const float* dt, int ld_dt, const float* bc, int ld_bc, const float* z, int ld_z,
-                                   const float* a, const float* skip, float* state, long long state_stride,
+                                   const float* dt_bias, const float* a, const float* skip, float* state, long long state_stride,
                                    void* out, int out_dtype, const int* query_start, const int* slots, int T, int S, int inner, int N,
                                    void* stream) {
     if (T <= 0 || S <= 0) return 0;
@@ -316,7 +338,7 @@ EMBER_API int ember_selective_scan(const float* x, int ld_x, const float* dt, in
     if (ld_x < inner || ld_dt < inner || ld_z < inner || ld_bc < 2 * N || state_stride < (long long)inner * N)
         return fail("selective_scan: rows of %d / %d / %d / %d, state rows of %lld do not hold %d channels of %d states", ld_x, ld_dt, ld_z, ld_bc, state_stride, inner, N);
     if (S > 65535) return fail("selective_scan: %d runs are too many for one launch", S);
-    SelectiveArgs p{x, ld_x, dt, ld_dt, bc, ld_bc, z, ld_z, a, skip, state, state_stride, out, query_start, slots, inner, N, 0};
+    SelectiveArgs p{x, ld_x, dt, ld_dt, bc, ld_bc, z, ld_z, dt_bias, a, skip, state, state_stride, out, query_start, slots, inner, N, 0};
     p.by16 = inner % 4 == 0 && ld_x % 4 == 0 && ld_dt % 4 == 0 && ld_z % 4 == 0 && ((((uintptr_t)x) | ((uintptr_t)dt) | ((uintptr_t)z)) & 15) == 0;
     cudaStream_t st = (cudaStream_t)stream;
     const bool single = T == S;

@@ -6,7 +6,7 @@
 //     rotated shared key part behind it into the token's single cache row [c | k_rot];
 //   * rotate_pairs:      rotation of neighbouring pairs (2i, 2i + 1) of a slice of every head, fp32 in, cache type out;
 //   * head_gemm:         out[t, h, :] = W[h] x[t, h, :] for every head (a product per head, weights [H, N, K]), with an
-//     optional bias, softplus and sigmoid gate on the result: folds a head's key up-projection into its query and takes a head's value
+//     optional sigmoid gate on the result: folds a head's key up-projection into its query and takes a head's value
 //     up-projection of the attended latent; fp32 multiply-adds in general, mma.sync tiles for bfloat16 weights;
 //   * sink_attention:    o = sum_j w_j v_j with w = softmax over the visible keys and one more term exp(sink[h]) in the
 //     denominator that has no key and no value; visible: j <= i and (no window, or i - j < window, or j < keep_first).
@@ -384,12 +384,9 @@ struct HeadGemmArgs {
     void* out; int ld_o, o_head, o_col;
     const float* gate; int ld_g, g_col;  // gate[t, g_col + h N + n] or null
     int T, H, N, K;
-    const float* bias; int softplus;     // bias [H N] or null joins the sum; then softplus of it (before a gate)
 };
 
 __device__ __forceinline__ float head_gemm_finish(const HeadGemmArgs& p, int t, int h, int n, float v) {
-    if (p.bias) v += p.bias[(size_t)h * p.N + n];
-    if (p.softplus) v = v > 20.0f ? v : log1pf(expf(v));
     if (p.gate) v *= sigmoidf_(p.gate[(size_t)t * p.ld_g + p.g_col + (size_t)h * p.N + n]);
     return v;
 }
@@ -1255,10 +1252,10 @@ EMBER_API int ember_rotate_pairs(const float* in, int ld_in, int in_head, int in
 
 EMBER_API int ember_head_gemm(const float* x, int ld_x, int x_head, int x_col, const void* w, int w_dtype, void* out, int out_dtype,
                               int ld_o, int o_head, int o_col, const float* gate, int ld_g, int g_col, int T, int H, int N, int K,
-                              const float* bias, int softplus, void* stream) {
+                              void* stream) {
     if (T <= 0) return 0;
     if (H <= 0 || N <= 0 || K <= 0 || H > 65535) return fail("head_gemm: %d heads of %d x %d", H, N, K);
-    HeadGemmArgs p{x, ld_x, x_head, x_col, w, out, ld_o, o_head, o_col, gate, ld_g, g_col, T, H, N, K, bias, softplus};
+    HeadGemmArgs p{x, ld_x, x_head, x_col, w, out, ld_o, o_head, o_col, gate, ld_g, g_col, T, H, N, K};
     cudaStream_t st = (cudaStream_t)stream;
     // bfloat16 weights with rows of whole 16-byte pieces (and x rows of whole float4s): the tensor-core form
     if (w_dtype == EMBER_BF16 && K % 8 == 0 && ld_x % 4 == 0 && x_head % 4 == 0 && x_col % 4 == 0 && (((uintptr_t)x) & 15) == 0 && (((uintptr_t)w) & 15) == 0 && (((uintptr_t)out) & 7) == 0 &&

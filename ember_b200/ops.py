@@ -21,8 +21,7 @@ EPI_RELU_MUL = 6  # the gated epilogue with relu: relu(c[2j]) * c[2j + 1]
 EPI_GELU_MUL = 7  # ... with the tanh form of gelu: 0.5 g (1 + tanh(sqrt(2 / pi) (g + 0.044715 g^3))) * c[2j + 1]
 EPI_GELU = 8      # gelu(c + bias) in its exact form, 0.5 z (1 + erf(z / sqrt 2)), stored like EPI_STORE
 EPI_SQUARE_RELU = 9      # max(c + bias, 0)^2, stored like EPI_STORE
-EPI_SOFTPLUS_F32 = 10    # log(1 + e^(c + bias)), stored in fp32
-PLAIN_EPILOGUES = (EPI_STORE, EPI_STORE_F32, EPI_ADD_F32, EPI_GELU, EPI_SQUARE_RELU, EPI_SOFTPLUS_F32)      # those that take a bias in both products
+PLAIN_EPILOGUES = (EPI_STORE, EPI_STORE_F32, EPI_ADD_F32, EPI_GELU, EPI_SQUARE_RELU)      # those that take a bias in both products
 GATED_EPILOGUES = (EPI_SILU_MUL, EPI_RELU_MUL, EPI_GELU_MUL)
 GATED_EPILOGUE_OF = {"silu": EPI_SILU_MUL, "relu": EPI_RELU_MUL, "gelu_tanh": EPI_GELU_MUL}
 
@@ -1030,25 +1029,25 @@ SELECTIVE_MAX_STATES = 256       # states a channel the selective scan takes
 
 
 def selective_scan(x: torch.Tensor, dt: torch.Tensor, bc: torch.Tensor, bc_col: int, z: torch.Tensor, z_col: int,
-                   a: torch.Tensor, skip: torch.Tensor, state: torch.Tensor, out: torch.Tensor, query_start: torch.Tensor,
+                   dt_bias: torch.Tensor, a: torch.Tensor, skip: torch.Tensor, state: torch.Tensor, out: torch.Tensor, query_start: torch.Tensor,
                    slots: torch.Tensor, T: int, S: int, stream: Optional[int] = None) -> None:
     """Selective scan with a diagonal state per channel over the step's runs (csrc/selective_scan.cu).  ``x`` fp32 [T, inner]
-    (after convolution and silu), ``dt`` fp32 [T, inner] the steps, ``bc`` fp32
+    (after convolution and silu), ``dt`` fp32 [T, inner] raw steps (softplus of them plus ``dt_bias`` is taken here), ``bc`` fp32
     with B and C behind one another from column ``bc_col`` on, ``z`` fp32 with the gate from column ``z_col`` on, ``a`` fp32
     [states, inner] = -exp(A_log) log2(e), ``skip`` [inner]; a request's state, [states, inner], is the first inner * states
     floats of its row of ``state``.  out [T, inner] (fp32 or bfloat16) = (S C + skip x) silu(z)."""
-    for t, n in ((x, "x"), (dt, "dt"), (bc, "bc"), (z, "z"), (a, "a"), (skip, "skip"), (state, "state")):
+    for t, n in ((x, "x"), (dt, "dt"), (bc, "bc"), (z, "z"), (dt_bias, "dt_bias"), (a, "a"), (skip, "skip"), (state, "state")):
         _check(t, n, torch.float32)
     _check(out, "out")
     _check_runs(query_start, slots, S)
     N, inner = a.shape
     if x.shape[-1] != inner or dt.shape[-1] != inner or z.shape[-1] < z_col + inner or bc.shape[-1] < bc_col + 2 * N or \
-            min(x.shape[0], dt.shape[0], z.shape[0], bc.shape[0]) < T or skip.numel() != inner or \
+            min(x.shape[0], dt.shape[0], z.shape[0], bc.shape[0]) < T or dt_bias.numel() != inner or skip.numel() != inner or \
             out.shape[-1] != inner or out.numel() < T * inner or state.dim() != 2 or state.shape[1] < inner * N:
         raise KernelError(f"selective_scan: buffers do not fit {inner} channels of {N} states")
     lib = _lib("selective_scan")
     _call(lib, lib.ember_selective_scan, _p(x), c_int(x.shape[-1]), _p(dt), c_int(dt.shape[-1]), _off(bc, bc_col), c_int(bc.shape[-1]),
-          _off(z, z_col), c_int(z.shape[-1]), _p(a), _p(skip), _p(state), c_longlong(state.shape[1]), _p(out),
+          _off(z, z_col), c_int(z.shape[-1]), _p(dt_bias), _p(a), _p(skip), _p(state), c_longlong(state.shape[1]), _p(out),
           c_int(dtype_code(out.dtype)), _p(query_start), _p(slots), c_int(T), c_int(S), c_int(inner), c_int(N), _stream(stream))
 
 
@@ -1371,15 +1370,9 @@ def rotate_pairs(x: torch.Tensor, x_head: int, x_col: int, out: torch.Tensor, ou
 
 
 def head_gemm(x: torch.Tensor, x_head: int, x_col: int, w: torch.Tensor, out: torch.Tensor, out_head: int, out_col: int, T: int,
-              gate: Optional[torch.Tensor] = None, gate_col: int = 0, stream: Optional[int] = None, bias: Optional[torch.Tensor] = None,
-              softplus: bool = False) -> None:
+              gate: Optional[torch.Tensor] = None, gate_col: int = 0, stream: Optional[int] = None) -> None:
     """out[t, h, out_col + n] = sum_k x[t, h, x_col + k] * w[h, n, k], a product per head (``w`` [heads, N, K]); with
-    ``gate`` (fp32 rows) the result is multiplied by sigmoid(gate[t, gate_col + h N + n]).  x fp32 2-D.  ``bias`` (fp32
-    [heads N]) joins the sum, and ``softplus`` is taken of it, before the gate."""
-    if bias is not None:
-        _check(bias, "bias", torch.float32)
-        if bias.numel() != w.shape[0] * w.shape[1]:
-            raise KernelError(f"head_gemm: a bias of {bias.numel()} for {tuple(w.shape)}")
+    ``gate`` (fp32 rows) the result is multiplied by sigmoid(gate[t, gate_col + h N + n]).  x fp32 2-D."""
     _check(x, "x", torch.float32)
     _check(w, "w")
     _check(out, "out")
@@ -1393,8 +1386,7 @@ def head_gemm(x: torch.Tensor, x_head: int, x_col: int, w: torch.Tensor, out: to
     lib = _lib("sink_attention")
     _call(lib, lib.ember_head_gemm, _p(x), c_int(x.shape[1]), c_int(x_head), c_int(x_col), _p(w), c_int(dtype_code(w.dtype)), _p(out),
           c_int(dtype_code(out.dtype)), c_int(out.shape[1]), c_int(out_head), c_int(out_col), _p(gate),
-          c_int(gate.shape[1] if gate is not None else 0), c_int(gate_col), c_int(T), c_int(H), c_int(N), c_int(K), _p(bias),
-          c_int(1 if softplus else 0), _stream(stream))
+          c_int(gate.shape[1] if gate is not None else 0), c_int(gate_col), c_int(T), c_int(H), c_int(N), c_int(K), _stream(stream))
 
 
 def sink_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: Optional[torch.Tensor], out: torch.Tensor, T: int, heads: int,

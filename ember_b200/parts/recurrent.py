@@ -432,8 +432,8 @@ class SelectiveScan(_StateMixer):
         S[c, n] <- exp(-dt_c exp(A_log[c, n])) S[c, n] + dt_c x_c B_n;  y_c = sum_n S[c, n] C_n + D_c x_c
 
     then y * silu(z) and the output product.  The products read bfloat16 operands on the bfloat16 path and leave fp32; steps,
-    decays, B, C and the state are fp32.  The step's projection adds its bias and takes the softplus where it stores (on the
-    tensor cores over a rounded copy of ``low``, else it reads ``low`` where the product before it left it).  The
+    decays, B, C and the state are fp32.  The step's projection goes over a rounded copy of ``low`` on the tensor cores, else
+    it reads ``low`` where the product before it left it; its bias and softplus are the scan's.  The
     state row of a request holds S [states, inner] and, behind it, the convolution's last inputs.  Tensors under the
     prefix: in, conv, conv.b, x, dt, dt.b, A_log, D, o."""
 
@@ -466,7 +466,7 @@ class SelectiveScan(_StateMixer):
         if w is None:
             return
         self.in_proj, self.x_proj, self.o = (Linear.from_host(w[p + n], rt) for n in ("in", "x", "o"))
-        self.dt_proj = Linear.from_host(w[p + "dt"], rt, w[p + "dt.b"])
+        self.dt_proj = Linear.from_host(w[p + "dt"], rt)
         # (off the tensor cores the step's product is the per-head one with a single head: it reads fp32 columns)
         self.dt_w = rt.to_device(w[p + "dt"], rt.dtype).view(1, s.inner, s.dt_rank)
         self.taps, self.conv_bias, self.dt_bias, self.skip = (rt.to_device(w[p + n], torch.float32) for n in ("conv", "conv.b", "dt.b", "D"))
@@ -487,13 +487,13 @@ class SelectiveScan(_StateMixer):
         ops.conv_silu(proj, 0, self.taps, self.conv_bias, cache.state, inner * N, ctx.seq_of, ctx.query_start, ctx.state_slots,
                       conv, T, ctx.S, stream=ctx.stream, rounded=conv_r if half else None)
         self.x_proj(ctx, conv_r, low, T, ops.EPI_STORE_F32)
-        if half and ops.gemm_tc_usable(y, self.dt_proj.weight, self.dt_proj.bias, ops.EPI_SOFTPLUS_F32):
+        if half and ops.gemm_tc_usable(y, self.dt_proj.weight, None, ops.EPI_STORE_F32):
             low_r = ctx.buf("mamba1.low_rounded", (mt, R), rt.dtype)
             ops.round_columns(low, 0, R, low_r, T, stream=ctx.stream)
-            self.dt_proj(ctx, low_r, dt, T, ops.EPI_SOFTPLUS_F32)
+            self.dt_proj(ctx, low_r, dt, T, ops.EPI_STORE_F32)
         else:
-            ops.head_gemm(low, R, 0, self.dt_w, dt, inner, 0, T, stream=ctx.stream, bias=self.dt_bias, softplus=True)
-        ops.selective_scan(conv, dt, low, R, proj, inner, self.a, self.skip, cache.state, y, ctx.query_start,
+            ops.head_gemm(low, R, 0, self.dt_w, dt, inner, 0, T, stream=ctx.stream)
+        ops.selective_scan(conv, dt, low, R, proj, inner, self.dt_bias, self.a, self.skip, cache.state, y, ctx.query_start,
                            ctx.state_slots, T, ctx.S, stream=ctx.stream)
         self._out(ctx, y, out, accumulate)
 

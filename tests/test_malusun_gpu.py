@@ -1,9 +1,9 @@
 """Malusun on the device against the plain implementation: each mechanism alone (fed in portions beside another request), the
 scan's state and the convolution's inputs carried from step to step, keys just inside and just outside a window in prompts
 and in decoding, a far key that dominates, distance slopes and the fixed sink in every attention kernel, values blended with
-an earlier layer's, experts weighed at their input beside a shared expert, relu squared and softplus in every path of the
-products, the norms around a sublayer in one kernel, whole models under every way of cutting the work, slots and pages used
-again, long decoding through captured graphs, and greedy generation through the entry point and its scheduler."""
+an earlier layer's, experts weighed at their input beside a shared expert, relu squared in every path of the products, the
+norms around a sublayer in one kernel, whole models under every way of cutting the work, slots and pages used again, long
+decoding through captured graphs, and greedy generation through the entry point and its scheduler."""
 import numpy as np
 import pytest
 import torch
@@ -496,28 +496,19 @@ def test_dense_feed_forward_alone(dtype, hidden, ff):
 @pytest.mark.parametrize("M,N,K", [(1, 128, 64), (7, 200, 72), (16, 2048, 512), (30, 300, 2048), (64, 2048, 6144), (128, 384, 128), (128, 1000, 4096),
                                    (129, 96, 64), (300, 2048, 512), (513, 250, 1024), (2048, 2048, 2048), (2304, 520, 640)])
 @pytest.mark.parametrize("split_mode", [0, 1, 2, 4])
-def test_square_relu_and_softplus_in_every_path_of_the_product(M, N, K, split_mode):
-    """K in one part and in several, token tiles of 16 to 128 and whole prompts, widths that are no multiple of a tile; softplus
-    keeps its relative precision where it is small."""
+def test_square_relu_in_every_path_of_the_product(M, N, K, split_mode):
+    """K in one part and in several, token tiles of 16 to 128 and whole prompts, widths that are no multiple of a tile."""
     from ember_b200 import ops
     g = torch.Generator().manual_seed(M + N)
-    a, w = torch.randn(M, K, generator=g).bfloat16(), (K ** -0.5 * torch.randn(N, K, generator=g)).bfloat16()
-    bias = 3.0 * torch.randn(N, generator=g) - 3.0
-    bias[0] = 40.0
-    ad, wd, bd = a.cuda(), w.cuda(), bias.cuda()
-    z = ad.double() @ wd.double().T
-    sp = torch.nn.functional.softplus(z + bd.double(), threshold=1e9)
-    for epi, b, want, dt in ((ops.EPI_SQUARE_RELU, None, torch.relu(z) ** 2, torch.bfloat16), (ops.EPI_SOFTPLUS_F32, bd, sp, torch.float32)):
-        for fn in ("tc",) + (("simt",) if split_mode == 0 else ()):
-            out = torch.zeros(M, N, dtype=dt, device="cuda")
-            if fn == "tc":
-                ops.gemm_tc(ad, wd, out, M, epi, split_mode=split_mode, bias=b)
-            else:
-                ops.gemm_simt(ad, wd, out, M, epi, bias=b)
-            if dt == torch.bfloat16:
-                assert _rel(out.cpu(), want.cpu()) < 5e-3, (epi, fn)
-            else:
-                assert float(((out.double() - want).abs() / want).max()) < 2e-5, (epi, fn)
+    a, w = torch.randn(M, K, generator=g).bfloat16().cuda(), (K ** -0.5 * torch.randn(N, K, generator=g)).bfloat16().cuda()
+    want = (torch.relu(a.double() @ w.double().T) ** 2).cpu()
+    for fn in ("tc",) + (("simt",) if split_mode == 0 else ()):
+        out = torch.zeros(M, N, dtype=torch.bfloat16, device="cuda")
+        if fn == "tc":
+            ops.gemm_tc(a, w, out, M, ops.EPI_SQUARE_RELU, split_mode=split_mode)
+        else:
+            ops.gemm_simt(a, w, out, M, ops.EPI_SQUARE_RELU)
+        assert _rel(out.cpu(), want) < 5e-3, fn
 
 
 ROUTED_CASES = [
