@@ -97,6 +97,14 @@ __global__ void place_columns_kernel(const float* __restrict__ x, TO* __restrict
     }
 }
 
+template <typename T>
+__global__ void zero_kernel(T* __restrict__ x, size_t n) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i < n) x[i] = T{};
+}
+
 // out[t, i] = x[t, i] for i < n: some columns of fp32 rows as rows of their own.
 template <typename TO>
 __global__ void round_columns_kernel(const float* __restrict__ x, int ldx, TO* __restrict__ out, int n, size_t total) {
@@ -523,6 +531,17 @@ EMBER_API int ember_embed_bigram(const int* tokens, const int* prev_ids, int n_p
         else run(embed_bigram_kernel<__nv_bfloat16, __nv_bfloat16>, (const __nv_bfloat16*)table);
     }
     return check_launch("embed_bigram");
+}
+
+// A buffer that a product adds into.
+EMBER_API int ember_zero(float* x, long long n, void* stream) {
+    if (n <= 0) return 0;
+    if ((((uintptr_t)x) & 15) == 0 && n % 4 == 0) {
+        launch_kernel(zero_kernel<float4>, (unsigned)((n / 4 + 255) / 256), 256, 0, (cudaStream_t)stream, (float4*)x, (size_t)(n / 4));
+    } else {
+        launch_kernel(zero_kernel<float>, (unsigned)((n + 255) / 256), 256, 0, (cudaStream_t)stream, x, (size_t)n);
+    }
+    return check_launch("zero");
 }
 
 EMBER_API int ember_round_columns(const float* x, int ldx, void* out, int out_dtype, int T, int n, void* stream) {

@@ -171,10 +171,19 @@ __device__ __forceinline__ void store_finished_chunk(const GemmTcParams& p, int 
 // ``first``: these are the sums of the first part of K (the one that brings the bias).
 template <bool FIN>
 __device__ __forceinline__ void store_chunk_normal(const GemmTcParams& p, int m, int n0, int nv, float* v, bool first) {
-    if (FIN && ((p.bias && first) || p.act >= 3)) {
+    if (FIN) {
+        if (p.bias && first) {
 #pragma unroll
-        for (int j = 0; j < 16; j++)
-            if (j < nv) v[j] = finish_sum<true>(p, n0 + j, v[j]);
+            for (int j = 0; j < 16; j++)
+                if (j < nv) v[j] += __ldg(p.bias + n0 + j);
+        }
+        if (p.act == 4) {
+#pragma unroll
+            for (int j = 0; j < 16; j++) { const float r = fmaxf(v[j], 0.0f); v[j] = r * r; }
+        } else if (p.act == 3) {
+#pragma unroll
+            for (int j = 0; j < 16; j++) v[j] = gelu_erf(v[j]);
+        }
     }
     store_finished_chunk(p, m, n0, nv, v);
 }

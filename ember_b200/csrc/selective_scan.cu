@@ -12,12 +12,10 @@
 // a whole warp, the loop over tokens has no exchange between threads at all, and a warp leaves its partials of sum_n S C in
 // shared memory for the pass that finishes a chunk of CT tokens, which adds the warps' partials in order.  (With neighbouring
 // lanes sharing a channel the B and C reads were four shared-memory wavefronts a warp and token and bounded the kernel.)
-// States go two by two through packed fp32 arithmetic.  As many warps again bring the inputs, by cp.async into a ring of
+// States go two by two through packed fp32 arithmetic.  More warps bring the inputs, by cp.async into a ring of
 // chunks some way ahead (what a block has in flight is what keeps the memory busy: with one chunk in flight the kernel waited
 // for it), and finish the chunk before (sums, gate, store) while a chunk is computed: one barrier a chunk.
 // A step whose runs are single tokens takes a kernel of its own, a thread a channel with all its states.
-#include <type_traits>
-
 #include "common.cuh"
 
 EMBER_DEFINE_LAST_ERROR
@@ -31,6 +29,7 @@ __device__ __forceinline__ float exp2_approx(float x) {
 }
 
 constexpr int SS_CHUNK = 32;          // tokens a chunk
+constexpr int SS_STEPS = 4;           // tokens a turn of the computing loop
 constexpr int SS_RING = 5;            // chunks of inputs in shared memory: one being finished, one computed, the rest on their way
 
 struct SelectiveArgs {
@@ -43,7 +42,7 @@ struct SelectiveArgs {
     void* out;                                 // [T, inner]
     const int* query_start; const int* slots;
     int inner, N;
-    int by16;                                  // rows of x, dt and z can be copied 16 bytes at a time
+    int by16, bc16;                            // rows of x, dt and z, and of B and C, can be copied 16 bytes at a time
 };
 
 // Packed fp32 pairs.
@@ -88,6 +87,23 @@ __device__ __forceinline__ float silu_<float>(float z) { return z / (1.0f + expf
 template <>
 __device__ __forceinline__ float silu_<__nv_bfloat16>(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
 
+// NS neighbouring floats of shared memory in the widest reads NS allows.
+template <int NS>
+__device__ __forceinline__ void read_row(const float* p, float (&v)[NS]) {
+    if (NS % 4 == 0) {
+#pragma unroll
+        for (int i = 0; i < NS / 4; i++) {
+            const float4 f = reinterpret_cast<const float4*>(p)[i];
+            v[4 * i] = f.x; v[4 * i + 1] = f.y; v[4 * i + 2] = f.z; v[4 * i + 3] = f.w;
+        }
+    } else {
+#pragma unroll
+        for (int i = 0; i < NS / 2; i++) {
+            const float2 f = reinterpret_cast<const float2*>(p)[i];
+            v[2 * i] = f.x; v[2 * i + 1] = f.y;
+        }
+    }
+}
 __device__ __forceinline__ void copy16(void* dst, const void* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
@@ -95,22 +111,23 @@ __device__ __forceinline__ void copy4(void* dst, const void* src) {
     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
 
-// NW warps compute, NW warps feed them and finish what they leave.
-template <int NW, int NS, int CT, int RING, typename TO>
-__global__ void __launch_bounds__(64 * NW) selective_scan_kernel(SelectiveArgs p) {
-    constexpr int THREADS = 32 * NW, NP = NW * NS, N2 = NS / 2;    // states a channel (with padding); pairs a thread
+// NW warps compute, NH warps feed them and finish what they leave.
+template <int NW, int NS, int NH, int CT, int RING, typename TO>
+__global__ void __launch_bounds__(32 * (NW + NH)) selective_scan_kernel(SelectiveArgs p) {
+    constexpr int THREADS = 32 * NW, FEED = 32 * NH, NP = NW * NS, N2 = NS / 2;    // states a channel (with padding); pairs a thread
     constexpr int TILE = CT * 32;                                  // a chunk's elements of x, of dt and of z
-    static_assert(NS % 2 == 0 && CT % NW == 0 && RING >= 4, "states go two by two, tokens are shared out evenly");
+    static_assert(NS % 2 == 0 && RING >= 4, "states go two by two");
     extern __shared__ __align__(16) float smem[];
     float* xs = smem;                                  // RING x [x | dt | z] x [CT][32]
-    float* bs = xs + RING * 3 * TILE;                  // RING x [CT][NP / 2] (B, B, C, C) of two states
+    float* bs = xs + RING * 3 * TILE;                  // RING x [CT][B (NP) | C (NP)]
     float* yp = bs + RING * CT * NP * 2;               // 2 x [CT][NW][32] partial read-outs
     pdl_launch_dependents();
     const int s = blockIdx.y, inner = p.inner, N = p.N;
     const int lane = threadIdx.x & 31, c0 = blockIdx.x * 32, c = c0 + lane;
     const bool feeds = threadIdx.x >= THREADS;
     const int warp = (threadIdx.x >> 5) - (feeds ? NW : 0), tid = threadIdx.x - (feeds ? THREADS : 0);
-    for (int i = threadIdx.x; i < RING * CT * NP * 2; i += 2 * THREADS) bs[i] = 0.0f;      // (B and C of padded states stay zero)
+    if (N < NP)                                        // (B and C of padded states stay zero)
+        for (int i = threadIdx.x; i < RING * CT * NP * 2; i += THREADS + FEED) bs[i] = 0.0f;
     __syncthreads();
     pdl_wait();
     const int first = p.query_start[s], end = p.query_start[s + 1];
@@ -118,32 +135,39 @@ __global__ void __launch_bounds__(64 * NW) selective_scan_kernel(SelectiveArgs p
     const bool live = c < inner;
     if (feeds) {
         const float skip = live ? p.skip[c] : 0.0f;
+        const int n4 = N / 4;
         auto issue = [&](int i) {              // the inputs of chunk i on their way
             const int t0 = first + i * CT, n_tok = min(CT, end - t0);
             if (n_tok > 0) {
                 float* xd = xs + (i % RING) * 3 * TILE;
-                if (p.by16) {
+                auto tile = [&](float* dst, const float* src, int ld) {
+                    src += (size_t)t0 * ld + c0;
+                    if (p.by16) {
 #pragma unroll
-                    for (int e = tid; e < 3 * CT * 8; e += THREADS) {
-                        const int which = e / (CT * 8), r = e % (CT * 8), tt = r / 8, ch = c0 + (r % 8) * 4;
-                        const float* base = which == 0 ? p.x : (which == 1 ? p.dt : p.z);
-                        const int ld = which == 0 ? p.ld_x : (which == 1 ? p.ld_dt : p.ld_z);
-                        if (tt < n_tok && ch < inner) copy16(xd + which * TILE + r * 4, base + (size_t)(t0 + tt) * ld + ch);
+                        for (int r = tid; r < CT * 8; r += FEED)
+                            if (r / 8 < n_tok && c0 + (r % 8) * 4 < inner) copy16(dst + r * 4, src + (r / 8) * (size_t)ld + (r % 8) * 4);
+                    } else {
+                        for (int r = tid; r < TILE; r += FEED)
+                            if (r / 32 < n_tok && live) copy4(dst + r, src + (r / 32) * (size_t)ld + lane);
+                    }
+                };
+                tile(xd, p.x, p.ld_x);
+                tile(xd + TILE, p.dt, p.ld_dt);
+                tile(xd + 2 * TILE, p.z, p.ld_z);
+                float* bd = bs + (i % RING) * CT * NP * 2;
+                const float* src = p.bc + (size_t)t0 * p.ld_bc;
+                if (p.bc16) {
+                    constexpr int P4 = NP / 2;                     // 16-byte pieces of a token's B and C (with padding)
+#pragma unroll
+                    for (int r = tid; r < CT * P4; r += FEED) {
+                        const int tt = r / P4, w = r % P4, n = w % (P4 / 2);
+                        if (tt < n_tok && n < n4) copy16(bd + r * 4, src + (size_t)tt * p.ld_bc + (w < P4 / 2 ? 0 : N) + n * 4);
                     }
                 } else {
-                    for (int e = tid; e < 3 * TILE; e += THREADS) {
-                        const int which = e / TILE, r = e % TILE, tt = r / 32;
-                        const float* base = which == 0 ? p.x : (which == 1 ? p.dt : p.z);
-                        const int ld = which == 0 ? p.ld_x : (which == 1 ? p.ld_dt : p.ld_z);
-                        if (tt < n_tok && live) copy4(xd + which * TILE + r, base + (size_t)(t0 + tt) * ld + c);
+                    for (int r = tid; r < CT * 2 * NP; r += FEED) {
+                        const int tt = r / (2 * NP), w = r % (2 * NP), n = w % NP;
+                        if (tt < n_tok && n < N) copy4(bd + r, src + (size_t)tt * p.ld_bc + (w < NP ? 0 : N) + n);
                     }
-                }
-                float* bd = bs + (i % RING) * CT * NP * 2;
-#pragma unroll 4
-                for (int e = tid; e < CT * 2 * NP; e += THREADS) {
-                    const int tt = e / (2 * NP), w = e % (2 * NP), n = w % NP;
-                    if (tt < n_tok && n < N)
-                        copy4(bd + tt * 2 * NP + (n >> 1) * 4 + (n & 1) + (w < NP ? 0 : 2), p.bc + (size_t)(t0 + tt) * p.ld_bc + (w < NP ? 0 : N) + n);
                 }
             }
             asm volatile("cp.async.commit_group;" ::: "memory");
@@ -151,11 +175,11 @@ __global__ void __launch_bounds__(64 * NW) selective_scan_kernel(SelectiveArgs p
         const float dt_bias = live ? p.dt_bias[c] : 0.0f;
         auto arrived = [&](int i) {            // chunk i is there: raw steps become steps
             asm volatile("cp.async.wait_group %0;" ::"n"(RING - 3) : "memory");
-            asm volatile("bar.sync 1, %0;" ::"n"(THREADS) : "memory");      // (pieces that other feeding threads copied)
+            asm volatile("bar.sync 1, %0;" ::"n"(FEED) : "memory");      // (pieces that other feeding threads copied)
             if (i < chunks) {
                 float* xd = xs + (i % RING) * 3 * TILE + TILE + lane;
 #pragma unroll
-                for (int tt = warp; tt < CT; tt += NW) xd[tt * 32] = softplus_<TO>(xd[tt * 32] + dt_bias);
+                for (int tt = warp; tt < CT; tt += NH) xd[tt * 32] = softplus_<TO>(xd[tt * 32] + dt_bias);
             }
         };
         auto finish = [&](int i) {             // chunk i: its partials, gate, store
@@ -163,7 +187,7 @@ __global__ void __launch_bounds__(64 * NW) selective_scan_kernel(SelectiveArgs p
             const float* xd = xs + (i % RING) * 3 * TILE + lane;
             const float* yc = yp + (i & 1) * CT * THREADS + lane;
 #pragma unroll
-            for (int tt = warp; tt < CT; tt += NW) {
+            for (int tt = warp; tt < CT; tt += NH) {
                 if (live && tt < n_tok) {
                     const float* part = yc + tt * THREADS;
                     float y0 = 0.0f, y1 = 0.0f;
@@ -202,47 +226,50 @@ __global__ void __launch_bounds__(64 * NW) selective_scan_kernel(SelectiveArgs p
     for (int i = 0; i < chunks; i++) {
         const int n_tok = min(CT, end - first - i * CT);
         const float* xc = xs + (i % RING) * 3 * TILE + lane;
-        const float4* bc = reinterpret_cast<const float4*>(bs + (i % RING) * CT * 2 * NP + 2 * n0);
+        const float* bc = bs + (i % RING) * CT * 2 * NP + n0;
         float* yc = yp + (i & 1) * CT * THREADS + warp * 32 + lane;
-        // a group of tokens: first everything that does not depend on the state (their operands, decays and inputs), then the
-        // chain through the state, then the stores (one between two tokens would keep the next one's operands from being
-        // fetched ahead of it)
-        auto group = [&](auto size, int g0) {
-            constexpr int GR = decltype(size)::value;
-            f32x2 decay[GR][N2], in[GR][N2], out[GR][N2];
-#pragma unroll
-            for (int k = 0; k < GR; k++) {
-                const float d = xc[TILE + (g0 + k) * 32], u = d * xc[(g0 + k) * 32];
-                const f32x2 dd = pk2(d, d), uu = pk2(u, u);
-#pragma unroll
-                for (int j = 0; j < N2; j++) {
-                    const float4 v = bc[(g0 + k) * (NP / 2) + j];                // the same address for the whole warp
-                    const float2 e = up2(mul2(dd, a[j]));
-                    decay[k][j] = pk2(exp2_approx(e.x), exp2_approx(e.y));
-                    in[k][j] = mul2(uu, pk2(v.x, v.y));
-                    out[k][j] = pk2(v.z, v.w);
-                }
-            }
-            float y[GR];
-#pragma unroll
-            for (int k = 0; k < GR; k++) {
-                f32x2 acc;
-#pragma unroll
-                for (int j = 0; j < N2; j++) {
-                    st[j] = fma2(decay[k][j], st[j], in[k][j]);
-                    acc = j == 0 ? mul2(st[j], out[k][j]) : fma2(st[j], out[k][j], acc);
-                }
-                const float2 r = up2(acc);
-                y[k] = r.x + r.y;
-            }
-#pragma unroll
-            for (int k = 0; k < GR; k++) yc[(g0 + k) * THREADS] = y[k];
+        // A token in three steps, each one token behind the one before: its operands from shared memory, its decays and inputs,
+        // the state.  (Left to the compiler the steps of a token follow one another, and a warp waits out every latency of
+        // it.)  The two tokens looked at past the chunk's end lie in the ring and are not used.
+        struct Operands { float d, x; float B[NS], C[NS]; };
+        struct Prepared { f32x2 decay[N2], in[N2], out[N2]; };
+        auto load = [&](int k) {
+            Operands o;
+            o.d = xc[TILE + k * 32];
+            o.x = xc[k * 32];
+            read_row<NS>(bc + k * 2 * NP, o.B);                                  // (the same addresses for the whole warp)
+            read_row<NS>(bc + k * 2 * NP + NP, o.C);
+            return o;
         };
-        if (n_tok == CT) {
-            constexpr int GR = NS > 8 ? 2 : (NS > 4 ? 4 : 8);
-            for (int g0 = 0; g0 < CT; g0 += GR) group(std::integral_constant<int, GR>{}, g0);
-        } else {
-            for (int tt = 0; tt < n_tok; tt++) group(std::integral_constant<int, 1>{}, tt);
+        auto prepare = [&](const Operands& o) {
+            Prepared t;
+            const float u = o.d * o.x;
+            const f32x2 dd = pk2(o.d, o.d), uu = pk2(u, u);
+#pragma unroll
+            for (int j = 0; j < N2; j++) {
+                const float2 e = up2(mul2(dd, a[j]));
+                t.decay[j] = pk2(exp2_approx(e.x), exp2_approx(e.y));
+                t.in[j] = mul2(uu, pk2(o.B[2 * j], o.B[2 * j + 1]));
+                t.out[j] = pk2(o.C[2 * j], o.C[2 * j + 1]);
+            }
+            return t;
+        };
+        Operands ahead = load(0);
+        Prepared ready = prepare(ahead);
+        ahead = load(1);
+#pragma unroll SS_STEPS
+        for (int k = 0; k < n_tok; k++) {
+            const Prepared t = ready;
+            ready = prepare(ahead);
+            ahead = load(k + 2);
+            f32x2 acc;
+#pragma unroll
+            for (int j = 0; j < N2; j++) {
+                st[j] = fma2(t.decay[j], st[j], t.in[j]);
+                acc = j == 0 ? mul2(st[j], t.out[j]) : fma2(st[j], t.out[j], acc);
+            }
+            const float2 r = up2(acc);
+            yc[k * THREADS] = r.x + r.y;
         }
         __syncthreads();
     }
@@ -290,20 +317,20 @@ __global__ void __launch_bounds__(SS_STEP_THREADS) selective_step_kernel(Selecti
     ((TO*)p.out)[(size_t)t * inner + c] = from_float<TO>(fmaf(skip, x, y0 + y1) * silu_<TO>(z));
 }
 
-template <int NW, int NS, int CT, typename TO, int RING = SS_RING>
+template <int NW, int NS, int NH, int CT, typename TO, int RING = SS_RING>
 int launch_selective(const SelectiveArgs& p, int S, cudaStream_t st) {
     const size_t smem = (size_t)(RING * 3 * CT * 32 + RING * 2 * CT * NW * NS + 2 * CT * NW * 32) * sizeof(float);
     if (smem > 48 * 1024) {
-        cudaError_t e = cudaFuncSetAttribute(selective_scan_kernel<NW, NS, CT, RING, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(selective_scan_kernel<NW, NS, NH, CT, RING, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return fail("selective_scan: shared memory %zu: %s", smem, cudaGetErrorString(e));
     }
-    launch_kernel(selective_scan_kernel<NW, NS, CT, RING, TO>, dim3((p.inner + 31) / 32, S), 64 * NW, smem, st, p);
+    launch_kernel(selective_scan_kernel<NW, NS, NH, CT, RING, TO>, dim3((p.inner + 31) / 32, S), 32 * (NW + NH), smem, st, p);
     return check_launch("selective_scan");
 }
 
-// Computing warps a block and states a thread by the number of states.  Sixteen states: eight warps of two states while every
-// block has an SM for itself (2,048 tokens of 4,096 channels: 98 us against 115), four warps of four, with fewer reads of
-// shared memory a state, when blocks share SMs (four runs of 512 tokens: 80 us against 102; 8,192 channels: 150 against 187).
+// Computing warps a block, states a thread and feeding warps by the number of states.  (Sixteen states, 2,048 tokens of 4,096
+// channels: four warps of four states 103 us, eight of two 105, and when blocks share SMs four runs of 512 tokens 86 us either
+// way: what is left is the instructions of both kinds of warps, 0.7 of the issue slots of the SMs that have a block.)
 template <typename TO>
 int pick_selective(const SelectiveArgs& p, int S, bool single, cudaStream_t st) {
     const int N = p.N;
@@ -313,13 +340,12 @@ int pick_selective(const SelectiveArgs& p, int S, bool single, cudaStream_t st) 
         else launch_kernel(selective_step_kernel<16, TO>, grid, SS_STEP_THREADS, 0, st, p);
         return check_launch("selective_step");
     }
-    if (N <= 8) return launch_selective<4, 2, SS_CHUNK, TO>(p, S, st);
-    if (N <= 16 && (long long)S * ((p.inner + 31) / 32) <= 148) return launch_selective<8, 2, SS_CHUNK, TO>(p, S, st);
-    if (N <= 16) return launch_selective<4, 4, SS_CHUNK, TO>(p, S, st);
-    if (N <= 32) return launch_selective<8, 4, SS_CHUNK, TO>(p, S, st);
-    if (N <= 64) return launch_selective<8, 8, SS_CHUNK, TO>(p, S, st);
-    if (N <= 128) return launch_selective<8, 16, 16, TO, 4>(p, S, st);
-    return launch_selective<16, 16, 16, TO, 4>(p, S, st);
+    if (N <= 8) return launch_selective<4, 2, 8, SS_CHUNK, TO>(p, S, st);
+    if (N <= 16) return launch_selective<4, 4, 8, SS_CHUNK, TO>(p, S, st);
+    if (N <= 32) return launch_selective<8, 4, 8, SS_CHUNK, TO>(p, S, st);
+    if (N <= 64) return launch_selective<8, 8, 8, SS_CHUNK, TO>(p, S, st);
+    if (N <= 128) return launch_selective<8, 16, 8, 16, TO, 4>(p, S, st);
+    return launch_selective<16, 16, 8, 16, TO, 4>(p, S, st);
 }
 
 }  // namespace ember
@@ -338,8 +364,9 @@ EMBER_API int ember_selective_scan(const float* x, int ld_x, const float* dt, in
     if (ld_x < inner || ld_dt < inner || ld_z < inner || ld_bc < 2 * N || state_stride < (long long)inner * N)
         return fail("selective_scan: rows of %d / %d / %d / %d, state rows of %lld do not hold %d channels of %d states", ld_x, ld_dt, ld_z, ld_bc, state_stride, inner, N);
     if (S > 65535) return fail("selective_scan: %d runs are too many for one launch", S);
-    SelectiveArgs p{x, ld_x, dt, ld_dt, bc, ld_bc, z, ld_z, dt_bias, a, skip, state, state_stride, out, query_start, slots, inner, N, 0};
+    SelectiveArgs p{x, ld_x, dt, ld_dt, bc, ld_bc, z, ld_z, dt_bias, a, skip, state, state_stride, out, query_start, slots, inner, N, 0, 0};
     p.by16 = inner % 4 == 0 && ld_x % 4 == 0 && ld_dt % 4 == 0 && ld_z % 4 == 0 && ((((uintptr_t)x) | ((uintptr_t)dt) | ((uintptr_t)z)) & 15) == 0;
+    p.bc16 = N % 4 == 0 && ld_bc % 4 == 0 && (((uintptr_t)bc) & 15) == 0;
     cudaStream_t st = (cudaStream_t)stream;
     const bool single = T == S;
     if (out_dtype == EMBER_F32) return pick_selective<float>(p, S, single, st);

@@ -138,6 +138,15 @@ def embed_bigram(tokens: torch.Tensor, table: torch.Tensor, bigram: torch.Tensor
           _p(state), c_int(state.stride(0)), _p(err), c_void_p(stream if stream is not None else current_stream_ptr()))
 
 
+def zero(x: torch.Tensor, n: int, stream: Optional[int] = None) -> None:
+    """x[:n] = 0 (fp32, in the buffer's order): what a product with an adding epilogue starts from."""
+    _check(x, "x", torch.float32)
+    if x.numel() < n:
+        raise KernelError(f"zero: {n} of {x.numel()} elements")
+    lib = _lib("elementwise")
+    _call(lib, lib.ember_zero, _p(x), c_longlong(n), _stream(stream))
+
+
 def round_columns(x: torch.Tensor, col: int, n: int, out: torch.Tensor, T: int, stream: Optional[int] = None) -> None:
     """out[t, :n] = x[t, col : col + n] in out's type (x fp32 [T, ld], out [T, n]): columns of one product made the operand of
     another."""

@@ -30,6 +30,18 @@ class Linear:
         b = rt.to_device(bias, torch.float32) if bias is not None else None
         return cls(dev, b)
 
+    # A prompt portion's product with so few columns has too few tiles for the SMs; added into zeros, K is cut as well.
+    NARROW = 512
+
+    def store_f32(self, ctx, x: torch.Tensor, out: torch.Tensor, m: int) -> None:
+        """out[:m] = the product in fp32, in whichever way fills the device: stored, or (narrow products of prompt portions on
+        the tensor cores) added into zeros in parts of K."""
+        if m > 128 and self.n <= self.NARROW and self.k >= 1024 and ops.gemm_tc_usable(x, self.weight, self.bias, ops.EPI_ADD_F32):
+            ops.zero(out, m * self.n, stream=ctx.stream)
+            self(ctx, x, out, m, ops.EPI_ADD_F32)
+        else:
+            self(ctx, x, out, m, ops.EPI_STORE_F32)
+
     def __call__(self, ctx, x: torch.Tensor, out: torch.Tensor, m: int, epilogue: int = ops.EPI_STORE) -> None:
         if m <= 0:
             return

@@ -486,7 +486,7 @@ class SelectiveScan(_StateMixer):
         self.in_proj(ctx, x, proj, T, ops.EPI_STORE_F32)
         ops.conv_silu(proj, 0, self.taps, self.conv_bias, cache.state, inner * N, ctx.seq_of, ctx.query_start, ctx.state_slots,
                       conv, T, ctx.S, stream=ctx.stream, rounded=conv_r if half else None)
-        self.x_proj(ctx, conv_r, low, T, ops.EPI_STORE_F32)
+        self.x_proj.store_f32(ctx, conv_r, low, T)
         if half and ops.gemm_tc_usable(y, self.dt_proj.weight, None, ops.EPI_STORE_F32):
             low_r = ctx.buf("mamba1.low_rounded", (mt, R), rt.dtype)
             ops.round_columns(low, 0, R, low_r, T, stream=ctx.stream)
