@@ -1,5 +1,5 @@
-"""Malusun: a decoder whose layers are listed one by one in config.json, every sublayer between two norms:
-``x = x + norm1b(mixer(norm1(x)))``, then ``x = x + norm2b(ff(norm2(x)))``; norm weights are stored around zero.  Three mixers: a
+"""Malusun: a decoder whose layers are listed one by one in config.json, every sublayer between two norms: the
+stream gains ``norm1b(mixer(norm1(.)))`` of itself and after it ``norm2b(ff(norm2(.)))``; norm weights are stored around zero.  Three mixers: a
 selective scan with a diagonal state per channel ("mamba1"); grouped-query softmax attention in a sliding window with a
 rotate-half rotation of part of each head ("attention"); and the same without a rotation, with biases, a linear distance
 bias on the scores and one added to the softmax's denominator ("attention_2").  Attention layers may blend their values

@@ -312,10 +312,10 @@ class StateSpaceSpec(PartSpec):
 
 @dataclass(frozen=True)
 class SelectiveScanSpec(PartSpec):
-    """Selective scan with a diagonal state per channel (Mamba): W_in h = [x | z], both of size ``inner``; x passes a short
-    causal convolution (``conv`` [inner, conv_taps], bias ``conv.b``) and silu; W_x x = [low | B | C] of sizes ``dt_rank``,
-    ``state_size``, ``state_size``; dt = softplus(W_dt low + dt.b), one per channel; S[c, n] <- exp(-dt_c exp(A_log[c, n])) S[c, n]
-    + dt_c x_c B_n; y_c = sum_n S[c, n] C_n + D_c x_c; W_o (y silu(z)).  Tensors: in, conv, conv.b, x, dt, dt.b, A_log, D, o."""
+    """Selective scan with a diagonal state per channel (Mamba): W_in h = [u | z], both of size ``inner``; u passes a short
+    causal convolution (``conv`` [inner, conv_taps], bias ``conv.b``) and silu; W_x u = [low | B | C] of sizes ``dt_rank``,
+    ``state_size``, ``state_size``; dt = softplus(W_dt low + dt.b), one per channel; M[n, c] <-
+    e^(-dt_c a[n, c]) M[n, c] + dt_c u_c B[n] with a = exp(A_log)^T; r_c = <M[:, c], C> + D_c u_c; W_o (r * silu(z)).  Tensors: in, conv, conv.b, x, dt, dt.b, A_log, D, o."""
 
     kind: ClassVar[str] = "mamba1"
     hidden_size: int = 0

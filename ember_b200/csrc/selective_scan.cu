@@ -1,15 +1,15 @@
-// Selective scan with a diagonal state per channel (Mamba) over a ragged batch.  Per channel c and state n, with
-// dt = softplus(raw step + bias) per token and channel and one B and one C row per token:
+// Selective scan with a diagonal state per channel (Mamba) over a ragged batch.  With a step d = softplus(raw step + bias) per
+// token and channel, and one B and one C row per token,
 //
-//     S[c, n] <- exp(-dt_c exp(A_log[c, n])) S[c, n] + dt_c x_c B_n;   y_c = sum_n S[c, n] C_n + D_c x_c
+//     M[n, c] <- e^(-d_c a[n, c]) M[n, c] + d_c u_c B[n];   r_c = <M[:, c], C> + D_c u_c
 //
-// and out = y * silu(z).  Everything is fp32 (`out` may be bfloat16: it is the operand of the next product).  The decay is
-// taken as 2^(dt a) with a = -exp(A_log) log2(e) made once when the weights are loaded.
+// and out = r * silu(z).  Everything is fp32 (`out` may be bfloat16: it is the operand of the next product).  The decay is
+// taken as a power of two, whose exponents' factor -a log2(e) is made once when the weights are loaded.
 //
-// A step's tokens are S runs (query_start [S + 1]); run s belongs to state slot slots[s], whose row holds S as [N, inner]
+// A step's tokens are S runs (query_start [S + 1]); run s belongs to state slot slots[s], whose row holds M as [N, inner]
 // (neighbouring channels side by side, like every other operand).  A block walks one run for 32 channels: a lane is a
 // channel, and the block's NW warps share its states, NS each, in registers.  A token's B and C are then the same address for
-// a whole warp, the loop over tokens has no exchange between threads at all, and a warp leaves its partials of sum_n S C in
+// a whole warp, the loop over tokens has no exchange between threads at all, and a warp leaves its partials of the read-out in
 // shared memory for the pass that finishes a chunk of CT tokens, which adds the warps' partials in order.  (With neighbouring
 // lanes sharing a channel the B and C reads were four shared-memory wavefronts a warp and token and bounded the kernel.)
 // States go two by two through packed fp32 arithmetic.  More warps bring the inputs, by cp.async into a ring of

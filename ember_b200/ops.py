@@ -1044,7 +1044,7 @@ def selective_scan(x: torch.Tensor, dt: torch.Tensor, bc: torch.Tensor, bc_col: 
     (after convolution and silu), ``dt`` fp32 [T, inner] raw steps (softplus of them plus ``dt_bias`` is taken here), ``bc`` fp32
     with B and C behind one another from column ``bc_col`` on, ``z`` fp32 with the gate from column ``z_col`` on, ``a`` fp32
     [states, inner] = -exp(A_log) log2(e), ``skip`` [inner]; a request's state, [states, inner], is the first inner * states
-    floats of its row of ``state``.  out [T, inner] (fp32 or bfloat16) = (S C + skip x) silu(z)."""
+    floats of its row of ``state``.  out [T, inner] (fp32 or bfloat16) = (read-out + skip x) silu(z)."""
     for t, n in ((x, "x"), (dt, "dt"), (bc, "bc"), (z, "z"), (dt_bias, "dt_bias"), (a, "a"), (skip, "skip"), (state, "state")):
         _check(t, n, torch.float32)
     _check(out, "out")

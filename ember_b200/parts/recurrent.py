@@ -426,15 +426,15 @@ class TimeMix(_StateMixer):
 
 # ---------------------------------------------------------------------------------------------- mamba1
 class SelectiveScan(_StateMixer):
-    """W_in h = [x | z]; x passes a short causal convolution (with bias) and silu; W_x x = [low | B | C];
-    dt = softplus(W_dt low + dt.b), one per channel; per channel c and state n
+    """W_in h = [u | z]; u passes a short causal convolution (with bias) and silu; W_x u = [low | B | C];
+    d = softplus(W_dt low + dt.b), one per channel; with a = exp(A_log)^T
 
-        S[c, n] <- exp(-dt_c exp(A_log[c, n])) S[c, n] + dt_c x_c B_n;  y_c = sum_n S[c, n] C_n + D_c x_c
+        M[n, c] <- e^(-d_c a[n, c]) M[n, c] + d_c u_c B[n];  r_c = <M[:, c], C> + D_c u_c
 
-    then y * silu(z) and the output product.  The products read bfloat16 operands on the bfloat16 path and leave fp32; steps,
+    then r * silu(z) and the output product.  The products read bfloat16 operands on the bfloat16 path and leave fp32; steps,
     decays, B, C and the state are fp32.  The step's projection goes over a rounded copy of ``low`` on the tensor cores, else
     it reads ``low`` where the product before it left it; its bias and softplus are the scan's.  The
-    state row of a request holds S [states, inner] and, behind it, the convolution's last inputs.  Tensors under the
+    state row of a request holds M [states, inner] and, behind it, the convolution's last inputs.  Tensors under the
     prefix: in, conv, conv.b, x, dt, dt.b, A_log, D, o."""
 
     def __init__(self, spec, prefix: str = ""):

@@ -511,6 +511,19 @@ def test_square_relu_in_every_path_of_the_product(M, N, K, split_mode):
         assert _rel(out.cpu(), want) < 5e-3, fn
 
 
+@pytest.mark.parametrize("M,N,K", [(129, 160, 1024), (300, 130, 2048), (2048, 160, 4096), (700, 512, 1088), (2100, 96, 1024), (64, 160, 4096), (300, 600, 2048)])
+@pytest.mark.parametrize("dtype", [torch.bfloat16, torch.float32])
+def test_narrow_products_of_prompt_portions(M, N, K, dtype):
+    """Few columns and many tokens: added into zeros with K in parts (whatever the buffer held), or stored."""
+    from types import SimpleNamespace
+    from ember_b200.parts.linear import Linear
+    g = torch.Generator().manual_seed(M + N)
+    a, w = torch.randn(M, K, generator=g).to(dtype).cuda(), (K ** -0.5 * torch.randn(N, K, generator=g)).to(dtype).cuda()
+    out = torch.full((M + 1, N), 7.0, device="cuda")
+    Linear(w).store_f32(SimpleNamespace(err=None, stream=None), a, out, M)
+    assert _rel(out[:M].cpu(), (a.double() @ w.double().T).cpu()) < 1e-5 and float((out[M] - 7.0).abs().max()) == 0.0
+
+
 ROUTED_CASES = [
     # hidden, ff, experts, top, shared
     (64, 40, 6, 2, 32), (100, 30, 3, 3, 50), (96, 24, 5, 1, 0), (128, 256, 48, 4, 128), (64, 50, 8, 1, 64), (64, 16, 1, 1, 8), (72, 20, 64, 6, 0)]
