@@ -157,7 +157,7 @@ def drawn_malusun(seed: int) -> dict:
             mix = pick(True, True, False, None)
             dim = pick(16, 32, 64, 128, 24, 20, vdim)
             own_kv, own_v = (kv, vdim) if mix else (pick(1, 2, 3), pick(16, 48, 64, dim, dim))
-            rot = (dim - dim % 2 if pick(True, False) else pick(2, 8, 16), pick(10000.0, 500.0, 1e6)) if kind == "attention" and rng.random() < 0.9 else None
+            rot = (dim - dim % 2 if pick(True, False) else min(dim - dim % 2, pick(2, 8, 16)), pick(10000.0, 500.0, 1e6)) if kind == "attention" and rng.random() < 0.9 else None
             mixer = _attention(own_kv * pick(1, 2, 4), own_kv, dim, own_v, float(dim ** -0.5 * pick(1.0, 0.7, 2.0)),
                                pick(None, 16, 24, 50, 64, 96, 7, 1, 130), rot, mix)
         layers.append(_layer(kind, mixer, mlp))

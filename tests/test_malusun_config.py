@@ -92,7 +92,7 @@ def test_random_folder_declares_what_the_plain_implementation_reads(name, tmp_pa
 
 def test_drawn_configurations_are_read():
     from ember_b200.config import config_from_dict
-    for seed in range(60):
+    for seed in range(200):
         c = drawn_malusun(seed)
         back = config_from_dict(config_from_dict(c).to_json()).to_json()
         assert all(back.get(k) == c.get(k) for k in ("layers", "embedding", "vocab", "width"))
